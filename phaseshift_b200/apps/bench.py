@@ -10,6 +10,8 @@ import statistics
 import sys
 from typing import List, Optional
 
+from ..models.registry import preset_names
+
 SUBCOMMANDS = ("pp", "tg", "batch", "gemm", "activation-quantize", "rmsnorm", "l2-normalize", "kv-append",
                "paged-attention", "rope", "gdn-recurrence", "gdn-conv1d", "elementwise", "embedding", "sampling", "mtp",
                "gpu-memory", "tp-reduce", "dflash2", "kld")
@@ -20,7 +22,7 @@ FUSED_INTO = {"l2-normalize": "gdn-recurrence",      # q/k L2 normalisation happ
 
 
 def _model_args(p):
-    p.add_argument("--model-dir"); p.add_argument("--random-model", default=None, choices=["tiny", "4b", "27b"])
+    p.add_argument("--model-dir"); p.add_argument("--random-model", default=None, choices=preset_names())
     p.add_argument("--preset", default=None); p.add_argument("--device", default=None)
     p.add_argument("--kv-cache-dtype", default="bf16", choices=["bf16", "fp8_e4m3", "nvfp4"])
     p.add_argument("--runs", type=int, default=3); p.add_argument("--warmup", type=int, default=1); p.add_argument("--output")
@@ -73,8 +75,7 @@ def build_parser() -> argparse.ArgumentParser:
 
 def _engine(a, max_seq_len: int, slots: int = 1, spec_rows: int = 0):
     import torch
-    from ..models.qwen35.config import PRESETS
-    from ..models.qwen35.weights import build_engine_weights, load_engine_weights, random_getter
+    from ..models import registry
     from ..runtime.engine import Engine
     from ..runtime.state import StateConfig
     dev = torch.device(a.device or ("cuda:0" if torch.cuda.is_available() else "cpu"))
@@ -89,10 +90,10 @@ def _engine(a, max_seq_len: int, slots: int = 1, spec_rows: int = 0):
         if tp.rank != 0:
             sys.stdout = open(os.devnull, "w")
     if a.model_dir:
-        ew = load_engine_weights(a.model_dir, dev, a.preset, keep_canonical=dev.type != "cuda", **tp_kw)
+        ew = registry.load_weights(a.model_dir, dev, a.preset, keep_canonical=dev.type != "cuda", **tp_kw)
     else:
-        cfg = PRESETS[a.random_model or "tiny"]()
-        ew = build_engine_weights(cfg, random_getter(cfg, 0, dev), a.preset or "bf16", dev, keep_canonical=dev.type != "cuda", **tp_kw)
+        cfg = registry.preset_config(a.random_model or "tiny")
+        ew = registry.random_weights(cfg, dev, a.preset or "bf16", keep_canonical=dev.type != "cuda", **tp_kw)
     extra = dict(conv_ring=max(16, 3 + spec_rows), spec_rows=spec_rows) if spec_rows else {}
     return Engine(ew, dev, StateConfig(max_slots=slots, max_seq_len=max_seq_len, kv_dtype=a.kv_cache_dtype, **extra), tp=tp), dev
 

@@ -22,11 +22,10 @@ def build_parser() -> argparse.ArgumentParser:
 
 def main(argv: Optional[List[str]] = None) -> int:
     a = build_parser().parse_args(argv)
-    import json
-    import os
+    from ..models.registry import config_from_dir
     from .server import load_tokenizer
     try:
-        vocab = int(json.load(open(os.path.join(a.model_dir, "config.json"))).get("vocab_size", 0)) or 259
+        vocab = config_from_dir(a.model_dir).vocab_size
     except (OSError, ValueError):
         vocab = 259
     # the directory's own tokenizer and chat template; directories without tokenizer assets (random test models) get the

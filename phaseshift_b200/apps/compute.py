@@ -14,14 +14,19 @@ import select
 import sys
 from typing import List, Optional
 
+from ..models.registry import DTYPES, preset_config, preset_names
+
 DEFAULT_PROMPT = [248041, 77091]
 
 
 def build_parser() -> argparse.ArgumentParser:
     ap = argparse.ArgumentParser(prog="phaseshift-compute", description=__doc__.split("\n")[0])
     ap.add_argument("--model-dir")
-    ap.add_argument("--random-model", choices=["tiny", "4b", "27b"], help="random-init weights instead of --model-dir")
+    ap.add_argument("--random-model", choices=preset_names(), help="random-init weights instead of --model-dir")
     ap.add_argument("--preset", default=None, choices=["bf16", "nvfp4", "mxfp8"], help="quantise a BF16 model on load")
+    ap.add_argument("--dtype", default=None, choices=sorted(DTYPES),
+                    help="precision of projections and activations (default: bfloat16 on a GPU, float32 on CPU; float32 on a GPU "
+                         "needs a model family with 32-bit kernels)")
     ap.add_argument("--input-ids-file")
     ap.add_argument("--max-new-tokens", type=int, default=32)
     ap.add_argument("--max-seq-len", type=int, default=512)
@@ -84,8 +89,7 @@ class ComputeRuntime:
 
     def __init__(self, a):
         import torch
-        from ..models.qwen35.config import PRESETS
-        from ..models.qwen35.weights import build_engine_weights, load_engine_weights, random_getter
+        from ..models import registry
         from ..runtime.engine import Engine
         from ..runtime.serving import ServingEngine
         from ..runtime.state import StateConfig
@@ -98,13 +102,17 @@ class ComputeRuntime:
             self.tp, self.device, self.host_group = init_tensor_parallel(self.device.type)
             self.rank = self.tp.rank
             tp_kw = dict(tp_rank=self.tp.rank, tp_size=self.tp.size)
-        if a.random_model:
-            cfg = PRESETS[a.random_model]()
-            ew = build_engine_weights(cfg, random_getter(cfg, 0, self.device), a.preset or "bf16", self.device,
-                                      keep_canonical=self.device.type != "cuda", **tp_kw)
-        else:
-            ew = load_engine_weights(a.model_dir, self.device, a.preset, verify_weights=bool(a.verify_weights),
-                                     keep_canonical=self.device.type != "cuda", **tp_kw)
+        dtype = DTYPES.get(getattr(a, "dtype", None) or "")
+        kw = dict(keep_canonical=self.device.type != "cuda", **tp_kw)
+        try:
+            if a.random_model:
+                ew = registry.random_weights(preset_config(a.random_model), self.device, a.preset, dtype, **kw)
+            else:
+                ew = registry.load_weights(a.model_dir, self.device, a.preset, dtype, verify_weights=bool(a.verify_weights), **kw)
+        except registry.UnsupportedOption as e:
+            raise SystemExit(f"phaseshift-compute: {e}")
+        if a.dflash2_model_dir and ew.cfg.family != "qwen35":
+            raise SystemExit("phaseshift-compute: speculative decoding (--dflash2-model-dir) needs the hybrid decoder")
         self.cfg = ew.cfg
         spec = bool(a.dflash2_model_dir)
         from ..runtime.state import KV_DTYPE_ALIASES

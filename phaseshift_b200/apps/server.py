@@ -21,6 +21,7 @@ import time
 import uuid
 from typing import Dict, List, Optional
 
+from ..models.registry import DTYPES, preset_names
 from ..serving import chat
 
 try:        # module-level names so FastAPI can resolve the handlers' (string) annotations
@@ -32,7 +33,8 @@ except Exception:  # pragma: no cover - the server app needs fastapi; everything
 
 def build_parser() -> argparse.ArgumentParser:
     ap = argparse.ArgumentParser(prog="phaseshift-server")
-    ap.add_argument("--model-dir"); ap.add_argument("--random-model", choices=["tiny", "4b", "27b"])
+    ap.add_argument("--model-dir"); ap.add_argument("--random-model", choices=preset_names())
+    ap.add_argument("--dtype", default=None, choices=sorted(DTYPES))
     ap.add_argument("--preset", default=None); ap.add_argument("--host", default="127.0.0.1")
     ap.add_argument("--port", type=int, default=8000); ap.add_argument("--max-seq-len", type=int, default=32768)
     ap.add_argument("--arena-gib", type=float, default=0); ap.add_argument("--device", default=None)
@@ -514,7 +516,7 @@ def load_tokenizer(model_dir: Optional[str], vocab_size: int):
 def build_runtime(a):
     from .compute import ComputeRuntime
     ns = argparse.Namespace(model_dir=a.model_dir, random_model=a.random_model, preset=a.preset, device=a.device,
-                            max_seq_len=a.max_seq_len, page_tokens=a.page_tokens, arena_gib=a.arena_gib,
+                            dtype=getattr(a, "dtype", None), max_seq_len=a.max_seq_len, page_tokens=a.page_tokens, arena_gib=a.arena_gib,
                             max_concurrent_requests=a.max_concurrent_requests,
                             kv_cache_capacity_tokens=a.kv_cache_capacity_tokens or (a.max_concurrent_requests + 1) * (a.max_seq_len + 1),
                             kv_cache_dtype=a.kv_cache_dtype, prefix_cache_capacity_tokens=a.prefix_cache_capacity_tokens,

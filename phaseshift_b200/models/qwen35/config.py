@@ -35,6 +35,7 @@ class Qwen35Config:
     layer_types: Optional[List[int]] = None       # 0 = GDN, 1 = full attention
     eos_token_ids: List[int] = field(default_factory=list)
     name: str = "qwen35"
+    family = "qwen35"
 
     def __post_init__(self):
         if self.layer_types is None:
@@ -81,6 +82,17 @@ class Qwen35Config:
     @property
     def attn_layers(self) -> List[int]:
         return [i for i, t in enumerate(self.layer_types) if t == 1]
+
+    def geometry(self, tp_rank: int = 0, tp_size: int = 1):
+        from .weights import TpGeometry
+        return TpGeometry.make(self, tp_rank, tp_size)
+
+    def state_specs(self, geo) -> list:
+        """Cache and state of every layer on one rank (runtime/state.py)."""
+        from ...runtime.state import KVSpec, RecurrentSpec, RunSpec
+        Dk, Dv = self.linear_key_head_dim, self.linear_value_head_dim
+        return [RunSpec(KVSpec(len(geo.kv_heads), self.head_dim), None) if t == 1 else
+                RunSpec(None, RecurrentSpec(len(geo.gdn_v_heads), Dk, Dv, 2 * Dk + Dv)) for t in self.layer_types]
 
     def param_count(self) -> int:
         h = self.hidden_size

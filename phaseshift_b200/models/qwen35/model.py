@@ -14,20 +14,12 @@ import torch
 
 from ...runtime.batch import StepBatch
 from ...runtime.state import ModelState
+from ..common import StepOutput
 from .config import Qwen35Config
 from .weights import EngineWeights
 
 
 FUSED_BA_MAX_ROWS = 8
-
-
-class StepOutput:
-    __slots__ = ("tokens", "logits", "hidden", "taps", "taps_cat", "read_back")
-
-    def __init__(self, tokens, logits, hidden, taps, taps_cat=None):
-        self.tokens, self.logits, self.hidden, self.taps = tokens, logits, hidden, taps
-        self.taps_cat = taps_cat        # the tapped hidden states side by side, [rows, taps * H] (taps are views of it)
-        self.read_back = None
 
 
 class Qwen35Runner:

@@ -16,25 +16,25 @@ import torch
 from .trace import OpTrace
 import torch.nn.functional as F
 
-from ..models.qwen35.config import Qwen35Config
 from ..models.qwen35.weights import AttnW, GdnW, LinearW
 from ..runtime.batch import StepBatch
 from ..runtime.state import GdnLayerState, KVLayer, ModelState
 from ..utils.sampling import sample_row_host
+from .specs import AttnSpec, GlaSpec, Pending
 
 
 class RefOps(OpTrace):
     act_dtype = torch.float32
     name = "ref"
 
-    def __init__(self, cfg: Qwen35Config, device, act_quant: bool = False, **_):
+    def __init__(self, cfg, device, act_quant: bool = False, **_):
         """``act_quant``: quantise the input of every block-quantised projection to the weights' block format
         (quant/act_quant.py), the arithmetic of the CUDA tensor-core layout; off = bf16/fp32 activations, the
         arithmetic of the streaming layout."""
         self.cfg, self.device = cfg, device
         self.act_quant = act_quant
-        half = cfg.rotary_dim // 2
-        self.inv_freq = cfg.rope_theta ** (-torch.arange(half, dtype=torch.float64) * 2.0 / cfg.rotary_dim)
+        half = getattr(cfg, "rotary_dim", 0) // 2
+        self.inv_freq = getattr(cfg, "rope_theta", 1.0) ** (-torch.arange(half, dtype=torch.float64) * 2.0 / max(1, 2 * half))
         self.launches = 0
         self.exact_rows = False
 
@@ -45,7 +45,7 @@ class RefOps(OpTrace):
         return self._dense(table)[b.ids[:rows].long()]
 
     def linear(self, x, W: LinearW, *, name: str, norm_w=None, eps: float = 0.0, residual=None, swiglu=False,
-               out_f32=False, out=None, ssq_in=None, ssq_out=None, prefetch=None, **_):
+               reglu=False, out_f32=False, out=None, ssq_in=None, ssq_out=None, prefetch=None, **_):
         x = x.float()
         if self.act_quant and W.fmt in ("nvfp4", "mxfp8"):
             # the tensor-core layout's arithmetic: quantise x (1 + w), apply the row factor 1/rms after the product
@@ -62,6 +62,8 @@ class RefOps(OpTrace):
             y = x @ self._dense(W).T
         if swiglu:
             y = F.silu(y[:, 0::2]) * y[:, 1::2]
+        if reglu:
+            y = F.relu(y[:, 0::2]) * y[:, 1::2]
         if residual is not None:
             y = y + residual.float()
         if out is not None:
@@ -222,3 +224,88 @@ class RefOps(OpTrace):
                 sum_out.copy_(x)
         ww = (1.0 + w.float()) if one_plus else w.float()
         return x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps) * ww
+
+    # ------------------------------------------------------------------ 32-bit residual stream
+    def embed_f32(self, b: StepBatch, rows: int, table: torch.Tensor, status) -> torch.Tensor:
+        return table[b.ids[:rows].long()].float()
+
+    def residual_norm(self, x, pend: Optional[Pending], *, add=None, step=None, norm_w=None, eps: float, scale: float = 1.0,
+                      width: int = 0, one: bool = False, name: str = ""):
+        """x + the pending contribution (+ add + step), and the normed row padded to `width` columns (column W holds 1 when
+        `one`).  Returns (new residual, normed row or None)."""
+        unit = lambda t: t.float() * torch.rsqrt(t.float().pow(2).mean(-1, keepdim=True) + eps)
+        if pend is not None:
+            y = pend.plain.float() if pend.plain is not None else unit(pend.branch_a) * pend.weight_a + unit(pend.branch_b) * pend.weight_b
+            x = x + pend.coef * y
+        if add is not None:
+            x = x + add
+        if step is not None:
+            x = x + step
+        h = None
+        if norm_w is not None:
+            h = x.new_zeros(x.shape[0], width)
+            h[:, :x.shape[1]] = unit(x) * norm_w * scale
+            if one:
+                h[:, x.shape[1]] = 1.0
+        return x, h
+
+    # ------------------------------------------------------------------ attention without rotation over paged keys
+    def attn_append(self, proj, spec: AttnSpec, b: StepBatch, kv: KVLayer, st: ModelState):
+        """proj rows start with [q heads | k heads]: the keys go to their pages, the queries are returned."""
+        rows, pt, D = proj.shape[0], st.sc.page_tokens, spec.dim
+        nq = spec.heads * D
+        k = proj[:, nq:nq + spec.kv_heads * D].reshape(rows, spec.kv_heads, D)
+        for r in range(rows):
+            slot, p = int(b.row_slot[r]), int(b.row_pos[r])
+            if slot < 0:
+                continue
+            page = int(st.block_table[slot, p // pt])
+            if page < 0:
+                raise RuntimeError("KV append into an unmapped page")
+            kv.k[page, :, p % pt, :] = k[r]
+        return proj[:, :nq]
+
+    def attention(self, q, spec: AttnSpec, b: StepBatch, kv: KVLayer, st: ModelState, max_visible: int):
+        rows, D, H = q.shape[0], spec.dim, spec.heads
+        pt = st.sc.page_tokens
+        out = q.new_zeros(rows, H, D)
+        qh = q.reshape(rows, H, D)
+        for r in range(rows):
+            slot, p = int(b.row_slot[r]), int(b.row_pos[r])
+            if slot < 0:
+                continue
+            lo = p - p % spec.chunk if spec.chunk > 0 else 0
+            tok = torch.arange(lo, p + 1)
+            pages = st.block_table[slot, tok // pt].long()
+            K = kv.k[pages, :, tok % pt].float().repeat_interleave(H // spec.kv_heads, 1)
+            V = kv.v[pages, :, tok % pt].float().repeat_interleave(H // spec.kv_heads, 1)
+            s = torch.einsum("hd,thd->ht", qh[r].float(), K) * spec.scale
+            if spec.sink is not None:
+                pr = torch.softmax(torch.cat([s, spec.sink[:, None]], 1), -1)[:, :-1]
+            else:
+                pr = torch.softmax(s, -1)
+            out[r] = torch.einsum("ht,thd->hd", pr, V)
+        return out.reshape(rows, H * D)
+
+    # ------------------------------------------------------------------ gated linear attention
+    def gla(self, proj, g: GlaSpec, b: StepBatch, gs: GdnLayerState, st: ModelState):
+        H, dk, dv = g.heads, g.dk, g.dv
+        out = proj.new_zeros(proj.shape[0], H * dv)
+        p = proj.float()
+        z = p[:, g.a_off:g.a_off + g.rank] @ g.a2.float().T + g.a2_bias
+        alpha = torch.exp(F.logsigmoid(z) * g.inv_tau).reshape(-1, H, dk)
+        q = p[:, g.q_off:g.q_off + H * dk].reshape(-1, H, dk) * g.q_scale
+        k = p[:, g.k_off:g.k_off + H * dk].reshape(-1, H, dk)
+        v = p[:, g.v_off:g.v_off + H * dv].reshape(-1, H, dv)
+        gate = F.silu(p[:, g.g_off:g.g_off + H * dv])
+        for s in range(b.n_seqs):
+            row0, n, slot, _ = (int(t) for t in b.seq_desc[s])
+            S = gs.rec[slot]
+            for row in range(row0, row0 + n):
+                S = S * alpha[row][:, :, None] + k[row][:, :, None] * v[row][:, None, :]
+                o = torch.einsum("hkv,hk->hv", S, q[row])
+                o = o * torch.rsqrt(o.pow(2).sum(-1, keepdim=True) / g.dv_true + g.eps) * g.norm_w
+                out[row] = o.reshape(-1) * gate[row]
+            if n > 0:
+                gs.rec[slot] = S
+        return out

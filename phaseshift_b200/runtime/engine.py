@@ -20,9 +20,8 @@ import torch
 
 from ..utils.graphs import capture as capture_graph
 
-from ..models.qwen35.config import Qwen35Config
-from ..models.qwen35.model import Qwen35Runner, StepOutput
-from ..models.qwen35.weights import EngineWeights, TpGeometry
+from ..models.common import StepOutput
+from ..models.registry import family_of
 from .batch import SeqRows, StepBatch, resolve_row_bucket
 from .state import ModelState, StateConfig
 
@@ -83,19 +82,23 @@ class PageAllocator:
 
 
 class Engine:
-    def __init__(self, weights: EngineWeights, device, state_cfg: StateConfig, backend: str = "auto", tp=None,
+    def __init__(self, weights, device, state_cfg: StateConfig, backend: str = "auto", tp=None,
                  use_graphs: bool = True, calibrate: bool = True, arena_gib: float = 0.0):
-        """``calibrate``: fix the activation scales of the block-scaled tensor-core projections from one forward
+        """``weights``: the engine weights of any registered model family (models/registry.py); its configuration picks the
+        family's runner, cache layout and precision.
+        ``calibrate``: fix the activation scales of the block-scaled tensor-core projections from one forward
         (once per weight set; see calibrate_act_scales)."""
-        self.cfg: Qwen35Config = weights.cfg
+        self.cfg = weights.cfg
+        self.family = family_of(self.cfg)
         self.device = torch.device(device)
         if backend == "auto":
             backend = "cuda" if self.device.type == "cuda" else "ref"
         self.backend = backend
-        geo = TpGeometry.make(self.cfg, weights.tp_rank, weights.tp_size)
+        geo = self.cfg.geometry(weights.tp_rank, weights.tp_size)
         if backend == "cuda":
             from ..ops.cuda_ops import CudaOps
-            self.ops = CudaOps(self.cfg, self.device, max_seq_len=state_cfg.max_seq_len)
+            self.ops = CudaOps(self.cfg, self.device, max_seq_len=state_cfg.max_seq_len,
+                               act_dtype=getattr(weights, "act_dtype", torch.bfloat16))
         else:
             from ..ops.ref_ops import RefOps
             self.ops = RefOps(self.cfg, self.device)
@@ -107,7 +110,7 @@ class Engine:
             self.arenas = ArenaSet(int(arena_gib * (1 << 30)), self.device.index or 0)
         self.state = ModelState(self.cfg, state_cfg, self.device, self.ops.act_dtype, geo, arenas=self.arenas)
         self._arm_checked_limits()
-        self.runner = Qwen35Runner(weights, self.state, self.ops, tp)
+        self.runner = self.family.runner(weights, self.state, self.ops, tp)
         self.tp = tp
         if tp is not None and hasattr(self.ops, "status"):
             tp.status_word = self.ops.status      # the transport's kernels report bounded-wait failures here
@@ -210,7 +213,7 @@ class Engine:
         projection kernel quantise K-panels independently inside its prologue.  Every rank calibrates its own slice."""
         from ..quant.act_quant import calibrate_act_scale
         from ..models.qwen35.weights import P as _P
-        w = self.runner.w
+        w = self.runner.w            # (only the hybrid decoder has block-quantised projections)
         sites: Dict[str, object] = {_P + "lm_head.weight": w.lm_head}
         for li, L in enumerate(w.layers):
             lp = f"{_P}layers.{li}."

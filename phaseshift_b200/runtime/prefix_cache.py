@@ -58,12 +58,15 @@ class PrefixCache:
             if l.k_scale is not None:
                 sshp = (self.pool_pages,) + tuple(l.k_scale.shape[1:])
                 ks, vs = torch.ones(sshp, dtype=l.k_scale.dtype, device=dev), torch.ones(sshp, dtype=l.k_scale.dtype, device=dev)
-            self.kv_pool.append((torch.zeros(shp, dtype=l.k.dtype, device=dev), torch.zeros(shp, dtype=l.k.dtype, device=dev), ks, vs))
+            pk = torch.zeros(shp, dtype=l.k.dtype, device=dev)
+            pv = pk if l.v is l.k else torch.zeros(shp, dtype=l.k.dtype, device=dev)       # keys that double as the values: one pool
+            self.kv_pool.append((pk, pv, ks, vs))
         for g in st.gdn:
             if g is None:
                 continue
             self.gdn_pool.append((torch.zeros((max_entries,) + tuple(g.rec.shape[1:]), dtype=g.rec.dtype, device=dev),
-                                  torch.zeros((max_entries,) + tuple(g.conv.shape[1:]), dtype=g.conv.dtype, device=dev)))
+                                  None if g.conv is None else torch.zeros((max_entries,) + tuple(g.conv.shape[1:]), dtype=g.conv.dtype,
+                                                                           device=dev)))
         pin = dev.type == "cuda"
         self._h_idx = torch.zeros(2, max(1, st.max_blocks), dtype=torch.long, pin_memory=pin)
         self._d_idx = torch.zeros(2, max(1, st.max_blocks), dtype=torch.long, device=dev)
@@ -71,9 +74,9 @@ class PrefixCache:
     def pool_bytes(self) -> int:
         n = 0
         for k, v, ks, vs in self.kv_pool:
-            n += 2 * k.numel() * k.element_size() + (2 * ks.numel() * ks.element_size() if ks is not None else 0)
+            n += (1 if v is k else 2) * k.numel() * k.element_size() + (2 * ks.numel() * ks.element_size() if ks is not None else 0)
         for rec, conv in self.gdn_pool:
-            n += rec.numel() * rec.element_size() + conv.numel() * conv.element_size()
+            n += rec.numel() * rec.element_size() + (conv.numel() * conv.element_size() if conv is not None else 0)
         return n
 
     def _index_pair(self, a: Sequence[int], b: Sequence[int]):
@@ -122,7 +125,8 @@ class PrefixCache:
             pk, pv, pks, pvs = self.kv_pool[ki]
             ki += 1
             pk.index_copy_(0, dst, l.k.index_select(0, src))
-            pv.index_copy_(0, dst, l.v.index_select(0, src))
+            if pv is not pk:
+                pv.index_copy_(0, dst, l.v.index_select(0, src))
             if pks is not None:
                 pks.index_copy_(0, dst, l.k_scale.index_select(0, src))
                 pvs.index_copy_(0, dst, l.v_scale.index_select(0, src))
@@ -133,7 +137,8 @@ class PrefixCache:
             rec, conv = self.gdn_pool[gi]
             gi += 1
             rec[ss].copy_(g.rec[slot])
-            conv[ss].copy_(g.conv[slot])
+            if conv is not None:
+                conv[ss].copy_(g.conv[slot])
         self.snaps[entry] = _Snapshot(n, mine, ss, extra)
         self.stats["saved_tokens"] += n
         return True
@@ -151,7 +156,8 @@ class PrefixCache:
             pk, pv, pks, pvs = self.kv_pool[ki]
             ki += 1
             l.k.index_copy_(0, dst, pk.index_select(0, src))
-            l.v.index_copy_(0, dst, pv.index_select(0, src))
+            if pv is not pk:
+                l.v.index_copy_(0, dst, pv.index_select(0, src))
             if pks is not None:
                 l.k_scale.index_copy_(0, dst, pks.index_select(0, src))
                 l.v_scale.index_copy_(0, dst, pvs.index_select(0, src))
@@ -162,7 +168,8 @@ class PrefixCache:
             rec, conv = self.gdn_pool[gi]
             gi += 1
             g.rec[slot].copy_(rec[snap.state_slot])
-            g.conv[slot].copy_(conv[snap.state_slot])
+            if conv is not None:
+                g.conv[slot].copy_(conv[snap.state_slot])
         self.stats["restored_tokens"] += snap.tokens
         return snap.extra
 

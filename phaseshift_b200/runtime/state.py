@@ -1,4 +1,8 @@
-"""Device-resident sequence state: paged KV pools, GDN conv/recurrent pools, block tables.
+"""Device-resident sequence state: paged KV pools, conv/recurrent pools, block tables.
+
+What a model keeps per sequence is described by its configuration (``cfg.state_specs(geometry)``): one `RunSpec` per layer
+execution, naming the attention pages and / or the recurrent state that execution owns.  A layer may own both (attention and
+a recurrence side by side), and a layer that runs several times in one forward owns one set per pass.
 
 Layouts (chosen for Blackwell: every (page, kv-head) tile is one contiguous 8 KB / 4 KB block that a
 single bulk copy can fetch; the reference interleaves heads inside a token,
@@ -7,6 +11,7 @@ include/phaseshift/models/qwen35/state/paged_kv_pool.h:59-140):
 * K/V pool per attention layer: ``[num_pages, Hkv, page_tokens, D]`` in bf16 or E4M3 bytes, FP8 pools
   carry ``[num_pages, Hkv, page_tokens]`` f32 scales (one per token x head, like the reference's
   FP8_E4M3 KV mode, state/kv_cache_types.h:11-46).
+  A shared spec (values are the keys) has one pool: ``v`` is ``k``.
 * GDN conv history per GDN layer: ``[slots, Hv, ring, 2*Dk+Dv]`` bf16, position p in slot p % ring.
 * GDN recurrent state per GDN layer: ``[slots, Hv, Dk, Dv]`` f32 (reference: gdn_state_pool.h:16-105).
 * Block table: ``[slots, max_blocks]`` int32, -1 = unmapped.
@@ -22,9 +27,6 @@ from typing import List, Optional
 
 import torch
 
-from ..models.qwen35.config import Qwen35Config
-from ..models.qwen35.weights import TpGeometry
-
 KV_DTYPES = ("bf16", "fp8_e4m3", "nvfp4")
 # names accepted on the command line for the reference's block-coded caches (src/apps/compute/main.hip:47-81): its 4-bit
 # format is served by the NVFP4 pools, its 8-bit format by the FP8 pools (same E4M3 codes, one scale per row instead of
@@ -38,6 +40,30 @@ def kv_row_bytes(kv_dtype: str, head_dim: int) -> int:
     if kv_dtype == "nvfp4":
         return ((head_dim // 2 + head_dim // 16) + 15) & ~15          # codes, block scales, padded to 16 bytes
     return head_dim * (1 if kv_dtype == "fp8_e4m3" else 2)
+
+
+@dataclass(frozen=True)
+class KVSpec:
+    """Attention pages of one layer execution: KV heads, head size, and whether the keys double as the values."""
+    heads: int
+    dim: int
+    shared: bool = False
+
+
+@dataclass(frozen=True)
+class RecurrentSpec:
+    """Recurrent state of one layer execution: ``[slots, heads, dk, dv]`` f32, and the channels of its short-conv history
+    per head (0 = none)."""
+    heads: int
+    dk: int
+    dv: int
+    conv_channels: int = 0
+
+
+@dataclass(frozen=True)
+class RunSpec:
+    kv: Optional[KVSpec]
+    rec: Optional[RecurrentSpec]
 
 
 @dataclass
@@ -66,6 +92,7 @@ class KVLayer:
 
 
 class GdnLayerState:
+    """Recurrent state of one layer execution; ``conv`` is None for recurrences without a short convolution."""
     __slots__ = ("conv", "rec", "rec_alt")
 
     def __init__(self, conv, rec, rec_alt):
@@ -75,8 +102,7 @@ class GdnLayerState:
 class ModelState:
     """All per-sequence device state of one rank."""
 
-    def __init__(self, cfg: Qwen35Config, sc: StateConfig, device, act_dtype=torch.bfloat16,
-                 geo: Optional[TpGeometry] = None, arenas=None):
+    def __init__(self, cfg, sc: StateConfig, device, act_dtype=torch.bfloat16, geo=None, arenas=None):
         """``arenas`` (a core.arena.ArenaSet, CUDA only): the KV pages and the recurrent / conv state are carved from
         the named arenas "kv" and "state" (stable virtual addresses, physical memory committed for exactly what the
         configuration needs, all under the set's byte budget) instead of the framework allocator."""
@@ -85,62 +111,67 @@ class ModelState:
         if sc.conv_ring < 4:
             raise ValueError("conv_ring must be >= 4")
         self.cfg, self.sc, self.device = cfg, sc, device
-        geo = geo or TpGeometry.make(cfg, 0, 1)
+        geo = geo or cfg.geometry(0, 1)
         self.geo = geo
-        self.hkv = len(geo.kv_heads)
-        self.hv = len(geo.gdn_v_heads)
+        self.specs: List[RunSpec] = cfg.state_specs(geo)
         self.num_pages = sc.num_pages()
         self.max_blocks = sc.max_blocks()
-        D, pt = cfg.head_dim, sc.page_tokens
-        fp8 = sc.kv_dtype == "fp8_e4m3"
-        self.kv_fp8 = fp8
+        pt = sc.page_tokens
+        self.kv_fp8 = sc.kv_dtype == "fp8_e4m3"
         self.kv_fmt = KV_FMT[sc.kv_dtype]            # 0 bf16, 1 FP8-E4M3 + row scale, 2 NVFP4 rows + row scale
-        Drow = D                                     # last extent of the pools
+        kv_specs = [s.kv for s in self.specs if s.kv is not None]
+        rec_specs = [s.rec for s in self.specs if s.rec is not None]
+        # heads of the (uniform) recurrent layers, for callers that log or replay their updates
+        self.hv = rec_specs[0].heads if rec_specs else 0
         if act_dtype == torch.float32:
-            kvt = torch.float32          # CPU reference keeps full precision
-            fp8 = self.kv_fp8 = False
+            kvt = torch.float32          # 32-bit engines keep full precision
+            self.kv_fp8 = False
             self.kv_fmt = 0
         elif self.kv_fmt == 2:
-            if D % 32 or D > 256:
+            if any(s.dim % 32 or s.dim > 256 for s in kv_specs):
                 raise ValueError("NVFP4 key/value pages need a head size that is a multiple of 32, at most 256")
-            kvt, Drow = torch.uint8, kv_row_bytes("nvfp4", D)
+            kvt = torch.uint8
         else:
-            kvt = torch.uint8 if fp8 else torch.bfloat16
+            kvt = torch.uint8 if self.kv_fp8 else torch.bfloat16
+        if self.kv_fmt != 0 and any(s.shared for s in kv_specs):
+            raise ValueError("pages whose keys double as the values are stored in bf16 (or 32-bit) only")
         scaled = self.kv_fmt != 0                    # pools with an fp32 scale per (page, head, token)
         self.kv: List[Optional[KVLayer]] = []
         self.gdn: List[Optional[GdnLayerState]] = []
-        Dk, Dv = cfg.linear_key_head_dim, cfg.linear_value_head_dim
         self.arenas = arenas
         esz = lambda dt: torch.empty(0, dtype=dt).element_size()
-        n_attn = sum(1 for lt in cfg.layer_types if lt == 1)
-        n_gdn = len(cfg.layer_types) - n_attn
-        kv_need = n_attn * (2 * self.num_pages * self.hkv * pt * Drow * esz(kvt) + (2 * self.num_pages * self.hkv * pt * 4 if scaled else 0) + 1024)
-        st_need = n_gdn * (sc.max_slots * self.hv * (sc.conv_ring * (2 * Dk + Dv) * esz(act_dtype)
-                                                      + Dk * Dv * 4 * (2 if sc.spec_rows > 0 else 1)) + 1024)
-        kv_arena = arenas.get("kv", kv_need + (2 << 20)) if arenas is not None and n_attn else None
-        st_arena = arenas.get("state", st_need + (2 << 20)) if arenas is not None and n_gdn else None
+        row_elems = lambda s: kv_row_bytes("nvfp4", s.dim) if self.kv_fmt == 2 else s.dim       # last extent of the pools
+        kv_need = sum((1 if s.shared else 2) * self.num_pages * s.heads * pt * (row_elems(s) * esz(kvt) + (4 if scaled else 0)) + 1024
+                      for s in kv_specs)
+        st_need = sum(sc.max_slots * s.heads * (sc.conv_ring * s.conv_channels * esz(act_dtype)
+                                                + s.dk * s.dv * 4 * (2 if sc.spec_rows > 0 else 1)) + 1024 for s in rec_specs)
+        kv_arena = arenas.get("kv", kv_need + (2 << 20)) if arenas is not None and kv_specs else None
+        st_arena = arenas.get("state", st_need + (2 << 20)) if arenas is not None and rec_specs else None
 
         def pool(arena, shape, dtype, fill=0):
             if arena is None:
                 return torch.full(shape, fill, dtype=dtype, device=device) if fill else torch.zeros(shape, dtype=dtype, device=device)
             t = arena.alloc(shape, dtype)
             return t.fill_(fill) if fill else t.zero_()
-        for lt in cfg.layer_types:
-            if lt == 1:
-                k = pool(kv_arena, (self.num_pages, self.hkv, pt, Drow), kvt)
-                v = pool(kv_arena, (self.num_pages, self.hkv, pt, Drow), kvt)
+        for spec in self.specs:
+            kv = rec = None
+            if spec.kv is not None:
+                shape = (self.num_pages, spec.kv.heads, pt, row_elems(spec.kv))
+                k = pool(kv_arena, shape, kvt)
+                v = k if spec.kv.shared else pool(kv_arena, shape, kvt)
                 ks = vs = None
                 if scaled:
-                    ks = pool(kv_arena, (self.num_pages, self.hkv, pt), torch.float32, 1)
-                    vs = pool(kv_arena, (self.num_pages, self.hkv, pt), torch.float32, 1)
-                self.kv.append(KVLayer(k, v, ks, vs))
-                self.gdn.append(None)
-            else:
-                conv = pool(st_arena, (sc.max_slots, self.hv, sc.conv_ring, 2 * Dk + Dv), act_dtype)
-                rec = pool(st_arena, (sc.max_slots, self.hv, Dk, Dv), torch.float32)
-                alt = pool(st_arena, (sc.max_slots, self.hv, Dk, Dv), torch.float32) if sc.spec_rows > 0 else None
-                self.gdn.append(GdnLayerState(conv, rec, alt))
-                self.kv.append(None)
+                    ks = pool(kv_arena, shape[:3], torch.float32, 1)
+                    vs = pool(kv_arena, shape[:3], torch.float32, 1)
+                kv = KVLayer(k, v, ks, vs)
+            if spec.rec is not None:
+                r = spec.rec
+                conv = pool(st_arena, (sc.max_slots, r.heads, sc.conv_ring, r.conv_channels), act_dtype) if r.conv_channels else None
+                main = pool(st_arena, (sc.max_slots, r.heads, r.dk, r.dv), torch.float32)
+                alt = pool(st_arena, (sc.max_slots, r.heads, r.dk, r.dv), torch.float32) if sc.spec_rows > 0 else None
+                rec = GdnLayerState(conv, main, alt)
+            self.kv.append(kv)
+            self.gdn.append(rec)
         self.block_table = torch.full((sc.max_slots, self.max_blocks), -1, dtype=torch.int32, device=device)
         self.status = torch.zeros(1, dtype=torch.int32, device=device)
 
@@ -148,7 +179,7 @@ class ModelState:
         n = 0
         for l in self.kv:
             if l is not None:
-                n += 2 * l.k.numel() * l.k.element_size()
+                n += (1 if l.v is l.k else 2) * l.k.numel() * l.k.element_size()
                 if l.k_scale is not None:
                     n += 2 * l.k_scale.numel() * 4
         return n
@@ -164,4 +195,5 @@ class ModelState:
         for g in self.gdn:
             if g is not None:
                 g.rec[dst].copy_(g.rec[src])
-                g.conv[dst].copy_(g.conv[src])
+                if g.conv is not None:
+                    g.conv[dst].copy_(g.conv[src])
