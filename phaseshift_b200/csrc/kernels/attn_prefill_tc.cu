@@ -55,6 +55,8 @@ struct AttnTcArgs {
     // decode / verify variant (DEC): split-KV partials in the layout of the per-row kernel's merge pass
     int split_tokens; int max_splits; int dec_max_rows;
     float* part_acc; float* part_ml;
+    int chunk;                   // > 0: position i sees only its own block of `chunk` positions (counted from position 0)
+    const float* sink;           // [Hq] or null: exp(sink[h]) joins head h's denominator (prefill; the merge pass does it for DEC)
     long long* prof;             // optional cycle stamps of CTA (0, 0, 0): [32 tiles][16], softmax slots 0-7, issuer slots 8-12
 };
 
@@ -137,8 +139,9 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         r_begin = 0; nq = 8 * n_rows; kvh = blockIdx.y; h = kvh * G;
         pos_q0 = pos_start; kv_end = pos_start + n_rows;
         const int tps = a.split_tokens / kTcTok;                         // tiles per split
-        t_first = (int)blockIdx.x * tps;
-        const int t_end = min((kv_end + kTcTok - 1) / kTcTok, t_first + tps);
+        const int t_lo = a.chunk > 0 ? pos_q0 / a.chunk * a.chunk / kTcTok : 0;      // tile of the first token any row sees
+        const int t_end = min((kv_end + kTcTok - 1) / kTcTok, ((int)blockIdx.x + 1) * tps);
+        t_first = max((int)blockIdx.x * tps, t_lo);
         if (t_first >= t_end) return;
         T = t_end - t_first;
     } else {
@@ -149,8 +152,8 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         h = blockIdx.y; kvh = h / G;
         pos_q0 = pos_start + r_begin;
         kv_end = pos_q0 + nq;
-        t_first = 0;
-        T = (kv_end + kTcTok - 1) / kTcTok;
+        t_first = a.chunk > 0 ? pos_q0 / a.chunk * a.chunk / kTcTok : 0;
+        T = (kv_end + kTcTok - 1) / kTcTok - t_first;
     }
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const bool cta_stamp = a.prof != nullptr && threadIdx.x == 0 && blockIdx.x == 0 && blockIdx.y == 0 && blockIdx.z == 0;
@@ -283,7 +286,10 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         const uint32_t lane_base = (uint32_t)(quad * 32) << 16;
         const int rp = DEC ? pos_q0 + (row >> 3) : pos_q0 + row;     // position of this thread's query row
         const float sc = a.scale_log2;
+        const int lo = a.chunk > 0 ? rp / a.chunk * a.chunk : 0;     // first token this row sees
+        const int lo_max = a.chunk > 0 ? (kv_end - 1) / a.chunk * a.chunk : 0;       // ... and the largest of any row
         float m_ref = 0.f, l_run = 0.f;
+        bool fresh = true;                                            // this row has not seen a token yet: m_ref is a placeholder
         bool ok = true;
         // the epilogue reads this tile's gate values (one 512-byte run per row): ask for them now, so that they come from
         // L2 then
@@ -307,6 +313,14 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
             tc::tmem_ld_32x32(tmem + lane_base + b * kTcTok + (half ^ 1) * 32, so);
             tc::tmem_ld_wait();
             if (stamp) a.prof[t * 16 + 2] = clock64();
+            if (tt * kTcTok < lo_max) {                               // tokens before some row's block
+                const int to = tt * kTcTok + (half ^ 1) * 32;
+#pragma unroll
+                for (int j = 0; j < 32; ++j) {
+                    if (t0 + j < lo) sr[j] = 0xff800000u;
+                    if (to + j < lo) so[j] = 0xff800000u;
+                }
+            }
             if (tt * kTcTok + kTcTok - 1 > pos_q0) {                  // some row of the tile does not see every token
                 const int to = tt * kTcTok + (half ^ 1) * 32;
 #pragma unroll
@@ -321,7 +335,9 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
             float mx = fmaxf(fmaxf(mq[0], mq[1]), fmaxf(mq[2], mq[3])) * sc;     // scale > 0, so the maximum commutes with it
             if (stamp) a.prof[t * 16 + 3] = clock64();
             float alpha = 1.f;
-            if (t == 0) m_ref = mx == -INFINITY ? 0.f : mx;           // (a row that sees nothing here keeps a finite reference)
+            if (fresh) {                                              // (a row that sees nothing yet keeps a finite reference)
+                if (mx != -INFINITY) { m_ref = mx; fresh = false; }
+            }
             else if (mx > m_ref + 8.f) { alpha = ex2_approx(m_ref - mx); m_ref = mx; }
             const bool rescale = __any_sync(0xffffffffu, alpha != 1.f);
             float sq[4] = {0.f, 0.f, 0.f, 0.f};
@@ -413,7 +429,8 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         } else {
         if (ok) {
             tc::fence_after_sync();
-            const float l = l_run + s_l[half ^ 1][row];
+            float l = l_run + s_l[half ^ 1][row];
+            if (a.sink != nullptr) l += ex2_approx(fmaf(a.sink[h], 1.4426950408889634f, -m_ref));
             const float inv = l > 0.f ? 1.f / l : 0.f;
             __nv_bfloat16* stg = reinterpret_cast<__nv_bfloat16*>(smem) + row * kTcOutPitch;
 #pragma unroll 1
@@ -609,7 +626,7 @@ int launch_attn_prefill_tc(const void* q, int q_rows, const void* k_pool, const 
                            int kv_fp8, const void* block_table, int max_blocks, int num_pages, int page_tokens, const void* seqs,
                            int n_seqs, int max_seq_rows, int min_rows, int Hq, int Hkv, float sm_scale, const void* gate, int ld_gate,
                            int gate_head_stride, int gate_offset, void* deq_k, void* deq_v, int deq_pages, void* deq_bt, void* deq_seqs,
-                           void* out, void* status, cudaStream_t stream) {
+                           void* out, void* status, int chunk, const void* sink, cudaStream_t stream) {
     if (kv_fp8) {
         // widen the step's pages into the bf16 scratch pool, then attend over that
         if (deq_k == nullptr || deq_v == nullptr || deq_bt == nullptr || deq_seqs == nullptr || deq_pages <= 0) return (int)cudaErrorInvalidValue;
@@ -635,6 +652,7 @@ int launch_attn_prefill_tc(const void* q, int q_rows, const void* k_pool, const 
     a.gate = (const __nv_bfloat16*)gate; a.ld_gate = ld_gate; a.gate_head_stride = gate_head_stride; a.gate_offset = gate_offset;
     a.out = (__nv_bfloat16*)out; a.status = (uint32_t*)status; a.budget = g_ps_wait_budget_cycles; a.prof = g_attn_tc_prof;
     a.split_tokens = 0; a.max_splits = 0; a.dec_max_rows = 0; a.part_acc = nullptr; a.part_ml = nullptr;
+    a.chunk = chunk; a.sink = (const float*)sink;
     const size_t smem = (size_t)kTcSmem;
     static bool set = false;
     if (!set) {
@@ -654,12 +672,13 @@ int launch_attn_prefill_tc(const void* q, int q_rows, const void* k_pool, const 
 // the caller runs ps_paged_attention_merge afterwards.  `split_tokens` is a multiple of 64, `q` is [q_rows, Hq, D] bf16.
 // Reference: src/phaseshift/models/qwen35/kernels/optimized/attention/paged_decode.hip (split-KV decode); the grouped-query
 // packing onto one MMA tile has no counterpart there.
-PS_API int ps_attn_decode_tc(const void* q, int q_rows, const void* k_pool, const void* v_pool, const void* block_table,
+// `chunk` > 0: a row sees only its own block of `chunk` positions; pass the same value to the merge pass (and a sink only there).
+PS_API int ps_attn_decode_tc_ex(const void* q, int q_rows, const void* k_pool, const void* v_pool, const void* block_table,
                              int max_blocks, int page_tokens, int num_pages, const void* seqs, int n_seqs, int dec_max_rows,
                              int Hq, int Hkv, int D, float sm_scale, int split_tokens, int max_splits, int max_visible,
-                             void* part_acc, void* part_ml, void* status, cudaStream_t stream) {
+                             void* part_acc, void* part_ml, void* status, int chunk, cudaStream_t stream) {
     using namespace ps;
-    if (D != kTcD || (page_tokens != 16 && page_tokens != 32 && page_tokens != 64) || Hkv <= 0 || (Hq % Hkv) || Hq / Hkv > 8 ||
+    if (chunk < 0 || D != kTcD || (page_tokens != 16 && page_tokens != 32 && page_tokens != 64) || Hkv <= 0 || (Hq % Hkv) || Hq / Hkv > 8 ||
         dec_max_rows < 1 || dec_max_rows > 16 || split_tokens < kTcTok || (split_tokens % kTcTok) || n_seqs <= 0 ||
         (((uintptr_t)q | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)part_acc) % 16))
         return (int)cudaErrorInvalidValue;
@@ -678,7 +697,7 @@ PS_API int ps_attn_decode_tc(const void* q, int q_rows, const void* k_pool, cons
     a.gate = nullptr; a.ld_gate = 0; a.gate_head_stride = 0; a.gate_offset = 0; a.out = nullptr;
     a.status = (uint32_t*)status; a.budget = g_ps_wait_budget_cycles; a.prof = nullptr;
     a.split_tokens = split_tokens; a.max_splits = max_splits; a.dec_max_rows = dec_max_rows;
-    a.part_acc = (float*)part_acc; a.part_ml = (float*)part_ml;
+    a.part_acc = (float*)part_acc; a.part_ml = (float*)part_ml; a.chunk = chunk; a.sink = nullptr;
     const size_t smem = (size_t)kTcSmem;
     static bool set = false;
     if (!set) {
@@ -687,6 +706,15 @@ PS_API int ps_attn_decode_tc(const void* q, int q_rows, const void* k_pool, cons
     }
     attn_tc_kernel<true><<<dim3(n_splits, Hkv, n_seqs), kTcThreads, smem, stream>>>(mq, mk, mv, a);
     return PS_LAUNCH_CHECK();
+}
+
+PS_API int ps_attn_decode_tc(const void* q, int q_rows, const void* k_pool, const void* v_pool, const void* block_table,
+                             int max_blocks, int page_tokens, int num_pages, const void* seqs, int n_seqs, int dec_max_rows,
+                             int Hq, int Hkv, int D, float sm_scale, int split_tokens, int max_splits, int max_visible,
+                             void* part_acc, void* part_ml, void* status, cudaStream_t stream) {
+    return ps_attn_decode_tc_ex(q, q_rows, k_pool, v_pool, block_table, max_blocks, page_tokens, num_pages, seqs, n_seqs,
+                                dec_max_rows, Hq, Hkv, D, sm_scale, split_tokens, max_splits, max_visible, part_acc, part_ml,
+                                status, 0, stream);
 }
 
 // Timing aid: a device buffer of 32 x 16 int64 that CTA (0, 0, 0) of later launches fills with cycle stamps of its softmax

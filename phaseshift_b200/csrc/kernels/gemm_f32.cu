@@ -1,0 +1,73 @@
+// 32-bit projection of the float32 engines: out[M,N] = epilogue(A[M,K] . W[N,K]^T), fp32 multiply-adds on the CUDA cores
+// (no TF32).  64 x 64 tiles, 4 x 4 outputs per thread; the gated epilogues combine interleaved (gate, up) columns as the
+// bf16 kernels do.  A precision mode, not a fast path.
+#include "ps_common.cuh"
+
+namespace ps {
+
+constexpr int kFT = 64, kFK = 16;
+
+struct GemmF32Args {
+    const float* a; int lda; const float* w; int ldw;
+    int M, N, K, epilogue;             // 0 store, 2 SwiGLU, 3 ReGLU
+    float* out; int ldo;
+};
+
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const GemmF32Args g) {
+    __shared__ float sa[kFK][kFT + 4], sw[kFK][kFT + 4];
+    const int m0 = blockIdx.y * kFT, n0 = blockIdx.x * kFT, t = threadIdx.x, tx = t & 15, ty = t >> 4;
+    float acc[4][4] = {};
+    for (int k0 = 0; k0 < g.K; k0 += kFK) {
+        for (int i = t; i < kFT * kFK; i += 256) {
+            const int r = i / kFK, k = i % kFK;
+            const bool kin = k0 + k < g.K;
+            sa[k][r] = kin && m0 + r < g.M ? g.a[(size_t)(m0 + r) * g.lda + k0 + k] : 0.f;
+            sw[k][r] = kin && n0 + r < g.N ? g.w[(size_t)(n0 + r) * g.ldw + k0 + k] : 0.f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < kFK; ++k) {
+            const float4 av = *reinterpret_cast<const float4*>(&sa[k][ty * 4]), wv = *reinterpret_cast<const float4*>(&sw[k][tx * 4]);
+            const float ar[4] = {av.x, av.y, av.z, av.w}, wr[4] = {wv.x, wv.y, wv.z, wv.w};
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(ar[i], wr[j], acc[i][j]);
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int m = m0 + ty * 4 + i;
+        if (m >= g.M) continue;
+        if (g.epilogue >= 2) {
+#pragma unroll
+            for (int j = 0; j < 4; j += 2) {
+                const int n = n0 + tx * 4 + j;
+                if (n + 1 < g.N) {
+                    const float gate = acc[i][j];
+                    const float act = g.epilogue == 3 ? fmaxf(gate, 0.f) : gate / (1.f + expf(-gate));
+                    g.out[(size_t)m * g.ldo + (n >> 1)] = act * acc[i][j + 1];
+                }
+            }
+        } else {
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const int n = n0 + tx * 4 + j;
+                if (n < g.N) g.out[(size_t)m * g.ldo + n] = acc[i][j];
+            }
+        }
+    }
+}
+
+}  // namespace ps
+
+PS_API int ps_gemm_f32(const void* a, int lda, const void* w, int ldw, int M, int N, int K, int epilogue, void* out, int ldo,
+                       cudaStream_t stream) {
+    using namespace ps;
+    if (M <= 0 || N <= 0 || K <= 0 || (epilogue != 0 && epilogue != 2 && epilogue != 3) || (epilogue >= 2 && (N & 1)))
+        return (int)cudaErrorInvalidValue;
+    GemmF32Args g{(const float*)a, lda, (const float*)w, ldw, M, N, K, epilogue, (float*)out, ldo};
+    gemm_f32_kernel<<<dim3((N + kFT - 1) / kFT, (M + kFT - 1) / kFT), 256, 0, stream>>>(g);
+    return PS_LAUNCH_CHECK();
+}

@@ -349,7 +349,7 @@ PS_API int ps_linear_stream(int wfmt, const void* x, int M, int N, int K, int ld
     stream_init_once();
     if (M < 1 || M > 8 || (K % 32) != 0 || (ldx % 8) != 0 || ((uintptr_t)w_tiled % 16) != 0)
         return (int)cudaErrorInvalidValue;
-    if (epilogue == EPI_SWIGLU && (N & 1)) return (int)cudaErrorInvalidValue;
+    if ((epilogue == EPI_SWIGLU || epilogue == EPI_REGLU) && (N & 1)) return (int)cudaErrorInvalidValue;
     LinearSmallArgs a;
     a.x = (const __nv_bfloat16*)x; a.M = M; a.N = N; a.K = K; a.ldx = ldx;
     a.w = (const uint8_t*)w_tiled; a.w_gscale = w_gscale;
@@ -360,7 +360,7 @@ PS_API int ps_linear_stream(int wfmt, const void* x, int M, int N, int K, int ld
     a.amax_best = nullptr; a.amax_ctl = nullptr; a.amax_tokens = nullptr;
     if (tp_combine != nullptr) {
         a.tp = *reinterpret_cast<const TpCombine*>(tp_combine);
-        if (a.tp.size > kTpMaxRanks || M > a.tp.max_rows || ((N + 3) / 4 * 4) > a.tp.n_pad || epilogue == EPI_SWIGLU)
+        if (a.tp.size > kTpMaxRanks || M > a.tp.max_rows || ((N + 3) / 4 * 4) > a.tp.n_pad || epilogue == EPI_SWIGLU || epilogue == EPI_REGLU)
             return (int)cudaErrorInvalidValue;
     } else {
         a.tp.size = 0;

@@ -7,7 +7,10 @@
 //     batch, so a row's result is bit-identical whether it is decoded alone, verified among 16
 //     speculative rows or batched with other requests (the reference gets this by forcing S=16);
 //   * the merge pass also applies the sigmoid output gate, so o_proj reads its input directly.
-// One CTA = (split, kv head, row) and serves all G = Hq/Hkv query heads that share the K/V tile.
+// One CTA = (split, kv head, row) and serves up to eight of the G = Hq/Hkv query heads that share the K/V tile.
+//
+// Two options of the mask and the denominator: `chunk` > 0 confines a row at position i to the positions of its own block of
+// `chunk` (blocks counted from position 0), and `sink` adds exp(sink[h]) to head h's denominator in the merge pass.
 //
 // K/V pools: [num_pages, Hkv, page_tokens, D]; FP8 pools carry one f32 scale per (page, head, token).
 #include <stdio.h>
@@ -32,6 +35,7 @@ struct PagedAttnArgs {
     float* part_acc;   // [rows, Hq, max_splits, D]
     float* part_ml;    // [rows, Hq, max_splits, 2]  (running max, running sum)
     uint32_t* status;
+    int chunk;         // > 0: a row sees only its own block of `chunk` positions
 };
 
 struct TileRegs { uint4 k[4]; uint4 v[4]; float ks, vs; };
@@ -125,7 +129,8 @@ __device__ __forceinline__ void tile_store(const PagedAttnArgs& a, const TileReg
 
 __global__ void __launch_bounds__(kAttnThreads) paged_attn_split_kernel(const PagedAttnArgs a) {
     extern __shared__ __align__(16) unsigned char smem[];
-    const int D = a.D, G = a.Hq / a.Hkv, kpitch = D + 8;
+    const int D = a.D, heads_per_kv = a.Hq / a.Hkv, kpitch = D + 8;
+    const int groups = (heads_per_kv + kAttnMaxG - 1) / kAttnMaxG;         // CTAs that share a KV head
     __nv_bfloat16* ks = reinterpret_cast<__nv_bfloat16*>(smem);            // [32][D+8]
     __nv_bfloat16* vs = ks + kAttnTile * kpitch;                           // [32][D]
     float* qs = reinterpret_cast<float*>(vs + kAttnTile * D);              // [G][D]
@@ -136,17 +141,20 @@ __global__ void __launch_bounds__(kAttnThreads) paged_attn_split_kernel(const Pa
 
     cudaTriggerProgrammaticLaunchCompletion();
     cudaGridDependencySynchronize();
-    const int split = blockIdx.x, kvh = blockIdx.y, row = blockIdx.z;
+    const int split = blockIdx.x, kvh = blockIdx.y / groups, row = blockIdx.z;
+    const int g_first = (blockIdx.y % groups) * kAttnMaxG;
+    const int G = min(kAttnMaxG, heads_per_kv - g_first), h0 = kvh * heads_per_kv + g_first;
     const int visible = a.row_pos[row] + 1;
-    const int tok_begin = split * a.split_tokens;
-    if (tok_begin >= visible) return;
-    const int tok_end = min(visible, tok_begin + a.split_tokens);
+    const int lo = a.chunk > 0 && visible > 0 ? (visible - 1) / a.chunk * a.chunk : 0;
+    const int tok_end = min(visible, (split + 1) * a.split_tokens);
+    const int tok_begin = max(split * a.split_tokens, lo);
+    if (tok_begin >= tok_end) return;
     const int slot = a.row_slot[row];
     const int t = threadIdx.x, warp = t >> 5, lane = t & 31;
 
     for (int i = t; i < G * D; i += kAttnThreads) {
         const int g = i / D, d = i % D;
-        qs[i] = bf16_to_f32(a.q[((size_t)row * a.Hq + kvh * G + g) * D + d]) * a.sm_scale;
+        qs[i] = bf16_to_f32(a.q[((size_t)row * a.Hq + h0 + g) * D + d]) * a.sm_scale;
     }
     if (t < kAttnTile) { kscale[t] = 1.f; vscale[t] = 1.f; }
     float acc[kAttnMaxG];
@@ -220,10 +228,10 @@ __global__ void __launch_bounds__(kAttnThreads) paged_attn_split_kernel(const Pa
     if (t < D) {
 #pragma unroll
         for (int g = 0; g < kAttnMaxG; ++g)
-            if (g < G) a.part_acc[(((size_t)row * a.Hq + kvh * G + g) * a.max_splits + split) * D + t] = acc[g];
+            if (g < G) a.part_acc[(((size_t)row * a.Hq + h0 + g) * a.max_splits + split) * D + t] = acc[g];
     }
     if (warp < G && lane == 0) {
-        float* ml = a.part_ml + (((size_t)row * a.Hq + kvh * G + warp) * a.max_splits + split) * 2;
+        float* ml = a.part_ml + (((size_t)row * a.Hq + h0 + warp) * a.max_splits + split) * 2;
         ml[0] = m_run; ml[1] = l_run;
     }
 }
@@ -233,6 +241,7 @@ struct AttnMergeArgs {
     int rows, Hq, D, split_tokens, max_splits;
     const __nv_bfloat16* gate; int ld_gate; int gate_head_stride; int gate_offset;   // optional sigmoid gate
     __nv_bfloat16* out;   // [rows, Hq*D]
+    int chunk; const float* sink;   // as in the split pass; sink [Hq] or null
 };
 
 // grid = (Hq, rows), block = D threads.  The split weights exp(m_s - max m) are computed once, in
@@ -248,21 +257,24 @@ __global__ void paged_attn_merge_kernel(const AttnMergeArgs a) {
     const int visible = a.row_pos[row] + 1;
     if (visible < 0) return;                                            // position -2: a row another kernel of the step owns
     const int n = (visible + a.split_tokens - 1) / a.split_tokens;      // 0 for a padding row
+    const int s0 = a.chunk > 0 && visible > 0 ? (visible - 1) / a.chunk * a.chunk / a.split_tokens : 0;
+    const float sink = a.sink != nullptr ? a.sink[h] : -3.0e38f;
     const float* ml = a.part_ml + ((size_t)row * a.Hq + h) * a.max_splits * 2;
     const float* pa = a.part_acc + ((size_t)row * a.Hq + h) * a.max_splits * a.D;
-    float m = -3.0e38f;
-    for (int s = d; s < n; s += blockDim.x) m = fmaxf(m, ml[2 * s]);
+    float m = sink;
+    for (int s = s0 + d; s < n; s += blockDim.x) m = fmaxf(m, ml[2 * s]);
     m = block_max(m, s_red);
     float l = 0.f;
-    for (int s = d; s < n; s += blockDim.x) {
+    for (int s = s0 + d; s < n; s += blockDim.x) {
         const float w = __expf(ml[2 * s] - m);
         s_w[s] = w;
         l = fmaf(w, ml[2 * s + 1], l);
     }
     l = block_sum(l, s_red + 32);      // its barriers also publish s_w
+    if (a.sink != nullptr) l += __expf(sink - m);
     float o = 0.f;
 #pragma unroll 4
-    for (int s = 0; s < n; ++s) o = fmaf(s_w[s], pa[(size_t)s * a.D + d], o);
+    for (int s = s0; s < n; ++s) o = fmaf(s_w[s], pa[(size_t)s * a.D + d], o);
     float v = l > 0.f ? o / l : 0.f;
     if (a.gate != nullptr) {
         v = bf16_to_f32(f32_to_bf16(v));
@@ -274,15 +286,16 @@ __global__ void paged_attn_merge_kernel(const AttnMergeArgs a) {
 
 }  // namespace ps
 
-PS_API int ps_paged_attention(const void* q, const void* k_pool, const void* v_pool, const void* k_scale,
+// `chunk` (0 = plain causal) and `sink` ([Hq] f32 or null) select the options named at the top of the file.
+PS_API int ps_paged_attention_ex(const void* q, const void* k_pool, const void* v_pool, const void* k_scale,
                               const void* v_scale, const void* block_table, int max_blocks, int page_tokens,
                               int num_pages, const void* row_slot, const void* row_pos, int rows, int Hq, int Hkv,
                               int D, float sm_scale, int kv_fp8, int split_tokens, int max_splits, int max_visible,
                               void* part_acc, void* part_ml, const void* gate, int ld_gate, int gate_head_stride,
-                              int gate_offset, void* out, void* status, cudaStream_t stream) {
+                              int gate_offset, void* out, void* status, int chunk, const void* sink, cudaStream_t stream) {
     using namespace ps;
     const int G = Hkv > 0 ? Hq / Hkv : 0;
-    if (G < 1 || G > kAttnMaxG || D > kAttnMaxD || (D % 32) || (split_tokens % kAttnTile) || rows <= 0)
+    if (G < 1 || (Hq % Hkv) || chunk < 0 || D > kAttnMaxD || (D % 32) || (split_tokens % kAttnTile) || rows <= 0)
         return (int)cudaErrorInvalidValue;
     PagedAttnArgs a;
     a.q = (const __nv_bfloat16*)q; a.k_pool = k_pool; a.v_pool = v_pool; a.k_scale = (const float*)k_scale;
@@ -290,7 +303,7 @@ PS_API int ps_paged_attention(const void* q, const void* k_pool, const void* v_p
     a.page_tokens = page_tokens; a.num_pages = num_pages; a.row_slot = (const int*)row_slot;
     a.row_pos = (const int*)row_pos; a.rows = rows; a.Hq = Hq; a.Hkv = Hkv; a.D = D; a.sm_scale = sm_scale;
     a.kv_fp8 = kv_fp8; a.split_tokens = split_tokens; a.max_splits = max_splits;
-    a.part_acc = (float*)part_acc; a.part_ml = (float*)part_ml; a.status = (uint32_t*)status;
+    a.part_acc = (float*)part_acc; a.part_ml = (float*)part_ml; a.status = (uint32_t*)status; a.chunk = chunk;
     int n_splits = (max_visible + split_tokens - 1) / split_tokens;
     if (n_splits < 1) n_splits = 1;
     if (n_splits > max_splits || max_splits > kAttnMaxSplits) return (int)cudaErrorInvalidValue;
@@ -301,30 +314,48 @@ PS_API int ps_paged_attention(const void* q, const void* k_pool, const void* v_p
         cudaFuncSetAttribute(paged_attn_split_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024);
         attr_set = true;
     }
-    dim3 grid(n_splits, Hkv, rows);
+    dim3 grid(n_splits, Hkv * ((G + kAttnMaxG - 1) / kAttnMaxG), rows);
     int err = launch_pdl(paged_attn_split_kernel, grid, dim3(kAttnThreads), smem, stream, a);
     if (err) return err;
     AttnMergeArgs m;
     m.part_acc = a.part_acc; m.part_ml = a.part_ml; m.row_pos = a.row_pos; m.rows = rows; m.Hq = Hq; m.D = D;
     m.split_tokens = split_tokens; m.max_splits = max_splits; m.gate = (const __nv_bfloat16*)gate;
     m.ld_gate = ld_gate; m.gate_head_stride = gate_head_stride; m.gate_offset = gate_offset;
-    m.out = (__nv_bfloat16*)out;
+    m.out = (__nv_bfloat16*)out; m.chunk = chunk; m.sink = (const float*)sink;
     return launch_pdl(paged_attn_merge_kernel, dim3(Hq, rows), dim3(D), 0, stream, m);
+}
+
+PS_API int ps_paged_attention(const void* q, const void* k_pool, const void* v_pool, const void* k_scale,
+                              const void* v_scale, const void* block_table, int max_blocks, int page_tokens,
+                              int num_pages, const void* row_slot, const void* row_pos, int rows, int Hq, int Hkv,
+                              int D, float sm_scale, int kv_fp8, int split_tokens, int max_splits, int max_visible,
+                              void* part_acc, void* part_ml, const void* gate, int ld_gate, int gate_head_stride,
+                              int gate_offset, void* out, void* status, cudaStream_t stream) {
+    return ps_paged_attention_ex(q, k_pool, v_pool, k_scale, v_scale, block_table, max_blocks, page_tokens, num_pages, row_slot,
+                                 row_pos, rows, Hq, Hkv, D, sm_scale, kv_fp8, split_tokens, max_splits, max_visible, part_acc,
+                                 part_ml, gate, ld_gate, gate_head_stride, gate_offset, out, status, 0, nullptr, stream);
 }
 
 // The merge pass alone: for partials produced by another split-KV kernel (attn_prefill_tc.cu's decode variant) in the same
 // layout.  Same arguments as the tail of ps_paged_attention.
-PS_API int ps_paged_attention_merge(const void* part_acc, const void* part_ml, const void* row_pos, int rows, int Hq, int D,
-                                    int split_tokens, int max_splits, const void* gate, int ld_gate, int gate_head_stride,
-                                    int gate_offset, void* out, cudaStream_t stream) {
+PS_API int ps_paged_attention_merge_ex(const void* part_acc, const void* part_ml, const void* row_pos, int rows, int Hq, int D,
+                                       int split_tokens, int max_splits, const void* gate, int ld_gate, int gate_head_stride,
+                                       int gate_offset, void* out, int chunk, const void* sink, cudaStream_t stream) {
     using namespace ps;
     if (rows <= 0 || Hq <= 0 || D <= 0 || D > kAttnMaxD || max_splits > kAttnMaxSplits) return (int)cudaErrorInvalidValue;
     AttnMergeArgs m;
     m.part_acc = (const float*)part_acc; m.part_ml = (const float*)part_ml; m.row_pos = (const int*)row_pos; m.rows = rows; m.Hq = Hq; m.D = D;
     m.split_tokens = split_tokens; m.max_splits = max_splits; m.gate = (const __nv_bfloat16*)gate;
     m.ld_gate = ld_gate; m.gate_head_stride = gate_head_stride; m.gate_offset = gate_offset;
-    m.out = (__nv_bfloat16*)out;
+    m.out = (__nv_bfloat16*)out; m.chunk = chunk; m.sink = (const float*)sink;
     return launch_pdl(paged_attn_merge_kernel, dim3(Hq, rows), dim3(D), 0, stream, m);
+}
+
+PS_API int ps_paged_attention_merge(const void* part_acc, const void* part_ml, const void* row_pos, int rows, int Hq, int D,
+                                    int split_tokens, int max_splits, const void* gate, int ld_gate, int gate_head_stride,
+                                    int gate_offset, void* out, cudaStream_t stream) {
+    return ps_paged_attention_merge_ex(part_acc, part_ml, row_pos, rows, Hq, D, split_tokens, max_splits, gate, ld_gate,
+                                       gate_head_stride, gate_offset, out, 0, nullptr, stream);
 }
 
 // ------------------------------------------------------------------------------------------------

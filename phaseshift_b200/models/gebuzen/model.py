@@ -59,7 +59,7 @@ class GebuzenRunner:
             with ops.range("norm"):
                 x, h = ops.residual_norm(x, pend, add=add, step=step, norm_w=L.norm1, eps=eps, width=L.in_proj.K, one=True, name="h_mix")
             with ops.range("mixer.in_proj"):
-                proj = ops.linear(h, L.in_proj, name="mix_proj")
+                proj = ops.linear(h, L.in_proj, name=f"mix_proj{L.in_proj.N}")
             attn, gla = self.attn[run.layer], self.gla[run.layer]
             with ops.range("attn.append"):
                 q = ops.attn_append(proj, attn, b, st.kv[j], st)
@@ -76,7 +76,7 @@ class GebuzenRunner:
                 with ops.range("norm"):
                     x, h = ops.residual_norm(x, pend, norm_w=L.norm2, eps=eps, width=L.gate_up.K, name="h_mlp")
                 with ops.range("mlp.gate_up"):
-                    act = ops.linear(h, L.gate_up, name="mlp_act", reglu=True)
+                    act = ops.linear(h, L.gate_up, name=f"mlp_act{L.gate_up.N}", reglu=True)
                 with ops.range("mlp.down"):
                     pend = Pending(m, plain=ops.linear(act, L.down, name="mlp_out", out_f32=True))
             if j in tap_layers:

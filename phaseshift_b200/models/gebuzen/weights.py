@@ -175,6 +175,7 @@ def build_engine_weights(cfg: GebuzenConfig, get: Callable[[str], torch.Tensor],
         return lw
 
     W = cfg.hidden_size
+    nout = pad(W, 4)                     # output rows of projections onto the residual width (paired fp32 stores need even pitches)
     kin = pad(W, 32)                     # input width of projections without a bias
     kin_b = pad(W + 1, 32)               # ... and with one: column W multiplies the constant 1
     layers = []
@@ -199,13 +200,13 @@ def build_engine_weights(cfg: GebuzenConfig, get: Callable[[str], torch.Tensor],
         in_proj = lin(rows, rows.shape[0], kin_b)
         del rows
         a2 = _pad_cols(_pad_heads(t(m + "right.a2"), r.heads, r.dim, dk), rp).contiguous()
-        left_o = lin(_pad_heads(t(m + "left.o").T.contiguous(), l.heads, l.dim, D).T, W, l.heads * D)
-        right_o = lin(_pad_heads(t(m + "right.o").T.contiguous(), r.heads, r.vdim, dv).T, W, r.heads * dv)
+        left_o = lin(_pad_heads(t(m + "left.o").T.contiguous(), l.heads, l.dim, D).T, nout, l.heads * D)
+        right_o = lin(_pad_heads(t(m + "right.o").T.contiguous(), r.heads, r.vdim, dv).T, nout, r.heads * dv)
         gate_up = down = norm2 = None
         if L.ff is not None:
             fp = pad(L.ff, 32)
             gu = torch.stack([_pad_rows(t(p + "mlp.gate"), fp), _pad_rows(t(p + "mlp.up"), fp)], 1).reshape(2 * fp, W)
-            gate_up, down, norm2 = lin(gu, 2 * fp, kin), lin(t(p + "mlp.down"), W, fp), f32(p + "norm2")
+            gate_up, down, norm2 = lin(gu, 2 * fp, kin), lin(t(p + "mlp.down"), nout, fp), f32(p + "norm2")
             del gu
         layers.append(ParallelLayerW(l, r, f32(p + "norm1"), in_proj, rp, a2,
                                      _pad_heads(f32(m + "right.a2.b"), r.heads, r.dim, dk).contiguous(), f32(m + "left.sink"),

@@ -17,16 +17,16 @@ import numpy as np
 import torch
 
 from .trace import OpTrace
-from ..models.qwen35.config import Qwen35Config
 from ..models.qwen35.weights import AttnW, GdnW, LinearW
 from ..runtime.batch import StepBatch
 from ..runtime.state import GdnLayerState, KVLayer, ModelState
 from . import _lib
+from .specs import AttnSpec, GlaSpec, Pending
 from ._lib import c_float, c_int, c_ll, ptr
 
 WFMT = {"bf16": 0, "nvfp4": 1, "mxfp8": 2}
 PRO_NONE, PRO_RMSNORM, PRO_SIGMOID_GATE = 0, 1, 2
-EPI_STORE, EPI_RESIDUAL, EPI_SWIGLU = 0, 1, 2
+EPI_STORE, EPI_RESIDUAL, EPI_SWIGLU, EPI_REGLU = 0, 1, 2, 3
 SMALL_M_MAX = 8
 
 
@@ -36,17 +36,18 @@ class CudaOps(OpTrace):
     GDN_CHUNKED_MIN_ROWS = 16      # steps with more rows than this use the chunked GDN kernels
     ATTN_PREFILL_MIN_ROWS = 16     # ... and the tiled tensor-core attention kernel
 
-    def __init__(self, cfg: Qwen35Config, device, attn_split_tokens: int = 64, attn_max_splits: int = 0,
-                 max_seq_len: int = 4096):
+    def __init__(self, cfg, device, attn_split_tokens: int = 64, attn_max_splits: int = 0,
+                 max_seq_len: int = 4096, act_dtype: torch.dtype = torch.bfloat16):
+        """``act_dtype``: bfloat16, or float32 for model families whose ops exist in 32-bit (see `linear`)."""
         if device.type != "cuda":
             raise ValueError("CudaOps needs a CUDA device")
         _lib.lib()      # fail loudly when the native library is missing
-        self.cfg, self.device = cfg, device
+        self.cfg, self.device, self.act_dtype = cfg, device, act_dtype
         self.ws: Dict[Tuple[str, int], torch.Tensor] = {}
         self.checked = _lib.checked_build()          # PS_CHECKED=1: descriptor assertions in the kernels + workspace canaries
         self._guarded: Dict[Tuple[str, int], torch.Tensor] = {}
-        half = cfg.rotary_dim // 2
-        inv = cfg.rope_theta ** (-np.arange(half, dtype=np.float64) * 2.0 / cfg.rotary_dim)
+        half = getattr(cfg, "rotary_dim", 0) // 2                    # 0: the model rotates nothing
+        inv = getattr(cfg, "rope_theta", 1.0) ** (-np.arange(half, dtype=np.float64) * 2.0 / max(1, 2 * half))
         self.inv_freq = torch.from_numpy(inv).to(device)
         # the split length is fixed per engine for steps of up to 8 rows and for Exact mode, so attention results there do not
         # depend on the batch; larger Fast-mode batches lengthen it (see paged_attention).  PS_ATTN_SPLIT_TOKENS overrides the
@@ -124,7 +125,7 @@ class CudaOps(OpTrace):
         return out
 
     def linear(self, x: torch.Tensor, W: LinearW, *, name: str, norm_w: Optional[torch.Tensor] = None,
-               eps: float = 0.0, residual: Optional[torch.Tensor] = None, swiglu: bool = False,
+               eps: float = 0.0, residual: Optional[torch.Tensor] = None, swiglu: bool = False, reglu: bool = False,
                out_f32: bool = False, out: Optional[torch.Tensor] = None,
                xn_out: Optional[torch.Tensor] = None, tp_combine=None, ssq_in=None,
                ssq_out: Optional[torch.Tensor] = None, prefetch: Optional[LinearW] = None, tp_scatter=None) -> torch.Tensor:
@@ -136,10 +137,14 @@ class CudaOps(OpTrace):
         ``prefetch``: the projection that will run next on the same rows; the tensor-core kernel warms L2 with the first
         bytes of its weights while it drains.
         ``tp_scatter`` (a parallel.tp.TpScatterStruct; tensor-core path with streamed activations only): instead of
-        storing to ``out`` the kernel pushes each bf16 output row to the receive buffer of the rank that owns it."""
+        storing to ``out`` the kernel pushes each bf16 output row to the receive buffer of the rank that owns it.
+        ``swiglu`` / ``reglu``: the weight's rows interleave (gate, up) and the output is silu / relu (gate) * up.
+        32-bit weights run in fp32 on the CUDA cores (plain and gated epilogues only)."""
         M, K = x.shape
+        if W.fmt == "f32":
+            return self._linear_f32(x, W, name, swiglu, reglu, out, plain=norm_w is None and residual is None)
         assert K == W.K and x.dtype == torch.bfloat16 and x.stride(1) == 1, (x.shape, W.K, x.dtype)
-        n_out = W.N // 2 if swiglu else W.N
+        n_out = W.N // 2 if swiglu or reglu else W.N
         if out is None:
             out = self.buf(name, M, n_out, torch.float32 if out_f32 else torch.bfloat16)
         assert out.shape[0] == M and out.shape[1] == n_out and out.stride(1) == 1
@@ -147,6 +152,8 @@ class CudaOps(OpTrace):
             raise ValueError(f"K={W.K} must be a multiple of 32 for the streaming / bf16 tensor-core kernels")
         sel = self.select_linear(W, M)
         if sel == "tc":
+            if reglu:
+                raise ValueError("the block-scaled projections have no ReGLU epilogue")
             # block-quantised codes straight into the tensor cores (any number of rows)
             return self.linear_bs(x, W, name=name, norm_w=norm_w, eps=eps, residual=residual, swiglu=swiglu,
                                   out_f32=out_f32, out=out, xn_out=xn_out, tp_combine=tp_combine, ssq_in=ssq_in,
@@ -162,9 +169,9 @@ class CudaOps(OpTrace):
         self.sel_counts["gemm" if (sel == "gemm" or batched) else "stream"] += 1
         if sel == "gemm" or batched:
             return self.linear_large(x, W, name=name, norm_w=norm_w, eps=eps, residual=residual, swiglu=swiglu,
-                                     out_f32=out_f32, out=out)
+                                     reglu=reglu, out_f32=out_f32, out=out)
         pro = PRO_RMSNORM if norm_w is not None else PRO_NONE
-        epi = EPI_SWIGLU if swiglu else (EPI_RESIDUAL if residual is not None else EPI_STORE)
+        epi = EPI_SWIGLU if swiglu else EPI_REGLU if reglu else (EPI_RESIDUAL if residual is not None else EPI_STORE)
         if W.tiled is None:
             W.make_tiled()
         L = _lib.lib()
@@ -187,7 +194,7 @@ class CudaOps(OpTrace):
 
     def can_fuse_argmax(self, W: LinearW, M: int) -> bool:
         """True when ``linear_argmax`` can serve these rows: the streaming kernel would be chosen and holds them in one launch."""
-        if M < 1 or M > SMALL_M_MAX or self.exact_rows or W.K % 32 or self.select_linear(W, M) != "stream":
+        if M < 1 or M > SMALL_M_MAX or self.exact_rows or W.fmt == "f32" or W.K % 32 or self.select_linear(W, M) != "stream":
             return False
         if M >= 2 and W.rowmajor_bf16 is not None and self.use_tc_gemm:
             return False
@@ -211,7 +218,20 @@ class CudaOps(OpTrace):
         self.sel_counts["stream"] += 1
         return tokens.view(-1)[:M]
 
-    def linear_large(self, x: torch.Tensor, W: LinearW, *, name: str, norm_w, eps, residual, swiglu, out_f32, out):
+    def _linear_f32(self, x: torch.Tensor, W: LinearW, name: str, swiglu: bool, reglu: bool, out, plain: bool) -> torch.Tensor:
+        M, K = x.shape
+        if not plain or x.dtype != torch.float32 or K != W.K or x.stride(1) != 1:
+            raise ValueError("32-bit projections take fp32 rows and have no fused norm or residual")
+        if out is None:
+            out = self.buf(name, M, W.N // 2 if swiglu or reglu else W.N, torch.float32)
+        w = W.q.codes
+        _lib.call("ps_gemm_f32", ptr(x), c_int(x.stride(0)), ptr(w), c_int(w.stride(0)), c_int(M), c_int(W.N), c_int(K),
+                  c_int(EPI_SWIGLU if swiglu else EPI_REGLU if reglu else EPI_STORE), ptr(out), c_int(out.stride(0)))
+        self.launches += 1
+        self.sel_counts["f32"] = self.sel_counts.get("f32", 0) + 1
+        return out
+
+    def linear_large(self, x: torch.Tensor, W: LinearW, *, name: str, norm_w, eps, residual, swiglu, out_f32, out, reglu=False):
         """Prefill-sized projection: (RMSNorm kernel) -> weight expansion to a bf16 scratch matrix -> tcgen05
         GEMM with the residual / SwiGLU / dtype epilogue fused."""
         M, K = x.shape
@@ -229,7 +249,7 @@ class CudaOps(OpTrace):
             _lib.call("ps_dequant_tiled", c_int(WFMT[W.fmt]), ptr(W.tiled), c_int(W.N), c_int(kp),
                       c_float(W.tensor_scale), ptr(wd), c_int(kp))
             self.launches += 1
-        epi = EPI_SWIGLU if swiglu else (EPI_RESIDUAL if residual is not None else EPI_STORE)
+        epi = EPI_SWIGLU if swiglu else EPI_REGLU if reglu else (EPI_RESIDUAL if residual is not None else EPI_STORE)
         if W.rowmajor_bf16 is not None and M <= 64 and W.N % 2 == 0:
             # batched decode: swap-AB split-K weight-streaming GEMM (gemm_smallm.cu)
             L = _lib.lib()
@@ -393,12 +413,31 @@ class CudaOps(OpTrace):
 
     def paged_attention(self, q: torch.Tensor, qkv: torch.Tensor, hq: int, hkv: int, b: StepBatch, kv: KVLayer,
                         st: ModelState, max_visible: int) -> torch.Tensor:
-        cfg = self.cfg
-        rows, D = q.shape[0], cfg.head_dim
-        out = self.buf("attn_ctx", rows, hq * D)
+        """The hybrid decoder's attention: plain causal, sigmoid output gate interleaved with the queries in `qkv`."""
+        D = self.cfg.head_dim
+        return self.attention(q, AttnSpec(hq, hkv, D, D ** -0.5, gate=qkv, gate_head_stride=2 * D, gate_offset=D), b, kv, st, max_visible)
+
+    def attention(self, q: torch.Tensor, spec: AttnSpec, b: StepBatch, kv: KVLayer, st: ModelState, max_visible: int) -> torch.Tensor:
+        """Softmax attention of the step's rows over their paged keys and values (ops/specs.py: AttnSpec)."""
+        rows, D, hq, hkv = q.shape[0], spec.dim, spec.heads, spec.kv_heads
+        sm, chunk, sink = c_float(spec.scale), c_int(spec.chunk), ptr(spec.sink)
+        gate = (ptr(spec.gate), c_int(spec.gate.stride(0) if spec.gate is not None else 0), c_int(spec.gate_head_stride),
+                c_int(spec.gate_offset))
+        if st.kv_fmt != 0 and (spec.chunk > 0 or spec.sink is not None):
+            raise ValueError("block-local masks and sinks need bf16 or 32-bit pages")
+        geom = f"{hq}x{D}"                      # layers of one model may differ in head geometry: one set of buffers for each
+        out = self.buf("attn_ctx" + geom, rows, hq * D, self.act_dtype)
+        if self.act_dtype == torch.float32 or D % 32 or D > 256:
+            if spec.gate is not None:
+                raise ValueError("the per-row attention kernel has no output gate")
+            _lib.call("ps_attn_rows", ptr(q), ptr(kv.k), ptr(kv.v), c_int(1 if self.act_dtype == torch.float32 else 0),
+                      ptr(st.block_table), c_int(st.max_blocks), c_int(st.sc.page_tokens), c_int(st.num_pages), ptr(b.row_slot),
+                      ptr(b.row_pos), c_int(rows), c_int(hq), c_int(hkv), c_int(D), sm, chunk, sink, ptr(out), ptr(st.status))
+            self.launches += 1
+            return out
         # the tiled kernel pays off when some sequence brings a long run of rows (a prefill chunk); steps made of
         # many sequences with a row or two each (batched decode) keep the per-row split-KV kernel
-        tiled = (not self.exact_rows and not b.graph_static and D in (64, 128, 256)
+        tiled = (not self.exact_rows and not b.graph_static
                  and any(len(sq.token_ids) > self.ATTN_PREFILL_MIN_ROWS for sq in b.seqs))
         row_pos = b.row_pos
         if tiled:
@@ -423,11 +462,10 @@ class CudaOps(OpTrace):
                 src = (dk, dv, None, None, dbt, dk.shape[0], dsq, 0)
             elif st.kv_fp8 and D == 256 and pt in (16, 32, 64):
                 deq = self._attn_scratch(n_long_pages(), hkv, pt, D, b.max_seqs, st.max_blocks)
-            _lib.call("ps_attn_prefill", ptr(q), ptr(src[0]), ptr(src[1]), ptr(src[2]), ptr(src[3]),
+            _lib.call("ps_attn_prefill_ex", ptr(q), ptr(src[0]), ptr(src[1]), ptr(src[2]), ptr(src[3]),
                       ptr(src[4]), c_int(st.max_blocks), c_int(pt), c_int(src[5]),
                       ptr(src[6]), c_int(b.n_seqs), c_int(rows), c_int(q.shape[0]), c_int(min_rows), c_int(hq), c_int(hkv), c_int(D),
-                      c_float(D ** -0.5), c_int(src[7]), ptr(qkv), c_int(qkv.stride(0)), c_int(2 * D), c_int(D),
-                      ptr(deq[0]), ptr(deq[1]), c_int(deq[2]), ptr(deq[3]), ptr(deq[4]), ptr(out), ptr(st.status))
+                      sm, c_int(src[7]), *gate, ptr(deq[0]), ptr(deq[1]), c_int(deq[2]), ptr(deq[3]), ptr(deq[4]), ptr(out), ptr(st.status), chunk, sink)
             self.launches += 2 if deq[0] is not None else 1
             if not any_short:
                 return out
@@ -439,8 +477,8 @@ class CudaOps(OpTrace):
         if rows > SMALL_M_MAX and not self.exact_rows:
             want = max(1, (4 * 148) // (rows * hkv))
             split_tokens = max(split_tokens, -(-(-(-max_visible // want)) // 32) * 32)
-        pacc = self.buf("attn_part_acc", rows, hq * self.max_splits * D, torch.float32)
-        pml = self.buf("attn_part_ml", rows, hq * self.max_splits * 2, torch.float32)
+        pacc = self.buf("attn_part_acc" + geom, rows, hq * self.max_splits * D, torch.float32)
+        pml = self.buf("attn_part_ml" + geom, rows, hq * self.max_splits * 2, torch.float32)
         # Decode / verify rows on the tensor cores: bf16 pages, head dim 256, every sequence handled here has at most 16 rows
         # (the query heads that share a KV head are packed into one MMA tile).  A row's result does not depend on the other
         # rows of its tile (every tile row has its own scores, reference maximum and accumulator lane), so Exact mode -- whose
@@ -450,29 +488,28 @@ class CudaOps(OpTrace):
                 and (b.graph_static or row_pos is b.row_pos_short or all(len(sq.token_ids) <= 16 for sq in b.seqs))):
             st_tok = -(-split_tokens // 64) * 64
             n_seqs = b.max_seqs if b.graph_static else b.n_seqs
-            _lib.call("ps_attn_decode_tc", ptr(q), c_int(q.shape[0]), ptr(kv.k), ptr(kv.v), ptr(st.block_table),
+            _lib.call("ps_attn_decode_tc_ex", ptr(q), c_int(q.shape[0]), ptr(kv.k), ptr(kv.v), ptr(st.block_table),
                       c_int(st.max_blocks), c_int(st.sc.page_tokens), c_int(st.num_pages), ptr(b.seq_desc), c_int(n_seqs),
-                      c_int(16), c_int(hq), c_int(hkv), c_int(D), c_float(D ** -0.5), c_int(st_tok), c_int(self.max_splits),
-                      c_int(max_visible), ptr(pacc), ptr(pml), ptr(st.status))
-            _lib.call("ps_paged_attention_merge", ptr(pacc), ptr(pml), ptr(row_pos), c_int(rows), c_int(hq), c_int(D),
-                      c_int(st_tok), c_int(self.max_splits), ptr(qkv), c_int(qkv.stride(0)), c_int(2 * D), c_int(D), ptr(out))
+                      c_int(16), c_int(hq), c_int(hkv), c_int(D), sm, c_int(st_tok), c_int(self.max_splits),
+                      c_int(max_visible), ptr(pacc), ptr(pml), ptr(st.status), chunk)
+            _lib.call("ps_paged_attention_merge_ex", ptr(pacc), ptr(pml), ptr(row_pos), c_int(rows), c_int(hq), c_int(D),
+                      c_int(st_tok), c_int(self.max_splits), *gate, ptr(out), chunk, sink)
             self.launches += 2
             return out
         if st.kv_fmt == 2:
             _lib.call("ps_paged_attention_fp4", ptr(q), ptr(kv.k), ptr(kv.v), ptr(kv.k_scale), ptr(kv.v_scale),
                       ptr(st.block_table), c_int(st.max_blocks), c_int(st.sc.page_tokens), c_int(st.num_pages),
-                      ptr(b.row_slot), ptr(row_pos), c_int(rows), c_int(hq), c_int(hkv), c_int(D), c_float(D ** -0.5),
+                      ptr(b.row_slot), ptr(row_pos), c_int(rows), c_int(hq), c_int(hkv), c_int(D), sm,
                       c_int(split_tokens), c_int(self.max_splits), c_int(max_visible), ptr(pacc), ptr(pml), ptr(st.status))
             _lib.call("ps_paged_attention_merge", ptr(pacc), ptr(pml), ptr(row_pos), c_int(rows), c_int(hq), c_int(D),
-                      c_int(split_tokens), c_int(self.max_splits), ptr(qkv), c_int(qkv.stride(0)), c_int(2 * D), c_int(D), ptr(out))
+                      c_int(split_tokens), c_int(self.max_splits), *gate, ptr(out))
             self.launches += 2
             return out
-        _lib.call("ps_paged_attention", ptr(q), ptr(kv.k), ptr(kv.v), ptr(kv.k_scale), ptr(kv.v_scale),
+        _lib.call("ps_paged_attention_ex", ptr(q), ptr(kv.k), ptr(kv.v), ptr(kv.k_scale), ptr(kv.v_scale),
                   ptr(st.block_table), c_int(st.max_blocks), c_int(st.sc.page_tokens), c_int(st.num_pages),
                   ptr(b.row_slot), ptr(row_pos), c_int(rows), c_int(hq), c_int(hkv), c_int(D),
-                  c_float(D ** -0.5), c_int(1 if st.kv_fp8 else 0), c_int(split_tokens),
-                  c_int(self.max_splits), c_int(max_visible), ptr(pacc), ptr(pml), ptr(qkv), c_int(qkv.stride(0)),
-                  c_int(2 * D), c_int(D), ptr(out), ptr(st.status))
+                  sm, c_int(1 if st.kv_fp8 else 0), c_int(split_tokens), c_int(self.max_splits), c_int(max_visible),
+                  ptr(pacc), ptr(pml), *gate, ptr(out), ptr(st.status), chunk, sink)
         self.launches += 2
         return out
 
@@ -581,3 +618,79 @@ class CudaOps(OpTrace):
                   c_int(rows), c_int(H), ptr(out), c_int(out.stride(0)), c_int(1 if one_plus else 0))
         self.launches += 1
         return out
+
+    # ------------------------------------------------------------------ 32-bit residual stream
+    def embed_f32(self, b: StepBatch, rows: int, table: torch.Tensor, status) -> torch.Tensor:
+        out = self.buf("x_embed", rows, table.shape[1], torch.float32)
+        _lib.call("ps_embed_f32", ptr(b.ids), ptr(table), c_int(1 if table.dtype == torch.float32 else 0), c_int(rows),
+                  c_int(table.shape[0]), c_int(table.shape[1]), ptr(out), ptr(status))
+        self.launches += 1
+        return out
+
+    def residual_norm(self, x: torch.Tensor, pend: Optional[Pending], *, add=None, step=None, norm_w=None, eps: float,
+                      scale: float = 1.0, width: int = 0, one: bool = False, name: str = ""):
+        """Add what is pending to the fp32 residual `x` (and `add` rows, a `step` vector), then norm the row for the next
+        projection: `width` columns, zero-padded, column W = 1 when `one` (ops/specs.py: Pending).  One launch.
+        Returns (residual, normed rows or None); the residual lives in one buffer of its own, `x` itself is only overwritten
+        when it is that buffer."""
+        rows, W = x.shape
+        changed = pend is not None or add is not None or step is not None
+        xo = self.buf("x_res", rows, W, torch.float32) if changed else None
+        h = self.buf(name, rows, width, self.act_dtype) if norm_w is not None else None
+        if xo is None and h is None:
+            return x, None
+        a = b = wa = wb = y = None
+        if pend is not None:
+            a, b, wa, wb, y = pend.branch_a, pend.branch_b, pend.weight_a, pend.weight_b, pend.plain
+        ld = lambda t: c_int(t.stride(0) if t is not None else 0)
+        _lib.call("ps_residual_norm", ptr(x), ptr(xo), c_int(rows), c_int(W), ptr(a), ld(a), ptr(wa), ptr(b), ld(b), ptr(wb),
+                  ptr(y), ld(y), c_float(pend.coef if pend is not None else 0.0), ptr(add), ptr(step), ptr(norm_w), c_float(eps),
+                  c_float(scale), ptr(h), c_int(1 if self.act_dtype == torch.float32 else 0), c_int(width), c_int(1 if one else 0))
+        self.launches += 1
+        return (xo if changed else x), h
+
+    # ------------------------------------------------------------------ attention without rotation: query copy + key append
+    def attn_append(self, proj: torch.Tensor, spec: AttnSpec, b: StepBatch, kv: KVLayer, st: ModelState) -> torch.Tensor:
+        rows = proj.shape[0]
+        q = self.buf(f"attn_q{spec.heads}x{spec.dim}", rows, spec.heads * spec.dim, self.act_dtype)
+        _lib.call("ps_attn_append", ptr(proj), c_int(proj.stride(0)), c_int(proj.element_size()), c_int(rows), c_int(spec.heads),
+                  c_int(spec.kv_heads), c_int(spec.dim), ptr(b.row_slot), ptr(b.row_pos), ptr(q), ptr(kv.k), ptr(st.block_table),
+                  c_int(st.max_blocks), c_int(st.sc.page_tokens), c_int(st.num_pages), ptr(st.status))
+        self.launches += 1
+        return q
+
+    # ------------------------------------------------------------------ gated linear attention
+    def gla(self, proj: torch.Tensor, g: GlaSpec, b: StepBatch, gs: GdnLayerState, st: ModelState) -> torch.Tensor:
+        """Sequences with many rows in the step take the chunked kernels, the others the row-sequential one."""
+        rows, f32 = proj.shape[0], self.act_dtype == torch.float32
+        out = self.buf(f"gla_o{g.heads}x{g.dv}", rows, g.heads * g.dv, self.act_dtype)
+        n_seqs = b.max_seqs if b.graph_static else b.n_seqs
+        T = self.GDN_CHUNKED_MIN_ROWS
+        L = _lib.lib()
+        chunk_ok = not f32 and not b.graph_static and bool(L.ps_gla_chunked_ok(c_int(g.dk), c_int(g.dv), c_int(g.rank)))
+        seq_rows = [len(sq.token_ids) for sq in b.seqs] if chunk_ok else []
+        long = [n for n in seq_rows if n > T]
+
+        def call(chunked: int, limit: int, blocks: int, scratch) -> None:
+            _lib.call("ps_gla", c_int(chunked), ptr(proj), c_int(proj.stride(0)), c_int(1 if f32 else 0), c_int(g.heads), c_int(g.dk),
+                      c_int(g.dv), c_int(g.dv_true), c_int(g.q_off), c_int(g.k_off), c_int(g.v_off), c_int(g.g_off), c_int(g.a_off),
+                      c_int(g.rank), c_float(g.q_scale), c_float(g.inv_tau), c_float(g.eps), ptr(g.a2), ptr(g.a2_bias), ptr(g.norm_w),
+                      ptr(gs.rec), ptr(b.seq_desc), c_int(n_seqs), c_int(limit), ptr(out), c_int(blocks), *[ptr(t) for t in scratch])
+        if long:
+            C = int(L.ps_gla_block_rows())
+            blocks = sum(-(-n // C) for n in long)
+            call(1, T, blocks, self._gla_scratch(blocks, g.heads, C, g.dk, g.dv))
+            self.launches += 3
+        if not long or len(long) < len(seq_rows):
+            call(0, T if long else 0, 0, (None,) * 4)
+            self.launches += 1
+        return out
+
+    def _gla_scratch(self, blocks: int, H: int, C: int, dk: int, dv: int):
+        """fp32 scratch of the chunked linear attention (decayed queries, A v, block states, block decays); one allocation that
+        grows to the largest step seen."""
+        sizes = [blocks * H * C * dk, blocks * H * C * dv, blocks * H * dk * dv, blocks * H * dk]
+        t = getattr(self, "_gla_buf", None)
+        if t is None or t.numel() < sum(sizes):
+            t = self._gla_buf = torch.empty(sum(sizes), dtype=torch.float32, device=self.device)
+        return torch.split(t[:sum(sizes)], sizes)

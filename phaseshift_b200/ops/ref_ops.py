@@ -235,7 +235,9 @@ class RefOps(OpTrace):
         `one`).  Returns (new residual, normed row or None)."""
         unit = lambda t: t.float() * torch.rsqrt(t.float().pow(2).mean(-1, keepdim=True) + eps)
         if pend is not None:
-            y = pend.plain.float() if pend.plain is not None else unit(pend.branch_a) * pend.weight_a + unit(pend.branch_b) * pend.weight_b
+            W = x.shape[1]                       # projections may carry padding columns behind the width
+            y = pend.plain[:, :W].float() if pend.plain is not None else \
+                unit(pend.branch_a[:, :W]) * pend.weight_a + unit(pend.branch_b[:, :W]) * pend.weight_b
             x = x + pend.coef * y
         if add is not None:
             x = x + add
