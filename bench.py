@@ -55,6 +55,10 @@ def _parse():
     ap.add_argument("--serving-slots", type=int, default=32,
                     help="sequence slots of the serving block (fewer than the requests, so that later admissions can hit "
                          "the prefix cache the earlier ones filled)")
+    ap.add_argument("--compare", default="", choices=["", "gebuzen"],
+                    help="instead of the headline workload: prefill and decode of a model family beside the hybrid decoder at equal "
+                         "layer shapes (random bf16 weights, 1 GPU), and the mixers' kernels against their rooflines")
+    ap.add_argument("--compare-layers", type=int, default=16)
     ap.add_argument("--watchdog", type=int, default=1500,
                     help="seconds after which a hung run dumps every thread's stack to stderr and exits")
     a = ap.parse_args()
@@ -360,10 +364,28 @@ def serving_block(ew, cfg, dev, tp, world, args):
             "timing": "CUDA events around the whole run, max over ranks; TTFT on the host clock of rank 0"}
 
 
+def compare_arm(args):
+    import torch
+    from phaseshift_b200.apps import compare_bench
+    torch.cuda.set_device(0)
+    peaks = {"hbm_gbs": 6650.0, "bf16_tflops": 1590.0}
+    try:
+        peaks = json.load(open(os.path.join(os.path.dirname(os.path.abspath(__file__)), "MEASURED_PEAKS.json")))
+    except Exception:
+        pass
+    sampler = ClockSampler(0)
+    res = compare_bench.run(peaks, layers=args.compare_layers, warmup=max(3, args.warmup // 2), sampler=sampler)
+    print(json.dumps({"compare": args.compare, **res, "clocks": sampler.stop(), "dtype": "bf16",
+                      "data": "synthetic (random-init weights, uniform-random prompt ids)"}), flush=True)
+    return 0
+
+
 def main():
     args = _parse()
     if args.impl == "reference":
         return reference_arm(args)
+    if args.compare:
+        return compare_arm(args)
 
     import faulthandler
     if args.watchdog > 0:

@@ -1,0 +1,215 @@
+"""Throughput of a model family beside the hybrid decoder at equal size (`bench.py --compare gebuzen`): prefill and decode of a
+stack of layers of real-model shapes with random bf16 weights, and the mixers' kernels alone against their rooflines.
+
+Every kernel row gives its time, the algorithmic bytes and FLOPs of one launch group, and the fraction of the roofline
+max(bytes / measured copy bandwidth, FLOPs / measured bf16 throughput) it reaches.  Kernel timings flush L2 between samples.
+"""
+from __future__ import annotations
+
+import statistics
+from typing import Dict, List
+
+import torch
+
+from ..models import registry
+from ..runtime.batch import SeqRows, StepBatch
+from ..runtime.engine import Engine
+from ..runtime.state import StateConfig
+
+
+def size_pairs(layers: int) -> List[tuple]:
+    """(label, Gebuzen configuration, hybrid configuration) of equal width, head and feed-forward shapes and depth."""
+    from ..models.gebuzen.config import ChunkAttention, ParallelLayer, gebuzen_27b_config, gebuzen_4b_config
+    from ..models.qwen35.config import qwen35_27b_config, qwen35_4b_config
+
+    def cut(cfg):
+        cfg.layers = cfg.layers[:layers]
+        return cfg
+
+    small128 = cut(gebuzen_4b_config(name="gebuzen-4b-d128"))
+    small128.layers = [ParallelLayer(ChunkAttention(32, 8, 128, 128 ** -0.5, 4096), L.right, L.ff) for L in small128.layers]
+    return [("4b", cut(gebuzen_4b_config()), qwen35_4b_config(num_hidden_layers=layers)),
+            ("4b, attention heads of 128", small128, None),
+            ("27b", cut(gebuzen_27b_config()), qwen35_27b_config(num_hidden_layers=layers))]
+
+
+def _events(fn, n: int) -> float:
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    torch.cuda.synchronize()
+    e0.record()
+    for _ in range(n):
+        fn()
+    e1.record()
+    torch.cuda.synchronize()
+    return e0.elapsed_time(e1) / n
+
+
+class _Flushed:
+    """Median device time of `fn` over samples, a buffer larger than L2 written before each."""
+
+    def __init__(self, device):
+        self.buf = torch.empty(256 << 20, dtype=torch.uint8, device=device)
+
+    def __call__(self, fn, samples: int = 15) -> float:
+        for _ in range(3):
+            fn()
+        ts = []
+        for _ in range(samples):
+            self.buf.zero_()
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record(); fn(); e1.record()
+            torch.cuda.synchronize()
+            ts.append(e0.elapsed_time(e1))
+        return statistics.median(ts) * 1e3
+
+
+def model_times(eng: Engine, prompt_tokens: int, steps: int, warmup: int, batch: int) -> Dict[str, float]:
+    """Prefill of one prompt, its continuation by as many tokens, and graph-replayed decode steps of 1 and `batch` rows."""
+    g = torch.Generator().manual_seed(1)
+    ids = torch.randint(0, eng.cfg.vocab_size, (2 * prompt_tokens,), generator=g).tolist()
+    out: Dict[str, float] = {}
+    first, second = [], []
+    for i in range(warmup + 3):
+        s = eng.open_sequence()
+        for store, part in ((first, ids[:prompt_tokens]), (second, ids[prompt_tokens:])):
+            t = _events(lambda: eng.step([SeqRows(s.slot, s.position, part, (len(part) - 1,))], [s]), 1)
+            if i >= warmup:
+                store.append(t)
+        eng.close_sequence(s)
+    out["prefill_ms"], out["prefill_cont_ms"] = statistics.median(first), statistics.median(second)
+    for rows in (1, batch):
+        seqs = [eng.open_sequence() for _ in range(rows)]
+        for s in seqs:
+            eng.step([SeqRows(s.slot, 0, ids[:prompt_tokens], (prompt_tokens - 1,))], [s])
+        for _ in range(3):
+            eng.step([SeqRows(s.slot, s.position, [7], (0,)) for s in seqs], seqs)
+        from ..runtime.batch import resolve_row_bucket
+        key = [k for k in eng.graphs if not isinstance(k, tuple) and eng.graph_key_bucket(k) == resolve_row_bucket(rows)][0]
+        graph = eng.graphs[key]
+        for _ in range(warmup):
+            graph.replay()
+        out[f"decode{rows}_ms"] = _events(graph.replay, steps)
+        out[f"launches{rows}"] = eng.launches_per_graph[key]
+        for s in seqs:
+            eng.close_sequence(s)
+    return out
+
+
+def _batch(eng: Engine, seqs) -> tuple:
+    """A step batch over fresh sequences [(first position, rows)] with mapped pages; returns (batch, open sequences)."""
+    opened = []
+    for p, n in seqs:
+        s = eng.open_sequence()
+        eng._reserve(s, p + n)
+        opened.append(s)
+    b = StepBatch(sum(n for _, n in seqs), len(seqs), eng.device)
+    b.max_context = eng.sc.max_seq_len + 1
+    b.fill([SeqRows(s.slot, p, [0] * n) for s, (p, n) in zip(opened, seqs)])
+    b.upload()
+    return b, opened
+
+
+def kernel_times(eng: Engine, timer: _Flushed, peaks: dict, rows: int, context: int, batch: int) -> Dict[str, dict]:
+    """The mixers' kernels alone.  `rows` = prefill rows, `context` = tokens before them / before a decoded row."""
+    hbm, tc = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    ops, st, r = eng.ops, eng.state, eng.runner
+    gz = eng.cfg.family == "gebuzen"
+    res: Dict[str, dict] = {}
+
+    def add(name, fn, nbytes, flops):
+        us = timer(fn)
+        floor = max(nbytes / hbm, flops / tc) * 1e6
+        res[name] = {"us": round(us, 1), "gb": round(nbytes / 1e9, 4), "gflop": round(flops / 1e9, 2), "roofline_us": round(floor, 2),
+                     "roofline_frac": round(floor / us, 4)}
+
+    def rand(n, width, dtype=torch.bfloat16):
+        return torch.randn(n, width, device=eng.device, dtype=torch.float32).to(dtype)
+
+    shapes = [("prefill", [(0, rows)]), ("prefill after context", [(context, rows)]), ("decode 1", [(context, 1)]),
+              (f"decode {batch}", [(context, 1)] * batch)]
+    if gz:
+        L, attn, gla = eng.w0, r.attn[0], r.gla[0]
+        H, G, D, width = attn.heads, attn.kv_heads, attn.dim, L.in_proj.N
+        rh, dk, dv = gla.heads, gla.dk, gla.dv
+        kv_bytes_tok = G * D * 2
+    else:
+        cfg = eng.cfg
+        la, lg = cfg.layer_types.index(1), cfg.layer_types.index(0)
+        m, gm = r.w.layers[la].mixer, r.w.layers[lg].mixer
+        H, G, D, width = r.hq, r.hkv, cfg.head_dim, m.qkv_proj.N
+        rh, dk, dv = r.hv, cfg.linear_key_head_dim, cfg.linear_value_head_dim
+        kv_bytes_tok = 2 * G * D * 2
+    for name, seqs in shapes:
+        b, opened = _batch(eng, seqs)
+        n = b.n_rows
+        vis = [list(range(p, p + k)) for p, k in seqs]
+        chunk = attn.chunk if gz else 0
+        pairs = sum((q % chunk + 1) if chunk else q + 1 for v in vis for q in v)
+        kv_tok = sum((v[-1] + 1 - (v[0] // chunk * chunk if chunk else 0)) for v in vis)
+        qkv = rand(n, width)
+        if gz:
+            q = ops.attn_append(qkv, attn, b, st.kv[0], st)
+            fa = lambda: ops.attention(q, attn, b, st.kv[0], st, b.max_visible_launch)
+        else:
+            q = ops.attn_prep(qkv, m, H, G, b, st.kv[la], st)
+            fa = lambda: ops.paged_attention(q, qkv, H, G, b, st.kv[la], st, b.max_visible_launch)
+        io = n * H * D * 2 * (2 if gz else 3)                       # queries, outputs (and the hybrid's output gate)
+        add("attention, " + name, fa, io + kv_tok * kv_bytes_tok, 4.0 * pairs * H * D)
+        state = len(seqs) * rh * dk * dv * 4 * 2
+        if gz:
+            fg = lambda: ops.gla(qkv, gla, b, st.gdn[0], st)
+            io = n * rh * (2 * dk + 3 * dv) * 2
+            flops = n * rh * (4.0 * dk * dv + 64.0 * (dk + dv))     # state update and read, the block-local triangle
+        else:
+            proj = rand(n, gm.in_proj.N + gm.ba_proj.N)
+            fg = lambda: ops.gdn(proj, gm, r.hk, rh, b, st.gdn[lg], st)
+            io = n * (2 * r.hk * dk + 3 * rh * dv) * 2
+            flops = n * rh * (6.0 * dk * dv + 64.0 * (2 * dk + dv))
+        add("recurrence, " + name, fg, io + state, flops)
+        if name in ("prefill", "decode 1"):
+            W = eng.cfg.hidden_size
+            if gz:
+                from ..ops.specs import Pending
+                x, a, c = rand(n, W, torch.float32), rand(n, W, torch.float32), rand(n, W, torch.float32)
+                pend = Pending(0.5, a, L.left_out, c, L.right_out)
+                add("norm, " + name, lambda: ops.residual_norm(x, pend, norm_w=L.norm2, eps=1e-6, width=L.gate_up.K, name="bench_h"),
+                    n * W * (4 * 4 + 2), 0.0)
+            else:
+                x = rand(n, W)
+                add("norm, " + name, lambda: ops.rmsnorm(x, r.w.layers[0].input_norm, 1e-6, "bench_h"), n * W * 4, 0.0)
+            w = L.gate_up if gz else r.w.layers[0].gate_up
+            xg = rand(n, w.K)
+            kw = {"reglu": True} if gz else {"swiglu": True}
+            add("gate_up, " + name, lambda: ops.linear(xg, w, name="bench_act", **kw), w.N * w.k_padded * 2 + n * (w.K + w.N // 2) * 2,
+                2.0 * n * w.N * w.K)
+        for s in opened:
+            eng.close_sequence(s)
+    return res
+
+
+def run(peaks: dict, layers: int = 16, prompt_tokens: int = 2048, steps: int = 50, warmup: int = 3, batch: int = 32, sampler=None) -> dict:
+    dev = torch.device("cuda:0")
+    timer = _Flushed(dev)
+    out = {"layers": layers, "prompt_tokens": prompt_tokens, "batch": batch, "sizes": {}}
+    for label, gz, hy in size_pairs(layers):
+        row = out["sizes"][label] = {}
+        for name, cfg in (("gebuzen", gz), ("hybrid", hy)):
+            if cfg is None:
+                continue
+            with torch.no_grad():
+                ew = registry.random_weights(cfg, dev, "bf16")
+                eng = Engine(ew, dev, StateConfig(max_slots=batch, max_seq_len=2 * prompt_tokens + 64, page_tokens=16))
+                if name == "gebuzen":
+                    eng.w0 = ew.layers[0]
+                if sampler is not None:
+                    sampler.begin()
+                t = model_times(eng, prompt_tokens, steps, warmup, batch)
+                k = kernel_times(eng, timer, peaks, prompt_tokens, prompt_tokens, batch)
+            rd = ew.decode_read_bytes()
+            row[name] = {**{a: round(v, 4) for a, v in t.items()},
+                         "prefill_tok_s": round(prompt_tokens / t["prefill_ms"] * 1e3), "decode1_tok_s": round(1e3 / t["decode1_ms"], 1),
+                         f"decode{batch}_tok_s": round(batch * 1e3 / t[f"decode{batch}_ms"]), "weights_gb": round(rd / 1e9, 3),
+                         "decode1_hbm_frac": round(rd / (t["decode1_ms"] * 1e-3) / (peaks["hbm_gbs"] * 1e9), 4), "kernels": k}
+            del eng, ew
+            torch.cuda.empty_cache()
+    return out

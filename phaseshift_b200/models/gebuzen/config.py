@@ -179,9 +179,9 @@ class GebuzenConfig:
         return GebuzenConfig.from_dict(raw, [eos] if isinstance(eos, int) else list(eos or []))
 
 
-def _uniform(name: str, vocab: int, width: int, n_layers: int, left: ChunkAttention, right: GatedLinear, ff: int, loop=None,
+def _uniform(preset: str, vocab: int, width: int, n_layers: int, left: ChunkAttention, right: GatedLinear, ff: int, loop=None,
              **over) -> GebuzenConfig:
-    kw = dict(residual_mult=0.5, name=name)
+    kw = dict(residual_mult=0.5, name=preset)
     kw.update(over)
     return GebuzenConfig(vocab, width, [ParallelLayer(left, right, ff)] * n_layers, loop=loop, **kw)
 

@@ -16,9 +16,9 @@ def rms_norm(x, w, eps):
     return rms(x, eps) * w
 
 
-def chunk_mask(n, size):
+def chunk_mask(n, size, device="cpu"):
     """allowed[i, j]: j is not after i and lies in the same block of `size` positions, blocks counted from position 0."""
-    i = torch.arange(n)
+    i = torch.arange(n, device=device)
     return (i[None, :] <= i[:, None]) & (i[None, :] // size == i[:, None] // size)
 
 
@@ -36,7 +36,7 @@ def chunk_attention_heads(q, k, scale, size, sink):
     G = k.shape[1]
     kk = k[:, [h // (H // G) for h in range(H)]]
     s = torch.einsum("ihd,jhd->hij", q, kk) * scale
-    p = softmax_with_sink(s, chunk_mask(n, size), sink)
+    p = softmax_with_sink(s, chunk_mask(n, size, q.device), sink)
     return torch.einsum("hij,jhd->ihd", p, kk)
 
 
