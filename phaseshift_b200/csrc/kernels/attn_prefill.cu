@@ -436,12 +436,12 @@ static int launch_prefill(const AttnPrefillArgs& a, int max_q_tiles, int n_seqs,
     return PS_LAUNCH_CHECK();
 }
 
-// attn_prefill_tc.cu: the tcgen05 kernel for head dim 256 and pages of 16 / 32 / 64 tokens (FP8 pools through a bf16 scratch pool)
+// attn_prefill_tc.cu: the tcgen05 kernel for head dims 64 / 128 / 192 / 256 and pages of 16 / 32 / 64 tokens (FP8 pools through a bf16 scratch pool)
 bool attn_prefill_tc_supported(int D, int page_tokens, int kv_fp8, const void* q, const void* k_pool, const void* v_pool,
                                const void* gate, int ld_gate, int gate_head_stride, int gate_offset, const void* deq_k);
 int launch_attn_prefill_tc(const void* q, int q_rows, const void* k_pool, const void* v_pool, const void* k_scale, const void* v_scale,
                            int kv_fp8, const void* block_table, int max_blocks, int num_pages, int page_tokens, const void* seqs,
-                           int n_seqs, int max_seq_rows, int min_rows, int Hq, int Hkv, float sm_scale, const void* gate, int ld_gate,
+                           int n_seqs, int max_seq_rows, int min_rows, int Hq, int Hkv, int D, float sm_scale, const void* gate, int ld_gate,
                            int gate_head_stride, int gate_offset, void* deq_k, void* deq_v, int deq_pages, void* deq_bt, void* deq_seqs,
                            void* out, void* status, int chunk, const void* sink, cudaStream_t stream);
 
@@ -463,7 +463,7 @@ PS_API int ps_attn_prefill_ex(const void* q, const void* k_pool, const void* v_p
     if (n_seqs <= 0 || max_seq_rows <= 0 || Hkv <= 0 || (Hq % Hkv) || q_rows < max_seq_rows) return (int)cudaErrorInvalidValue;
     if (attn_prefill_tc_supported(D, page_tokens, kv_fp8, q, k_pool, v_pool, gate, ld_gate, gate_head_stride, gate_offset, deq_k))
         return launch_attn_prefill_tc(q, q_rows, k_pool, v_pool, k_scale, v_scale, kv_fp8, block_table, max_blocks, num_pages, page_tokens,
-                                      seqs, n_seqs, max_seq_rows, min_rows, Hq, Hkv, sm_scale, gate, ld_gate, gate_head_stride, gate_offset,
+                                      seqs, n_seqs, max_seq_rows, min_rows, Hq, Hkv, D, sm_scale, gate, ld_gate, gate_head_stride, gate_offset,
                                       deq_k, deq_v, deq_pages, deq_bt, deq_seqs, out, status, chunk, sink, stream);
     AttnPrefillArgs a;
     a.chunk = chunk; a.sink = (const float*)sink;

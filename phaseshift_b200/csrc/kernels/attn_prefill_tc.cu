@@ -1,5 +1,7 @@
-// Causal paged attention for prefill-sized steps on the fifth-generation tensor cores (head dim 256, bf16 pools,
-// pages of 16, 32 or 64 tokens): one CTA = 128 consecutive query rows of one sequence and one query head.
+// Causal paged attention for prefill-sized steps on the fifth-generation tensor cores (head dims 64, 128, 192 and 256, bf16
+// pools, pages of 16, 32 or 64 tokens): one CTA = 128 consecutive query rows of one sequence and one query head.  Optionally
+// confined to blocks of positions (`chunk`), with a sink per head in the denominator, and with keys that are the values.
+// Described for head dim 256; other sizes have fewer 64-column groups:
 //
 //   warp 8   TMA producer for Q (once) and the K tiles: a 64-token tile is four pages, each fetched as four
 //            64-column boxes (128-byte swizzle) straight from the paged pool through a tensor map over
@@ -19,6 +21,9 @@
 //            result is the exact softmax).  The epilogue normalises, applies the sigmoid output gate and writes
 //            bf16 through shared memory with coalesced 16-byte stores.
 //
+// Keys that are the values (SHARED, one pool): every tile is fetched once into one of four stages, read by S(t) as the K-major
+// operand and by P V(t) as the MN-major one, and freed by the latter; warp 9 has nothing to do.
+//
 // Every wait is bounded; a timeout raises the CTA's abort flag, every role unwinds, outstanding copies get a
 // bounded chance to land, tensor memory is freed and PS_DEV_WAIT_TIMEOUT is recorded.  Token rows of the last
 // tile that lie beyond the sequence's end are zeroed in shared memory before the P V product (their
@@ -34,14 +39,19 @@
 
 namespace ps {
 
-constexpr int kTcRows = 128, kTcTok = 64, kTcD = 256;
+constexpr int kTcRows = 128, kTcTok = 64;
 constexpr int kTcThreads = 416;                      // warps 0-7 softmax, 8 Q / K producer, 9 V producer, 10-11 S issuers, 12 P V issuer
-constexpr int kTcQBytes = kTcRows * kTcD * 2;         // 64 KB: four 64-column boxes of 128 rows
-constexpr int kTcKvStage = kTcTok * kTcD * 2;         // 32 KB: four 64-column boxes of 64 tokens
 constexpr int kTcPBuf = kTcRows * kTcTok * 2;         // 16 KB: 128 rows x 64 tokens
-constexpr int kTcSmem = kTcQBytes + 4 * kTcKvStage + 2 * kTcPBuf;
-constexpr int kTcOutPitch = kTcD + 8;                 // staging pitch of the epilogue (elements)
-constexpr uint32_t kTcTmemCols = 512;                 // S0 | S1 (64 each) | O (256)
+template <int D> struct TcShape {
+    static_assert(D % 64 == 0 && D >= 64 && D <= 256, "head dims of 64-column groups");
+    static constexpr int kGroups = D / 64;                        // 64-column boxes per row
+    static constexpr int kQBytes = kTcRows * D * 2;               // D = 256: 64 KB, four 64-column boxes of 128 rows
+    static constexpr int kKvStage = kTcTok * D * 2;               // D = 256: 32 KB, four 64-column boxes of 64 tokens
+    static constexpr int kSmem = kQBytes + 4 * kKvStage + 2 * kTcPBuf;
+    static constexpr int kOutPitch = D + 8;                       // staging pitch of the epilogue (elements)
+    static constexpr uint32_t kTmemCols = D <= 128 ? 256 : 512;   // S0 | S1 (64 each) | O (D)
+    static_assert(kTcRows * kOutPitch * 2 <= kSmem, "the output staging lies inside the tile buffers");
+};
 
 struct AttnTcArgs {
     const int* block_table; int max_blocks; int num_pages; int page_tokens;     // page_tokens: 16, 32 or 64
@@ -109,12 +119,17 @@ __device__ __forceinline__ float sigmoid_fast(float x) {
 // and one KV head: tile row 8 r + g is query head g of that KV head for the sequence's row r (grouped-query packing: the G <= 8
 // heads that share the KV head ride in one MMA tile, so K and V are read once for all of them), over the tokens of its
 // split; it leaves unnormalised partial outputs and (maximum, sum) pairs for the merge pass of paged_attention.cu.
-template <bool DEC>
+template <int D, bool DEC, bool SHARED>
 __global__ void __launch_bounds__(kTcThreads, 1)
 attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                const __grid_constant__ CUtensorMap map_v, const AttnTcArgs a) {
     extern __shared__ __align__(1024) unsigned char smem_raw[];
-    // Q, two K and two V stages, two P buffers: 224 KB, which with the static part below is the whole 227 KB of the SM;
+    using Shape = TcShape<D>;
+    constexpr int kTcD = D, kTcQBytes = Shape::kQBytes, kTcKvStage = Shape::kKvStage, kTcOutPitch = Shape::kOutPitch, kNB = Shape::kGroups;
+    constexpr uint32_t kTcTmemCols = Shape::kTmemCols;
+    constexpr int kStageMask = SHARED ? 3 : 1;       // stages of one operand (a shared tile's four stages cover both operands' space)
+    constexpr int kStageLog = SHARED ? 2 : 1;
+    // Q, two K and two V stages, two P buffers: 224 KB at D = 256, which with the static part below is the whole 227 KB of the SM;
     // the swizzled tiles need the 1024-byte alignment that the declaration asks for (checked, not assumed)
     unsigned char* smem = smem_raw;
     if ((tc::smem_u32(smem) & 1023u) != 0) {
@@ -125,7 +140,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
     unsigned char* sK = sQ + kTcQBytes;
     unsigned char* sV = sK + 2 * kTcKvStage;
     unsigned char* sP = sV + 2 * kTcKvStage;
-    __shared__ __align__(8) uint64_t q_full, k_full[2], v_full[2], s_full[2], p_full[2], pv_done[2];
+    __shared__ __align__(8) uint64_t q_full, k_full[4], v_full[2], s_full[2], p_full[2], pv_done[2], kv_free[4];
     __shared__ float s_l[2][kTcRows];            // row sums of the two column halves, exchanged once at the end
     __shared__ uint32_t tmem_base_slot;
     __shared__ int s_abort, s_bad, k_issued, k_consumed, v_issued, v_consumed, q_issued, q_consumed;
@@ -165,6 +180,10 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
             tc::mbar_init(&k_full[s], 1); tc::mbar_init(&v_full[s], 1); tc::mbar_init(&s_full[s], 1);
             tc::mbar_init(&p_full[s], 8); tc::mbar_init(&pv_done[s], 1);
         }
+        if constexpr (SHARED) {
+            tc::mbar_init(&k_full[2], 1); tc::mbar_init(&k_full[3], 1);
+            for (int s = 0; s < 4; ++s) tc::mbar_init(&kv_free[s], 1);
+        }
         tc::fence_barrier_init();
         s_abort = 0; s_bad = 0; k_issued = k_consumed = v_issued = v_consumed = q_issued = q_consumed = 0;
         tc::tma_prefetch_desc(&map_q); tc::tma_prefetch_desc(&map_k); tc::tma_prefetch_desc(&map_v);
@@ -179,7 +198,9 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
     const uint32_t tmem = tmem_base_slot;
     const uint32_t tmem_o = tmem + 128;
 
-    if (warp == 8 || warp == 9) {
+    if (SHARED && warp == 9) {
+        // the values arrive with the keys
+    } else if (warp == 8 || warp == 9) {
         // ------------------------------------------------ TMA producers: warp 8 = Q and K, warp 9 = V.  One lane per box (a
         // tile is up to 16 boxes: pages x four 64-column groups): issuing them from one thread one after the other costs
         // more than a thousand cycles, and the stage's consumer is waiting for them.
@@ -188,36 +209,40 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
             if constexpr (DEC) {
                 // one 8-row box per (row of the sequence, 64-column group): the G heads of this KV head are consecutive rows
                 // of the [rows * Hq, D] view of q; tile rows 8 r + g with g >= G hold other heads' values and are never used
-                if (lane == 0) tc::mbar_expect_tx(&q_full, (uint32_t)n_rows * 4u * 1024u);
+                if (lane == 0) tc::mbar_expect_tx(&q_full, (uint32_t)n_rows * (uint32_t)kNB * 1024u);
                 __syncwarp();
-                for (int i = lane; i < 4 * n_rows; i += 32) {
-                    const int r = i >> 2, c4 = i & 3;
+                for (int i = lane; i < kNB * n_rows; i += 32) {
+                    const int r = i / kNB, c4 = i % kNB;
                     tc::tma_load_2d(sQ + c4 * (kTcRows * 128) + (8 * r) * 128, &map_q, c4 * 64, (row_start + r) * a.Hq + h, &q_full);
                 }
             } else {
                 if (lane == 0) tc::mbar_expect_tx(&q_full, kTcQBytes);
                 __syncwarp();
-                if (lane < 4) tc::tma_load_2d(sQ + lane * (kTcRows * 128), &map_q, h * kTcD + lane * 64, row_start + r_begin, &q_full);
+                if (lane < kNB) tc::tma_load_2d(sQ + lane * (kTcRows * 128), &map_q, h * kTcD + lane * 64, row_start + r_begin, &q_full);
             }
             if (lane == 0) q_issued = 1;
         }
         const int* bt = a.block_table + (size_t)slot * a.max_blocks;
         const int pt = a.page_tokens, ppt = kTcTok / pt;            // a page is one box of pt token rows per 64-column group
-        const int pg = lane >> 2, cb = lane & 3;
+        const int pg = lane / kNB, cb = lane % kNB;
         const bool active = pg < ppt;
         unsigned char* stage0 = isK ? sK : sV;
         uint64_t* full = isK ? k_full : v_full;
         uint64_t* freed = isK ? s_full : pv_done;                   // a K stage is free once S(t) has read it, a V stage after P V(t)
         const CUtensorMap* map = isK ? &map_k : &map_v;
         for (int t = 0; t < T; ++t) {
-            const int b = t & 1;
+            const int b = t & kStageMask;
             int page = 0;
             const int blk = (t_first + t) * ppt + pg;
             if (active && blk * pt < kv_end) {
                 page = bt[blk];
                 if (page < 0 || page >= a.num_pages) { s_bad = 1; page = 0; }
             }
-            if (t >= 2 && !__all_sync(0xffffffffu, tc::mbar_wait_abortable(&freed[b], (uint32_t)((t - 2) >> 1) & 1u, a.budget, &s_abort))) break;
+            if constexpr (SHARED) {
+                if (t >= 4 && !__all_sync(0xffffffffu, tc::mbar_wait_abortable(&kv_free[b], (uint32_t)((t - 4) >> 2) & 1u, a.budget, &s_abort))) break;
+            } else {
+                if (t >= 2 && !__all_sync(0xffffffffu, tc::mbar_wait_abortable(&freed[b], (uint32_t)((t - 2) >> 1) & 1u, a.budget, &s_abort))) break;
+            }
             if (lane == 0) tc::mbar_expect_tx(&full[b], kTcKvStage);
             __syncwarp();
             if (active)
@@ -231,7 +256,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         if (lane == 0) {
             constexpr uint32_t idesc_s = tc::idesc_bf16_f32(kTcRows, kTcTok);
             const int b = warp - 10;
-            const uint32_t q_addr = tc::smem_u32(sQ), k_addr = tc::smem_u32(sK) + b * kTcKvStage;
+            const uint32_t q_addr = tc::smem_u32(sQ), k_addr0 = tc::smem_u32(sK);
             bool ok = tc::mbar_wait_abortable(&q_full, 0, a.budget, &s_abort);
             if (ok) q_consumed = 1;
             for (int t = b; t < T && ok; t += 2) {
@@ -240,7 +265,9 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
                 if (stamp) a.prof[t * 16 + 8] = clock64();
                 // the score buffer is free once the softmax warps have read S(t - 2), which they signal with P(t - 2)
                 if (t >= 2 && !tc::mbar_wait_abortable(&p_full[b], ph ^ 1u, a.budget, &s_abort)) { ok = false; break; }
-                if (!tc::mbar_wait_abortable(&k_full[b], ph, a.budget, &s_abort)) { ok = false; break; }
+                const int ks_ = t & kStageMask;                                          // the tile's stage
+                const uint32_t k_addr = k_addr0 + ks_ * kTcKvStage;
+                if (!tc::mbar_wait_abortable(&k_full[ks_], (uint32_t)(t >> kStageLog) & 1u, a.budget, &s_abort)) { ok = false; break; }
                 if (stamp) a.prof[t * 16 + 9] = clock64();
                 atomicMax(&k_consumed, t + 1);
                 tc::fence_after_sync();
@@ -258,22 +285,24 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         // ------------------------------------------------ output issuer: O += P(t) V(t)
         if (lane == 0) {
             constexpr uint32_t idesc_o = tc::idesc_bf16_f32_bmn(kTcRows, kTcD);
-            const uint32_t v_addr = tc::smem_u32(sV), p_addr = tc::smem_u32(sP);
+            const uint32_t v_addr0 = tc::smem_u32(SHARED ? sK : sV), p_addr = tc::smem_u32(sP);
             for (int t = 0; t < T; ++t) {
                 const int b = t & 1;
                 const uint32_t ph = (uint32_t)(t >> 1) & 1u;
                 const bool stamp = a.prof != nullptr && blockIdx.x == 0 && blockIdx.y == 0 && blockIdx.z == 0 && t < 32;
                 if (!tc::mbar_wait_abortable(&p_full[b], ph, a.budget, &s_abort)) break;
                 if (stamp) a.prof[t * 16 + 11] = clock64();
-                if (!tc::mbar_wait_abortable(&v_full[b], ph, a.budget, &s_abort)) break;
+                const uint32_t v_addr = v_addr0 + (t & kStageMask) * kTcKvStage;
+                if (!tc::mbar_wait_abortable(SHARED ? &k_full[t & 3] : &v_full[b], SHARED ? (uint32_t)(t >> 2) & 1u : ph, a.budget, &s_abort)) break;
                 v_consumed = t + 1;
                 tc::fence_after_sync();
 #pragma unroll
                 for (int kk = 0; kk < kTcTok / 16; ++kk) {
                     const uint64_t adesc = tc::smem_desc_sw128(p_addr + b * kTcPBuf + kk * 32);
-                    const uint64_t bdesc = tc::smem_desc_sw128_mn(v_addr + b * kTcKvStage + kk * (16 * 128), kTcTok * 128, 1024);
+                    const uint64_t bdesc = tc::smem_desc_sw128_mn(v_addr + kk * (16 * 128), kTcTok * 128, 1024);
                     tc::mma_bf16_ss(tmem_o, adesc, bdesc, idesc_o, (t > 0 || kk > 0) ? 1u : 0u);
                 }
+                if constexpr (SHARED) tc::mma_commit(&kv_free[t & 3]);
                 tc::mma_commit(&pv_done[b]);
                 if (stamp) a.prof[t * 16 + 12] = clock64();
             }
@@ -362,12 +391,14 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
             if (t == T - 1 && kv_end < (tt + 1) * kTcTok) {
                 // token rows of the last V tile beyond the sequence's end: zero them (whole 128-byte rows, so the swizzle
                 // does not matter)
-                ok = __all_sync(0xffffffffu, tc::mbar_wait_abortable(&v_full[b], ph, a.budget, &s_abort));
+                // (a shared tile has been read by S(t) already: the scores are here)
+                ok = __all_sync(0xffffffffu, tc::mbar_wait_abortable(SHARED ? &k_full[t & 3] : &v_full[b], SHARED ? (uint32_t)(t >> 2) & 1u : ph,
+                                                                     a.budget, &s_abort));
                 if (!ok) break;
                 const int jz = kv_end - tt * kTcTok;
-                unsigned char* vs = sV + b * kTcKvStage;
-                for (int i = (int)threadIdx.x; i < (kTcTok - jz) * 32; i += 2 * kTcRows) {
-                    const int r = jz + (i >> 5), cb = (i & 31) >> 3, c = i & 7;
+                unsigned char* vs = (SHARED ? sK : sV) + (t & kStageMask) * kTcKvStage;
+                for (int i = (int)threadIdx.x; i < (kTcTok - jz) * kNB * 8; i += 2 * kTcRows) {
+                    const int r = jz + i / (kNB * 8), cb = i % (kNB * 8) >> 3, c = i & 7;
                     *reinterpret_cast<uint4*>(vs + cb * (kTcTok * 128) + r * 128 + c * 16) = make_uint4(0, 0, 0, 0);
                 }
             }
@@ -462,14 +493,14 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
                     const int i = i0 + u * 2 * kTcRows;
                     g[u] = make_uint4(0, 0, 0, 0);
                     if (a.gate != nullptr && i < n_items)
-                        g[u] = __ldg(reinterpret_cast<const uint4*>(a.gate + (size_t)(row_start + r_begin + (i >> 5)) * a.ld_gate +
-                                                                    (size_t)h * a.gate_head_stride + a.gate_offset + (i & 31) * 8));
+                        g[u] = __ldg(reinterpret_cast<const uint4*>(a.gate + (size_t)(row_start + r_begin + i / (kTcD / 8)) * a.ld_gate +
+                                                                    (size_t)h * a.gate_head_stride + a.gate_offset + i % (kTcD / 8) * 8));
                 }
 #pragma unroll
                 for (int u = 0; u < 4; ++u) {
                     const int i = i0 + u * 2 * kTcRows;
                     if (i >= n_items) break;
-                    const int r = i >> 5, c = i & 31;
+                    const int r = i / (kTcD / 8), c = i % (kTcD / 8);
                     uint4 v = *reinterpret_cast<const uint4*>(stg0 + r * kTcOutPitch + c * 8);
                     if (a.gate != nullptr) {
                         const uint32_t vw[4] = {v.x, v.y, v.z, v.w}, gw[4] = {g[u].x, g[u].y, g[u].z, g[u].w};
@@ -497,7 +528,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
             // copies still in flight get a bounded chance to land before the shared memory goes back to the next CTA
             const long long bd = a.budget < 4000000ll ? a.budget : 4000000ll;
             if (q_issued > q_consumed) tc::mbar_wait(&q_full, 0, bd);
-            for (int c = k_consumed; c < k_issued; ++c) tc::mbar_wait(&k_full[c & 1], (uint32_t)(c >> 1) & 1u, bd);
+            for (int c = k_consumed; c < k_issued; ++c) tc::mbar_wait(&k_full[c & kStageMask], (uint32_t)(c >> kStageLog) & 1u, bd);
             for (int c = v_consumed; c < v_issued; ++c) tc::mbar_wait(&v_full[c & 1], (uint32_t)(c >> 1) & 1u, bd);
         }
     }
@@ -513,6 +544,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
 // (values times their per-token scale), with its own block table (scratch page = running index) and sequence descriptors
 // (slot = sequence index), and the tensor-core kernel runs on that.  The copy moves 3 bytes per cached element; the
 // attention it feeds is an order of magnitude faster than the mma.sync kernel on FP8 pages.
+constexpr int kDeqD = 256;     // the only head size whose FP8 pools come this way
 struct AttnDeqArgs {
     const uint8_t* k_pool; const uint8_t* v_pool; const float* k_scale; const float* v_scale;
     const int* block_table; int max_blocks; int num_pages; int page_tokens; int Hkv;
@@ -549,8 +581,8 @@ __global__ void __launch_bounds__(256) attn_kv_dequant_kernel(const AttnDeqArgs 
     if (!ok && threadIdx.x == 0) set_status(a.status, PS_DEV_BAD_INDEX);
     const size_t src = ((size_t)(ok ? page : 0) * a.Hkv + kvh) * pt;          // token rows of the source page
     const size_t dst = ((size_t)p * a.Hkv + kvh) * pt;
-    for (int i = threadIdx.x; i < pt * (kTcD / 16); i += blockDim.x) {
-        const int tok = i / (kTcD / 16), c = i % (kTcD / 16);
+    for (int i = threadIdx.x; i < pt * (kDeqD / 16); i += blockDim.x) {
+        const int tok = i / (kDeqD / 16), c = i % (kDeqD / 16);
         const bool live = ok && blk * pt + tok < kv_end;
 #pragma unroll
         for (int which = 0; which < 2; ++which) {
@@ -559,7 +591,7 @@ __global__ void __launch_bounds__(256) attn_kv_dequant_kernel(const AttnDeqArgs 
             __nv_bfloat16* out = which ? a.v_out : a.k_out;
             uint32_t o[8] = {0, 0, 0, 0, 0, 0, 0, 0};
             if (live) {
-                const uint4 v = __ldg(reinterpret_cast<const uint4*>(pool + (src + tok) * kTcD) + c);
+                const uint4 v = __ldg(reinterpret_cast<const uint4*>(pool + (src + tok) * kDeqD) + c);
                 const float sc = sp[src + tok];
                 const uint32_t w[4] = {v.x, v.y, v.z, v.w};
 #pragma unroll
@@ -569,7 +601,7 @@ __global__ void __launch_bounds__(256) attn_kv_dequant_kernel(const AttnDeqArgs 
                     o[j] = f32x2_to_bf16x2_bits(lo, hi);
                 }
             }
-            uint4* d = reinterpret_cast<uint4*>(out + (dst + tok) * kTcD + c * 16);
+            uint4* d = reinterpret_cast<uint4*>(out + (dst + tok) * kDeqD + c * 16);
             d[0] = make_uint4(o[0], o[1], o[2], o[3]);
             d[1] = make_uint4(o[4], o[5], o[6], o[7]);
         }
@@ -616,15 +648,38 @@ bool attn_prefill_tc_supported(int D, int page_tokens, int kv_fp8, const void* q
         const char* e = getenv("PS_ATTN_PREFILL");                 // "legacy": always the mma.sync kernel
         enabled = (e != nullptr && e[0] == 'l') ? 0 : 1;
     }
-    if (!enabled || D != kTcD || (page_tokens != 16 && page_tokens != 32 && page_tokens != 64) || (kv_fp8 && deq_k == nullptr)) return false;
+    if (!enabled || D % 64 || D < 64 || D > 256 || (page_tokens != 16 && page_tokens != 32 && page_tokens != 64) || (kv_fp8 && (deq_k == nullptr || D != kDeqD))) return false;
     if (((uintptr_t)q | (uintptr_t)k_pool | (uintptr_t)v_pool) % 16) return false;
     if (gate != nullptr && (((uintptr_t)gate % 16) || (ld_gate % 8) || (gate_head_stride % 8) || (gate_offset % 8))) return false;
     return true;
 }
 
+template <int D, bool DEC, bool SHARED>
+static int launch_attn_tc(dim3 grid, const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const AttnTcArgs& a, cudaStream_t stream) {
+    constexpr size_t smem = TcShape<D>::kSmem;
+    static bool set = false;
+    if (!set) {
+        cudaFuncSetAttribute(attn_tc_kernel<D, DEC, SHARED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        set = true;
+    }
+    attn_tc_kernel<D, DEC, SHARED><<<grid, kTcThreads, smem, stream>>>(mq, mk, mv, a);
+    return PS_LAUNCH_CHECK();
+}
+template <bool DEC>
+static int launch_attn_tc_any(int D, bool shared, dim3 grid, const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv,
+                              const AttnTcArgs& a, cudaStream_t stream) {
+    switch (D) {
+        case 64: return shared ? launch_attn_tc<64, DEC, true>(grid, mq, mk, mv, a, stream) : launch_attn_tc<64, DEC, false>(grid, mq, mk, mv, a, stream);
+        case 128: return shared ? launch_attn_tc<128, DEC, true>(grid, mq, mk, mv, a, stream) : launch_attn_tc<128, DEC, false>(grid, mq, mk, mv, a, stream);
+        case 192: return shared ? launch_attn_tc<192, DEC, true>(grid, mq, mk, mv, a, stream) : launch_attn_tc<192, DEC, false>(grid, mq, mk, mv, a, stream);
+        case 256: return shared ? launch_attn_tc<256, DEC, true>(grid, mq, mk, mv, a, stream) : launch_attn_tc<256, DEC, false>(grid, mq, mk, mv, a, stream);
+        default: return (int)cudaErrorInvalidValue;
+    }
+}
+
 int launch_attn_prefill_tc(const void* q, int q_rows, const void* k_pool, const void* v_pool, const void* k_scale, const void* v_scale,
                            int kv_fp8, const void* block_table, int max_blocks, int num_pages, int page_tokens, const void* seqs,
-                           int n_seqs, int max_seq_rows, int min_rows, int Hq, int Hkv, float sm_scale, const void* gate, int ld_gate,
+                           int n_seqs, int max_seq_rows, int min_rows, int Hq, int Hkv, int D, float sm_scale, const void* gate, int ld_gate,
                            int gate_head_stride, int gate_offset, void* deq_k, void* deq_v, int deq_pages, void* deq_bt, void* deq_seqs,
                            void* out, void* status, int chunk, const void* sink, cudaStream_t stream) {
     if (kv_fp8) {
@@ -641,11 +696,11 @@ int launch_attn_prefill_tc(const void* q, int q_rows, const void* k_pool, const 
         k_pool = deq_k; v_pool = deq_v; block_table = deq_bt; seqs = deq_seqs; num_pages = deq_pages;
     }
     CUtensorMap mq, mk, mv;
-    int err = attn_map_2d(&mq, q, (uint64_t)q_rows, (uint64_t)Hq * kTcD, (uint64_t)Hq * kTcD, kTcRows);
+    int err = attn_map_2d(&mq, q, (uint64_t)q_rows, (uint64_t)Hq * D, (uint64_t)Hq * D, kTcRows);
     if (err) return err;
     const uint64_t pool_rows = (uint64_t)num_pages * Hkv * page_tokens;
-    if ((err = attn_map_2d(&mk, k_pool, pool_rows, kTcD, kTcD, (uint32_t)page_tokens))) return err;
-    if ((err = attn_map_2d(&mv, v_pool, pool_rows, kTcD, kTcD, (uint32_t)page_tokens))) return err;
+    if ((err = attn_map_2d(&mk, k_pool, pool_rows, D, D, (uint32_t)page_tokens))) return err;
+    if ((err = attn_map_2d(&mv, v_pool, pool_rows, D, D, (uint32_t)page_tokens))) return err;
     AttnTcArgs a;
     a.block_table = (const int*)block_table; a.max_blocks = max_blocks; a.num_pages = num_pages; a.page_tokens = page_tokens; a.seqs = (const int*)seqs;
     a.Hq = Hq; a.Hkv = Hkv; a.scale_log2 = sm_scale * 1.4426950408889634f; a.min_rows = min_rows;
@@ -653,20 +708,13 @@ int launch_attn_prefill_tc(const void* q, int q_rows, const void* k_pool, const 
     a.out = (__nv_bfloat16*)out; a.status = (uint32_t*)status; a.budget = g_ps_wait_budget_cycles; a.prof = g_attn_tc_prof;
     a.split_tokens = 0; a.max_splits = 0; a.dec_max_rows = 0; a.part_acc = nullptr; a.part_ml = nullptr;
     a.chunk = chunk; a.sink = (const float*)sink;
-    const size_t smem = (size_t)kTcSmem;
-    static bool set = false;
-    if (!set) {
-        cudaFuncSetAttribute(attn_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        set = true;
-    }
     const int tiles = (max_seq_rows + kTcRows - 1) / kTcRows;
-    attn_tc_kernel<false><<<dim3(tiles, Hq, n_seqs), kTcThreads, smem, stream>>>(mq, mk, mv, a);
-    return PS_LAUNCH_CHECK();
+    return launch_attn_tc_any<false>(D, k_pool == v_pool, dim3(tiles, Hq, n_seqs), mq, mk, mv, a, stream);
 }
 
 }  // namespace ps
 
-// Decode / verify attention on the tensor cores (bf16 pools, head dim 256, pages of 16 / 32 / 64 tokens, at most 8 query
+// Decode / verify attention on the tensor cores (bf16 pools, head dim 64 / 128 / 192 / 256, pages of 16 / 32 / 64 tokens, at most 8 query
 // heads per KV head): split-KV partials for every sequence of the step with at most `dec_max_rows` (<= 16) rows, in the
 // layout of ps_paged_attention's merge pass (`part_acc` [rows, Hq, max_splits, D] fp32, `part_ml` [rows, Hq, max_splits, 2]);
 // the caller runs ps_paged_attention_merge afterwards.  `split_tokens` is a multiple of 64, `q` is [q_rows, Hq, D] bf16.
@@ -678,7 +726,7 @@ PS_API int ps_attn_decode_tc_ex(const void* q, int q_rows, const void* k_pool, c
                              int Hq, int Hkv, int D, float sm_scale, int split_tokens, int max_splits, int max_visible,
                              void* part_acc, void* part_ml, void* status, int chunk, cudaStream_t stream) {
     using namespace ps;
-    if (chunk < 0 || D != kTcD || (page_tokens != 16 && page_tokens != 32 && page_tokens != 64) || Hkv <= 0 || (Hq % Hkv) || Hq / Hkv > 8 ||
+    if (chunk < 0 || D % 64 || D < 64 || D > 256 || (page_tokens != 16 && page_tokens != 32 && page_tokens != 64) || Hkv <= 0 || (Hq % Hkv) || Hq / Hkv > 8 ||
         dec_max_rows < 1 || dec_max_rows > 16 || split_tokens < kTcTok || (split_tokens % kTcTok) || n_seqs <= 0 ||
         (((uintptr_t)q | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)part_acc) % 16))
         return (int)cudaErrorInvalidValue;
@@ -686,11 +734,11 @@ PS_API int ps_attn_decode_tc_ex(const void* q, int q_rows, const void* k_pool, c
     if (n_splits < 1) n_splits = 1;
     if (n_splits > max_splits) return (int)cudaErrorInvalidValue;
     CUtensorMap mq, mk, mv;
-    int err = attn_map_2d(&mq, q, (uint64_t)q_rows * Hq, kTcD, kTcD, 8);                 // the [rows * Hq, D] view, 8-row boxes
+    int err = attn_map_2d(&mq, q, (uint64_t)q_rows * Hq, D, D, 8);                 // the [rows * Hq, D] view, 8-row boxes
     if (err) return err;
     const uint64_t pool_rows = (uint64_t)num_pages * Hkv * page_tokens;
-    if ((err = attn_map_2d(&mk, k_pool, pool_rows, kTcD, kTcD, (uint32_t)page_tokens))) return err;
-    if ((err = attn_map_2d(&mv, v_pool, pool_rows, kTcD, kTcD, (uint32_t)page_tokens))) return err;
+    if ((err = attn_map_2d(&mk, k_pool, pool_rows, D, D, (uint32_t)page_tokens))) return err;
+    if ((err = attn_map_2d(&mv, v_pool, pool_rows, D, D, (uint32_t)page_tokens))) return err;
     AttnTcArgs a;
     a.block_table = (const int*)block_table; a.max_blocks = max_blocks; a.num_pages = num_pages; a.page_tokens = page_tokens; a.seqs = (const int*)seqs;
     a.Hq = Hq; a.Hkv = Hkv; a.scale_log2 = sm_scale * 1.4426950408889634f; a.min_rows = 0;
@@ -698,14 +746,7 @@ PS_API int ps_attn_decode_tc_ex(const void* q, int q_rows, const void* k_pool, c
     a.status = (uint32_t*)status; a.budget = g_ps_wait_budget_cycles; a.prof = nullptr;
     a.split_tokens = split_tokens; a.max_splits = max_splits; a.dec_max_rows = dec_max_rows;
     a.part_acc = (float*)part_acc; a.part_ml = (float*)part_ml; a.chunk = chunk; a.sink = nullptr;
-    const size_t smem = (size_t)kTcSmem;
-    static bool set = false;
-    if (!set) {
-        cudaFuncSetAttribute(attn_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        set = true;
-    }
-    attn_tc_kernel<true><<<dim3(n_splits, Hkv, n_seqs), kTcThreads, smem, stream>>>(mq, mk, mv, a);
-    return PS_LAUNCH_CHECK();
+    return launch_attn_tc_any<true>(D, k_pool == v_pool, dim3(n_splits, Hkv, n_seqs), mq, mk, mv, a, stream);
 }
 
 PS_API int ps_attn_decode_tc(const void* q, int q_rows, const void* k_pool, const void* v_pool, const void* block_table,

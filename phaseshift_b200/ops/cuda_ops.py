@@ -484,7 +484,7 @@ class CudaOps(OpTrace):
         # rows of its tile (every tile row has its own scores, reference maximum and accumulator lane), so Exact mode -- whose
         # verified rows must reproduce single-row decoding bit for bit -- uses it as well.  FP8 pages and other shapes keep the
         # per-row kernel.  PS_ATTN_DECODE=legacy switches it off.
-        if (self.attn_decode_tc and D == 256 and st.kv_fmt == 0 and st.sc.page_tokens in (16, 32, 64) and hq // hkv <= 8
+        if (self.attn_decode_tc and D % 64 == 0 and st.kv_fmt == 0 and st.sc.page_tokens in (16, 32, 64) and hq // hkv <= 8
                 and (b.graph_static or row_pos is b.row_pos_short or all(len(sq.token_ids) <= 16 for sq in b.seqs))):
             st_tok = -(-split_tokens // 64) * 64
             n_seqs = b.max_seqs if b.graph_static else b.n_seqs

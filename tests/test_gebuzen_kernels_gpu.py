@@ -152,7 +152,7 @@ def attention_case(H, G, D, chunk, seqs, dtype, sink=True, page=16, graph=False,
         at += w.shape[0]
 
 
-HEADS = [(4, 4, 32), (6, 2, 96), (16, 1, 64), (24, 2, 128), (4, 2, 256), (2, 1, 288), (8, 2, 160), (3, 3, 192), (20, 2, 256)]
+HEADS = [(8, 2, 128), (4, 4, 64), (4, 4, 32), (6, 2, 96), (16, 1, 64), (24, 2, 128), (4, 2, 256), (2, 1, 288), (8, 2, 160), (3, 3, 192), (20, 2, 256)]
 
 
 @pytest.mark.parametrize("H,G,D", HEADS)
@@ -163,14 +163,14 @@ def test_attention_of_a_mixed_batch(H, G, D, chunk, dtype):
     attention_case(H, G, D, chunk, [(37, 150), (130, 1), (0, 2), (63, 3), (199, 16)], dtype)
 
 
-@pytest.mark.parametrize("H,G,D", [(6, 2, 96), (4, 2, 256), (16, 1, 64)])
+@pytest.mark.parametrize("H,G,D", [(6, 2, 96), (4, 2, 256), (16, 1, 64), (8, 2, 128), (3, 3, 192), (4, 4, 64)])
 @pytest.mark.parametrize("graph", [False, True])
 def test_decoded_rows_alone(H, G, D, graph):
     for chunk in (50, 128, 0):
         attention_case(H, G, D, chunk, [(127, 1), (128, 1), (49, 1), (50, 1), (0, 1), (700, 1)], BF, graph=graph)
 
 
-@pytest.mark.parametrize("H,G,D", [(6, 2, 96), (4, 2, 256), (2, 1, 288), (24, 2, 128)])
+@pytest.mark.parametrize("H,G,D", [(6, 2, 96), (4, 2, 256), (2, 1, 288), (24, 2, 128), (8, 2, 128), (8, 1, 64)])
 @pytest.mark.parametrize("standout", [0, 15, 16, 63, 64, 99, 100, 127, 128, 199, 200, 255])
 def test_a_standout_key_counts_exactly_inside_its_chunk(H, G, D, standout):
     """Rows on both sides of every border of 100-position chunks and of pages, in a prompt's portion and decoded alone."""
@@ -179,7 +179,7 @@ def test_a_standout_key_counts_exactly_inside_its_chunk(H, G, D, standout):
     attention_case(H, G, D, 100, [(0, 260)], F32 if D != 256 else BF, standout=standout)
 
 
-@pytest.mark.parametrize("D", [64, 256])
+@pytest.mark.parametrize("D", [64, 128, 192, 256])
 @pytest.mark.parametrize("page", [16, 32, 64])
 def test_page_sizes(D, page):
     attention_case(4, 2, D, 90, [(50, 200), (89, 1), (90, 1), (91, 2)], BF, page=page)
