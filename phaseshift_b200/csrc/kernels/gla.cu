@@ -212,6 +212,33 @@ __global__ void __launch_bounds__(kGPrepThreads) gla_prepare_kernel(const GlaArg
         const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(a.a2) + (size_t)h * dk * a.rank;
         for (int i = t; i < dk * a.rank; i += kGPrepThreads) s2[(i / a.rank) * pw + i % a.rank] = bf16_to_f32(w[i]);
         __syncthreads();
+        if constexpr (DKT > 0) {
+            // a thread owns one channel and every (512 / dk)-th row: eight weights at a time in registers, a1 as broadcast vectors
+            constexpr int kStep = kGPrepThreads / DKT, kRows = kGC / kStep;
+            const int d = t % DKT, r0 = t / DKT;
+            float z[kRows];
+#pragma unroll
+            for (int j = 0; j < kRows; ++j) z[j] = a.a2_bias[h * dk + d];
+            for (int c0 = 0; c0 < a.rank; c0 += 8) {
+                float wv[8];
+#pragma unroll
+                for (int c = 0; c < 8; ++c) wv[c] = s2[d * pw + c0 + c];
+#pragma unroll
+                for (int j = 0; j < kRows; ++j) {
+                    const float4 x = *reinterpret_cast<const float4*>(s1 + (r0 + j * kStep) * a.rank + c0);
+                    const float4 y = *reinterpret_cast<const float4*>(s1 + (r0 + j * kStep) * a.rank + c0 + 4);
+                    float acc = z[j];
+                    acc = fmaf(wv[0], x.x, acc); acc = fmaf(wv[1], x.y, acc); acc = fmaf(wv[2], x.z, acc); acc = fmaf(wv[3], x.w, acc);
+                    acc = fmaf(wv[4], y.x, acc); acc = fmaf(wv[5], y.y, acc); acc = fmaf(wv[6], y.z, acc); acc = fmaf(wv[7], y.w, acc);
+                    z[j] = acc;
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < kRows; ++j) {
+                const int r = r0 + j * kStep;
+                sB[r * PQ + d] = r < n ? gla_log_decay(z[j], a.inv_tau) : 0.f;
+            }
+        } else
         for (int i = t; i < kGC * dk; i += kGPrepThreads) {
             const int r = i / dk, d = i % dk;
             float la = 0.f;
@@ -252,7 +279,29 @@ __global__ void __launch_bounds__(kGPrepThreads) gla_prepare_kernel(const GlaArg
 #pragma unroll 1
     for (int blk = 0; blk < 4; ++blk) {
         const int il = (blk & 1) ? 15 - warp : warp, i = blk * 16 + il;
-        constexpr int kU = DKT > 0 ? (DKT + 31) / 32 : 8;
+        if constexpr (DKT > 0) {
+            constexpr int kU = DKT / 32;                // consecutive channels of a lane
+            const int d = lane * kU;
+            float qi[kU], bi[kU];
+#pragma unroll
+            for (int u = 0; u < kU; ++u) { qi[u] = sQ[i * PQ + d + u]; bi[u] = sB[i * PQ + d + u]; }
+            for (int jl = 0; jl <= il; ++jl) {
+                const int j = blk * 16 + jl;
+                float kj[kU], bj[kU], s = 0.f;
+                if constexpr (kU == 4) {
+                    *reinterpret_cast<float4*>(kj) = *reinterpret_cast<const float4*>(sK + j * PK + d);
+                    *reinterpret_cast<float4*>(bj) = *reinterpret_cast<const float4*>(sB + j * PQ + d);
+                } else {
+#pragma unroll
+                    for (int u = 0; u < kU; ++u) { kj[u] = sK[j * PK + d + u]; bj[u] = sB[j * PQ + d + u]; }
+                }
+#pragma unroll
+                for (int u = 0; u < kU; ++u) s = fmaf(qi[u] * kj[u], __expf(bi[u] - bj[u]), s);
+                s = warp_sum(s);
+                if (lane == 0) sA[i * kGAPitch + j] = s;
+            }
+        } else {
+        constexpr int kU = 8;
         float qi[kU], bi[kU];
 #pragma unroll
         for (int u = 0; u < kU; ++u) {
@@ -270,6 +319,7 @@ __global__ void __launch_bounds__(kGPrepThreads) gla_prepare_kernel(const GlaArg
             }
             s = warp_sum(s);
             if (lane == 0) sA[i * kGAPitch + j] = s;
+        }
         }
         if (lane > il && lane < 16) sA[i * kGAPitch + blk * 16 + lane] = 0.f;
     }
@@ -428,6 +478,10 @@ __global__ void __launch_bounds__(256) gla_scan_kernel(const GlaArgs a) {
     *st = S;
 }
 
+__device__ __forceinline__ void gla_cp_async16(void* dst, const void* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+
 // grid = (blocks, H)
 template <int DKT, int DVT>
 __global__ void __launch_bounds__(kGOutThreads) gla_output_kernel(const GlaArgs a) {
@@ -444,14 +498,13 @@ __global__ void __launch_bounds__(kGOutThreads) gla_output_kernel(const GlaArgs 
     const float* qd = a.qd + bh * kGC * dk;
     for (int i = t; i < kGC * dk / 4; i += kGOutThreads) {
         const int r = i / (dk / 4), c = (i % (dk / 4)) * 4;
-        *reinterpret_cast<float4*>(sQ + r * PQ + c) = *reinterpret_cast<const float4*>(qd + r * dk + c);
+        gla_cp_async16(sQ + r * PQ + c, qd + r * dk + c);
     }
     const float* S = a.u + bh * dk * dv;
     for (int i = t; i < dk * dv / 4; i += kGOutThreads) {
         const int r = i / (dv / 4), c = (i % (dv / 4)) * 4;
-        *reinterpret_cast<float4*>(sS + r * PS + c) = *reinterpret_cast<const float4*>(S + (size_t)r * dv + c);
+        gla_cp_async16(sS + r * PS + c, S + (size_t)r * dv + c);
     }
-    __syncthreads();
     constexpr int kNT = DVT > 0 ? DVT / 16 : 16;           // column tiles of eight per warp (half of the head)
     const int m = warp & 3, half = warp >> 2, nt = dv / 16;
     float acc[kNT][4];
@@ -463,6 +516,8 @@ __global__ void __launch_bounds__(kGOutThreads) gla_output_kernel(const GlaArgs 
             acc[j][0] = x.x; acc[j][1] = x.y; acc[j][2] = y.x; acc[j][3] = y.y;
         } else acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
     }
+    asm volatile("cp.async.wait_all;" ::: "memory");
+    __syncthreads();
     const float* q0 = sQ + (m * 16 + g) * PQ + tq;
     const float* s0 = sS + tq * PS + half * (dv / 2) + g;
     for (int k = 0; k < dk; k += 8) {
