@@ -24,9 +24,9 @@ def _doc_flags(name: str):
 
 
 def test_every_app_flag_is_documented_and_no_documented_flag_is_missing():
-    from phaseshift_b200.apps import bench, compute, gpu_test_runner, quantizer, server, tools
+    from phaseshift_b200.apps import bench, compute, gpu_test_runner, quantizer, server, tools, trace_run
     for mod, doc in ((compute, "compute.md"), (server, "server.md"), (quantizer, "quantizer.md"), (bench, "bench.md"),
-                     (tools, "tools.md"), (gpu_test_runner, "gpu_test_runner.md")):
+                     (tools, "tools.md"), (gpu_test_runner, "gpu_test_runner.md"), (trace_run, "trace_run.md")):
         have, said = _flags(mod.build_parser()), _doc_flags(doc)
         assert have - said == set(), (doc, "undocumented", sorted(have - said))
         assert said - have == set(), (doc, "documented but absent", sorted(said - have))
