@@ -16,12 +16,9 @@ from pathlib import Path
 from typing import List, NamedTuple, Optional, Sequence
 
 from ...runtime.state import KVSpec, RecurrentSpec, RunSpec
+from ..common import SingleRank, eos_ids_of_dir, pad
 
 ARCHITECTURE = "Gebuzen"
-
-
-def pad(n: int, to: int) -> int:
-    return -(-n // to) * to
 
 
 @dataclass(frozen=True)
@@ -76,11 +73,6 @@ class LayerRun(NamedTuple):
     layer: int
     pass_index: Optional[int]
     opens_pass: bool
-
-
-class SingleRank:
-    """Tensor-parallel geometry of a model that runs on one rank."""
-    tp_rank, tp_size = 0, 1
 
 
 @dataclass
@@ -171,12 +163,7 @@ class GebuzenConfig:
 
     @staticmethod
     def from_dir(model_dir) -> "GebuzenConfig":
-        raw = json.loads((Path(model_dir) / "config.json").read_text())
-        eos: object = []
-        gen = Path(model_dir) / "generation_config.json"
-        if gen.exists():
-            eos = json.loads(gen.read_text()).get("eos_token_id", [])
-        return GebuzenConfig.from_dict(raw, [eos] if isinstance(eos, int) else list(eos or []))
+        return GebuzenConfig.from_dict(json.loads((Path(model_dir) / "config.json").read_text()), eos_ids_of_dir(model_dir))
 
 
 def _uniform(preset: str, vocab: int, width: int, n_layers: int, left: ChunkAttention, right: GatedLinear, ff: int, loop=None,

@@ -20,8 +20,9 @@ from typing import Callable, Dict, List, Optional
 import torch
 
 from ...quant.formats import QuantizedTensor
+from ..common import pad, pad_cols, pad_heads, pad_rows, plain_linear
 from ..qwen35.weights import LinearW
-from .config import ChunkAttention, GatedLinear, GebuzenConfig, pad
+from .config import ChunkAttention, GatedLinear, GebuzenConfig
 
 DECAY_RANK = 16          # rank of the decay projection in random-init models (a loaded model's tensors give theirs)
 
@@ -134,29 +135,11 @@ class GebuzenWeights:
         return esz * (self.embed.numel() + sum(w.N * w.k_padded for w in self.linears()) + sum(l.a2.numel() for l in self.layers))
 
 
-def _pad_heads(t: torch.Tensor, heads: int, dim: int, to: int) -> torch.Tensor:
-    """[heads * dim, ...] -> [heads * to, ...], zero rows at the end of every head."""
-    if dim == to:
-        return t
-    out = t.new_zeros((heads, to) + tuple(t.shape[1:]))
-    out[:, :dim] = t.reshape((heads, dim) + tuple(t.shape[1:]))
-    return out.reshape((heads * to,) + tuple(t.shape[1:]))
-
-
-def _pad_rows(t: torch.Tensor, to: int) -> torch.Tensor:
-    return t if t.shape[0] == to else torch.cat([t, t.new_zeros((to - t.shape[0],) + tuple(t.shape[1:]))], 0)
-
-
-def _pad_cols(t: torch.Tensor, to: int) -> torch.Tensor:
-    return t if t.shape[1] == to else torch.cat([t, t.new_zeros(t.shape[0], to - t.shape[1])], 1)
-
-
 def build_engine_weights(cfg: GebuzenConfig, get: Callable[[str], torch.Tensor], device="cpu",
                          dtype: Optional[torch.dtype] = None) -> GebuzenWeights:
     """``dtype``: what projections and activations run in, bfloat16 or float32 (default: bfloat16 on a CUDA device)."""
     dev = torch.device(device)
-    on_cuda = dev.type == "cuda"
-    dtype = dtype or (torch.bfloat16 if on_cuda else torch.float32)
+    dtype = dtype or (torch.bfloat16 if dev.type == "cuda" else torch.float32)
     if dtype not in (torch.bfloat16, torch.float32):
         raise ValueError(f"Gebuzen runs in bfloat16 or float32, not {dtype}")
     fmt = "bf16" if dtype == torch.bfloat16 else "f32"
@@ -168,11 +151,7 @@ def build_engine_weights(cfg: GebuzenConfig, get: Callable[[str], torch.Tensor],
         return get(name).to(device=dev, dtype=torch.float32).contiguous()
 
     def lin(w: torch.Tensor, n: int, k: int) -> LinearW:
-        w = _pad_cols(_pad_rows(w, n), k).contiguous()
-        lw = LinearW(QuantizedTensor(fmt, (n, k), k, w))
-        if on_cuda and fmt == "bf16":
-            lw.make_tiled(True)          # both forms stay: streaming tiles for single rows, row-major for the tensor-core GEMMs
-        return lw
+        return plain_linear(w, n, k, fmt)
 
     W = cfg.hidden_size
     nout = pad(W, 4)                     # output rows of projections onto the residual width (paired fp32 stores need even pitches)
@@ -187,30 +166,30 @@ def build_engine_weights(cfg: GebuzenConfig, get: Callable[[str], torch.Tensor],
 
         def with_bias(name: str, heads: int, dim: int, to: int) -> torch.Tensor:
             wb = torch.cat([t(name), t(name + ".b")[:, None]], 1)
-            return _pad_cols(_pad_heads(wb, heads, dim, to), kin_b)
+            return pad_cols(pad_heads(wb, heads, dim, to), kin_b)
 
         def plain(name: str, heads: int, dim: int, to: int) -> torch.Tensor:
-            return _pad_cols(_pad_heads(t(name), heads, dim, to), kin_b)
+            return pad_cols(pad_heads(t(name), heads, dim, to), kin_b)
 
         D, dk, dv = l.dim_padded, r.dim_padded, r.vdim_padded
         rows = torch.cat([with_bias(m + "left.q", l.heads, l.dim, D), with_bias(m + "left.k", l.kv_heads, l.dim, D),
                           plain(m + "right.q", r.heads, r.dim, dk), plain(m + "right.k", r.heads, r.dim, dk),
                           plain(m + "right.v", r.heads, r.vdim, dv), plain(m + "right.g", r.heads, r.vdim, dv),
-                          _pad_cols(_pad_rows(t(m + "right.a1"), rp), kin_b)], 0)
+                          pad_cols(pad_rows(t(m + "right.a1"), rp), kin_b)], 0)
         in_proj = lin(rows, rows.shape[0], kin_b)
         del rows
-        a2 = _pad_cols(_pad_heads(t(m + "right.a2"), r.heads, r.dim, dk), rp).contiguous()
-        left_o = lin(_pad_heads(t(m + "left.o").T.contiguous(), l.heads, l.dim, D).T, nout, l.heads * D)
-        right_o = lin(_pad_heads(t(m + "right.o").T.contiguous(), r.heads, r.vdim, dv).T, nout, r.heads * dv)
+        a2 = pad_cols(pad_heads(t(m + "right.a2"), r.heads, r.dim, dk), rp).contiguous()
+        left_o = lin(pad_heads(t(m + "left.o").T.contiguous(), l.heads, l.dim, D).T, nout, l.heads * D)
+        right_o = lin(pad_heads(t(m + "right.o").T.contiguous(), r.heads, r.vdim, dv).T, nout, r.heads * dv)
         gate_up = down = norm2 = None
         if L.ff is not None:
             fp = pad(L.ff, 32)
-            gu = torch.stack([_pad_rows(t(p + "mlp.gate"), fp), _pad_rows(t(p + "mlp.up"), fp)], 1).reshape(2 * fp, W)
+            gu = torch.stack([pad_rows(t(p + "mlp.gate"), fp), pad_rows(t(p + "mlp.up"), fp)], 1).reshape(2 * fp, W)
             gate_up, down, norm2 = lin(gu, 2 * fp, kin), lin(t(p + "mlp.down"), nout, fp), f32(p + "norm2")
             del gu
         layers.append(ParallelLayerW(l, r, f32(p + "norm1"), in_proj, rp, a2,
-                                     _pad_heads(f32(m + "right.a2.b"), r.heads, r.dim, dk).contiguous(), f32(m + "left.sink"),
-                                     _pad_rows(f32(m + "right.norm"), dv).contiguous(), left_o, right_o,
+                                     pad_heads(f32(m + "right.a2.b"), r.heads, r.dim, dk).contiguous(), f32(m + "left.sink"),
+                                     pad_rows(f32(m + "right.norm"), dv).contiguous(), left_o, right_o,
                                      f32(m + "left.out"), f32(m + "right.out"), norm2, gate_up, down))
     head = lin(t("head"), pad(cfg.vocab_size, 2), kin)
     return GebuzenWeights(cfg, t("embed").contiguous(), f32("loop.step") if cfg.loop is not None else None, layers,

@@ -7,6 +7,7 @@ per layer execution, runtime/state.py) and ``family`` (the name it is registered
 """
 from __future__ import annotations
 
+import importlib
 import json
 from dataclasses import dataclass
 from pathlib import Path
@@ -70,42 +71,33 @@ def _qwen_runner(weights, state, ops, tp=None):
     return Qwen35Runner(weights, state, ops, tp)
 
 
-# ---------------------------------------------------------------- Gebuzen
-def _gebuzen_config(model_dir):
-    from .gebuzen.config import GebuzenConfig
-    return GebuzenConfig.from_dir(model_dir)
+# ---------------------------------------------------------------- decoders with plain weights that run on one rank
+def _plain_family(name: str, architecture: str) -> ModelFamily:
+    """Family of ``models/<name>``: its modules ``config`` (<Architecture>Config, PRESETS), ``weights`` (load_engine_weights,
+    build_engine_weights, random_getter) and ``model`` (<Architecture>Runner); bf16 or 32-bit weights, no tensor parallelism."""
+    def module(which):
+        return importlib.import_module(f".{name}.{which}", __package__)
 
+    def options(preset, kw) -> None:
+        _reject(preset not in (None, "bf16"), f"{architecture} models have no {preset!r} weight preset (bf16, or 32-bit with dtype=float32)")
+        _reject(kw.get("tp_size", 1) != 1, f"{architecture} models run on one rank")
 
-def _gebuzen_presets():
-    from .gebuzen.config import PRESETS
-    return PRESETS
+    def load(model_dir, device, preset=None, dtype=None, **kw):
+        options(preset, kw)
+        return module("weights").load_engine_weights(model_dir, device, dtype)
 
+    def rand(cfg, device, preset=None, dtype=None, **kw):
+        options(preset, kw)
+        return module("weights").build_engine_weights(cfg, module("weights").random_getter(cfg, 0, device), device, dtype)
 
-def _gebuzen_options(preset, kw) -> None:
-    _reject(preset not in (None, "bf16"), f"Gebuzen models have no {preset!r} weight preset (bf16, or 32-bit with dtype=float32)")
-    _reject(kw.get("tp_size", 1) != 1, "Gebuzen models run on one rank")
-
-
-def _gebuzen_load(model_dir, device, preset=None, dtype=None, **kw):
-    from .gebuzen.weights import load_engine_weights
-    _gebuzen_options(preset, kw)
-    return load_engine_weights(model_dir, device, dtype)
-
-
-def _gebuzen_random(cfg, device, preset=None, dtype=None, **kw):
-    from .gebuzen.weights import build_engine_weights, random_getter
-    _gebuzen_options(preset, kw)
-    return build_engine_weights(cfg, random_getter(cfg, 0, device), device, dtype)
-
-
-def _gebuzen_runner(weights, state, ops, tp=None):
-    from .gebuzen.model import GebuzenRunner
-    return GebuzenRunner(weights, state, ops, tp)
+    return ModelFamily(name, lambda raw: raw.get("architecture") == architecture,
+                       lambda d: getattr(module("config"), architecture + "Config").from_dir(d), lambda: module("config").PRESETS, load, rand,
+                       lambda weights, state, ops, tp=None: getattr(module("model"), architecture + "Runner")(weights, state, ops, tp))
 
 
 FAMILIES: List[ModelFamily] = [
-    ModelFamily("gebuzen", lambda raw: raw.get("architecture") == "Gebuzen", _gebuzen_config, _gebuzen_presets, _gebuzen_load,
-                _gebuzen_random, _gebuzen_runner),
+    _plain_family("luvutar", "Luvutar"),
+    _plain_family("gebuzen", "Gebuzen"),
     # the first family of the framework; a config.json without an architecture of another family is read as its own
     ModelFamily("qwen35", lambda raw: "architecture" not in raw, _qwen_config, _qwen_presets, _qwen_load, _qwen_random, _qwen_runner),
 ]

@@ -9,6 +9,7 @@ speculative decoding and tensor-parallel logic be tested without a GPU.
 """
 from __future__ import annotations
 
+import math
 from typing import Optional
 
 import torch
@@ -20,7 +21,7 @@ from ..models.qwen35.weights import AttnW, GdnW, LinearW
 from ..runtime.batch import StepBatch
 from ..runtime.state import GdnLayerState, KVLayer, ModelState
 from ..utils.sampling import sample_row_host
-from .specs import AttnSpec, GlaSpec, Pending
+from .specs import AttnSpec, GlaSpec, LatentSpec, Pending, StreamWrite
 
 
 class RefOps(OpTrace):
@@ -45,7 +46,7 @@ class RefOps(OpTrace):
         return self._dense(table)[b.ids[:rows].long()]
 
     def linear(self, x, W: LinearW, *, name: str, norm_w=None, eps: float = 0.0, residual=None, swiglu=False,
-               reglu=False, out_f32=False, out=None, ssq_in=None, ssq_out=None, prefetch=None, **_):
+               reglu=False, gelu=False, out_f32=False, out=None, ssq_in=None, ssq_out=None, prefetch=None, **_):
         x = x.float()
         if self.act_quant and W.fmt in ("nvfp4", "mxfp8"):
             # the tensor-core layout's arithmetic: quantise x (1 + w), apply the row factor 1/rms after the product
@@ -64,6 +65,8 @@ class RefOps(OpTrace):
             y = F.silu(y[:, 0::2]) * y[:, 1::2]
         if reglu:
             y = F.relu(y[:, 0::2]) * y[:, 1::2]
+        if gelu:
+            y = F.gelu(y, approximate="tanh")
         if residual is not None:
             y = y + residual.float()
         if out is not None:
@@ -251,23 +254,47 @@ class RefOps(OpTrace):
                 h[:, x.shape[1]] = 1.0
         return x, h
 
+    # ------------------------------------------------------------------ parallel residual streams
+    def stream_norm(self, x, pend: Optional[StreamWrite], *, read=None, norm_w=None, eps: float, width: int = 0, name: str = "",
+                    last: bool = False):
+        """x [rows, streams, W]: write what is pending into all streams, then read the next sublayer's input from them and norm
+        it, padded to `width` columns.  Returns (new streams, normed row or None)."""
+        W = x.shape[2]
+        if pend is not None:
+            x = torch.einsum("st,rsw->rtw", pend.mix, x) + pend.out[:, None] * pend.y[:, None, :W].float()
+        h = None
+        if norm_w is not None:
+            u = torch.einsum("s,rsw->rw", read, x)
+            h = x.new_zeros(x.shape[0], width)
+            h[:, :W] = u * torch.rsqrt(u.pow(2).mean(-1, keepdim=True) + eps) * norm_w
+        return x, h
+
     # ------------------------------------------------------------------ attention without rotation over paged keys
-    def attn_append(self, proj, spec: AttnSpec, b: StepBatch, kv: KVLayer, st: ModelState):
-        """proj rows start with [q heads | k heads]: the keys go to their pages, the queries are returned."""
-        rows, pt, D = proj.shape[0], st.sc.page_tokens, spec.dim
-        nq = spec.heads * D
-        k = proj[:, nq:nq + spec.kv_heads * D].reshape(rows, spec.kv_heads, D)
-        for r in range(rows):
-            slot, p = int(b.row_slot[r]), int(b.row_pos[r])
-            if slot < 0:
+    def _page_of(self, b: StepBatch, r: int, st: ModelState):
+        """(page, offset) of row r's position, or None for a padding row."""
+        slot, p, pt = int(b.row_slot[r]), int(b.row_pos[r]), st.sc.page_tokens
+        if slot < 0:
+            return None
+        page = int(st.block_table[slot, p // pt])
+        if page < 0:
+            raise RuntimeError("KV append into an unmapped page")
+        return page, p % pt
+
+    def attn_append(self, proj, spec: AttnSpec, b: StepBatch, kv: Optional[KVLayer], st: ModelState):
+        """proj rows start with [q heads | k heads (| v heads)]: keys and values go to their pages, the queries are returned.
+        ``kv`` None: the layer has no keys of its own."""
+        rows, D, G = proj.shape[0], spec.dim, spec.kv_heads
+        nq, nk = spec.heads * D, spec.kv_heads * D
+        for r in range(rows if kv is not None else 0):
+            at = self._page_of(b, r, st)
+            if at is None:
                 continue
-            page = int(st.block_table[slot, p // pt])
-            if page < 0:
-                raise RuntimeError("KV append into an unmapped page")
-            kv.k[page, :, p % pt, :] = k[r]
+            kv.k[at[0], :, at[1], :] = proj[r, nq:nq + nk].reshape(G, D)
+            if kv.v is not kv.k:
+                kv.v[at[0], :, at[1], :] = proj[r, nq + nk:nq + 2 * nk].reshape(G, D)
         return proj[:, :nq]
 
-    def attention(self, q, spec: AttnSpec, b: StepBatch, kv: KVLayer, st: ModelState, max_visible: int):
+    def attention(self, q, spec: AttnSpec, b: StepBatch, kv: KVLayer, st: ModelState, max_visible: int, gate=None):
         rows, D, H = q.shape[0], spec.dim, spec.heads
         pt = st.sc.page_tokens
         out = q.new_zeros(rows, H, D)
@@ -276,18 +303,58 @@ class RefOps(OpTrace):
             slot, p = int(b.row_slot[r]), int(b.row_pos[r])
             if slot < 0:
                 continue
-            lo = p - p % spec.chunk if spec.chunk > 0 else 0
-            tok = torch.arange(lo, p + 1)
+            tok = torch.arange(spec.first_visible(p), p + 1)
             pages = st.block_table[slot, tok // pt].long()
             K = kv.k[pages, :, tok % pt].float().repeat_interleave(H // spec.kv_heads, 1)
             V = kv.v[pages, :, tok % pt].float().repeat_interleave(H // spec.kv_heads, 1)
             s = torch.einsum("hd,thd->ht", qh[r].float(), K) * spec.scale
+            if spec.temp_coef != 0.0:
+                s = s * (1.0 + spec.temp_coef * math.log(math.floor((p + 1) / spec.temp_every) + 1))
+            if spec.bias is not None:
+                s = s + spec.bias[:, (p - tok).clamp(max=spec.bias.shape[1] - 1)]
             if spec.sink is not None:
                 pr = torch.softmax(torch.cat([s, spec.sink[:, None]], 1), -1)[:, :-1]
             else:
                 pr = torch.softmax(s, -1)
             out[r] = torch.einsum("ht,thd->hd", pr, V)
+        gate = spec.gate if gate is None else gate
+        if gate is not None:
+            cols = spec.gate_offset + torch.arange(H)[:, None] * spec.gate_head_stride
+            out = out * torch.sigmoid(gate[:, cols if spec.gate_per_head else cols + torch.arange(D)].float())
         return out.reshape(rows, H * D)
+
+    # ------------------------------------------------------------------ latent attention
+    @staticmethod
+    def _turn_pairs(t, pos, inv_freq):
+        """Neighbouring elements of the first 2 * len(inv_freq) columns of t [rows, ..., R] turn by pos * inv_freq."""
+        n = 2 * inv_freq.numel()
+        ang = (pos.double()[:, None] * inv_freq).reshape((-1,) + (1,) * (t.dim() - 2) + (n // 2,))
+        u, v = t[..., 0:n:2].double(), t[..., 1:n:2].double()
+        t = t.clone()
+        t[..., 0:n:2], t[..., 1:n:2] = (u * ang.cos() - v * ang.sin()).float(), (v * ang.cos() + u * ang.sin()).float()
+        return t
+
+    def latent_down(self, proj, s: LatentSpec, b: StepBatch, kv: KVLayer, st: ModelState):
+        """proj rows are [query latent | latent | rotated key part | ...]: the latent and the turned key part go to their page,
+        the normed query latent is returned."""
+        unit = lambda t, true: t * torch.rsqrt(t.pow(2).sum(-1, keepdim=True) / true + s.eps)
+        p = proj.float()
+        c = unit(p[:, s.c_off:s.c_off + s.kv_rank], s.kv_rank_true) * s.kv_norm
+        r = self._turn_pairs(p[:, s.c_off + s.kv_rank:s.c_off + s.row], b.row_pos[:proj.shape[0]], s.inv_freq)
+        for i in range(proj.shape[0]):
+            at = self._page_of(b, i, st)
+            if at is not None:
+                kv.k[at[0], 0, at[1]] = torch.cat([c[i], r[i]])
+        return unit(p[:, :s.q_rank], s.q_rank_true) * s.q_norm
+
+    def latent_attention(self, q, s: LatentSpec, b: StepBatch, kv: KVLayer, st: ModelState, gate):
+        rows, H = q.shape[0], s.heads
+        qh = q.float().reshape(rows, H, s.dim + s.rot)
+        into = torch.einsum("rhd,hcd->rhc", qh[..., :s.dim], s.uk_t.float().reshape(H, s.kv_rank, s.dim))
+        qe = torch.cat([into, self._turn_pairs(qh[..., s.dim:], b.row_pos[:rows], s.inv_freq)], -1)
+        o = self.attention(qe.reshape(rows, -1), s.shared_keys(), b, kv, st, b.max_visible_launch).reshape(rows, H, s.row)[..., :s.kv_rank]
+        o = torch.einsum("rhc,hvc->rhv", o, s.uv.float().reshape(H, s.vdim, s.kv_rank)).reshape(rows, H * s.vdim)
+        return o * torch.sigmoid(gate[:, s.gate_off:s.gate_off + H * s.vdim].float())
 
     # ------------------------------------------------------------------ gated linear attention
     def gla(self, proj, g: GlaSpec, b: StepBatch, gs: GdnLayerState, st: ModelState):
