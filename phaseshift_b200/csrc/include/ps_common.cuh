@@ -142,6 +142,8 @@ __device__ __forceinline__ uint32_t f32x2_to_bf16x2_bits(float a, float b) {
 }
 
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + __expf(-x)); }
+// z/2 (1 + tanh u) with u = sqrt(2/pi) (z + 0.044715 z^3), written as z / (1 + exp(-2u)).
+__device__ __forceinline__ float gelu_tanh_f(float z) { return z / (1.f + __expf(-1.5957691216057308f * fmaf(0.044715f * z * z, z, z))); }
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + __expf(-x)); }
 __device__ __forceinline__ float softplus_f(float x) { return x > 20.f ? x : log1pf(__expf(x)); }
 

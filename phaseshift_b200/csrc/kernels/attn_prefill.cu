@@ -12,6 +12,7 @@
 // the six query heads that share a KV head run as neighbouring CTAs so their K/V tiles hit in L2.
 // Decode and speculative verification stay on the split-KV kernel (paged_attention.cu), whose per-row
 // arithmetic does not depend on the batch.
+#include "attn_options.cuh"
 #include "ps_common.cuh"
 
 namespace ps {
@@ -29,12 +30,8 @@ struct AttnPrefillArgs {
     const __nv_bfloat16* gate; int ld_gate; int gate_head_stride; int gate_offset;
     __nv_bfloat16* out;          // [rows, Hq*D]
     uint32_t* status;
-    int chunk;                   // > 0: position i sees only its own block of `chunk` positions (counted from position 0)
-    const float* sink;           // [Hq] or null: exp(sink[h]) joins head h's denominator
+    AttnOptions opt; int transform;      // mask and sink; `transform`: query temperature or distance bias
 };
-
-// First position a query at `pos` sees.
-__device__ __forceinline__ int chunk_start(int pos, int chunk) { return chunk > 0 ? pos / chunk * chunk : 0; }
 
 __device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], const void* p) {
     const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
@@ -298,7 +295,7 @@ __global__ void __launch_bounds__(kPfThreads) attn_prefill_async_kernel(const At
     const int t = threadIdx.x, warp = t >> 5, lane = t & 31;
     bool bad = false;
 
-    const int t_first = chunk_start(pos_q0, a.chunk) / kPfTok * kPfTok;      // tile of the first token the first row sees
+    const int t_first = attn_first(a.opt, pos_q0) / kPfTok * kPfTok;      // tile of the first token the first row sees
     issue_tile<D>(a, a.k_pool, sK, slot, kvh, t_first, kv_end, bad);
     issue_tile<D>(a, a.v_pool, sV, slot, kvh, t_first, kv_end, bad);
     for (int p = t; p < kPfRows * (D / 8); p += kPfThreads) {
@@ -313,8 +310,9 @@ __global__ void __launch_bounds__(kPfThreads) attn_prefill_async_kernel(const At
     for (int j = 0; j < D / 8; ++j) { o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f; }
     float m_run[2] = {-1.0e30f, -1.0e30f}, l_run[2] = {0.f, 0.f};
     const int rpos0 = pos_q0 + warp * 16 + (lane >> 2);
-    const int lo[2] = {chunk_start(rpos0, a.chunk), chunk_start(rpos0 + 8, a.chunk)};
-    const int warp_lo = chunk_start(pos_q0 + warp * 16, a.chunk);            // no row of this warp sees an earlier token
+    const int lo[2] = {attn_first(a.opt, rpos0), attn_first(a.opt, rpos0 + 8)};
+    const float row_scale[2] = {a.scale_log2 * attn_temperature(a.opt, rpos0), a.scale_log2 * attn_temperature(a.opt, rpos0 + 8)};
+    const int warp_lo = attn_first(a.opt, pos_q0 + warp * 16);              // no row of this warp sees an earlier token
 
     for (int t0 = t_first; t0 < kv_end; t0 += kPfTok) {
         const bool live = t0 <= pos_q0 + warp * 16 + 15 && t0 + kPfTok > warp_lo;       // some row of this warp sees this tile
@@ -348,7 +346,8 @@ __global__ void __launch_bounds__(kPfThreads) attn_prefill_async_kernel(const At
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     const int tok = t0 + 8 * j + (lane & 3) * 2 + (e & 1);
-                    float v = s[j][e] * a.scale_log2;
+                    float v = s[j][e] * row_scale[e >> 1];
+                    if (a.transform) v = fmaf(attn_bias(a.opt, h, max(rpos0 + (e >> 1) * 8 - tok, 0)), 1.4426950408889634f, v);
                     if (tok > rpos0 + (e >> 1) * 8 || tok < lo[e >> 1]) v = -1.0e30f;
                     s[j][e] = v;
                     mx[e >> 1] = fmaxf(mx[e >> 1], v);
@@ -406,15 +405,17 @@ __global__ void __launch_bounds__(kPfThreads) attn_prefill_async_kernel(const At
         const int lr = warp * 16 + (lane >> 2) + r * 8;
         if (lr >= nq) continue;
         const size_t row = (size_t)(row_start + r_begin + lr);
-        if (a.sink != nullptr) l_run[r] += exp2f(fmaf(a.sink[h], 1.4426950408889634f, -m_run[r]));
+        if (a.opt.sink != nullptr) l_run[r] += exp2f(fmaf(a.opt.sink[h], 1.4426950408889634f, -m_run[r]));
         const float inv = l_run[r] > 0.f ? 1.f / l_run[r] : 0.f;
 #pragma unroll
         for (int j = 0; j < D / 8; ++j) {
             const int d = 8 * j + (lane & 3) * 2;
             float v0 = bf16_to_f32(f32_to_bf16(o[j][2 * r] * inv)), v1 = bf16_to_f32(f32_to_bf16(o[j][2 * r + 1] * inv));
             if (a.gate != nullptr) {
-                const float2 gv = bf16x2_bits_to_f32x2(*reinterpret_cast<const uint32_t*>(
-                    a.gate + row * a.ld_gate + (size_t)h * a.gate_head_stride + a.gate_offset + d));
+                const __nv_bfloat16* gr = a.gate + row * a.ld_gate + (size_t)h * a.gate_head_stride + a.gate_offset;
+                float2 gv;
+                if (a.opt.gate_per_head) gv.x = gv.y = bf16_to_f32(*gr);
+                else gv = bf16x2_bits_to_f32x2(*reinterpret_cast<const uint32_t*>(gr + d));
                 v0 *= sigmoid_f(gv.x); v1 *= sigmoid_f(gv.y);
             }
             *reinterpret_cast<uint32_t*>(a.out + (row * a.Hq + h) * D + d) = f32x2_to_bf16x2_bits(v0, v1);
@@ -438,12 +439,12 @@ static int launch_prefill(const AttnPrefillArgs& a, int max_q_tiles, int n_seqs,
 
 // attn_prefill_tc.cu: the tcgen05 kernel for head dims 64 / 128 / 192 / 256 and pages of 16 / 32 / 64 tokens (FP8 pools through a bf16 scratch pool)
 bool attn_prefill_tc_supported(int D, int page_tokens, int kv_fp8, const void* q, const void* k_pool, const void* v_pool,
-                               const void* gate, int ld_gate, int gate_head_stride, int gate_offset, const void* deq_k);
+                               const void* gate, int ld_gate, int gate_head_stride, int gate_offset, const void* deq_k, const AttnOptions& opt);
 int launch_attn_prefill_tc(const void* q, int q_rows, const void* k_pool, const void* v_pool, const void* k_scale, const void* v_scale,
                            int kv_fp8, const void* block_table, int max_blocks, int num_pages, int page_tokens, const void* seqs,
                            int n_seqs, int max_seq_rows, int min_rows, int Hq, int Hkv, int D, float sm_scale, const void* gate, int ld_gate,
                            int gate_head_stride, int gate_offset, void* deq_k, void* deq_v, int deq_pages, void* deq_bt, void* deq_seqs,
-                           void* out, void* status, int chunk, const void* sink, cudaStream_t stream);
+                           void* out, void* status, const AttnOptions& opt, cudaStream_t stream);
 
 }  // namespace ps
 
@@ -451,22 +452,25 @@ int launch_attn_prefill_tc(const void* q, int q_rows, const void* k_pool, const 
 // `min_rows`: sequences with at most this many rows are skipped (the caller runs the split-KV kernel on their rows);
 // `deq_*`: optional bf16 scratch pool ([deq_pages, Hkv, page_tokens, D] twice), block table [n_seqs, max_blocks] and
 // sequence descriptors [n_seqs, 4] that let FP8 pools take the tensor-core kernel.
-// `chunk`, `sink`: see AttnPrefillArgs (bf16 pools only).
+// `options`: an AttnOptions (attn_options.cuh) or null; mask, sink and score transforms on bf16 pools only.
 PS_API int ps_attn_prefill_ex(const void* q, const void* k_pool, const void* v_pool, const void* k_scale, const void* v_scale,
                            const void* block_table, int max_blocks, int page_tokens, int num_pages, const void* seqs,
                            int n_seqs, int max_seq_rows, int q_rows, int min_rows, int Hq, int Hkv, int D, float sm_scale, int kv_fp8,
                            const void* gate, int ld_gate, int gate_head_stride, int gate_offset, void* deq_k, void* deq_v,
-                           int deq_pages, void* deq_bt, void* deq_seqs, void* out, void* status, int chunk, const void* sink,
+                           int deq_pages, void* deq_bt, void* deq_seqs, void* out, void* status, const void* options,
                            cudaStream_t stream) {
     using namespace ps;
-    if (chunk < 0 || (kv_fp8 && (chunk > 0 || sink != nullptr))) return (int)cudaErrorInvalidValue;
+    const AttnOptions opt = attn_options(options);
+    if (!attn_options_ok(opt)) return (int)cudaErrorInvalidValue;
+    if (kv_fp8 && (opt.chunk > 0 || opt.window > 0 || opt.sink != nullptr || opt.gate_per_head || attn_transforms_scores(opt)))
+        return (int)cudaErrorInvalidValue;
     if (n_seqs <= 0 || max_seq_rows <= 0 || Hkv <= 0 || (Hq % Hkv) || q_rows < max_seq_rows) return (int)cudaErrorInvalidValue;
-    if (attn_prefill_tc_supported(D, page_tokens, kv_fp8, q, k_pool, v_pool, gate, ld_gate, gate_head_stride, gate_offset, deq_k))
+    if (attn_prefill_tc_supported(D, page_tokens, kv_fp8, q, k_pool, v_pool, gate, ld_gate, gate_head_stride, gate_offset, deq_k, opt))
         return launch_attn_prefill_tc(q, q_rows, k_pool, v_pool, k_scale, v_scale, kv_fp8, block_table, max_blocks, num_pages, page_tokens,
                                       seqs, n_seqs, max_seq_rows, min_rows, Hq, Hkv, D, sm_scale, gate, ld_gate, gate_head_stride, gate_offset,
-                                      deq_k, deq_v, deq_pages, deq_bt, deq_seqs, out, status, chunk, sink, stream);
+                                      deq_k, deq_v, deq_pages, deq_bt, deq_seqs, out, status, opt, stream);
     AttnPrefillArgs a;
-    a.chunk = chunk; a.sink = (const float*)sink;
+    a.opt = opt; a.transform = attn_transforms_scores(opt) ? 1 : 0;
     a.q = (const __nv_bfloat16*)q; a.k_pool = k_pool; a.v_pool = v_pool; a.k_scale = (const float*)k_scale;
     a.v_scale = (const float*)v_scale; a.block_table = (const int*)block_table; a.max_blocks = max_blocks;
     a.page_tokens = page_tokens; a.num_pages = num_pages; a.seqs = (const int*)seqs; a.Hq = Hq; a.Hkv = Hkv;
@@ -494,5 +498,5 @@ PS_API int ps_attn_prefill(const void* q, const void* k_pool, const void* v_pool
                            int deq_pages, void* deq_bt, void* deq_seqs, void* out, void* status, cudaStream_t stream) {
     return ps_attn_prefill_ex(q, k_pool, v_pool, k_scale, v_scale, block_table, max_blocks, page_tokens, num_pages, seqs, n_seqs,
                               max_seq_rows, q_rows, min_rows, Hq, Hkv, D, sm_scale, kv_fp8, gate, ld_gate, gate_head_stride,
-                              gate_offset, deq_k, deq_v, deq_pages, deq_bt, deq_seqs, out, status, 0, nullptr, stream);
+                              gate_offset, deq_k, deq_v, deq_pages, deq_bt, deq_seqs, out, status, nullptr, stream);
 }

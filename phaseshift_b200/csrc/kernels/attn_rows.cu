@@ -1,9 +1,10 @@
-// Key append without rotation, and per-row attention for any head size in bf16 or 32-bit.
+// Key (and value) append without rotation, and per-row attention for any head size in bf16 or 32-bit.
 //
-// ps_attn_append copies the query columns of a projection row to the dense query buffer and its key columns to their page.
-// ps_attn_rows is the plain form of the masked attention (block-local mask, sink) that paged_attention.cu and
+// ps_attn_append copies the query columns of a projection row to the dense query buffer and its key and value columns to their
+// page.  ps_attn_rows is the plain form of the attention (with the options of attn_options.cuh) that paged_attention.cu and
 // attn_prefill*.cu serve for bf16 pools and head sizes up to 256: one CTA per (row, query head), scores and softmax in
 // 32-bit.  The 32-bit engines run on it, and head sizes that the tiled kernels do not take.
+#include "attn_options.cuh"
 #include "ps_common.cuh"
 
 namespace ps {
@@ -11,7 +12,7 @@ namespace ps {
 struct AttnAppendArgs {
     const uint4* proj; int ld16;                 // row pitch in 16-byte units
     int q16, head16, Hkv;                        // 16-byte units of the query columns and of one key head
-    uint4* q_out; uint4* k_pool;
+    uint4* q_out; uint4* k_pool; uint4* v_pool;   // v_pool null: the keys are the values
     const int* row_slot; const int* row_pos; const int* block_table; int max_blocks, page_tokens, num_pages;
     uint32_t* status;
 };
@@ -22,6 +23,7 @@ __global__ void attn_append_kernel(const AttnAppendArgs a) {
     const int row = blockIdx.x;
     const uint4* src = a.proj + (size_t)row * a.ld16;
     for (int i = threadIdx.x; i < a.q16; i += blockDim.x) a.q_out[(size_t)row * a.q16 + i] = src[i];
+    if (a.Hkv == 0) return;                      // the layer reads another one's keys
     const int slot = a.row_slot[row], pos = a.row_pos[row];
     if (slot < 0 || pos < 0) return;             // padding row
     const int blk = pos / a.page_tokens, off = pos % a.page_tokens;
@@ -29,7 +31,9 @@ __global__ void attn_append_kernel(const AttnAppendArgs a) {
     if (page < 0 || page >= a.num_pages) { if (threadIdx.x == 0) set_status(a.status, PS_DEV_BAD_INDEX); return; }
     for (int i = threadIdx.x; i < a.Hkv * a.head16; i += blockDim.x) {
         const int head = i / a.head16, c = i % a.head16;
-        a.k_pool[(((size_t)page * a.Hkv + head) * a.page_tokens + off) * a.head16 + c] = src[a.q16 + i];
+        const size_t at = (((size_t)page * a.Hkv + head) * a.page_tokens + off) * a.head16 + c;
+        a.k_pool[at] = src[a.q16 + i];
+        if (a.v_pool != nullptr) a.v_pool[at] = src[a.q16 + a.Hkv * a.head16 + i];
     }
 }
 
@@ -41,11 +45,12 @@ struct AttnRowsArgs {
     const void* q; const void* k_pool; const void* v_pool;
     const int* block_table; int max_blocks, page_tokens, num_pages;
     const int* row_slot; const int* row_pos;
-    int Hq, Hkv, D; float scale; int chunk; const float* sink;
+    int Hq, Hkv, D; float scale; AttnOptions opt;
+    const void* gate; int ld_gate, gate_head_stride, gate_offset;    // optional sigmoid gate
     void* out; uint32_t* status;
 };
 
-constexpr int kArThreads = 128, kArTile = 128, kArMaxD = 1024;
+constexpr int kArThreads = 128, kArTile = 128, kArMaxD = 2048;
 
 // grid = (Hq, rows)
 template <typename T>
@@ -66,9 +71,10 @@ __global__ void __launch_bounds__(kArThreads) attn_rows_kernel(const AttnRowsArg
         s_q[d] = (float)reinterpret_cast<const T*>(a.q)[((size_t)row * a.Hq + h) * D + d];
         s_o[d] = 0.f;
     }
-    const int lo = a.chunk > 0 ? pos / a.chunk * a.chunk : 0;
-    float m = a.sink != nullptr ? a.sink[h] : -3.0e38f;
-    float l = a.sink != nullptr ? 1.f : 0.f;
+    const int lo = attn_first(a.opt, pos);
+    const float scale = a.scale * attn_temperature(a.opt, pos);
+    float m = a.opt.sink != nullptr ? a.opt.sink[h] : -3.0e38f;
+    float l = a.opt.sink != nullptr ? 1.f : 0.f;
     for (int t0 = lo; t0 <= pos; t0 += kArTile) {
         const int n = min(kArTile, pos + 1 - t0);
         __syncthreads();
@@ -86,7 +92,7 @@ __global__ void __launch_bounds__(kArThreads) attn_rows_kernel(const AttnRowsArg
                 for (int d = lane; d < D; d += 32) s = fmaf(s_q[d], (float)k[d], s);
             }
             s = warp_sum(s);
-            if (lane == 0) s_p[j] = s_page[j] >= 0 ? s * a.scale : -INFINITY;
+            if (lane == 0) s_p[j] = s_page[j] >= 0 ? fmaf(s, scale, attn_bias(a.opt, h, pos - t0 - j)) : -INFINITY;
         }
         __syncthreads();
         const float s = t < n ? s_p[t] : -INFINITY;
@@ -109,35 +115,47 @@ __global__ void __launch_bounds__(kArThreads) attn_rows_kernel(const AttnRowsArg
         }
     }
     const float inv = l > 0.f ? 1.f / l : 0.f;
-    for (int d = t; d < D; d += kArThreads) out[d] = ar_cast<T>(s_o[d] * inv);
+    const T* gate = a.gate == nullptr ? nullptr
+                                      : reinterpret_cast<const T*>(a.gate) + (size_t)row * a.ld_gate + (size_t)h * a.gate_head_stride + a.gate_offset;
+    for (int d = t; d < D; d += kArThreads) {
+        float o = s_o[d] * inv;
+        if (gate != nullptr) o *= 1.f / (1.f + expf(-(float)gate[a.opt.gate_per_head ? 0 : d]));
+        out[d] = ar_cast<T>(o);
+    }
 }
 
 }  // namespace ps
 
-// proj: rows of [Hq * D queries | Hkv * D keys | ...] of `esz`-byte elements; D * esz a multiple of 16.
+// proj: rows of [Hq * D queries | Hkv * D keys (| Hkv * D values, with a value pool) | ...] of `esz`-byte elements; D * esz a
+// multiple of 16.  Hkv 0: nothing is appended.
 PS_API int ps_attn_append(const void* proj, int ld, int esz, int rows, int Hq, int Hkv, int D, const void* row_slot, const void* row_pos,
-                          void* q_out, void* k_pool, const void* block_table, int max_blocks, int page_tokens, int num_pages,
+                          void* q_out, void* k_pool, void* v_pool, const void* block_table, int max_blocks, int page_tokens, int num_pages,
                           void* status, cudaStream_t stream) {
     using namespace ps;
-    if (rows <= 0 || (D * esz) % 16 || ((size_t)ld * esz) % 16 || ((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)k_pool) % 16)
+    if (rows <= 0 || Hkv < 0 || (D * esz) % 16 || ((size_t)ld * esz) % 16 ||
+        ((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)k_pool | (uintptr_t)v_pool) % 16)
         return (int)cudaErrorInvalidValue;
     AttnAppendArgs a;
     a.proj = (const uint4*)proj; a.ld16 = (int)((size_t)ld * esz / 16); a.head16 = D * esz / 16; a.q16 = Hq * a.head16; a.Hkv = Hkv;
-    a.q_out = (uint4*)q_out; a.k_pool = (uint4*)k_pool; a.row_slot = (const int*)row_slot; a.row_pos = (const int*)row_pos;
-    a.block_table = (const int*)block_table; a.max_blocks = max_blocks; a.page_tokens = page_tokens; a.num_pages = num_pages;
-    a.status = (uint32_t*)status;
+    a.q_out = (uint4*)q_out; a.k_pool = (uint4*)k_pool; a.v_pool = (uint4*)v_pool; a.row_slot = (const int*)row_slot;
+    a.row_pos = (const int*)row_pos; a.block_table = (const int*)block_table; a.max_blocks = max_blocks; a.page_tokens = page_tokens;
+    a.num_pages = num_pages; a.status = (uint32_t*)status;
     return launch_pdl(attn_append_kernel, dim3(rows), dim3(256), 0, stream, a);
 }
 
+// `options`: an AttnOptions or null.  The gate has the pools' element type.
 PS_API int ps_attn_rows(const void* q, const void* k_pool, const void* v_pool, int f32, const void* block_table, int max_blocks,
                         int page_tokens, int num_pages, const void* row_slot, const void* row_pos, int rows, int Hq, int Hkv, int D,
-                        float scale, int chunk, const void* sink, void* out, void* status, cudaStream_t stream) {
+                        float scale, const void* options, const void* gate, int ld_gate, int gate_head_stride, int gate_offset,
+                        void* out, void* status, cudaStream_t stream) {
     using namespace ps;
-    if (rows <= 0 || rows > 65535 || Hkv <= 0 || (Hq % Hkv) || D <= 0 || D > kArMaxD || chunk < 0) return (int)cudaErrorInvalidValue;
+    const AttnOptions opt = attn_options(options);
+    if (rows <= 0 || rows > 65535 || Hkv <= 0 || (Hq % Hkv) || D <= 0 || D > kArMaxD || !attn_options_ok(opt)) return (int)cudaErrorInvalidValue;
     AttnRowsArgs a;
     a.q = q; a.k_pool = k_pool; a.v_pool = v_pool; a.block_table = (const int*)block_table; a.max_blocks = max_blocks;
     a.page_tokens = page_tokens; a.num_pages = num_pages; a.row_slot = (const int*)row_slot; a.row_pos = (const int*)row_pos;
-    a.Hq = Hq; a.Hkv = Hkv; a.D = D; a.scale = scale; a.chunk = chunk; a.sink = (const float*)sink; a.out = out; a.status = (uint32_t*)status;
+    a.Hq = Hq; a.Hkv = Hkv; a.D = D; a.scale = scale; a.opt = opt; a.gate = gate; a.ld_gate = ld_gate;
+    a.gate_head_stride = gate_head_stride; a.gate_offset = gate_offset; a.out = out; a.status = (uint32_t*)status;
     if (f32) return launch_pdl(attn_rows_kernel<float>, dim3(Hq, rows), dim3(kArThreads), 0, stream, a);
     return launch_pdl(attn_rows_kernel<__nv_bfloat16>, dim3(Hq, rows), dim3(kArThreads), 0, stream, a);
 }

@@ -8,7 +8,7 @@
 //     lives in tensor memory (128 lanes x BN columns);
 //   * `tcgen05.commit` releases ring slots back to the producer and finally signals the epilogue;
 //   * four epilogue warps read the accumulator with `tcgen05.ld` (each warp its own 32-lane quadrant),
-//     apply the fused epilogue (residual add / SwiGLU on interleaved gate-up columns / f32 or bf16
+//     apply the fused epilogue (residual add / SwiGLU on interleaved gate-up columns / tanh-gelu / f32 or bf16
 //     store) and write to global memory.
 // Warp roles: warp 0 = TMA producer, warp 1 = MMA issuer + TMEM owner, warps 2..5 = epilogue.
 // Every mbarrier wait is bounded; a timeout sets PS_DEV_WAIT_TIMEOUT in the status word, the CTA
@@ -21,7 +21,7 @@
 
 namespace ps {
 
-enum GemmEpilogue : int { GEPI_STORE = 0, GEPI_RESIDUAL = 1, GEPI_SWIGLU = 2, GEPI_REGLU = 3 };
+enum GemmEpilogue : int { GEPI_STORE = 0, GEPI_RESIDUAL = 1, GEPI_SWIGLU = 2, GEPI_REGLU = 3, GEPI_GELU = 4 };
 
 constexpr int kBM = 128, kBK = 64;
 constexpr int kGemmThreads = 192;
@@ -161,12 +161,14 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                                     v0 = bf16_to_f32(f32_to_bf16(v0)) + rs.x;
                                     v1 = bf16_to_f32(f32_to_bf16(v1)) + rs.y;
                                 }
+                                if (g.epilogue == GEPI_GELU) { v0 = gelu_tanh_f(v0); v1 = gelu_tanh_f(v1); }
                                 if (g.out_f32) *reinterpret_cast<float2*>(reinterpret_cast<float*>(g.out) + (size_t)row * g.ldo + col) = make_float2(v0, v1);
                                 else *reinterpret_cast<uint32_t*>(reinterpret_cast<__nv_bfloat16*>(g.out) + (size_t)row * g.ldo + col) = f32x2_to_bf16x2_bits(v0, v1);
                             } else if (col < g.N) {
                                 float v0 = __uint_as_float(r[j]);
                                 if (g.epilogue == GEPI_RESIDUAL)
                                     v0 = bf16_to_f32(f32_to_bf16(v0)) + bf16_to_f32(g.residual[(size_t)row * g.ld_res + col]);
+                                if (g.epilogue == GEPI_GELU) v0 = gelu_tanh_f(v0);
                                 if (g.out_f32) reinterpret_cast<float*>(g.out)[(size_t)row * g.ldo + col] = v0;
                                 else reinterpret_cast<__nv_bfloat16*>(g.out)[(size_t)row * g.ldo + col] = f32_to_bf16(v0);
                             }

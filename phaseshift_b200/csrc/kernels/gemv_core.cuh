@@ -32,7 +32,7 @@ namespace ps {
 
 enum WeightFormat : int { W_BF16 = 0, W_NVFP4 = 1, W_MXFP8 = 2 };
 enum LinearPrologue : int { PRO_NONE = 0, PRO_RMSNORM_ONEPLUS = 1, PRO_SIGMOID_GATE = 2 };
-enum LinearEpilogue : int { EPI_STORE = 0, EPI_RESIDUAL = 1, EPI_SWIGLU = 2, EPI_REGLU = 3 };     // gated: silu / relu (gate) * up
+enum LinearEpilogue : int { EPI_STORE = 0, EPI_RESIDUAL = 1, EPI_SWIGLU = 2, EPI_REGLU = 3, EPI_GELU = 4 };     // gated: silu / relu (gate) * up
 
 constexpr int kTpMaxRanks = 8;
 // Tensor-parallel combine fused into a row-parallel projection's epilogue (one-shot all-reduce over
@@ -451,6 +451,7 @@ __device__ __forceinline__ void quad_epilogue(const LinearSmallArgs& a, int n0, 
         float y = v[r];
         if (a.epilogue == EPI_RESIDUAL)   // y rounded to bf16 before the add, like projection-then-add
             y = bf16_to_f32(f32_to_bf16(y)) + bf16_to_f32(a.residual[(size_t)m * a.ld_res + n]);
+        if (a.epilogue == EPI_GELU) y = gelu_tanh_f(y);
         if (a.out_f32) reinterpret_cast<float*>(a.out)[(size_t)m * a.ldo + n] = y;
         else reinterpret_cast<__nv_bfloat16*>(a.out)[(size_t)m * a.ldo + n] = f32_to_bf16(y);
     }

@@ -9,12 +9,12 @@
 //   * the merge pass also applies the sigmoid output gate, so o_proj reads its input directly.
 // One CTA = (split, kv head, row) and serves up to eight of the G = Hq/Hkv query heads that share the K/V tile.
 //
-// Two options of the mask and the denominator: `chunk` > 0 confines a row at position i to the positions of its own block of
-// `chunk` (blocks counted from position 0), and `sink` adds exp(sink[h]) to head h's denominator in the merge pass.
+// The options of attn_options.cuh: mask, query temperature and distance bias in the split pass, sink and gate in the merge pass.
 //
 // K/V pools: [num_pages, Hkv, page_tokens, D]; FP8 pools carry one f32 scale per (page, head, token).
 #include <stdio.h>
 
+#include "attn_options.cuh"
 #include "ps_common.cuh"
 #include "ps_noalloc.h"
 
@@ -35,7 +35,7 @@ struct PagedAttnArgs {
     float* part_acc;   // [rows, Hq, max_splits, D]
     float* part_ml;    // [rows, Hq, max_splits, 2]  (running max, running sum)
     uint32_t* status;
-    int chunk;         // > 0: a row sees only its own block of `chunk` positions
+    AttnOptions opt;
 };
 
 struct TileRegs { uint4 k[4]; uint4 v[4]; float ks, vs; };
@@ -145,16 +145,17 @@ __global__ void __launch_bounds__(kAttnThreads) paged_attn_split_kernel(const Pa
     const int g_first = (blockIdx.y % groups) * kAttnMaxG;
     const int G = min(kAttnMaxG, heads_per_kv - g_first), h0 = kvh * heads_per_kv + g_first;
     const int visible = a.row_pos[row] + 1;
-    const int lo = a.chunk > 0 && visible > 0 ? (visible - 1) / a.chunk * a.chunk : 0;
+    const int lo = visible > 0 ? attn_first(a.opt, visible - 1) : 0;
     const int tok_end = min(visible, (split + 1) * a.split_tokens);
     const int tok_begin = max(split * a.split_tokens, lo);
     if (tok_begin >= tok_end) return;
     const int slot = a.row_slot[row];
     const int t = threadIdx.x, warp = t >> 5, lane = t & 31;
 
+    const float q_scale = a.sm_scale * attn_temperature(a.opt, visible - 1);
     for (int i = t; i < G * D; i += kAttnThreads) {
         const int g = i / D, d = i % D;
-        qs[i] = bf16_to_f32(a.q[((size_t)row * a.Hq + h0 + g) * D + d]) * a.sm_scale;
+        qs[i] = bf16_to_f32(a.q[((size_t)row * a.Hq + h0 + g) * D + d]) * q_scale;
     }
     if (t < kAttnTile) { kscale[t] = 1.f; vscale[t] = 1.f; }
     float acc[kAttnMaxG];
@@ -188,6 +189,7 @@ __global__ void __launch_bounds__(kAttnThreads) paged_attn_split_kernel(const Pa
             }
             s *= kscale[lane];
             const bool live = tok < tok_end;
+            if (live) s += attn_bias(a.opt, h0 + warp, visible - 1 - tok);
             if (!live) s = -3.0e38f;
             const float m_new = fmaxf(m_run, warp_max(s));
             const float p = live ? __expf(s - m_new) : 0.f;
@@ -241,7 +243,8 @@ struct AttnMergeArgs {
     int rows, Hq, D, split_tokens, max_splits;
     const __nv_bfloat16* gate; int ld_gate; int gate_head_stride; int gate_offset;   // optional sigmoid gate
     __nv_bfloat16* out;   // [rows, Hq*D]
-    int chunk; const float* sink;   // as in the split pass; sink [Hq] or null
+    AttnOptions opt;
+    int ring;             // > 0: split s of a row lies in slot s % ring of the partials
 };
 
 // grid = (Hq, rows), block = D threads.  The split weights exp(m_s - max m) are computed once, in
@@ -257,28 +260,33 @@ __global__ void paged_attn_merge_kernel(const AttnMergeArgs a) {
     const int visible = a.row_pos[row] + 1;
     if (visible < 0) return;                                            // position -2: a row another kernel of the step owns
     const int n = (visible + a.split_tokens - 1) / a.split_tokens;      // 0 for a padding row
-    const int s0 = a.chunk > 0 && visible > 0 ? (visible - 1) / a.chunk * a.chunk / a.split_tokens : 0;
-    const float sink = a.sink != nullptr ? a.sink[h] : -3.0e38f;
+    const int s0 = visible > 0 ? attn_first(a.opt, visible - 1) / a.split_tokens : 0;
+    const int ring = a.ring > 0 ? a.ring : kAttnMaxSplits;
+    const float sink = a.opt.sink != nullptr ? a.opt.sink[h] : -3.0e38f;
     const float* ml = a.part_ml + ((size_t)row * a.Hq + h) * a.max_splits * 2;
     const float* pa = a.part_acc + ((size_t)row * a.Hq + h) * a.max_splits * a.D;
     float m = sink;
-    for (int s = s0 + d; s < n; s += blockDim.x) m = fmaxf(m, ml[2 * s]);
+    for (int s = s0 + d; s < n; s += blockDim.x) m = fmaxf(m, ml[2 * (s % ring)]);
     m = block_max(m, s_red);
     float l = 0.f;
     for (int s = s0 + d; s < n; s += blockDim.x) {
-        const float w = __expf(ml[2 * s] - m);
-        s_w[s] = w;
-        l = fmaf(w, ml[2 * s + 1], l);
+        const float w = __expf(ml[2 * (s % ring)] - m);
+        s_w[s % ring] = w;
+        l = fmaf(w, ml[2 * (s % ring) + 1], l);
     }
     l = block_sum(l, s_red + 32);      // its barriers also publish s_w
-    if (a.sink != nullptr) l += __expf(sink - m);
+    if (a.opt.sink != nullptr) l += __expf(sink - m);
     float o = 0.f;
+    int at = s0 % ring;
 #pragma unroll 4
-    for (int s = s0; s < n; ++s) o = fmaf(s_w[s], pa[(size_t)s * a.D + d], o);
+    for (int s = s0; s < n; ++s) {
+        o = fmaf(s_w[at], pa[(size_t)at * a.D + d], o);
+        at = at + 1 == ring ? 0 : at + 1;
+    }
     float v = l > 0.f ? o / l : 0.f;
     if (a.gate != nullptr) {
         v = bf16_to_f32(f32_to_bf16(v));
-        const float g = bf16_to_f32(a.gate[(size_t)row * a.ld_gate + h * a.gate_head_stride + a.gate_offset + d]);
+        const float g = bf16_to_f32(a.gate[(size_t)row * a.ld_gate + h * a.gate_head_stride + a.gate_offset + (a.opt.gate_per_head ? 0 : d)]);
         v *= sigmoid_f(g);
     }
     a.out[((size_t)row * a.Hq + h) * a.D + d] = f32_to_bf16(v);
@@ -286,16 +294,17 @@ __global__ void paged_attn_merge_kernel(const AttnMergeArgs a) {
 
 }  // namespace ps
 
-// `chunk` (0 = plain causal) and `sink` ([Hq] f32 or null) select the options named at the top of the file.
+// `options`: an AttnOptions (attn_options.cuh) or null.
 PS_API int ps_paged_attention_ex(const void* q, const void* k_pool, const void* v_pool, const void* k_scale,
                               const void* v_scale, const void* block_table, int max_blocks, int page_tokens,
                               int num_pages, const void* row_slot, const void* row_pos, int rows, int Hq, int Hkv,
                               int D, float sm_scale, int kv_fp8, int split_tokens, int max_splits, int max_visible,
                               void* part_acc, void* part_ml, const void* gate, int ld_gate, int gate_head_stride,
-                              int gate_offset, void* out, void* status, int chunk, const void* sink, cudaStream_t stream) {
+                              int gate_offset, void* out, void* status, const void* options, cudaStream_t stream) {
     using namespace ps;
     const int G = Hkv > 0 ? Hq / Hkv : 0;
-    if (G < 1 || (Hq % Hkv) || chunk < 0 || D > kAttnMaxD || (D % 32) || (split_tokens % kAttnTile) || rows <= 0)
+    const AttnOptions opt = attn_options(options);
+    if (G < 1 || (Hq % Hkv) || !attn_options_ok(opt) || D > kAttnMaxD || (D % 32) || (split_tokens % kAttnTile) || rows <= 0)
         return (int)cudaErrorInvalidValue;
     PagedAttnArgs a;
     a.q = (const __nv_bfloat16*)q; a.k_pool = k_pool; a.v_pool = v_pool; a.k_scale = (const float*)k_scale;
@@ -303,7 +312,7 @@ PS_API int ps_paged_attention_ex(const void* q, const void* k_pool, const void* 
     a.page_tokens = page_tokens; a.num_pages = num_pages; a.row_slot = (const int*)row_slot;
     a.row_pos = (const int*)row_pos; a.rows = rows; a.Hq = Hq; a.Hkv = Hkv; a.D = D; a.sm_scale = sm_scale;
     a.kv_fp8 = kv_fp8; a.split_tokens = split_tokens; a.max_splits = max_splits;
-    a.part_acc = (float*)part_acc; a.part_ml = (float*)part_ml; a.status = (uint32_t*)status; a.chunk = chunk;
+    a.part_acc = (float*)part_acc; a.part_ml = (float*)part_ml; a.status = (uint32_t*)status; a.opt = opt;
     int n_splits = (max_visible + split_tokens - 1) / split_tokens;
     if (n_splits < 1) n_splits = 1;
     if (n_splits > max_splits || max_splits > kAttnMaxSplits) return (int)cudaErrorInvalidValue;
@@ -321,7 +330,7 @@ PS_API int ps_paged_attention_ex(const void* q, const void* k_pool, const void* 
     m.part_acc = a.part_acc; m.part_ml = a.part_ml; m.row_pos = a.row_pos; m.rows = rows; m.Hq = Hq; m.D = D;
     m.split_tokens = split_tokens; m.max_splits = max_splits; m.gate = (const __nv_bfloat16*)gate;
     m.ld_gate = ld_gate; m.gate_head_stride = gate_head_stride; m.gate_offset = gate_offset;
-    m.out = (__nv_bfloat16*)out; m.chunk = chunk; m.sink = (const float*)sink;
+    m.out = (__nv_bfloat16*)out; m.opt = opt; m.ring = 0;
     return launch_pdl(paged_attn_merge_kernel, dim3(Hq, rows), dim3(D), 0, stream, m);
 }
 
@@ -333,21 +342,25 @@ PS_API int ps_paged_attention(const void* q, const void* k_pool, const void* v_p
                               int gate_offset, void* out, void* status, cudaStream_t stream) {
     return ps_paged_attention_ex(q, k_pool, v_pool, k_scale, v_scale, block_table, max_blocks, page_tokens, num_pages, row_slot,
                                  row_pos, rows, Hq, Hkv, D, sm_scale, kv_fp8, split_tokens, max_splits, max_visible, part_acc,
-                                 part_ml, gate, ld_gate, gate_head_stride, gate_offset, out, status, 0, nullptr, stream);
+                                 part_ml, gate, ld_gate, gate_head_stride, gate_offset, out, status, nullptr, stream);
 }
 
 // The merge pass alone: for partials produced by another split-KV kernel (attn_prefill_tc.cu's decode variant) in the same
-// layout.  Same arguments as the tail of ps_paged_attention.
+// layout.  Same arguments as the tail of ps_paged_attention.  `ring` > 0: `max_splits` partials per row and head are kept in
+// a ring, split s in slot s % ring (kernels whose rows see a bounded number of splits).
 PS_API int ps_paged_attention_merge_ex(const void* part_acc, const void* part_ml, const void* row_pos, int rows, int Hq, int D,
                                        int split_tokens, int max_splits, const void* gate, int ld_gate, int gate_head_stride,
-                                       int gate_offset, void* out, int chunk, const void* sink, cudaStream_t stream) {
+                                       int gate_offset, void* out, const void* options, int ring, cudaStream_t stream) {
     using namespace ps;
-    if (rows <= 0 || Hq <= 0 || D <= 0 || D > kAttnMaxD || max_splits > kAttnMaxSplits) return (int)cudaErrorInvalidValue;
+    const AttnOptions opt = attn_options(options);
+    if (rows <= 0 || rows > 65535 || Hq <= 0 || D <= 0 || D > 1024 || max_splits > kAttnMaxSplits || ring < 0 || ring > max_splits ||
+        !attn_options_ok(opt))
+        return (int)cudaErrorInvalidValue;
     AttnMergeArgs m;
     m.part_acc = (const float*)part_acc; m.part_ml = (const float*)part_ml; m.row_pos = (const int*)row_pos; m.rows = rows; m.Hq = Hq; m.D = D;
     m.split_tokens = split_tokens; m.max_splits = max_splits; m.gate = (const __nv_bfloat16*)gate;
     m.ld_gate = ld_gate; m.gate_head_stride = gate_head_stride; m.gate_offset = gate_offset;
-    m.out = (__nv_bfloat16*)out; m.chunk = chunk; m.sink = (const float*)sink;
+    m.out = (__nv_bfloat16*)out; m.opt = opt; m.ring = ring;
     return launch_pdl(paged_attn_merge_kernel, dim3(Hq, rows), dim3(D), 0, stream, m);
 }
 
@@ -355,7 +368,7 @@ PS_API int ps_paged_attention_merge(const void* part_acc, const void* part_ml, c
                                     int split_tokens, int max_splits, const void* gate, int ld_gate, int gate_head_stride,
                                     int gate_offset, void* out, cudaStream_t stream) {
     return ps_paged_attention_merge_ex(part_acc, part_ml, row_pos, rows, Hq, D, split_tokens, max_splits, gate, ld_gate,
-                                       gate_head_stride, gate_offset, out, 0, nullptr, stream);
+                                       gate_head_stride, gate_offset, out, nullptr, 0, stream);
 }
 
 // ------------------------------------------------------------------------------------------------

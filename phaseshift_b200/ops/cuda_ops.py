@@ -21,13 +21,27 @@ from ..models.qwen35.weights import AttnW, GdnW, LinearW
 from ..runtime.batch import StepBatch
 from ..runtime.state import GdnLayerState, KVLayer, ModelState
 from . import _lib
-from .specs import AttnSpec, GlaSpec, Pending
+from .specs import AttnSpec, GlaSpec, LatentSpec, Pending, StreamWrite
 from ._lib import c_float, c_int, c_ll, ptr
 
 WFMT = {"bf16": 0, "nvfp4": 1, "mxfp8": 2}
 PRO_NONE, PRO_RMSNORM, PRO_SIGMOID_GATE = 0, 1, 2
-EPI_STORE, EPI_RESIDUAL, EPI_SWIGLU, EPI_REGLU = 0, 1, 2, 3
+EPI_STORE, EPI_RESIDUAL, EPI_SWIGLU, EPI_REGLU, EPI_GELU = 0, 1, 2, 3, 4
 SMALL_M_MAX = 8
+
+
+class AttnOptions(ctypes.Structure):
+    """csrc/include/attn_options.cuh: AttnOptions."""
+    _fields_ = [("chunk", ctypes.c_int), ("window", ctypes.c_int), ("temp_coef", ctypes.c_float), ("temp_every", ctypes.c_float),
+                ("bias", ctypes.c_void_p), ("bias_len", ctypes.c_int), ("gate_per_head", ctypes.c_int), ("sink", ctypes.c_void_p)]
+
+    @staticmethod
+    def of(s: AttnSpec) -> "AttnOptions":
+        for t in (s.bias, s.sink):
+            if t is not None and (t.dtype != torch.float32 or not t.is_contiguous() or t.shape[0] != s.heads):
+                raise ValueError("attention biases and sinks are contiguous f32 tensors, one row per head")
+        return AttnOptions(s.chunk, s.window, s.temp_coef, s.temp_every, None if s.bias is None else s.bias.data_ptr(),
+                           0 if s.bias is None else s.bias.shape[1], int(s.gate_per_head), None if s.sink is None else s.sink.data_ptr())
 
 
 class CudaOps(OpTrace):
@@ -125,7 +139,7 @@ class CudaOps(OpTrace):
         return out
 
     def linear(self, x: torch.Tensor, W: LinearW, *, name: str, norm_w: Optional[torch.Tensor] = None,
-               eps: float = 0.0, residual: Optional[torch.Tensor] = None, swiglu: bool = False, reglu: bool = False,
+               eps: float = 0.0, residual: Optional[torch.Tensor] = None, swiglu: bool = False, reglu: bool = False, gelu: bool = False,
                out_f32: bool = False, out: Optional[torch.Tensor] = None,
                xn_out: Optional[torch.Tensor] = None, tp_combine=None, ssq_in=None,
                ssq_out: Optional[torch.Tensor] = None, prefetch: Optional[LinearW] = None, tp_scatter=None) -> torch.Tensor:
@@ -139,10 +153,11 @@ class CudaOps(OpTrace):
         ``tp_scatter`` (a parallel.tp.TpScatterStruct; tensor-core path with streamed activations only): instead of
         storing to ``out`` the kernel pushes each bf16 output row to the receive buffer of the rank that owns it.
         ``swiglu`` / ``reglu``: the weight's rows interleave (gate, up) and the output is silu / relu (gate) * up.
-        32-bit weights run in fp32 on the CUDA cores (plain and gated epilogues only)."""
+        ``gelu``: the tanh form of gelu is applied to every output.
+        32-bit weights run in fp32 on the CUDA cores (activation epilogues only)."""
         M, K = x.shape
         if W.fmt == "f32":
-            return self._linear_f32(x, W, name, swiglu, reglu, out, plain=norm_w is None and residual is None)
+            return self._linear_f32(x, W, name, swiglu, reglu, gelu, out, plain=norm_w is None and residual is None)
         assert K == W.K and x.dtype == torch.bfloat16 and x.stride(1) == 1, (x.shape, W.K, x.dtype)
         n_out = W.N // 2 if swiglu or reglu else W.N
         if out is None:
@@ -152,8 +167,8 @@ class CudaOps(OpTrace):
             raise ValueError(f"K={W.K} must be a multiple of 32 for the streaming / bf16 tensor-core kernels")
         sel = self.select_linear(W, M)
         if sel == "tc":
-            if reglu:
-                raise ValueError("the block-scaled projections have no ReGLU epilogue")
+            if reglu or gelu:
+                raise ValueError("the block-scaled projections have no ReGLU or gelu epilogue")
             # block-quantised codes straight into the tensor cores (any number of rows)
             return self.linear_bs(x, W, name=name, norm_w=norm_w, eps=eps, residual=residual, swiglu=swiglu,
                                   out_f32=out_f32, out=out, xn_out=xn_out, tp_combine=tp_combine, ssq_in=ssq_in,
@@ -169,9 +184,9 @@ class CudaOps(OpTrace):
         self.sel_counts["gemm" if (sel == "gemm" or batched) else "stream"] += 1
         if sel == "gemm" or batched:
             return self.linear_large(x, W, name=name, norm_w=norm_w, eps=eps, residual=residual, swiglu=swiglu,
-                                     reglu=reglu, out_f32=out_f32, out=out)
+                                     reglu=reglu, gelu=gelu, out_f32=out_f32, out=out)
         pro = PRO_RMSNORM if norm_w is not None else PRO_NONE
-        epi = EPI_SWIGLU if swiglu else EPI_REGLU if reglu else (EPI_RESIDUAL if residual is not None else EPI_STORE)
+        epi = self._epilogue(swiglu, reglu, gelu, residual)
         if W.tiled is None:
             W.make_tiled()
         L = _lib.lib()
@@ -191,6 +206,12 @@ class CudaOps(OpTrace):
                       ctypes.byref(tp_combine) if tp_combine is not None else ptr(None), ptr(self.status))
             self.launches += 1
         return out
+
+    @staticmethod
+    def _epilogue(swiglu: bool, reglu: bool, gelu: bool, residual) -> int:
+        if gelu and residual is not None:
+            raise ValueError("a projection has either an activation or a residual in its epilogue")
+        return EPI_SWIGLU if swiglu else EPI_REGLU if reglu else EPI_GELU if gelu else EPI_RESIDUAL if residual is not None else EPI_STORE
 
     def can_fuse_argmax(self, W: LinearW, M: int) -> bool:
         """True when ``linear_argmax`` can serve these rows: the streaming kernel would be chosen and holds them in one launch."""
@@ -218,7 +239,7 @@ class CudaOps(OpTrace):
         self.sel_counts["stream"] += 1
         return tokens.view(-1)[:M]
 
-    def _linear_f32(self, x: torch.Tensor, W: LinearW, name: str, swiglu: bool, reglu: bool, out, plain: bool) -> torch.Tensor:
+    def _linear_f32(self, x: torch.Tensor, W: LinearW, name: str, swiglu: bool, reglu: bool, gelu: bool, out, plain: bool) -> torch.Tensor:
         M, K = x.shape
         if not plain or x.dtype != torch.float32 or K != W.K or x.stride(1) != 1:
             raise ValueError("32-bit projections take fp32 rows and have no fused norm or residual")
@@ -226,12 +247,13 @@ class CudaOps(OpTrace):
             out = self.buf(name, M, W.N // 2 if swiglu or reglu else W.N, torch.float32)
         w = W.q.codes
         _lib.call("ps_gemm_f32", ptr(x), c_int(x.stride(0)), ptr(w), c_int(w.stride(0)), c_int(M), c_int(W.N), c_int(K),
-                  c_int(EPI_SWIGLU if swiglu else EPI_REGLU if reglu else EPI_STORE), ptr(out), c_int(out.stride(0)))
+                  c_int(self._epilogue(swiglu, reglu, gelu, None)), ptr(out), c_int(out.stride(0)))
         self.launches += 1
         self.sel_counts["f32"] = self.sel_counts.get("f32", 0) + 1
         return out
 
-    def linear_large(self, x: torch.Tensor, W: LinearW, *, name: str, norm_w, eps, residual, swiglu, out_f32, out, reglu=False):
+    def linear_large(self, x: torch.Tensor, W: LinearW, *, name: str, norm_w, eps, residual, swiglu, out_f32, out, reglu=False,
+                     gelu=False):
         """Prefill-sized projection: (RMSNorm kernel) -> weight expansion to a bf16 scratch matrix -> tcgen05
         GEMM with the residual / SwiGLU / dtype epilogue fused."""
         M, K = x.shape
@@ -249,7 +271,7 @@ class CudaOps(OpTrace):
             _lib.call("ps_dequant_tiled", c_int(WFMT[W.fmt]), ptr(W.tiled), c_int(W.N), c_int(kp),
                       c_float(W.tensor_scale), ptr(wd), c_int(kp))
             self.launches += 1
-        epi = EPI_SWIGLU if swiglu else EPI_REGLU if reglu else (EPI_RESIDUAL if residual is not None else EPI_STORE)
+        epi = self._epilogue(swiglu, reglu, gelu, residual)
         if W.rowmajor_bf16 is not None and M <= 64 and W.N % 2 == 0:
             # batched decode: swap-AB split-K weight-streaming GEMM (gemm_smallm.cu)
             L = _lib.lib()
@@ -417,24 +439,21 @@ class CudaOps(OpTrace):
         D = self.cfg.head_dim
         return self.attention(q, AttnSpec(hq, hkv, D, D ** -0.5, gate=qkv, gate_head_stride=2 * D, gate_offset=D), b, kv, st, max_visible)
 
-    def attention(self, q: torch.Tensor, spec: AttnSpec, b: StepBatch, kv: KVLayer, st: ModelState, max_visible: int) -> torch.Tensor:
+    def attention(self, q: torch.Tensor, spec: AttnSpec, b: StepBatch, kv: KVLayer, st: ModelState, max_visible: int,
+                  gate: Optional[torch.Tensor] = None) -> torch.Tensor:
         """Softmax attention of the step's rows over their paged keys and values (ops/specs.py: AttnSpec)."""
         rows, D, hq, hkv = q.shape[0], spec.dim, spec.heads, spec.kv_heads
-        sm, chunk, sink = c_float(spec.scale), c_int(spec.chunk), ptr(spec.sink)
-        gate = (ptr(spec.gate), c_int(spec.gate.stride(0) if spec.gate is not None else 0), c_int(spec.gate_head_stride),
-                c_int(spec.gate_offset))
-        if st.kv_fmt != 0 and (spec.chunk > 0 or spec.sink is not None):
-            raise ValueError("block-local masks and sinks need bf16 or 32-bit pages")
+        sm, opts = c_float(spec.scale), AttnOptions.of(spec)
+        opt = ctypes.byref(opts)
+        gate_t = spec.gate if gate is None else gate
+        gate = (ptr(gate_t), c_int(gate_t.stride(0) if gate_t is not None else 0), c_int(spec.gate_head_stride), c_int(spec.gate_offset))
+        if st.kv_fmt != 0 and (spec.chunk > 0 or spec.window > 0 or spec.sink is not None or spec.bias is not None or spec.temp_coef != 0.0
+                               or spec.gate_per_head):
+            raise ValueError("masks, sinks, score transforms and per-head gates need bf16 or 32-bit pages")
         geom = f"{hq}x{D}"                      # layers of one model may differ in head geometry: one set of buffers for each
         out = self.buf("attn_ctx" + geom, rows, hq * D, self.act_dtype)
         if self.act_dtype == torch.float32 or D % 32 or D > 256:
-            if spec.gate is not None:
-                raise ValueError("the per-row attention kernel has no output gate")
-            _lib.call("ps_attn_rows", ptr(q), ptr(kv.k), ptr(kv.v), c_int(1 if self.act_dtype == torch.float32 else 0),
-                      ptr(st.block_table), c_int(st.max_blocks), c_int(st.sc.page_tokens), c_int(st.num_pages), ptr(b.row_slot),
-                      ptr(b.row_pos), c_int(rows), c_int(hq), c_int(hkv), c_int(D), sm, chunk, sink, ptr(out), ptr(st.status))
-            self.launches += 1
-            return out
+            return self._attn_rows(q, spec, b, kv, st, out, gate)
         # the tiled kernel pays off when some sequence brings a long run of rows (a prefill chunk); steps made of
         # many sequences with a row or two each (batched decode) keep the per-row split-KV kernel
         tiled = (not self.exact_rows and not b.graph_static
@@ -465,7 +484,7 @@ class CudaOps(OpTrace):
             _lib.call("ps_attn_prefill_ex", ptr(q), ptr(src[0]), ptr(src[1]), ptr(src[2]), ptr(src[3]),
                       ptr(src[4]), c_int(st.max_blocks), c_int(pt), c_int(src[5]),
                       ptr(src[6]), c_int(b.n_seqs), c_int(rows), c_int(q.shape[0]), c_int(min_rows), c_int(hq), c_int(hkv), c_int(D),
-                      sm, c_int(src[7]), *gate, ptr(deq[0]), ptr(deq[1]), c_int(deq[2]), ptr(deq[3]), ptr(deq[4]), ptr(out), ptr(st.status), chunk, sink)
+                      sm, c_int(src[7]), *gate, ptr(deq[0]), ptr(deq[1]), c_int(deq[2]), ptr(deq[3]), ptr(deq[4]), ptr(out), ptr(st.status), opt)
             self.launches += 2 if deq[0] is not None else 1
             if not any_short:
                 return out
@@ -485,15 +504,16 @@ class CudaOps(OpTrace):
         # verified rows must reproduce single-row decoding bit for bit -- uses it as well.  FP8 pages and other shapes keep the
         # per-row kernel.  PS_ATTN_DECODE=legacy switches it off.
         if (self.attn_decode_tc and D % 64 == 0 and st.kv_fmt == 0 and st.sc.page_tokens in (16, 32, 64) and hq // hkv <= 8
+                and not (kv.k is kv.v and (spec.bias is not None or spec.temp_coef != 0.0))
                 and (b.graph_static or row_pos is b.row_pos_short or all(len(sq.token_ids) <= 16 for sq in b.seqs))):
             st_tok = -(-split_tokens // 64) * 64
             n_seqs = b.max_seqs if b.graph_static else b.n_seqs
             _lib.call("ps_attn_decode_tc_ex", ptr(q), c_int(q.shape[0]), ptr(kv.k), ptr(kv.v), ptr(st.block_table),
                       c_int(st.max_blocks), c_int(st.sc.page_tokens), c_int(st.num_pages), ptr(b.seq_desc), c_int(n_seqs),
                       c_int(16), c_int(hq), c_int(hkv), c_int(D), sm, c_int(st_tok), c_int(self.max_splits),
-                      c_int(max_visible), ptr(pacc), ptr(pml), ptr(st.status), chunk)
+                      c_int(max_visible), ptr(pacc), ptr(pml), ptr(st.status), opt)
             _lib.call("ps_paged_attention_merge_ex", ptr(pacc), ptr(pml), ptr(row_pos), c_int(rows), c_int(hq), c_int(D),
-                      c_int(st_tok), c_int(self.max_splits), *gate, ptr(out), chunk, sink)
+                      c_int(st_tok), c_int(self.max_splits), *gate, ptr(out), opt, c_int(0))
             self.launches += 2
             return out
         if st.kv_fmt == 2:
@@ -509,8 +529,18 @@ class CudaOps(OpTrace):
                   ptr(st.block_table), c_int(st.max_blocks), c_int(st.sc.page_tokens), c_int(st.num_pages),
                   ptr(b.row_slot), ptr(row_pos), c_int(rows), c_int(hq), c_int(hkv), c_int(D),
                   sm, c_int(1 if st.kv_fp8 else 0), c_int(split_tokens), c_int(self.max_splits), c_int(max_visible),
-                  ptr(pacc), ptr(pml), *gate, ptr(out), ptr(st.status), chunk, sink)
+                  ptr(pacc), ptr(pml), *gate, ptr(out), ptr(st.status), opt)
         self.launches += 2
+        return out
+
+    def _attn_rows(self, q, spec: AttnSpec, b: StepBatch, kv: KVLayer, st: ModelState, out: torch.Tensor, gate) -> torch.Tensor:
+        """One CTA per row and head, any head size, bf16 or 32-bit."""
+        opts = AttnOptions.of(spec)
+        _lib.call("ps_attn_rows", ptr(q), ptr(kv.k), ptr(kv.v), c_int(1 if self.act_dtype == torch.float32 else 0),
+                  ptr(st.block_table), c_int(st.max_blocks), c_int(st.sc.page_tokens), c_int(st.num_pages), ptr(b.row_slot),
+                  ptr(b.row_pos), c_int(q.shape[0]), c_int(spec.heads), c_int(spec.kv_heads), c_int(spec.dim), c_float(spec.scale),
+                  ctypes.byref(opts), *gate, ptr(out), ptr(st.status))
+        self.launches += 1
         return out
 
     def _attn_scratch(self, pages: int, hkv: int, pt: int, D: int, max_seqs: int, max_blocks: int):
@@ -649,15 +679,158 @@ class CudaOps(OpTrace):
         self.launches += 1
         return (xo if changed else x), h
 
-    # ------------------------------------------------------------------ attention without rotation: query copy + key append
-    def attn_append(self, proj: torch.Tensor, spec: AttnSpec, b: StepBatch, kv: KVLayer, st: ModelState) -> torch.Tensor:
+    # ------------------------------------------------------------------ parallel residual streams
+    def stream_norm(self, x: torch.Tensor, pend: Optional[StreamWrite], *, read: Optional[torch.Tensor] = None,
+                    norm_w: Optional[torch.Tensor] = None, eps: float, width: int = 0, name: str = "", last: bool = False):
+        """Write what is pending into the fp32 streams `x` [rows, streams, W], read the next sublayer's input from them and norm it
+        for the next projection (`width` columns, zero-padded).  One launch.  Returns (streams, normed rows or None); the
+        streams live in one buffer of their own.  ``last``: they are not needed again."""
+        rows, S, W = x.shape
+        xo = None
+        if pend is not None and not last:
+            xo = self.buf("x_streams", rows, S * W, torch.float32).view(rows, S, W)
+        h = self.buf(name, rows, width, self.act_dtype) if norm_w is not None else None
+        if xo is None and h is None:
+            return x, None
+        mix, out, y = (pend.mix, pend.out, pend.y) if pend is not None else (None, None, None)
+        _lib.call("ps_stream_norm", ptr(x), c_ll(x.stride(0)), c_ll(x.stride(1)), ptr(xo), c_int(rows), c_int(W), c_int(S), ptr(mix), ptr(out),
+                  ptr(y), c_int(y.stride(0) if y is not None else 0), ptr(read), ptr(norm_w), c_float(eps), ptr(h),
+                  c_int(1 if self.act_dtype == torch.float32 else 0), c_int(width))
+        self.launches += 1
+        return (xo if xo is not None else x), h
+
+    # ------------------------------------------------------------------ attention without rotation: query copy + key / value append
+    def attn_append(self, proj: torch.Tensor, spec: AttnSpec, b: StepBatch, kv: Optional[KVLayer], st: ModelState) -> torch.Tensor:
+        """``kv`` None: the layer reads another one's keys, only the queries are copied."""
         rows = proj.shape[0]
         q = self.buf(f"attn_q{spec.heads}x{spec.dim}", rows, spec.heads * spec.dim, self.act_dtype)
+        k = kv.k if kv is not None else None
+        v = kv.v if kv is not None and kv.v is not kv.k else None
         _lib.call("ps_attn_append", ptr(proj), c_int(proj.stride(0)), c_int(proj.element_size()), c_int(rows), c_int(spec.heads),
-                  c_int(spec.kv_heads), c_int(spec.dim), ptr(b.row_slot), ptr(b.row_pos), ptr(q), ptr(kv.k), ptr(st.block_table),
-                  c_int(st.max_blocks), c_int(st.sc.page_tokens), c_int(st.num_pages), ptr(st.status))
+                  c_int(spec.kv_heads if kv is not None else 0), c_int(spec.dim), ptr(b.row_slot), ptr(b.row_pos), ptr(q), ptr(k), ptr(v),
+                  ptr(st.block_table), c_int(st.max_blocks), c_int(st.sc.page_tokens), c_int(st.num_pages), ptr(st.status))
         self.launches += 1
         return q
+
+    # ------------------------------------------------------------------ latent attention
+    def latent_down(self, proj: torch.Tensor, s: LatentSpec, b: StepBatch, kv: KVLayer, st: ModelState) -> torch.Tensor:
+        """Norm both latents of the projection rows, turn the shared key part, append; returns the query latents."""
+        rows = proj.shape[0]
+        cq = self.buf(f"latent_cq{s.q_rank}", rows, s.q_rank, self.act_dtype)
+        _lib.call("ps_latent_down", ptr(proj), c_int(proj.stride(0)), c_int(1 if self.act_dtype == torch.float32 else 0), c_int(rows),
+                  c_int(s.q_rank), c_int(s.kv_rank), c_int(s.rot), c_int(s.q_rank_true), c_int(s.kv_rank_true), c_int(s.rot_true // 2),
+                  ptr(s.q_norm), ptr(s.kv_norm), c_float(s.eps), ptr(s.inv_freq), ptr(cq), ptr(kv.k), ptr(b.row_slot), ptr(b.row_pos),
+                  ptr(st.block_table), c_int(st.max_blocks), c_int(st.sc.page_tokens), c_int(st.num_pages), ptr(st.status))
+        self.launches += 1
+        return cq
+
+    def _latent_turn(self, q, head: int, off: int, out, ohead: int, ooff: int, s: LatentSpec, b: StepBatch) -> None:
+        _lib.call("ps_latent_turn", ptr(q), c_int(q.stride(0)), c_int(head), c_int(off), ptr(out), c_int(out.stride(0)), c_int(ohead),
+                  c_int(ooff), c_int(1 if q.dtype == torch.float32 else 0), c_int(q.shape[0]), c_int(s.heads), c_int(s.rot),
+                  c_int(s.rot_true // 2), ptr(s.inv_freq), ptr(b.row_pos))
+        self.launches += 1
+
+    def _gemm_heads(self, x, x_head: int, w, heads: int, N: int, K: int, out, o_head: int, gate=None, g_head: int = 0) -> None:
+        """out[:, h] = x[:, h] w[h]^T (* sigmoid(gate[:, h])); `x_head` / `o_head` / `g_head`: columns between heads."""
+        M, ldg = x.shape[0], gate.stride(0) if gate is not None else 0
+        if self.act_dtype == torch.float32:
+            _lib.call("ps_gemm_f32_batched", ptr(x), c_int(x.stride(0)), c_ll(x_head), ptr(w), c_int(K), c_ll(N * K), c_int(heads), c_int(M),
+                      c_int(N), c_int(K), ptr(gate), c_int(ldg), c_ll(g_head), ptr(out), c_int(out.stride(0)), c_ll(o_head))
+        else:
+            _lib.call("ps_gemm_heads", ptr(x), c_int(x.stride(0)), c_int(x_head), ptr(w), c_int(heads), c_int(M), c_int(N), c_int(K),
+                      ptr(gate), c_int(ldg), c_int(g_head), ptr(out), c_int(out.stride(0)), c_int(o_head), ptr(self.status))
+        self.launches += 1
+
+    def latent_attention(self, q: torch.Tensor, s: LatentSpec, b: StepBatch, kv: KVLayer, st: ModelState, gate: torch.Tensor) -> torch.Tensor:
+        """Attention of query rows [rows, heads * (dim + rot)] (not turned yet; turned in place) over the cached latents, values back
+        in the heads and gated with the projection rows `gate`.  Sequences with many rows in the step attend over expanded keys
+        and values, the others in the latent space."""
+        rows, H, T = q.shape[0], s.heads, self.ATTN_PREFILL_MIN_ROWS
+        out = self.buf(f"latent_ctx{H}x{s.vdim}", rows, H * s.vdim, self.act_dtype)
+        L = _lib.lib()
+        long = []
+        if (self.act_dtype == torch.bfloat16 and not self.exact_rows and not b.graph_static and T == StepBatch.SHORT_SEQ_ROWS
+                and L.ps_latent_prefill_ok(c_int(s.dim), c_int(s.rot), c_int(s.vdim))):
+            long = [sq for sq in b.seqs if len(sq.token_ids) > T]
+        if not long or any(len(sq.token_ids) <= T for sq in b.seqs):
+            self._latent_absorbed(q, s, b, kv, st, gate, out, short_only=bool(long))
+        if long:
+            self._latent_expanded(q, s, b, kv, st, gate, out, long)
+        return out
+
+    def _latent_absorbed(self, q, s: LatentSpec, b: StepBatch, kv: KVLayer, st: ModelState, gate, out, short_only: bool) -> None:
+        """Queries into the latent space, attention with the cached rows as the keys and values of all heads, outputs back to the
+        heads with the gate.  ``short_only``: the rows of longer sequences come later and overwrite what this leaves there."""
+        rows, H, L = q.shape[0], s.heads, _lib.lib()
+        spec = s.shared_keys()
+        qe = self.buf(f"latent_qe{H}x{s.row}", rows, H * s.row, self.act_dtype)
+        self._gemm_heads(q, s.dim + s.rot, s.uk_t, H, s.kv_rank, s.dim, qe, s.row)
+        self._latent_turn(q, s.dim + s.rot, s.dim, qe, s.row, s.kv_rank, s, b)
+        pt = st.sc.page_tokens
+        tc = (self.act_dtype == torch.bfloat16 and self.attn_decode_tc and bool(L.ps_latent_decode_ok(c_int(s.kv_rank), c_int(s.rot), c_int(pt)))
+              and (short_only or b.graph_static or all(len(sq.token_ids) <= 16 for sq in b.seqs)))
+        if tc:
+            o, head = self._latent_decode(qe, s, spec, b, kv, st, b.row_pos_short if short_only else b.row_pos), s.kv_rank
+        else:
+            o, head = self.buf(f"latent_or{H}x{s.row}", rows, H * s.row, self.act_dtype), s.row
+            self._attn_rows(qe, spec, b, kv, st, o, (ptr(None), c_int(0), c_int(0), c_int(0)))
+        self._gemm_heads(o, head, s.uv, H, s.vdim, s.kv_rank, out, s.vdim, gate[:, s.gate_off:], s.vdim)
+
+    def _latent_decode(self, qe, s: LatentSpec, spec: AttnSpec, b: StepBatch, kv: KVLayer, st: ModelState, row_pos) -> torch.Tensor:
+        """Split-KV pass and merge.  The split length is a function of the step's row bucket and of the longest reach of a row
+        (the window, or the engine's longest context), so buffers and captured graphs stay valid."""
+        rows, H, L = qe.shape[0], s.heads, _lib.lib()
+        if b.graph_static:
+            n_seqs, seq_rows = b.max_seqs, b.max_rows if b.max_rows <= 16 else 1        # larger captured steps are pure decode batches
+        else:
+            n_seqs, seq_rows = b.n_seqs, max(n for n in (len(sq.token_ids) for sq in b.seqs) if n <= 16)
+        reach = min(s.window, b.max_context) if s.window > 0 else b.max_context
+        ctas = b.max_seqs * L.ps_latent_decode_ctas(c_int(H), c_int(s.kv_rank), c_int(1))
+        split = max(64, -(-reach // max(1, 296 // ctas) // 64) * 64)
+        while -(-(reach + 80) // split) + 1 > 512:
+            split *= 2
+        ring = -(-(reach + 80) // split) + 1                 # a tile of up to 16 rows, from the tile of its first visible token on
+        pacc = self.buf(f"latent_acc{H}x{s.kv_rank}x{ring}", rows, H * ring * s.kv_rank, torch.float32)
+        pml = self.buf(f"latent_ml{H}x{ring}", rows, H * ring * 2, torch.float32)
+        out = self.buf(f"latent_o{H}x{s.kv_rank}", rows, H * s.kv_rank)
+        opts = AttnOptions.of(spec)
+        _lib.call("ps_latent_decode", ptr(qe), c_int(rows), ptr(kv.k), ptr(st.block_table), c_int(st.max_blocks), c_int(st.sc.page_tokens),
+                  c_int(st.num_pages), ptr(b.seq_desc), c_int(n_seqs), c_int(seq_rows), c_int(H), c_int(s.kv_rank), c_int(s.rot),
+                  c_float(s.scale), c_int(split), c_int(ring), c_int(ring), ctypes.byref(opts), ptr(pacc), ptr(pml), ptr(st.status))
+        _lib.call("ps_paged_attention_merge_ex", ptr(pacc), ptr(pml), ptr(row_pos), c_int(rows), c_int(H), c_int(s.kv_rank), c_int(split),
+                  c_int(ring), ptr(None), c_int(0), c_int(0), c_int(0), ptr(out), ctypes.byref(opts), c_int(ring))
+        self.launches += 2
+        return out
+
+    def _latent_expanded(self, q, s: LatentSpec, b: StepBatch, kv: KVLayer, st: ModelState, gate, out, long) -> None:
+        """The tokens that the long sequences see, gathered into consecutive rows and expanded to keys and values per head."""
+        H, T, L = s.heads, self.ATTN_PREFILL_MIN_ROWS, _lib.lib()
+        spec = s.shared_keys()
+        tile = int(L.ps_latent_tile())
+        n = sum(-(-(sq.pos_start + len(sq.token_ids) - spec.first_visible(sq.pos_start) // tile * tile) // tile) * tile for sq in long)
+        lat, rot, exp = self._latent_scratch(n, s)
+        opts = AttnOptions.of(spec)
+        _lib.call("ps_latent_gather", ptr(kv.k), c_int(s.kv_rank), c_int(s.rot), ptr(st.block_table), c_int(st.max_blocks),
+                  c_int(st.sc.page_tokens), c_int(st.num_pages), ptr(b.seq_desc), c_int(b.n_seqs), c_int(T), ctypes.byref(opts), c_int(n),
+                  ptr(lat), ptr(rot), ptr(st.status))
+        N = s.ukv.shape[0]
+        _lib.call("ps_gemm_bf16_tc", ptr(lat), c_int(s.kv_rank), ptr(s.ukv), c_int(s.kv_rank), c_int(n), c_int(N), c_int(s.kv_rank),
+                  c_int(EPI_STORE), ptr(None), c_int(0), ptr(exp), c_int(N), c_int(0), ptr(self.status))
+        self.launches += 2
+        self._latent_turn(q, s.dim + s.rot, s.dim, q, s.dim + s.rot, s.dim, s, b)
+        g = gate[:, s.gate_off:]
+        _lib.call("ps_latent_prefill", ptr(q), c_int(q.shape[0]), ptr(exp), ptr(rot), c_int(n), ptr(b.seq_desc), c_int(b.n_seqs),
+                  c_int(max(len(sq.token_ids) for sq in long)), c_int(T), c_int(H), c_int(s.dim), c_int(s.rot), c_int(s.vdim), c_float(s.scale),
+                  ctypes.byref(opts), ptr(g), c_int(g.stride(0)), c_int(s.vdim), c_int(0), ptr(out), ptr(st.status))
+        self.launches += 1
+
+    def _latent_scratch(self, n: int, s: LatentSpec):
+        """bf16 scratch of the expanded form (latents, rotated parts, keys and values); one allocation that grows to the largest step seen."""
+        sizes = [n * s.kv_rank, n * s.rot, n * s.ukv.shape[0]]
+        t = getattr(self, "_latent_buf", None)
+        if t is None or t.numel() < sum(sizes):
+            t = self._latent_buf = torch.empty(sum(sizes), dtype=torch.bfloat16, device=self.device)
+        return torch.split(t[:sum(sizes)], sizes)
 
     # ------------------------------------------------------------------ gated linear attention
     def gla(self, proj: torch.Tensor, g: GlaSpec, b: StepBatch, gs: GdnLayerState, st: ModelState) -> torch.Tensor:
