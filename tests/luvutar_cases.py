@@ -37,8 +37,8 @@ WIDE = model(520, 192, 4, [latent(6, 128, 64, 128, 96, 512, 150, 160), attention
                            attention(6, 2, 128, 128, 64, 100, 0.7, 16, kv_from=1), latent(20, 64, 64, 64, 64, 256, 64, 128),
                            attention(8, 1, 256, 256, 128, scale=0.05)])
 # one of everything: one stream, one head, a window of the position itself, two buckets, a temperature step at every position
-UNIT = model(64, 64, 1, [latent(1, 32, 2, 32, 32, 32, 1, 64, scale=1.0), attention(1, 1, 32, 32, 64, bias_max=2, coef=1.0, every=1, scale=1.0),
-                         attention(1, 1, 32, 32, None, bias_max=2, every=1, kv_from=1)])
+UNIT = model(64, 64, 1, [latent(1, 32, 2, 32, 32, 32, 1, 64, scale=1.0), attention(1, 1, 32, 32, 64, bias_max=2, coef=1.0, every=1, scale=0.05),
+                         attention(1, 1, 32, 32, None, bias_max=2, every=1, scale=0.05, kv_from=1)])
 # sizes beyond the tiled kernels: many streams, a wide latent, wide heads, many query heads on one key head, several row tiles
 TAIL = model(200, 128, 5, [latent(2, 200, 40, 72, 48, 600, 90, 100), attention(16, 1, 32, 32, None, bias_max=200),
                            attention(2, 2, 288, 264, 96, every=50), latent(40, 16, 16, 16, 40, 64, 300, 128),
