@@ -55,9 +55,10 @@ def _parse():
     ap.add_argument("--serving-slots", type=int, default=32,
                     help="sequence slots of the serving block (fewer than the requests, so that later admissions can hit "
                          "the prefix cache the earlier ones filled)")
-    ap.add_argument("--compare", default="", choices=["", "gebuzen"],
-                    help="instead of the headline workload: prefill and decode of a model family beside the hybrid decoder at equal "
-                         "layer shapes (random bf16 weights, 1 GPU), and the mixers' kernels against their rooflines")
+    ap.add_argument("--compare", default="", choices=["", "gebuzen", "luvutar"],
+                    help="instead of the headline workload: prefill and decode of a model family beside the closest other one (Gebuzen: the "
+                         "hybrid decoder; Luvutar: Gebuzen) at equal layer shapes (random bf16 weights, 1 GPU), and the mixers' kernels "
+                         "against their rooflines")
     ap.add_argument("--compare-layers", type=int, default=16)
     ap.add_argument("--watchdog", type=int, default=1500,
                     help="seconds after which a hung run dumps every thread's stack to stderr and exits")
@@ -374,7 +375,8 @@ def compare_arm(args):
     except Exception:
         pass
     sampler = ClockSampler(0)
-    res = compare_bench.run(peaks, layers=args.compare_layers, warmup=max(3, args.warmup // 2), sampler=sampler)
+    res = compare_bench.run(peaks, layers=args.compare_layers, warmup=max(3, args.warmup // 2), sampler=sampler,
+                            which=args.compare)
     print(json.dumps({"compare": args.compare, **res, "clocks": sampler.stop(), "dtype": "bf16",
                       "data": "synthetic (random-init weights, uniform-random prompt ids)"}), flush=True)
     return 0

@@ -1,5 +1,6 @@
-"""Throughput of a model family beside the hybrid decoder at equal size (`bench.py --compare gebuzen`): prefill and decode of a
-stack of layers of real-model shapes with random bf16 weights, and the mixers' kernels alone against their rooflines.
+"""Throughput of a model family beside the closest other one at equal size (`bench.py --compare gebuzen`: the hybrid decoder;
+`--compare luvutar`: Gebuzen): prefill and decode of a stack of layers of real-model shapes with random bf16 weights, and the
+mixers' kernels alone against their rooflines.
 
 Every kernel row gives its time, the algorithmic bytes and FLOPs of one launch group, and the fraction of the roofline
 max(bytes / measured copy bandwidth, FLOPs / measured bf16 throughput) it reaches.  Kernel timings flush L2 between samples.
@@ -17,7 +18,28 @@ from ..runtime.engine import Engine
 from ..runtime.state import StateConfig
 
 
-def size_pairs(layers: int) -> List[tuple]:
+def luvutar_pairs(layers: int) -> List[tuple]:
+    """(label, Luvutar configuration, Gebuzen configuration) of equal width, attention heads, feed-forward weights and depth."""
+    from ..models.gebuzen.config import gebuzen_27b_config, gebuzen_4b_config
+    from ..models.luvutar.config import BiasedAttention, LatentAttention, Layer, luvutar_27b_config, luvutar_4b_config
+
+    def cut(cfg):
+        cfg.layers = cfg.layers[:layers]
+        return cfg
+
+    def narrow(m):
+        """Half the head size, twice the heads; a latent half as wide."""
+        if isinstance(m, LatentAttention):
+            return LatentAttention(40, 64, 32, 64, 768, 256, 96 ** -0.5, m.rot_base, m.window)
+        return BiasedAttention(32, 8, 128, 128, 128 ** -0.5, m.bias_max, m.temp_coef, m.temp_every, m.kv_from)
+
+    small = cut(luvutar_4b_config(name="luvutar-4b-d128"))
+    small.layers = [Layer(narrow(L.mixer), L.ff) for L in small.layers]
+    return [("4b", cut(luvutar_4b_config()), cut(gebuzen_4b_config())), ("4b, attention heads of 128, latents of 256", small, None),
+            ("27b", cut(luvutar_27b_config()), cut(gebuzen_27b_config()))]
+
+
+def gebuzen_pairs(layers: int) -> List[tuple]:
     """(label, Gebuzen configuration, hybrid configuration) of equal width, head and feed-forward shapes and depth."""
     from ..models.gebuzen.config import ChunkAttention, ParallelLayer, gebuzen_27b_config, gebuzen_4b_config
     from ..models.qwen35.config import qwen35_27b_config, qwen35_4b_config
@@ -187,13 +209,92 @@ def kernel_times(eng: Engine, timer: _Flushed, peaks: dict, rows: int, context: 
     return res
 
 
-def run(peaks: dict, layers: int = 16, prompt_tokens: int = 2048, steps: int = 50, warmup: int = 3, batch: int = 32, sampler=None) -> dict:
+def luvutar_kernel_times(eng: Engine, timer: _Flushed, peaks: dict, rows: int, context: int, batch: int) -> Dict[str, dict]:
+    """As `kernel_times`, for the parts of both mixers and the residual streams."""
+    from ..ops.specs import LatentSpec, StreamWrite
+    hbm, tc = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    ops, st, w = eng.ops, eng.state, eng.runner.w
+    res: Dict[str, dict] = {}
+
+    def add(name, fn, nbytes, flops):
+        us = timer(fn)
+        floor = max(nbytes / hbm, flops / tc) * 1e6
+        res[name] = {"us": round(us, 1), "gb": round(nbytes / 1e9, 4), "gflop": round(flops / 1e9, 2), "roofline_us": round(floor, 2),
+                     "roofline_frac": round(floor / us, 4)}
+
+    def rand(n, width, dtype=torch.bfloat16):
+        return torch.randn(n, width, device=eng.device, dtype=torch.float32).to(dtype)
+
+    la = next(i for i, L in enumerate(w.layers) if isinstance(L.attn, LatentSpec))
+    lb = next(i for i, L in enumerate(w.layers) if not isinstance(L.attn, LatentSpec))
+    A, B = w.layers[la], w.layers[lb]
+    s, f = A.attn, B.attn
+    S, W = eng.cfg.streams, eng.cfg.hidden_size
+    shapes = [("prefill", [(0, rows)]), ("prefill after context", [(context, rows)]), ("decode 1", [(context, 1)]),
+              (f"decode {batch}", [(context, 1)] * batch)]
+    for name, seqs in shapes:
+        b, opened = _batch(eng, seqs)
+        n = b.n_rows
+        vis = [(p, k) for p, k in seqs]
+        full = sum(q + 1 for p, k in vis for q in range(p, p + k))
+        win = sum(min(q + 1, s.window) for p, k in vis for q in range(p, p + k))
+        kv_full = sum(p + k for p, k in vis)
+        kv_win = sum(p + k - max(0, p - s.window + 1) for p, k in vis)
+        qkv = rand(n, B.in_proj.N)
+        q = ops.attn_append(qkv, f, b, st.kv[lb], st)
+        add("attention, " + name, lambda: ops.attention(q, f, b, st.kv[lb], st, b.max_visible_launch, gate=qkv),
+            2 * n * f.heads * f.dim * 2 + kv_full * 2 * f.kv_heads * f.dim * 2, 4.0 * full * f.heads * f.dim)
+        proj = rand(n, A.in_proj.N)
+        add("latents, " + name, lambda: ops.latent_down(proj, s, b, st.kv[la], st), n * (2 * s.q_rank + 2 * s.row) * 2, 0.0)
+        lq = rand(n, A.uq.N)
+        H = s.heads
+        io = n * H * (s.dim + s.rot + 2 * s.vdim) * 2
+        if name.startswith("prefill"):
+            # keys and values are products of the latents of every visible token
+            flops = 2.0 * win * H * (s.dim + s.rot + s.vdim) + 2.0 * kv_win * s.ukv.numel()
+            add("latent attention, " + name, lambda: ops.latent_attention(lq, s, b, st.kv[la], st, proj), io + kv_win * s.row * 2, flops)
+            add("latent attention core, " + name, _prefill_core(ops, lq, s, b, st, st.kv[la], proj),
+                io + kv_win * (H * (s.dim + s.vdim) + s.rot) * 2, 2.0 * win * H * (s.dim + s.rot + s.vdim))
+        else:
+            weights = (s.uk_t.numel() + s.uv.numel()) * 2
+            add("latent attention, " + name, lambda: ops.latent_attention(lq, s, b, st.kv[la], st, proj), io + kv_win * s.row * 2 + weights,
+                2.0 * win * H * (s.row + s.kv_rank) + 2.0 * n * weights / 2)
+            qe = rand(n, H * s.row)
+            add("latent attention core, " + name, lambda: ops._latent_decode(qe, s, s.shared_keys(), b, st.kv[la], st, b.row_pos),
+                n * H * (s.row + s.kv_rank) * 2 + kv_win * s.row * 2, 2.0 * win * H * (s.row + s.kv_rank))
+            add("queries into the latent space, " + name,
+                lambda: ops._gemm_heads(lq, s.dim + s.rot, s.uk_t, H, s.kv_rank, s.dim, qe, s.row), s.uk_t.numel() * 2 + n * H * (s.dim + s.kv_rank) * 2,
+                2.0 * n * s.uk_t.numel())
+        if name != "prefill after context":
+            x, y = rand(n, S * W, torch.float32).view(n, S, W), rand(n, W, torch.float32)
+            hc = A.hc2
+            pend = StreamWrite(A.hc1.mix, A.hc1.out, y)
+            add("streams + norm, " + name, lambda: ops.stream_norm(x, pend, read=hc.read, norm_w=hc.norm, eps=1e-6, width=A.up.K, name="bench_h"),
+                n * W * (8 * S + 4 + 2), 0.0)
+            xg = rand(n, A.up.K)
+            add("up, " + name, lambda: ops.linear(xg, A.up, name="bench_act", gelu=True),
+                A.up.N * A.up.k_padded * 2 + n * (A.up.K + A.up.N) * 2, 2.0 * n * A.up.N * A.up.K)
+        for o in opened:
+            eng.close_sequence(o)
+    return res
+
+
+def _prefill_core(ops, q, s, b, st, kv, gate):
+    """The attention over keys and values that one call of `latent_attention` has gathered and expanded."""
+    out = ops.latent_attention(q, s, b, kv, st, gate)
+    long = list(b.seqs)
+    lat, rot, exp = ops._latent_scratch(ops.latent_rows(s, long), s)
+    return lambda: ops._latent_prefill(q, s, b, st, gate, out, rot, exp, long)
+
+
+def run(peaks: dict, layers: int = 16, prompt_tokens: int = 2048, steps: int = 50, warmup: int = 3, batch: int = 32, sampler=None,
+        which: str = "gebuzen") -> dict:
     dev = torch.device("cuda:0")
     timer = _Flushed(dev)
     out = {"layers": layers, "prompt_tokens": prompt_tokens, "batch": batch, "sizes": {}}
-    for label, gz, hy in size_pairs(layers):
+    for label, *cfgs in (luvutar_pairs if which == "luvutar" else gebuzen_pairs)(layers):
         row = out["sizes"][label] = {}
-        for name, cfg in (("gebuzen", gz), ("hybrid", hy)):
+        for name, cfg in zip(("luvutar", "gebuzen") if which == "luvutar" else ("gebuzen", "hybrid"), cfgs):
             if cfg is None:
                 continue
             with torch.no_grad():
@@ -204,7 +305,7 @@ def run(peaks: dict, layers: int = 16, prompt_tokens: int = 2048, steps: int = 5
                 if sampler is not None:
                     sampler.begin()
                 t = model_times(eng, prompt_tokens, steps, warmup, batch)
-                k = kernel_times(eng, timer, peaks, prompt_tokens, prompt_tokens, batch)
+                k = (luvutar_kernel_times if name == "luvutar" else kernel_times)(eng, timer, peaks, prompt_tokens, prompt_tokens, batch)
             rd = ew.decode_read_bytes()
             row[name] = {**{a: round(v, 4) for a, v in t.items()},
                          "prefill_tok_s": round(prompt_tokens / t["prefill_ms"] * 1e3), "decode1_tok_s": round(1e3 / t["decode1_ms"], 1),

@@ -7,14 +7,9 @@
 // consecutive rows, one GEMM expands them, and ps_latent_prefill attends over the result on the tensor cores (attn_tc.cuh).
 // Rows of short sequences attend in the latent space instead (attn_latent_decode.cu).
 #include "attn_tc.cuh"
+#include "turn_angle.cuh"
 
 namespace ps {
-
-// sine and cosine of pos * freq: the angle is reduced to one turn in double precision
-__device__ __forceinline__ void turn_angle(int pos, double freq, float* s, float* c) {
-    const double a = (double)pos * freq;
-    sincosf((float)(a - 6.283185307179586 * rint(a * 0.15915494309189535)), s, c);
-}
 
 template <typename T> __device__ __forceinline__ T la_cast(float v);
 template <> __device__ __forceinline__ float la_cast<float>(float v) { return v; }
@@ -29,7 +24,21 @@ struct LatentDownArgs {
     uint32_t* status;
 };
 
-// one CTA per row
+// four elements at once (16- or 8-byte accesses)
+__device__ __forceinline__ float4 la_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 la_load4(const __nv_bfloat16* p) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    const float2 a = bf16x2_bits_to_f32x2(v.x), b = bf16x2_bits_to_f32x2(v.y);
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void la_store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void la_store4(__nv_bfloat16* p, float4 v) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(f32x2_to_bf16x2_bits(v.x, v.y), f32x2_to_bf16x2_bits(v.z, v.w));
+}
+__device__ __forceinline__ float la_sq4(float4 v) { return fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w))); }
+__device__ __forceinline__ float4 la_scale4(float4 v, float s, float4 w) { return make_float4(v.x * s * w.x, v.y * s * w.y, v.z * s * w.z, v.w * s * w.w); }
+
+// one CTA per row; QR, KR, R and the row pitch are multiples of 4
 template <typename T>
 __global__ void __launch_bounds__(256) latent_down_kernel(const LatentDownArgs a) {
     __shared__ float red[64];
@@ -39,21 +48,21 @@ __global__ void __launch_bounds__(256) latent_down_kernel(const LatentDownArgs a
     const T* src = reinterpret_cast<const T*>(a.proj) + (size_t)row * a.ld;
     const T* lat = src + a.QR;
     const T* rot = lat + a.KR;
+    const int slot = a.row_slot[row], pos = a.row_pos[row], blk = pos / a.page_tokens;
+    const bool real = slot >= 0 && pos >= 0;                                      // (not a padding row)
+    const int page = real && blk < a.max_blocks ? a.block_table[(size_t)slot * a.max_blocks + blk] : -1;
     float ss[2] = {0.f, 0.f};
-    for (int i = t; i < a.QR; i += n) { const float v = (float)src[i]; ss[0] = fmaf(v, v, ss[0]); }
-    for (int i = t; i < a.KR; i += n) { const float v = (float)lat[i]; ss[1] = fmaf(v, v, ss[1]); }
+    for (int i = 4 * t; i < a.QR; i += 4 * n) ss[0] += la_sq4(la_load4(src + i));
+    for (int i = 4 * t; i < a.KR; i += 4 * n) ss[1] += la_sq4(la_load4(lat + i));
     block_sum_n<2>(ss, red);
     const float iq = rsqrtf(ss[0] / (float)a.q_true + a.eps), ik = rsqrtf(ss[1] / (float)a.kv_true + a.eps);
     T* cq = reinterpret_cast<T*>(a.cq) + (size_t)row * a.QR;
-    for (int i = t; i < a.QR; i += n) cq[i] = la_cast<T>((float)src[i] * iq * a.q_norm[i]);
-    const int slot = a.row_slot[row], pos = a.row_pos[row];
-    if (slot < 0 || pos < 0) return;             // padding row
-    const int blk = pos / a.page_tokens;
-    const int page = blk < a.max_blocks ? a.block_table[(size_t)slot * a.max_blocks + blk] : -1;
+    for (int i = 4 * t; i < a.QR; i += 4 * n) la_store4(cq + i, la_scale4(la_load4(src + i), iq, *reinterpret_cast<const float4*>(a.q_norm + i)));
+    if (!real) return;
     if (page < 0 || page >= a.num_pages) { if (t == 0) set_status(a.status, PS_DEV_BAD_INDEX); return; }
     T* dst = reinterpret_cast<T*>(a.pool) + ((size_t)page * a.page_tokens + pos % a.page_tokens) * (a.KR + a.R);
-    for (int i = t; i < a.KR; i += n) dst[i] = la_cast<T>((float)lat[i] * ik * a.kv_norm[i]);
-    for (int i = t; i < a.R / 2; i += n) {
+    for (int i = 4 * t; i < a.KR; i += 4 * n) la_store4(dst + i, la_scale4(la_load4(lat + i), ik, *reinterpret_cast<const float4*>(a.kv_norm + i)));
+    for (int i = n - 1 - t; i < a.R / 2; i += n) {                                // from the last thread on: the first ones have the latents
         float u = (float)rot[2 * i], v = (float)rot[2 * i + 1];
         if (i < a.pairs) {
             float s, c;
@@ -84,13 +93,13 @@ __global__ void __launch_bounds__(256) latent_turn_kernel(const LatentTurnArgs a
         s_sin[i] = s; s_cos[i] = c;
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < a.H * half; i += blockDim.x) {
-        const int h = i / half, j = i % half;
-        const T* src = reinterpret_cast<const T*>(a.q) + (size_t)row * a.ld + (size_t)h * a.head + a.off + 2 * j;
-        T* dst = reinterpret_cast<T*>(a.out) + (size_t)row * a.ldo + (size_t)h * a.ohead + a.ooff + 2 * j;
-        const float u = (float)src[0], v = (float)src[1];
-        dst[0] = la_cast<T>(u * s_cos[j] - v * s_sin[j]);
-        dst[1] = la_cast<T>(v * s_cos[j] + u * s_sin[j]);
+    const int quads = half / 2;                                                   // two pairs at once
+    for (int i = threadIdx.x; i < a.H * quads; i += blockDim.x) {
+        const int h = i / quads, j = 2 * (i % quads);
+        const float4 x = la_load4(reinterpret_cast<const T*>(a.q) + (size_t)row * a.ld + (size_t)h * a.head + a.off + 2 * j);
+        la_store4(reinterpret_cast<T*>(a.out) + (size_t)row * a.ldo + (size_t)h * a.ohead + a.ooff + 2 * j,
+                  make_float4(x.x * s_cos[j] - x.y * s_sin[j], x.y * s_cos[j] + x.x * s_sin[j],
+                              x.z * s_cos[j + 1] - x.w * s_sin[j + 1], x.w * s_cos[j + 1] + x.z * s_sin[j + 1]));
     }
 }
 
@@ -149,7 +158,8 @@ PS_API int ps_latent_down(const void* proj, int ld, int f32, int rows, int QR, i
                           const void* row_slot, const void* row_pos, const void* block_table, int max_blocks, int page_tokens,
                           int num_pages, void* status, cudaStream_t stream) {
     using namespace ps;
-    if (rows <= 0 || QR <= 0 || KR <= 0 || R < 0 || (R & 1) || 2 * pairs > R || q_true <= 0 || kv_true <= 0 || ld < QR + KR + R)
+    if (rows <= 0 || QR <= 0 || KR <= 0 || R < 0 || ((QR | KR | R | ld) & 3) || 2 * pairs > R || q_true <= 0 || kv_true <= 0 || ld < QR + KR + R ||
+        (((uintptr_t)proj | (uintptr_t)cq | (uintptr_t)pool | (uintptr_t)q_norm | (uintptr_t)kv_norm) % 16))
         return (int)cudaErrorInvalidValue;
     LatentDownArgs a;
     a.proj = proj; a.ld = ld; a.QR = QR; a.KR = KR; a.R = R; a.q_true = q_true; a.kv_true = kv_true; a.pairs = pairs;
@@ -164,7 +174,9 @@ PS_API int ps_latent_down(const void* proj, int ld, int f32, int rows, int QR, i
 PS_API int ps_latent_turn(const void* q, int ld, int head, int off, void* out, int ldo, int ohead, int ooff, int f32, int rows, int H, int R,
                           int pairs, const void* inv_freq, const void* row_pos, cudaStream_t stream) {
     using namespace ps;
-    if (rows <= 0 || H <= 0 || R <= 0 || (R & 1) || R > 512 || 2 * pairs > R) return (int)cudaErrorInvalidValue;
+    if (rows <= 0 || H <= 0 || R <= 0 || R > 512 || 2 * pairs > R || ((R | ld | head | off | ldo | ohead | ooff) & 3) ||
+        (((uintptr_t)q | (uintptr_t)out) % 16))
+        return (int)cudaErrorInvalidValue;
     LatentTurnArgs a;
     a.q = q; a.ld = ld; a.head = head; a.off = off; a.out = out; a.ldo = ldo; a.ohead = ohead; a.ooff = ooff; a.H = H; a.R = R;
     a.pairs = pairs; a.inv_freq = (const double*)inv_freq; a.row_pos = (const int*)row_pos;

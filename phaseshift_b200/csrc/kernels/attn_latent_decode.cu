@@ -1,13 +1,14 @@
 // Latent attention for decode rows and short portions, in the latent space: all heads share the cached rows [latent | rotated
 // part] as keys, and the latent part as values (bf16 pool, one head per token, pages of 16, 32 or 64 tokens).
 //
-// One CTA = up to 128 (row, head) pairs of one sequence as one MMA tile -- tile row r * hp + g is head g of the CTA's row r --,
-// one KV split, and up to 256 of the value columns (tensor memory holds 128 score columns and 256 output columns; wider latents
+// One CTA = up to 128 (row, head) pairs of one sequence as one MMA tile -- tile row r * hp + g is head g of the CTA's row r; rows
+// beyond the used ones read whatever lies behind the queries in shared memory, and nobody reads their results --, one KV split, and up to 256 of the value columns (tensor memory holds 128 score columns and 256 output columns; wider latents
 // take two CTAs that both compute the scores):
 //
 //   warp 4   TMA producer: the queries once, then per tile of 64 tokens every 64-column group of the cached rows, once, into a
 //            ring of 8 KB stages (a group is one box per page).  The groups that are this CTA's values come last.
-//   warp 5   one thread issues S(t) += Q_g K_g^T group by group as they land (tcgen05.mma), two score accumulators; a group that
+//   warps 5, 7 one thread each issues S(t) += Q_g K_g^T group by group as they land (tcgen05.mma) into one of two score
+//            accumulators, warp 5 for even t and warp 7 for odd t (rings of fewer than two tiles: warp 5 for all); a group that
 //            is no value gives its stage back at once.
 //   warp 6   one thread issues O_g += P(t) V_g for the value groups, still in their stages (an MN-major operand), and gives these
 //            back.
@@ -21,14 +22,14 @@
 
 namespace ps {
 
-constexpr int kLdThreads = 224, kLdGroup = kTcTok * 64 * 2, kLdMaxStages = 12;
+constexpr int kLdThreads = 256, kLdGroup = kTcTok * 64 * 2, kLdMaxStages = 24;
 
 struct LatentDecodeArgs {
     const int* block_table; int max_blocks, num_pages, page_tokens;
     const int* seqs;             // [n_seqs][4] = row_start, n_rows, slot, pos_start
     int H, heads_per_tile, hp, rows_per_tile, row_tiles, head_tiles;
     int ng, krg;                 // 64-column groups of a cached row, of its latent
-    int stages;
+    int stages, q_group;         // stages of the ring; bytes of the queries' rows of one group
     float scale_log2; AttnOptions opt;
     int split_tokens, ring, max_rows;
     float* part_acc; float* part_ml;
@@ -63,8 +64,8 @@ attn_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
         if (threadIdx.x == 0) set_status(a.status, PS_DEV_BAD_INDEX);
         return;
     }
-    unsigned char* sQ = smem;                    // ng groups of 128 rows x 64 columns
-    unsigned char* sP = sQ + (size_t)ng * (kTcRows * 128);
+    unsigned char* sQ = smem;                    // ng groups of the used rows x 64 columns (the MMA reads 128 rows from each)
+    unsigned char* sP = sQ + (size_t)ng * a.q_group;
     unsigned char* sS = sP + kTcPBuf;
 
     if (threadIdx.x == 0) {
@@ -93,7 +94,7 @@ attn_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
         __syncwarp();
         for (int i = lane; i < n_box; i += 32) {
             const int g = i % ng, rb = i / ng, r = rb / blocks, b8 = rb % blocks;
-            tc::tma_load_2d(sQ + (size_t)g * (kTcRows * 128) + (r * a.hp + 8 * b8) * 128, &map_q, g * 64,
+            tc::tma_load_2d(sQ + (size_t)g * a.q_group + (r * a.hp + 8 * b8) * 128, &map_q, g * 64,
                             (row_start + r0 + r) * a.H + h0 + 8 * b8, &q_full);
         }
         if (lane == 0) q_issued = 1;
@@ -121,27 +122,30 @@ attn_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
                 if (lane == 0) s_issued = p + 1;
             }
         }
-    } else if (warp == 5) {
+    } else if (warp == 5 || warp == 7) {
         // ------------------------------------------------ scores
         if (lane == 0) {
             constexpr uint32_t idesc = tc::idesc_bf16_f32(kTcRows, kTcTok);
             const uint32_t q_addr = tc::smem_u32(sQ), s_addr = tc::smem_u32(sS);
-            bool ok = tc::mbar_wait_abortable(&q_full, 0, a.budget, &s_abort);
+            // A wait for a stage's next fill must not begin before its last one has landed (the parity would read as done).  A fill
+            // of tile t replaces one of tile t - 2 or earlier in a ring of two tiles, and P(t - 2) has been waited for; a smaller
+            // ring has one issuer, which takes the fills in order.
+            const int issuers = ns >= 2 * ng ? 2 : 1;
+            bool ok = (warp == 5 || issuers == 2) && tc::mbar_wait_abortable(&q_full, 0, a.budget, &s_abort);
             if (ok) q_consumed = 1;
-            int p = 0;
-            for (int t = 0; t < T && ok; ++t) {
+            for (int t = warp == 5 ? 0 : 1; t < T && ok; t += issuers) {
                 const int b = t & 1;
                 // the accumulator is free once the softmax warps have read S(t - 2), which they signal with P(t - 2)
                 if (t >= 2 && !tc::mbar_wait_abortable(&p_full[b], ((uint32_t)(t >> 1) & 1u) ^ 1u, a.budget, &s_abort)) break;
-                for (int i = 0; i < ng; ++i, ++p) {
-                    const int st = p % ns;
+                for (int i = 0; i < ng; ++i) {
+                    const int p = t * ng + i, st = p % ns;
                     const int g = i < 4 * vp ? i : i < ng - nv ? i + nv : 4 * vp + i - (ng - nv);
                     if (!tc::mbar_wait_abortable(&full[st], (uint32_t)(p / ns) & 1u, a.budget, &s_abort)) { ok = false; break; }
-                    s_consumed = p + 1;
+                    atomicMax(&s_consumed, p + 1);
                     tc::fence_after_sync();
 #pragma unroll
                     for (int kk = 0; kk < 4; ++kk)
-                        tc::mma_bf16_ss(tmem + b * kTcTok, tc::smem_desc_sw128(q_addr + g * (kTcRows * 128) + kk * 32),
+                        tc::mma_bf16_ss(tmem + b * kTcTok, tc::smem_desc_sw128(q_addr + g * a.q_group + kk * 32),
                                         tc::smem_desc_sw128(s_addr + st * kLdGroup + kk * 32), idesc, (i > 0 || kk > 0) ? 1u : 0u);
                     if (i < ng - nv) tc::mma_commit(&freed[st]);
                 }
@@ -296,8 +300,9 @@ attn_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
     }
 }
 
-static int latent_decode_stages(int ng) {
-    const int left = 227 * 1024 - 2048 - kTcPBuf - ng * kTcRows * 128;            // 2 KB for the static part
+// Stages beside `rows` query rows per group; the 2 KB are the static part.
+static int latent_decode_stages(int ng, int rows) {
+    const int left = 227 * 1024 - 2048 - kTcPBuf - ng * rows * 128;
     const int n = left / kLdGroup;
     return n > kLdMaxStages ? kLdMaxStages : n;
 }
@@ -307,7 +312,7 @@ static int latent_decode_stages(int ng) {
 // Whether a cached row of KR + R elements fits the kernel (queries and at least two free stages beside the value groups).
 PS_API int ps_latent_decode_ok(int KR, int R, int page_tokens) {
     return KR > 0 && R > 0 && KR % 64 == 0 && R % 64 == 0 && (page_tokens == 16 || page_tokens == 32 || page_tokens == 64) &&
-           ps::latent_decode_stages((KR + R) / 64) >= 6;
+           ps::latent_decode_stages((KR + R) / 64, ps::kTcRows) >= 6;
 }
 
 // CTAs of one split (value parts x head tiles x row tiles of `max_rows` rows) per sequence: what a caller sizes splits with.
@@ -335,16 +340,17 @@ PS_API int ps_latent_decode(const void* q, int q_rows, const void* pool, const v
     a.head_tiles = (H + kTcRows - 1) / kTcRows;
     a.heads_per_tile = (H + a.head_tiles - 1) / a.head_tiles;
     a.hp = (a.heads_per_tile + 7) / 8 * 8;
-    a.rows_per_tile = kTcRows / a.hp;
+    a.rows_per_tile = kTcRows / a.hp < max_rows ? kTcRows / a.hp : max_rows;
+    a.q_group = a.rows_per_tile * a.hp * 128;
     a.row_tiles = (max_rows + a.rows_per_tile - 1) / a.rows_per_tile;
-    a.ng = (KR + R) / 64; a.krg = KR / 64; a.stages = latent_decode_stages(a.ng);
+    a.ng = (KR + R) / 64; a.krg = KR / 64; a.stages = latent_decode_stages(a.ng, a.rows_per_tile * a.hp);
     a.scale_log2 = scale * 1.4426950408889634f; a.opt = opt; a.split_tokens = split_tokens; a.ring = ring; a.max_rows = max_rows;
     a.part_acc = (float*)part_acc; a.part_ml = (float*)part_ml; a.status = (uint32_t*)status; a.budget = g_ps_wait_budget_cycles;
     CUtensorMap mq, mkv;
     int err = attn_map_2d(&mq, q, (uint64_t)q_rows * H, (uint64_t)(KR + R), (uint64_t)(KR + R), 8);
     if (err) return err;
     if ((err = attn_map_2d(&mkv, pool, (uint64_t)num_pages * page_tokens, (uint64_t)(KR + R), (uint64_t)(KR + R), (uint32_t)page_tokens))) return err;
-    const size_t smem = (size_t)a.ng * kTcRows * 128 + kTcPBuf + (size_t)a.stages * kLdGroup;
+    const size_t smem = (size_t)a.ng * a.q_group + kTcPBuf + (size_t)a.stages * kLdGroup;
     static bool attr_set = false;
     if (!attr_set) {
         cudaFuncSetAttribute(attn_latent_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 225 * 1024);

@@ -5,7 +5,11 @@
 // the stages hold mostly weights.  One CTA per (128 weight rows, head, 64 rows); K (64 to 512 here) runs through a four-stage TMA
 // ring and the accumulator in tensor memory goes straight to the output, lane = weight row.  The weight tiles of the first stages
 // are requested before the predecessor kernel has finished (programmatic dependent launch).  Every wait is bounded.
+//
+// With `turn_r`, one more CTA per head and 64 rows copies the rotated part of x's head (behind its K columns) behind the head's
+// outputs, turned by the row's position, so that the latent queries leave this kernel complete.
 #include "ps_tcgen05.cuh"
+#include "turn_angle.cuh"
 
 namespace ps {
 
@@ -16,6 +20,7 @@ struct GemmHeadsArgs {
     int nb, box_rows;            // MMA N; rows of an x box
     __nv_bfloat16* out; int ldo, o_head;
     const __nv_bfloat16* gate; int ldg, g_head;
+    int turn_r, turn_pairs; const double* inv_freq; const int* row_pos; const __nv_bfloat16* x; int ldx;
     uint32_t* status; long long budget;
 };
 
@@ -33,6 +38,18 @@ gemm_heads_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_consta
     const int n0 = blockIdx.x * kGhM, h = blockIdx.y, m0 = blockIdx.z * kGhRows, iters = g.K / kGhK;
 
     cudaTriggerProgrammaticLaunchCompletion();
+    if (g.turn_r > 0 && blockIdx.x == gridDim.x - 1) {
+        cudaGridDependencySynchronize();
+        const int half = g.turn_r / 2;
+        for (int i = threadIdx.x; i < min(kGhRows, g.M - m0) * half; i += kGhThreads) {
+            const int m = m0 + i / half, j = i % half;
+            const float2 v = bf16x2_bits_to_f32x2(*reinterpret_cast<const uint32_t*>(g.x + (size_t)m * g.ldx + (size_t)h * g.x_head + g.K + 2 * j));
+            float s = 0.f, c = 1.f;
+            if (j < g.turn_pairs) turn_angle(max(g.row_pos[m], 0), g.inv_freq[j], &s, &c);
+            *reinterpret_cast<uint32_t*>(g.out + (size_t)m * g.ldo + (size_t)h * g.o_head + g.N + 2 * j) = f32x2_to_bf16x2_bits(v.x * c - v.y * s, v.y * c + v.x * s);
+        }
+        return;
+    }
     if (threadIdx.x == 0) {
         for (int s = 0; s < kGhStages; ++s) { tc::mbar_init(&full[s], 1); tc::mbar_init(&empty[s], 1); }
         tc::mbar_init(&acc_bar, 1);
@@ -148,11 +165,14 @@ static int gh_map_2d(CUtensorMap* map, const void* base, uint64_t rows, uint64_t
 }  // namespace ps
 
 // x [M, ldx] bf16, head h at column h * x_head; w [heads * N, K] bf16 row-major; out [M, ldo], head h at column h * o_head; gate
-// (optional) likewise.  K, x_head multiples of 64, ldx of 8, 16-byte aligned bases.
+// (optional) likewise.  K, x_head multiples of 64, ldx of 8, 16-byte aligned bases.  `turn_r` > 0 columns behind each head's K are
+// turned by the row's position (pairs of neighbours, `inv_freq` f64 radians per position) and stored behind its N outputs.
 PS_API int ps_gemm_heads(const void* x, int ldx, int x_head, const void* w, int heads, int M, int N, int K, const void* gate, int ldg,
-                         int g_head, void* out, int ldo, int o_head, void* status, cudaStream_t stream) {
+                         int g_head, void* out, int ldo, int o_head, int turn_r, int turn_pairs, const void* inv_freq, const void* row_pos,
+                         void* status, cudaStream_t stream) {
     using namespace ps;
-    if (heads <= 0 || heads > 65535 || M <= 0 || N <= 0 || K <= 0 || K % kGhK || x_head % kGhK || ldx % 8 || ldx < (heads - 1) * x_head + K ||
+    if (heads <= 0 || heads > 65535 || M <= 0 || N <= 0 || K <= 0 || K % kGhK || x_head % kGhK || ldx % 8 || ldx < (heads - 1) * x_head + K + turn_r ||
+        turn_r < 0 || (turn_r & 1) || 2 * turn_pairs > turn_r || (turn_r > 0 && ((ldo | o_head | N) & 1)) ||
         (((uintptr_t)x | (uintptr_t)w) % 16))
         return (int)cudaErrorInvalidValue;
     GemmHeadsArgs g;
@@ -161,6 +181,8 @@ PS_API int ps_gemm_heads(const void* x, int ldx, int x_head, const void* w, int 
     g.nb = rows <= 16 ? 16 : rows <= 32 ? 32 : 64;
     g.box_rows = (rows + 7) / 8 * 8;
     g.gate = (const __nv_bfloat16*)gate; g.ldg = ldg; g.g_head = g_head; g.status = (uint32_t*)status; g.budget = g_ps_wait_budget_cycles;
+    g.turn_r = turn_r; g.turn_pairs = turn_pairs; g.inv_freq = (const double*)inv_freq; g.row_pos = (const int*)row_pos;
+    g.x = (const __nv_bfloat16*)x; g.ldx = ldx;
     CUtensorMap mw, mx;
     int err = gh_map_2d(&mw, w, (uint64_t)heads * N, (uint64_t)K, (uint64_t)K, kGhM);
     if (err) return err;
@@ -171,6 +193,6 @@ PS_API int ps_gemm_heads(const void* x, int ldx, int x_head, const void* w, int 
         cudaFuncSetAttribute(gemm_heads_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         attr_set = true;
     }
-    return launch_pdl(gemm_heads_kernel, dim3((N + kGhM - 1) / kGhM, heads, (M + kGhRows - 1) / kGhRows), dim3(kGhThreads), smem, stream,
+    return launch_pdl(gemm_heads_kernel, dim3((N + kGhM - 1) / kGhM + (turn_r > 0 ? 1 : 0), heads, (M + kGhRows - 1) / kGhRows), dim3(kGhThreads), smem, stream,
                       mw, mx, g);
 }

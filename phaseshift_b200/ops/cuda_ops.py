@@ -730,16 +730,22 @@ class CudaOps(OpTrace):
                   c_int(s.rot_true // 2), ptr(s.inv_freq), ptr(b.row_pos))
         self.launches += 1
 
-    def _gemm_heads(self, x, x_head: int, w, heads: int, N: int, K: int, out, o_head: int, gate=None, g_head: int = 0) -> None:
-        """out[:, h] = x[:, h] w[h]^T (* sigmoid(gate[:, h])); `x_head` / `o_head` / `g_head`: columns between heads."""
+    def _gemm_heads(self, x, x_head: int, w, heads: int, N: int, K: int, out, o_head: int, gate=None, g_head: int = 0,
+                    turn: Optional[Tuple[LatentSpec, StepBatch]] = None) -> None:
+        """out[:, h] = x[:, h] w[h]^T (* sigmoid(gate[:, h])); `x_head` / `o_head` / `g_head`: columns between heads.  ``turn``: the
+        rotated part behind each head's `K` columns is turned by the row's position and stored behind its `N` outputs."""
         M, ldg = x.shape[0], gate.stride(0) if gate is not None else 0
         if self.act_dtype == torch.float32:
             _lib.call("ps_gemm_f32_batched", ptr(x), c_int(x.stride(0)), c_ll(x_head), ptr(w), c_int(K), c_ll(N * K), c_int(heads), c_int(M),
                       c_int(N), c_int(K), ptr(gate), c_int(ldg), c_ll(g_head), ptr(out), c_int(out.stride(0)), c_ll(o_head))
         else:
+            s, b = turn if turn is not None else (None, None)
             _lib.call("ps_gemm_heads", ptr(x), c_int(x.stride(0)), c_int(x_head), ptr(w), c_int(heads), c_int(M), c_int(N), c_int(K),
-                      ptr(gate), c_int(ldg), c_int(g_head), ptr(out), c_int(out.stride(0)), c_int(o_head), ptr(self.status))
+                      ptr(gate), c_int(ldg), c_int(g_head), ptr(out), c_int(out.stride(0)), c_int(o_head), c_int(s.rot if s else 0),
+                      c_int(s.rot_true // 2 if s else 0), ptr(s.inv_freq if s else None), ptr(b.row_pos if s else None), ptr(self.status))
         self.launches += 1
+        if turn is not None and self.act_dtype == torch.float32:
+            self._latent_turn(x, x_head, K, out, o_head, N, *turn)
 
     def latent_attention(self, q: torch.Tensor, s: LatentSpec, b: StepBatch, kv: KVLayer, st: ModelState, gate: torch.Tensor) -> torch.Tensor:
         """Attention of query rows [rows, heads * (dim + rot)] (not turned yet; turned in place) over the cached latents, values back
@@ -764,8 +770,7 @@ class CudaOps(OpTrace):
         rows, H, L = q.shape[0], s.heads, _lib.lib()
         spec = s.shared_keys()
         qe = self.buf(f"latent_qe{H}x{s.row}", rows, H * s.row, self.act_dtype)
-        self._gemm_heads(q, s.dim + s.rot, s.uk_t, H, s.kv_rank, s.dim, qe, s.row)
-        self._latent_turn(q, s.dim + s.rot, s.dim, qe, s.row, s.kv_rank, s, b)
+        self._gemm_heads(q, s.dim + s.rot, s.uk_t, H, s.kv_rank, s.dim, qe, s.row, turn=(s, b))
         pt = st.sc.page_tokens
         tc = (self.act_dtype == torch.bfloat16 and self.attn_decode_tc and bool(L.ps_latent_decode_ok(c_int(s.kv_rank), c_int(s.rot), c_int(pt)))
               and (short_only or b.graph_static or all(len(sq.token_ids) <= 16 for sq in b.seqs)))
@@ -786,7 +791,7 @@ class CudaOps(OpTrace):
             n_seqs, seq_rows = b.n_seqs, max(n for n in (len(sq.token_ids) for sq in b.seqs) if n <= 16)
         reach = min(s.window, b.max_context) if s.window > 0 else b.max_context
         ctas = b.max_seqs * L.ps_latent_decode_ctas(c_int(H), c_int(s.kv_rank), c_int(1))
-        split = max(64, -(-reach // max(1, 296 // ctas) // 64) * 64)
+        split = max(128, -(-reach // max(1, 296 // ctas) // 64) * 64)
         while -(-(reach + 80) // split) + 1 > 512:
             split *= 2
         ring = -(-(reach + 80) // split) + 1                 # a tile of up to 16 rows, from the tile of its first visible token on
@@ -804,10 +809,8 @@ class CudaOps(OpTrace):
 
     def _latent_expanded(self, q, s: LatentSpec, b: StepBatch, kv: KVLayer, st: ModelState, gate, out, long) -> None:
         """The tokens that the long sequences see, gathered into consecutive rows and expanded to keys and values per head."""
-        H, T, L = s.heads, self.ATTN_PREFILL_MIN_ROWS, _lib.lib()
-        spec = s.shared_keys()
-        tile = int(L.ps_latent_tile())
-        n = sum(-(-(sq.pos_start + len(sq.token_ids) - spec.first_visible(sq.pos_start) // tile * tile) // tile) * tile for sq in long)
+        T, spec = self.ATTN_PREFILL_MIN_ROWS, s.shared_keys()
+        n = self.latent_rows(s, long)
         lat, rot, exp = self._latent_scratch(n, s)
         opts = AttnOptions.of(spec)
         _lib.call("ps_latent_gather", ptr(kv.k), c_int(s.kv_rank), c_int(s.rot), ptr(st.block_table), c_int(st.max_blocks),
@@ -818,11 +821,21 @@ class CudaOps(OpTrace):
                   c_int(EPI_STORE), ptr(None), c_int(0), ptr(exp), c_int(N), c_int(0), ptr(self.status))
         self.launches += 2
         self._latent_turn(q, s.dim + s.rot, s.dim, q, s.dim + s.rot, s.dim, s, b)
-        g = gate[:, s.gate_off:]
-        _lib.call("ps_latent_prefill", ptr(q), c_int(q.shape[0]), ptr(exp), ptr(rot), c_int(n), ptr(b.seq_desc), c_int(b.n_seqs),
-                  c_int(max(len(sq.token_ids) for sq in long)), c_int(T), c_int(H), c_int(s.dim), c_int(s.rot), c_int(s.vdim), c_float(s.scale),
-                  ctypes.byref(opts), ptr(g), c_int(g.stride(0)), c_int(s.vdim), c_int(0), ptr(out), ptr(st.status))
+        self._latent_prefill(q, s, b, st, gate, out, rot, exp, long)
+
+    def _latent_prefill(self, q, s: LatentSpec, b: StepBatch, st: ModelState, gate, out, rot, exp, long) -> None:
+        """Attention of turned queries over expanded keys and values."""
+        T, g, opts = self.ATTN_PREFILL_MIN_ROWS, gate[:, s.gate_off:], AttnOptions.of(s.shared_keys())
+        _lib.call("ps_latent_prefill", ptr(q), c_int(q.shape[0]), ptr(exp), ptr(rot), c_int(rot.numel() // s.rot), ptr(b.seq_desc), c_int(b.n_seqs),
+                  c_int(max(len(sq.token_ids) for sq in long)), c_int(T), c_int(s.heads), c_int(s.dim), c_int(s.rot), c_int(s.vdim),
+                  c_float(s.scale), ctypes.byref(opts), ptr(g), c_int(g.stride(0)), c_int(s.vdim), c_int(0), ptr(out), ptr(st.status))
         self.launches += 1
+
+    @staticmethod
+    def latent_rows(s: LatentSpec, long) -> int:
+        """Gathered rows of the step's long sequences: what their rows see, in whole tiles."""
+        tile, spec = int(_lib.lib().ps_latent_tile()), s.shared_keys()
+        return sum(-(-(sq.pos_start + len(sq.token_ids) - spec.first_visible(sq.pos_start) // tile * tile) // tile) * tile for sq in long)
 
     def _latent_scratch(self, n: int, s: LatentSpec):
         """bf16 scratch of the expanded form (latents, rotated parts, keys and values); one allocation that grows to the largest step seen."""

@@ -20,7 +20,7 @@ from phaseshift_b200.ops.specs import distance_bias_table
 from phaseshift_b200.runtime.serving import ServingEngine
 
 ROOT = Path(__file__).resolve().parents[1]
-TOL = 4e-5
+TOL = 6e-5
 
 
 # ------------------------------------------------------------------ configuration, registry, loading

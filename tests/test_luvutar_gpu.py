@@ -14,7 +14,7 @@ from phaseshift_b200.runtime.batch import SeqRows
 from phaseshift_b200.runtime.serving import ServingEngine
 
 pytestmark = pytest.mark.gpu
-TOL = {torch.float32: 4e-5, torch.bfloat16: 5e-2}
+TOL = {torch.float32: 1e-4, torch.bfloat16: 5e-2}
 PEAK = {torch.float32: 2.0, torch.bfloat16: 1.0}         # attention that bf16 rounding does not amplify from layer to layer
 DTYPES = [torch.float32, torch.bfloat16]
 _ref = {}
