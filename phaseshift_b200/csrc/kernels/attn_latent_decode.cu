@@ -1,16 +1,18 @@
 // Latent attention for decode rows and short portions, in the latent space: all heads share the cached rows [latent | rotated
 // part] as keys, and the latent part as values (bf16 pool, one head per token, pages of 16, 32 or 64 tokens).
 //
-// One CTA = up to 128 (row, head) pairs of one sequence as one MMA tile -- tile row r * hp + g is head g of the CTA's row r; rows
-// beyond the used ones read whatever lies behind the queries in shared memory, and nobody reads their results --, one KV split, and up to 256 of the value columns (tensor memory holds 128 score columns and 256 output columns; wider latents
-// take two CTAs that both compute the scores):
+// One CTA = up to 128 (row, head) pairs of one sequence as one MMA tile (fewer with wide rows: two tiles of the ring come first) --
+// tile row r * hp + g is head g of the CTA's row r; rows beyond the used ones read whatever lies behind the queries in shared
+// memory, and nobody reads their results --, one KV split, and up to 256 of the value columns (tensor memory holds four score
+// tiles and 256 output columns; wider latents take two CTAs that both compute the scores):
 //
-//   warp 4   TMA producer: the queries once, then per tile of 64 tokens every 64-column group of the cached rows, once, into a
-//            ring of 8 KB stages (a group is one box per page).  The groups that are this CTA's values come last.
-//   warps 5, 7 one thread each issues S(t) += Q_g K_g^T group by group as they land (tcgen05.mma) into one of two score
-//            accumulators, warp 5 for even t and warp 7 for odd t (rings of fewer than two tiles: warp 5 for all); a group that
-//            is no value gives its stage back at once.
-//   warp 6   one thread issues O_g += P(t) V_g for the value groups, still in their stages (an MN-major operand), and gives these
+//   warps 4-7 TMA producers: the queries once, then per tile of 64 tokens every 64-column group of the cached rows, once, into a
+//            ring of 8 KB stages (a group is one box per page).  The groups that are this CTA's values come last.  Fills take
+//            turns among the four warps (waiting, arming and issuing one costs several hundred cycles); the ring is a multiple
+//            of four stages, so a stage always belongs to the same warp.
+//   warps 8, 9 one thread each issues S(t) += Q_g K_g^T group by group as they land (tcgen05.mma) into one of four
+//            score accumulators, warp 8 for even t and warp 9 for odd t; a group that is no value gives its stage back at once.
+//   warp 10  one thread issues O_g += P(t) V_g for the value groups, still in their stages (an MN-major operand), and gives these
 //            back.
 //   warps 0-3 softmax: one thread per (row, head) with its window, reference maximum and sum in 32-bit; probabilities go to
 //            shared memory as a bf16 operand; the output accumulator is rescaled only when the maximum has grown by 2^8.
@@ -22,7 +24,7 @@
 
 namespace ps {
 
-constexpr int kLdThreads = 256, kLdGroup = kTcTok * 64 * 2, kLdMaxStages = 24;
+constexpr int kLdThreads = 352, kLdProducers = 4, kLdGroup = kTcTok * 64 * 2, kLdMaxStages = 24;
 
 struct LatentDecodeArgs {
     const int* block_table; int max_blocks, num_pages, page_tokens;
@@ -40,9 +42,9 @@ struct LatentDecodeArgs {
 __global__ void __launch_bounds__(kLdThreads, 1)
 attn_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv, const LatentDecodeArgs a) {
     extern __shared__ __align__(1024) unsigned char smem[];
-    __shared__ __align__(8) uint64_t q_full, full[kLdMaxStages], freed[kLdMaxStages], s_full[2], p_full[2], pv_done[2];
+    __shared__ __align__(8) uint64_t q_full, full[kLdMaxStages], freed[kLdMaxStages], s_full[4], s_free[4], p_full[2], pv_done[2];
     __shared__ uint32_t tmem_slot;
-    __shared__ int s_abort, s_bad, s_issued, s_consumed, q_issued, q_consumed;
+    __shared__ int s_abort, s_bad, s_fills[kLdMaxStages], q_issued;
 
     const int vp = (int)blockIdx.y / a.head_tiles, ht = (int)blockIdx.y % a.head_tiles;
     const int seq = (int)blockIdx.z / a.row_tiles, r0 = ((int)blockIdx.z % a.row_tiles) * a.rows_per_tile;
@@ -65,116 +67,127 @@ attn_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
         return;
     }
     unsigned char* sQ = smem;                    // ng groups of the used rows x 64 columns (the MMA reads 128 rows from each)
-    unsigned char* sP = sQ + (size_t)ng * a.q_group;
-    unsigned char* sS = sP + kTcPBuf;
+    unsigned char* sP = sQ + (size_t)ng * a.q_group;             // two buffers of the used rows x 64 tokens
+    unsigned char* sS = sP + 2 * a.q_group;
 
     if (threadIdx.x == 0) {
         tc::mbar_init(&q_full, 1);
         for (int s = 0; s < ns; ++s) { tc::mbar_init(&full[s], 1); tc::mbar_init(&freed[s], 1); }
-        for (int s = 0; s < 2; ++s) { tc::mbar_init(&s_full[s], 1); tc::mbar_init(&p_full[s], 4); tc::mbar_init(&pv_done[s], 1); }
+        for (int s = 0; s < 4; ++s) { tc::mbar_init(&s_full[s], 1); tc::mbar_init(&s_free[s], 4); }
+        for (int s = 0; s < 2; ++s) { tc::mbar_init(&p_full[s], 4); tc::mbar_init(&pv_done[s], 1); }
         tc::fence_barrier_init();
-        s_abort = 0; s_bad = 0; s_issued = s_consumed = q_issued = q_consumed = 0;
+        for (int s = 0; s < ns; ++s) s_fills[s] = 0;
+        s_abort = 0; s_bad = 0; q_issued = 0;
         tc::tma_prefetch_desc(&map_q); tc::tma_prefetch_desc(&map_kv);
     }
-    if (warp == 6) {
+    if (warp == 10) {
         tc::tmem_alloc(&tmem_slot, 512);
         tc::tmem_relinquish();
     }
     tc::fence_before_sync();
     __syncthreads();
     tc::fence_after_sync();
-    const uint32_t tmem = tmem_slot, tmem_o = tmem + 128;
+    const uint32_t tmem = tmem_slot, tmem_o = tmem + 256;
     cudaGridDependencySynchronize();
 
-    if (warp == 4) {
-        // ------------------------------------------------ producer
-        const int blocks = (nh + 7) / 8;                                          // boxes of 8 heads per row and group
-        const int n_box = nr * blocks * ng;
-        if (lane == 0) tc::mbar_expect_tx(&q_full, (uint32_t)n_box * 1024u);
-        __syncwarp();
-        for (int i = lane; i < n_box; i += 32) {
-            const int g = i % ng, rb = i / ng, r = rb / blocks, b8 = rb % blocks;
-            tc::tma_load_2d(sQ + (size_t)g * a.q_group + (r * a.hp + 8 * b8) * 128, &map_q, g * 64,
-                            (row_start + r0 + r) * a.H + h0 + 8 * b8, &q_full);
+    // group of the cached row that comes i-th in a tile: values last
+    auto group_at = [&](int i) { return i < 4 * vp ? i : i < ng - nv ? i + nv : 4 * vp + i - (ng - nv); };
+    if (warp >= 4 && warp < 4 + kLdProducers) {
+        // ------------------------------------------------ producers
+        if (warp == 4) {
+            const int blocks = (nh + 7) / 8;                                      // boxes of 8 heads per row and group
+            const int n_box = nr * blocks * ng;
+            if (lane == 0) tc::mbar_expect_tx(&q_full, (uint32_t)n_box * 1024u);
+            __syncwarp();
+            for (int i = lane; i < n_box; i += 32) {
+                const int g = i % ng, rb = i / ng, r = rb / blocks, b8 = rb % blocks;
+                tc::tma_load_2d(sQ + (size_t)g * a.q_group + (r * a.hp + 8 * b8) * 128, &map_q, g * 64,
+                                (row_start + r0 + r) * a.H + h0 + 8 * b8, &q_full);
+            }
+            if (lane == 0) q_issued = 1;
         }
-        if (lane == 0) q_issued = 1;
         const int* bt = a.block_table + (size_t)slot * a.max_blocks;
         const int pt = a.page_tokens, ppt = kTcTok / pt;
-        int p = 0;
-        bool ok = true;
-        for (int t = 0; t < T && ok; ++t) {
-            int page = 0;
+        auto page_of = [&](int t) {                                               // this lane's page of tile t
             const int blk = (t_first + t) * ppt + lane;
-            if (lane < ppt && blk * pt < kv_end) {
-                page = bt[blk];
-                if (page < 0 || page >= a.num_pages) { s_bad = 1; page = 0; }
-            }
-            for (int i = 0; i < ng; ++i, ++p) {
-                const int st = p % ns;
-                const int g = i < 4 * vp ? i : i < ng - nv ? i + nv : 4 * vp + i - (ng - nv);     // values last
-                if (p >= ns) {
-                    ok = __all_sync(0xffffffffu, tc::mbar_wait_abortable(&freed[st], (uint32_t)(p / ns - 1) & 1u, a.budget, &s_abort));
-                    if (!ok) break;
-                }
-                if (lane == 0) tc::mbar_expect_tx(&full[st], kLdGroup);
-                __syncwarp();
-                if (lane < ppt) tc::tma_load_2d(sS + st * kLdGroup + lane * (pt * 128), &map_kv, g * 64, page * pt, &full[st]);
-                if (lane == 0) s_issued = p + 1;
-            }
+            if (t >= T || lane >= ppt || blk * pt >= kv_end) return 0;
+            const int page = bt[blk];
+            if (page < 0 || page >= a.num_pages) { s_bad = 1; return 0; }
+            return page;
+        };
+        int i = warp - 4, st = warp - 4, fill = 0, t = 0;
+        while (i >= ng) { i -= ng; ++t; }
+        int page = page_of(t), next = page_of(t + 1);
+        while (t < T) {
+            if (fill > 0 && !__all_sync(0xffffffffu, tc::mbar_wait_abortable(&freed[st], (uint32_t)(fill - 1) & 1u, a.budget, &s_abort))) break;
+            if (lane == 0) tc::mbar_expect_tx(&full[st], kLdGroup);
+            __syncwarp();
+            if (lane < ppt) tc::tma_load_2d(sS + st * kLdGroup + lane * (pt * 128), &map_kv, group_at(i) * 64, page * pt, &full[st]);
+            if (lane == 0) s_fills[st] = fill + 1;
+            st += kLdProducers;
+            if (st >= ns) { st -= ns; ++fill; }
+            i += kLdProducers;
+            while (i >= ng) { i -= ng; ++t; page = next; next = page_of(t + 1); }
         }
-    } else if (warp == 5 || warp == 7) {
+    } else if (warp == 8 || warp == 9) {
         // ------------------------------------------------ scores
         if (lane == 0) {
             constexpr uint32_t idesc = tc::idesc_bf16_f32(kTcRows, kTcTok);
             const uint32_t q_addr = tc::smem_u32(sQ), s_addr = tc::smem_u32(sS);
-            // A wait for a stage's next fill must not begin before its last one has landed (the parity would read as done).  A fill
-            // of tile t replaces one of tile t - 2 or earlier in a ring of two tiles, and P(t - 2) has been waited for; a smaller
-            // ring has one issuer, which takes the fills in order.
-            const int issuers = ns >= 2 * ng ? 2 : 1;
-            bool ok = (warp == 5 || issuers == 2) && tc::mbar_wait_abortable(&q_full, 0, a.budget, &s_abort);
-            if (ok) q_consumed = 1;
-            for (int t = warp == 5 ? 0 : 1; t < T && ok; t += issuers) {
-                const int b = t & 1;
-                // the accumulator is free once the softmax warps have read S(t - 2), which they signal with P(t - 2)
-                if (t >= 2 && !tc::mbar_wait_abortable(&p_full[b], ((uint32_t)(t >> 1) & 1u) ^ 1u, a.budget, &s_abort)) break;
+            bool ok = tc::mbar_wait_abortable(&q_full, 0, a.budget, &s_abort);
+            int st = 0;
+            uint32_t ph = 0;
+            if (warp == 9) { st = ng; while (st >= ns) { st -= ns; ph ^= 1u; } }
+            for (int t = warp - 8; t < T && ok; t += 2) {
+                const int b = t & 3;
+                // A wait for a stage's next fill must not begin before its last one has landed (the parity would read as done): the
+                // ring holds two tiles, so a fill of tile t replaces one of tile t - 2 or earlier, which must have been multiplied.
+                if (t >= 2 && !tc::mbar_wait_abortable(&s_full[(t - 2) & 3], (uint32_t)((t - 2) >> 2) & 1u, a.budget, &s_abort)) break;
+                if (t >= 4 && !tc::mbar_wait_abortable(&s_free[b], ((uint32_t)(t >> 2) & 1u) ^ 1u, a.budget, &s_abort)) break;
                 for (int i = 0; i < ng; ++i) {
-                    const int p = t * ng + i, st = p % ns;
-                    const int g = i < 4 * vp ? i : i < ng - nv ? i + nv : 4 * vp + i - (ng - nv);
-                    if (!tc::mbar_wait_abortable(&full[st], (uint32_t)(p / ns) & 1u, a.budget, &s_abort)) { ok = false; break; }
-                    atomicMax(&s_consumed, p + 1);
+                    if (!tc::mbar_wait_abortable(&full[st], ph, a.budget, &s_abort)) { ok = false; break; }
                     tc::fence_after_sync();
+                    const uint32_t qa = q_addr + group_at(i) * a.q_group, ka = s_addr + st * kLdGroup;
 #pragma unroll
                     for (int kk = 0; kk < 4; ++kk)
-                        tc::mma_bf16_ss(tmem + b * kTcTok, tc::smem_desc_sw128(q_addr + g * a.q_group + kk * 32),
-                                        tc::smem_desc_sw128(s_addr + st * kLdGroup + kk * 32), idesc, (i > 0 || kk > 0) ? 1u : 0u);
+                        tc::mma_bf16_ss(tmem + b * kTcTok, tc::smem_desc_sw128(qa + kk * 32), tc::smem_desc_sw128(ka + kk * 32), idesc,
+                                        (i > 0 || kk > 0) ? 1u : 0u);
                     if (i < ng - nv) tc::mma_commit(&freed[st]);
+                    if (++st == ns) { st = 0; ph ^= 1u; }
                 }
                 if (ok) tc::mma_commit(&s_full[b]);
+                st += ng;
+                while (st >= ns) { st -= ns; ph ^= 1u; }
             }
         }
-    } else if (warp == 6) {
+    } else if (warp == 10) {
         // ------------------------------------------------ outputs
         if (lane == 0) {
             constexpr uint32_t idesc = tc::idesc_bf16_f32_bmn(kTcRows, 64);
             const uint32_t p_addr = tc::smem_u32(sP), s_addr = tc::smem_u32(sS);
+            int st = ng - nv;
+            uint32_t ph = 0;
+            while (st >= ns) { st -= ns; ph ^= 1u; }
             for (int t = 0; t < T; ++t) {
                 const int b = t & 1;
                 if (!tc::mbar_wait_abortable(&p_full[b], (uint32_t)(t >> 1) & 1u, a.budget, &s_abort)) break;
                 bool ok = true;
                 for (int j = 0; j < nv && ok; ++j) {
-                    const int p = t * ng + ng - nv + j, st = p % ns;
-                    ok = tc::mbar_wait_abortable(&full[st], (uint32_t)(p / ns) & 1u, a.budget, &s_abort);      // landed: S(t) has read it
+                    ok = tc::mbar_wait_abortable(&full[st], ph, a.budget, &s_abort);                  // landed: S(t) has read it
                     if (!ok) break;
                     tc::fence_after_sync();
+                    const uint32_t va = s_addr + st * kLdGroup, pa = p_addr + b * a.q_group;
 #pragma unroll
                     for (int kk = 0; kk < kTcTok / 16; ++kk)
-                        tc::mma_bf16_ss(tmem_o + j * 64, tc::smem_desc_sw128(p_addr + kk * 32),
-                                        tc::smem_desc_sw128_mn(s_addr + st * kLdGroup + kk * (16 * 128), kTcTok * 128, 1024), idesc,
-                                        (t > 0 || kk > 0) ? 1u : 0u);
+                        tc::mma_bf16_ss(tmem_o + j * 64, tc::smem_desc_sw128(pa + kk * 32),
+                                        tc::smem_desc_sw128_mn(va + kk * (16 * 128), kTcTok * 128, 1024), idesc, (t > 0 || kk > 0) ? 1u : 0u);
                     tc::mma_commit(&freed[st]);
+                    if (++st == ns) { st = 0; ph ^= 1u; }
                 }
                 if (!ok) break;
                 tc::mma_commit(&pv_done[b]);
+                st += ng - nv;
+                while (st >= ns) { st -= ns; ph ^= 1u; }
             }
         }
     } else {
@@ -188,17 +201,21 @@ attn_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
         float m_ref = 0.f, l_run = 0.f;
         bool fresh = true, ok = true;
         for (int t = 0; t < T; ++t) {
-            const int b = t & 1, tok0 = (t_first + t) * kTcTok;
-            ok = __all_sync(0xffffffffu, tc::mbar_wait_abortable(&s_full[b], (uint32_t)(t >> 1) & 1u, a.budget, &s_abort));
+            const int b = t & 1, sb = t & 3, tok0 = (t_first + t) * kTcTok;
+            ok = __all_sync(0xffffffffu, tc::mbar_wait_abortable(&s_full[sb], (uint32_t)(t >> 2) & 1u, a.budget, &s_abort));
             if (!ok) break;
             tc::fence_after_sync();
             float alpha = 1.f;
-            uint32_t pk[32];
+            uint32_t pk[32], s0[32], s1[32];
             if (live) {
-                uint32_t s0[32], s1[32];
-                tc::tmem_ld_32x32(tmem + lane_base + b * kTcTok, s0);
-                tc::tmem_ld_32x32(tmem + lane_base + b * kTcTok + 32, s1);
+                tc::tmem_ld_32x32(tmem + lane_base + sb * kTcTok, s0);
+                tc::tmem_ld_32x32(tmem + lane_base + sb * kTcTok + 32, s1);
                 tc::tmem_ld_wait();
+                tc::fence_before_sync();
+            }
+            __syncwarp();
+            if (lane == 0) tc::mbar_arrive(&s_free[sb]);                          // the accumulator may take S(t + 4)
+            if (live) {
                 if (tok0 < lo || tok0 + kTcTok - 1 > rp) {
 #pragma unroll
                     for (int j = 0; j < 32; ++j) {
@@ -224,13 +241,13 @@ attn_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
                 }
                 l_run = l_run * alpha + ((sq[0] + sq[1]) + (sq[2] + sq[3]));
             }
-            if (t >= 1) {                                                         // P V(t - 1) has read P, and O is complete up to it
-                ok = __all_sync(0xffffffffu, tc::mbar_wait_abortable(&pv_done[b ^ 1], (uint32_t)((t - 1) >> 1) & 1u, a.budget, &s_abort));
+            const bool rescale = t >= 1 && __any_sync(0xffffffffu, alpha != 1.f);
+            if (t >= 2) {                                                         // P V(t - 2) has read this buffer
+                ok = __all_sync(0xffffffffu, tc::mbar_wait_abortable(&pv_done[b], (uint32_t)((t - 2) >> 1) & 1u, a.budget, &s_abort));
                 if (!ok) break;
-                tc::fence_after_sync();
             }
-            if (live) {
-                unsigned char* prow = sP + row * 128;
+            if (row * 128 < a.q_group) {                                          // (rows behind the used ones have no place)
+                unsigned char* prow = sP + b * a.q_group + row * 128;
 #pragma unroll
                 for (int c = 0; c < 8; ++c)
                     *reinterpret_cast<uint4*>(prow + ((c ^ (row & 7)) << 4)) = make_uint4(pk[4 * c], pk[4 * c + 1], pk[4 * c + 2], pk[4 * c + 3]);
@@ -244,7 +261,10 @@ attn_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
                 }
             }
             tc::fence_proxy_async_smem();
-            if (__any_sync(0xffffffffu, alpha != 1.f)) {
+            if (rescale) {                                                        // O must be complete up to P V(t - 1)
+                ok = __all_sync(0xffffffffu, tc::mbar_wait_abortable(&pv_done[b ^ 1], (uint32_t)((t - 1) >> 1) & 1u, a.budget, &s_abort));
+                if (!ok) break;
+                tc::fence_after_sync();
 #pragma unroll 1
                 for (int c0 = 0; c0 < nv * 64; c0 += 32) {
                     uint32_t o[32];
@@ -289,36 +309,54 @@ attn_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
             set_status(a.status, PS_DEV_WAIT_TIMEOUT);
             // copies still in flight get a bounded chance to land before the shared memory goes back to the next CTA
             const long long bd = a.budget < 4000000ll ? a.budget : 4000000ll;
-            if (q_issued > q_consumed) tc::mbar_wait(&q_full, 0, bd);
-            for (int c = s_consumed; c < s_issued; ++c) tc::mbar_wait(&full[c % ns], (uint32_t)(c / ns) & 1u, bd);
+            if (q_issued) tc::mbar_wait(&q_full, 0, bd);
+            for (int s = 0; s < ns; ++s)
+                if (s_fills[s] > 0) tc::mbar_wait(&full[s], (uint32_t)(s_fills[s] - 1) & 1u, bd);
         }
     }
     __syncthreads();
-    if (warp == 6) {
+    if (warp == 10) {
         tc::fence_after_sync();
         tc::tmem_dealloc(tmem, 512);
     }
 }
 
-// Stages beside `rows` query rows per group; the 2 KB are the static part.
+constexpr int kLdSmem = 225 * 1024;              // of the 227 KB; the rest is the static part
+
+// Query rows (a multiple of 8) that leave room for a ring of two tiles: they take ng query groups and two probability buffers.
+static int latent_decode_rows(int ng) {
+    const int ring = (2 * ng + kLdProducers - 1) / kLdProducers * kLdProducers;
+    const int rows = (kLdSmem - ring * kLdGroup) / (128 * (ng + 2)) / 8 * 8;
+    return rows > kTcRows ? kTcRows : rows;
+}
 static int latent_decode_stages(int ng, int rows) {
-    const int left = 227 * 1024 - 2048 - kTcPBuf - ng * rows * 128;
-    const int n = left / kLdGroup;
+    const int n = (kLdSmem - (ng + 2) * rows * 128) / kLdGroup / kLdProducers * kLdProducers;
     return n > kLdMaxStages ? kLdMaxStages : n;
+}
+struct LatentDecodeTile { int heads, hp, rows, row_tiles, head_tiles; };
+static LatentDecodeTile latent_decode_tile(int H, int ng, int max_rows) {
+    LatentDecodeTile t;
+    const int room = latent_decode_rows(ng);
+    t.head_tiles = (H + room - 1) / room;
+    t.heads = (H + t.head_tiles - 1) / t.head_tiles;
+    t.hp = (t.heads + 7) / 8 * 8;
+    t.rows = room / t.hp < max_rows ? room / t.hp : max_rows;
+    t.row_tiles = (max_rows + t.rows - 1) / t.rows;
+    return t;
 }
 
 }  // namespace ps
 
-// Whether a cached row of KR + R elements fits the kernel (queries and at least two free stages beside the value groups).
+// Whether a cached row of KR + R elements fits the kernel (a ring of two tiles beside at least eight query rows).
 PS_API int ps_latent_decode_ok(int KR, int R, int page_tokens) {
     return KR > 0 && R > 0 && KR % 64 == 0 && R % 64 == 0 && (page_tokens == 16 || page_tokens == 32 || page_tokens == 64) &&
-           ps::latent_decode_stages((KR + R) / 64, ps::kTcRows) >= 6;
+           2 * ((KR + R) / 64) <= ps::kLdMaxStages && ps::latent_decode_rows((KR + R) / 64) >= 8;
 }
 
 // CTAs of one split (value parts x head tiles x row tiles of `max_rows` rows) per sequence: what a caller sizes splits with.
-PS_API int ps_latent_decode_ctas(int H, int KR, int max_rows) {
-    const int ht = (H + 127) / 128, per = (H + ht - 1) / ht, hp = (per + 7) / 8 * 8, rpt = 128 / hp;
-    return ht * ((KR / 64 + 3) / 4) * ((max_rows + rpt - 1) / rpt);
+PS_API int ps_latent_decode_ctas(int H, int KR, int R, int max_rows) {
+    const ps::LatentDecodeTile t = ps::latent_decode_tile(H, (KR + R) / 64, max_rows);
+    return t.head_tiles * t.row_tiles * ((KR / 64 + 3) / 4);
 }
 
 // q [q_rows, H, KR + R] bf16 (latent queries, turned rotated parts); partial outputs part_acc [q_rows, H, ring, KR] f32 and part_ml
@@ -337,23 +375,21 @@ PS_API int ps_latent_decode(const void* q, int q_rows, const void* pool, const v
     LatentDecodeArgs a;
     a.block_table = (const int*)block_table; a.max_blocks = max_blocks; a.num_pages = num_pages; a.page_tokens = page_tokens;
     a.seqs = (const int*)seqs; a.H = H;
-    a.head_tiles = (H + kTcRows - 1) / kTcRows;
-    a.heads_per_tile = (H + a.head_tiles - 1) / a.head_tiles;
-    a.hp = (a.heads_per_tile + 7) / 8 * 8;
-    a.rows_per_tile = kTcRows / a.hp < max_rows ? kTcRows / a.hp : max_rows;
-    a.q_group = a.rows_per_tile * a.hp * 128;
-    a.row_tiles = (max_rows + a.rows_per_tile - 1) / a.rows_per_tile;
-    a.ng = (KR + R) / 64; a.krg = KR / 64; a.stages = latent_decode_stages(a.ng, a.rows_per_tile * a.hp);
+    a.ng = (KR + R) / 64; a.krg = KR / 64;
+    const LatentDecodeTile tile = latent_decode_tile(H, a.ng, max_rows);
+    a.head_tiles = tile.head_tiles; a.heads_per_tile = tile.heads; a.hp = tile.hp; a.rows_per_tile = tile.rows; a.row_tiles = tile.row_tiles;
+    a.q_group = tile.rows * tile.hp * 128;
+    a.stages = latent_decode_stages(a.ng, tile.rows * tile.hp);
     a.scale_log2 = scale * 1.4426950408889634f; a.opt = opt; a.split_tokens = split_tokens; a.ring = ring; a.max_rows = max_rows;
     a.part_acc = (float*)part_acc; a.part_ml = (float*)part_ml; a.status = (uint32_t*)status; a.budget = g_ps_wait_budget_cycles;
     CUtensorMap mq, mkv;
     int err = attn_map_2d(&mq, q, (uint64_t)q_rows * H, (uint64_t)(KR + R), (uint64_t)(KR + R), 8);
     if (err) return err;
     if ((err = attn_map_2d(&mkv, pool, (uint64_t)num_pages * page_tokens, (uint64_t)(KR + R), (uint64_t)(KR + R), (uint32_t)page_tokens))) return err;
-    const size_t smem = (size_t)a.ng * a.q_group + kTcPBuf + (size_t)a.stages * kLdGroup;
+    const size_t smem = (size_t)(a.ng + 2) * a.q_group + (size_t)a.stages * kLdGroup;
     static bool attr_set = false;
     if (!attr_set) {
-        cudaFuncSetAttribute(attn_latent_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 225 * 1024);
+        cudaFuncSetAttribute(attn_latent_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kLdSmem);
         attr_set = true;
     }
     const int vparts = (a.krg + 3) / 4;

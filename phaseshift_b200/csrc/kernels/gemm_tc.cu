@@ -31,12 +31,13 @@ struct GemmArgs {
     int epilogue;
     const __nv_bfloat16* residual; int ld_res;
     void* out; int ldo; int out_f32;
+    int vec;             // rows of `out` take 16-byte stores
     uint32_t* status;
     long long budget;    // clock-cycle budget of every mbarrier wait
     int a_box_rows;      // rows fetched per A tile (a multiple of 8, <= 128); the rest of the tile stays zero
 };
 
-// BN x kGemmStages x CTAs per SM: <256, 4, 1> / <128, 4, 1> for prefill-sized M; <32, 5, 2> for M <= 128 (batched decode
+// BN x kGemmStages x CTAs per SM: <256, 4, 1> / <128, 4, 1> for prefill-sized M (<128, 3, 2> up to K = 1024); <32, 5, 2> for M <= 128 (batched decode
 // on resident bf16 weights), where the problem is a weight stream: narrow N tiles give every SM a slice even
 // when N is 5120, and two co-resident CTAs per SM keep ~40 KB of weights in flight without wave quantisation.
 template <int BN, int kGemmStages, int kMinBlocks>
@@ -149,6 +150,21 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                                 o[j] = f32_to_bf16((g.epilogue == GEPI_REGLU ? fmaxf(gt, 0.f) : silu_f(gt)) * up);
                             }
                         }
+                    } else if (g.vec && g.epilogue != GEPI_RESIDUAL && col0 + 31 < g.N) {
+                        if (g.epilogue == GEPI_GELU) {
+#pragma unroll
+                            for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(gelu_tanh_f(__uint_as_float(r[j])));
+                        }
+                        if (g.out_f32) {
+                            uint4* o = reinterpret_cast<uint4*>(reinterpret_cast<float*>(g.out) + (size_t)row * g.ldo + col0);
+#pragma unroll
+                            for (int j = 0; j < 8; ++j) o[j] = make_uint4(r[4 * j], r[4 * j + 1], r[4 * j + 2], r[4 * j + 3]);
+                        } else {
+                            uint4* o = reinterpret_cast<uint4*>(reinterpret_cast<__nv_bfloat16*>(g.out) + (size_t)row * g.ldo + col0);
+                            auto two = [&](int i) { return f32x2_to_bf16x2_bits(__uint_as_float(r[i]), __uint_as_float(r[i + 1])); };
+#pragma unroll
+                            for (int j = 0; j < 4; ++j) o[j] = make_uint4(two(8 * j), two(8 * j + 2), two(8 * j + 4), two(8 * j + 6));
+                        }
                     } else {
 #pragma unroll
                         for (int j = 0; j < 32; j += 2) {
@@ -258,8 +274,11 @@ PS_API int ps_gemm_bf16_tc(const void* a, int lda, const void* w, int ldw, int M
     g.M = M; g.N = N; g.K = K; g.epilogue = epilogue; g.residual = (const __nv_bfloat16*)residual; g.ld_res = ld_res;
     g.out = out; g.ldo = ldo; g.out_f32 = out_f32; g.status = (uint32_t*)status;
     g.budget = g_ps_wait_budget_cycles;
+    g.vec = ((uintptr_t)out % 16 == 0) && (ldo % (out_f32 ? 4 : 8) == 0);
     g.a_box_rows = M >= kBM ? kBM : ((M + 7) / 8) * 8;
     if (M <= kBM && N >= 512) return launch_gemm<32, 5, 2>(a, lda, w, ldw, g, stream);
+    // short sums: the store of a tile takes longer than its products, so two CTAs per SM overlap them
+    if (K <= 1024) return launch_gemm<128, 3, 2>(a, lda, w, ldw, g, stream);
     if (N >= 256) return launch_gemm<256, 4, 1>(a, lda, w, ldw, g, stream);
     return launch_gemm<128, 4, 1>(a, lda, w, ldw, g, stream);
 }

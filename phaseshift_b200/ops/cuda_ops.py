@@ -790,7 +790,7 @@ class CudaOps(OpTrace):
         else:
             n_seqs, seq_rows = b.n_seqs, max(n for n in (len(sq.token_ids) for sq in b.seqs) if n <= 16)
         reach = min(s.window, b.max_context) if s.window > 0 else b.max_context
-        ctas = b.max_seqs * L.ps_latent_decode_ctas(c_int(H), c_int(s.kv_rank), c_int(1))
+        ctas = b.max_seqs * L.ps_latent_decode_ctas(c_int(H), c_int(s.kv_rank), c_int(s.rot), c_int(1))
         split = max(128, -(-reach // max(1, 296 // ctas) // 64) * 64)
         while -(-(reach + 80) // split) + 1 > 512:
             split *= 2
