@@ -4,14 +4,15 @@
 // One CTA = up to 128 (row, head) pairs of one sequence as one MMA tile (fewer with wide rows: two tiles of the ring come first) --
 // tile row r * hp + g is head g of the CTA's row r; rows beyond the used ones read whatever lies behind the queries in shared
 // memory, and nobody reads their results --, one KV split, and up to 256 of the value columns (tensor memory holds four score
-// tiles and 256 output columns; wider latents take two CTAs that both compute the scores):
+// accumulators and 256 output columns; wider latents take two CTAs that both compute the scores):
 //
 //   warps 4-7 TMA producers: the queries once, then per tile of 64 tokens every 64-column group of the cached rows, once, into a
 //            ring of 8 KB stages (a group is one box per page).  The groups that are this CTA's values come last.  Fills take
 //            turns among the four warps (waiting, arming and issuing one costs several hundred cycles); the ring is a multiple
 //            of four stages, so a stage always belongs to the same warp.
-//   warps 8, 9 one thread each issues S(t) += Q_g K_g^T group by group as they land (tcgen05.mma) into one of four
-//            score accumulators, warp 8 for even t and warp 9 for odd t; a group that is no value gives its stage back at once.
+//   warps 8, 9 one thread each issues half of S(t) = sum_g Q_g K_g^T (every other group, as they land) into an accumulator of
+//            its own, since issuing a product costs a thread more than the product itself; the softmax adds the two.  Two pairs
+//            of accumulators take turns.  A group that is no value gives its stage back at once.
 //   warp 10  one thread issues O_g += P(t) V_g for the value groups, still in their stages (an MN-major operand), and gives these
 //            back.
 //   warps 0-3 softmax: one thread per (row, head) with its window, reference maximum and sum in 32-bit; probabilities go to
@@ -42,7 +43,7 @@ struct LatentDecodeArgs {
 __global__ void __launch_bounds__(kLdThreads, 1)
 attn_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv, const LatentDecodeArgs a) {
     extern __shared__ __align__(1024) unsigned char smem[];
-    __shared__ __align__(8) uint64_t q_full, full[kLdMaxStages], freed[kLdMaxStages], s_full[4], s_free[4], p_full[2], pv_done[2];
+    __shared__ __align__(8) uint64_t q_full, full[kLdMaxStages], freed[kLdMaxStages], s_full[2], s_free[2], p_full[2], pv_done[2];
     __shared__ uint32_t tmem_slot;
     __shared__ int s_abort, s_bad, s_fills[kLdMaxStages], q_issued;
 
@@ -73,8 +74,9 @@ attn_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
     if (threadIdx.x == 0) {
         tc::mbar_init(&q_full, 1);
         for (int s = 0; s < ns; ++s) { tc::mbar_init(&full[s], 1); tc::mbar_init(&freed[s], 1); }
-        for (int s = 0; s < 4; ++s) { tc::mbar_init(&s_full[s], 1); tc::mbar_init(&s_free[s], 4); }
-        for (int s = 0; s < 2; ++s) { tc::mbar_init(&p_full[s], 4); tc::mbar_init(&pv_done[s], 1); }
+        for (int s = 0; s < 2; ++s) {
+            tc::mbar_init(&s_full[s], 2); tc::mbar_init(&s_free[s], 4); tc::mbar_init(&p_full[s], 4); tc::mbar_init(&pv_done[s], 1);
+        }
         tc::fence_barrier_init();
         for (int s = 0; s < ns; ++s) s_fills[s] = 0;
         s_abort = 0; s_bad = 0; q_issued = 0;
@@ -135,35 +137,37 @@ attn_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
             constexpr uint32_t idesc = tc::idesc_bf16_f32(kTcRows, kTcTok);
             const uint32_t q_addr = tc::smem_u32(sQ), s_addr = tc::smem_u32(sS);
             bool ok = tc::mbar_wait_abortable(&q_full, 0, a.budget, &s_abort);
-            int st = 0;
-            uint32_t ph = 0;
-            if (warp == 9) { st = ng; while (st >= ns) { st -= ns; ph ^= 1u; } }
-            for (int t = warp - 8; t < T && ok; t += 2) {
-                const int b = t & 3;
-                // A wait for a stage's next fill must not begin before its last one has landed (the parity would read as done): the
-                // ring holds two tiles, so a fill of tile t replaces one of tile t - 2 or earlier, which must have been multiplied.
-                if (t >= 2 && !tc::mbar_wait_abortable(&s_full[(t - 2) & 3], (uint32_t)((t - 2) >> 2) & 1u, a.budget, &s_abort)) break;
-                if (t >= 4 && !tc::mbar_wait_abortable(&s_free[b], ((uint32_t)(t >> 2) & 1u) ^ 1u, a.budget, &s_abort)) break;
-                for (int i = 0; i < ng; ++i) {
-                    if (!tc::mbar_wait_abortable(&full[st], ph, a.budget, &s_abort)) { ok = false; break; }
+            const int mine = warp - 8;
+            int st0 = 0;                                                          // stage and phase of the tile's first group
+            uint32_t ph0 = 0;
+            for (int t = 0; t < T && ok; ++t) {
+                const int b = t & 1;
+                const uint32_t acc = tmem + b * (2 * kTcTok) + mine * kTcTok;
+                // The accumulators are free once the softmax warps have read S(t - 2).  The same wait keeps the ones below from
+                // beginning before a stage's last fill has landed (the parity would read as done): the ring holds two tiles, so a
+                // fill of tile t replaces one of tile t - 2 or earlier.
+                if (t >= 2 && !tc::mbar_wait_abortable(&s_free[b], ((uint32_t)(t >> 1) & 1u) ^ 1u, a.budget, &s_abort)) break;
+                for (int i = mine; i < ng; i += 2) {
+                    const int st = st0 + i < ns ? st0 + i : st0 + i - ns;
+                    if (!tc::mbar_wait_abortable(&full[st], st0 + i < ns ? ph0 : ph0 ^ 1u, a.budget, &s_abort)) { ok = false; break; }
                     tc::fence_after_sync();
                     const uint32_t qa = q_addr + group_at(i) * a.q_group, ka = s_addr + st * kLdGroup;
 #pragma unroll
                     for (int kk = 0; kk < 4; ++kk)
-                        tc::mma_bf16_ss(tmem + b * kTcTok, tc::smem_desc_sw128(qa + kk * 32), tc::smem_desc_sw128(ka + kk * 32), idesc,
-                                        (i > 0 || kk > 0) ? 1u : 0u);
+                        tc::mma_bf16_ss(acc, tc::smem_desc_sw128(qa + kk * 32), tc::smem_desc_sw128(ka + kk * 32), idesc,
+                                        (i > mine || kk > 0) ? 1u : 0u);
                     if (i < ng - nv) tc::mma_commit(&freed[st]);
-                    if (++st == ns) { st = 0; ph ^= 1u; }
                 }
                 if (ok) tc::mma_commit(&s_full[b]);
-                st += ng;
-                while (st >= ns) { st -= ns; ph ^= 1u; }
+                st0 += ng;
+                while (st0 >= ns) { st0 -= ns; ph0 ^= 1u; }
             }
         }
     } else if (warp == 10) {
         // ------------------------------------------------ outputs
         if (lane == 0) {
-            constexpr uint32_t idesc = tc::idesc_bf16_f32_bmn(kTcRows, 64);
+            const uint32_t idesc_all = tc::idesc_bf16_f32_bmn(kTcRows, 64 * nv);
+            constexpr uint32_t idesc_one = tc::idesc_bf16_f32_bmn(kTcRows, 64);
             const uint32_t p_addr = tc::smem_u32(sP), s_addr = tc::smem_u32(sS);
             int st = ng - nv;
             uint32_t ph = 0;
@@ -171,17 +175,23 @@ attn_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
             for (int t = 0; t < T; ++t) {
                 const int b = t & 1;
                 if (!tc::mbar_wait_abortable(&p_full[b], (uint32_t)(t >> 1) & 1u, a.budget, &s_abort)) break;
+                const uint32_t pa = p_addr + b * a.q_group;
+                const bool together = st + nv <= ns;                              // the value groups' stages follow one another: one wide product
+                const int first = st;
                 bool ok = true;
                 for (int j = 0; j < nv && ok; ++j) {
                     ok = tc::mbar_wait_abortable(&full[st], ph, a.budget, &s_abort);                  // landed: S(t) has read it
                     if (!ok) break;
                     tc::fence_after_sync();
-                    const uint32_t va = s_addr + st * kLdGroup, pa = p_addr + b * a.q_group;
+                    if (!together || j == nv - 1) {
+                        const uint32_t va = s_addr + (together ? first : st) * kLdGroup, o = tmem_o + (together ? 0 : j * 64);
 #pragma unroll
-                    for (int kk = 0; kk < kTcTok / 16; ++kk)
-                        tc::mma_bf16_ss(tmem_o + j * 64, tc::smem_desc_sw128(pa + kk * 32),
-                                        tc::smem_desc_sw128_mn(va + kk * (16 * 128), kTcTok * 128, 1024), idesc, (t > 0 || kk > 0) ? 1u : 0u);
-                    tc::mma_commit(&freed[st]);
+                        for (int kk = 0; kk < kTcTok / 16; ++kk)
+                            tc::mma_bf16_ss(o, tc::smem_desc_sw128(pa + kk * 32), tc::smem_desc_sw128_mn(va + kk * (16 * 128), kTcTok * 128, 1024),
+                                            together ? idesc_all : idesc_one, (t > 0 || kk > 0) ? 1u : 0u);
+                        if (together) { for (int k = first; k < first + nv; ++k) tc::mma_commit(&freed[k]); }
+                        else tc::mma_commit(&freed[st]);
+                    }
                     if (++st == ns) { st = 0; ph ^= 1u; }
                 }
                 if (!ok) break;
@@ -201,20 +211,29 @@ attn_latent_decode_kernel(const __grid_constant__ CUtensorMap map_q, const __gri
         float m_ref = 0.f, l_run = 0.f;
         bool fresh = true, ok = true;
         for (int t = 0; t < T; ++t) {
-            const int b = t & 1, sb = t & 3, tok0 = (t_first + t) * kTcTok;
-            ok = __all_sync(0xffffffffu, tc::mbar_wait_abortable(&s_full[sb], (uint32_t)(t >> 2) & 1u, a.budget, &s_abort));
+            const int b = t & 1, tok0 = (t_first + t) * kTcTok;
+            ok = __all_sync(0xffffffffu, tc::mbar_wait_abortable(&s_full[b], (uint32_t)(t >> 1) & 1u, a.budget, &s_abort));
             if (!ok) break;
             tc::fence_after_sync();
             float alpha = 1.f;
             uint32_t pk[32], s0[32], s1[32];
             if (live) {
-                tc::tmem_ld_32x32(tmem + lane_base + sb * kTcTok, s0);
-                tc::tmem_ld_32x32(tmem + lane_base + sb * kTcTok + 32, s1);
+                const uint32_t acc = tmem + lane_base + b * (2 * kTcTok);
+                uint32_t h[32];
+                tc::tmem_ld_32x32(acc, s0);
+                tc::tmem_ld_32x32(acc + kTcTok, h);
+                tc::tmem_ld_32x32(acc + 32, s1);
                 tc::tmem_ld_wait();
+#pragma unroll
+                for (int j = 0; j < 32; ++j) s0[j] = __float_as_uint(__uint_as_float(s0[j]) + __uint_as_float(h[j]));
+                tc::tmem_ld_32x32(acc + kTcTok + 32, h);
+                tc::tmem_ld_wait();
+#pragma unroll
+                for (int j = 0; j < 32; ++j) s1[j] = __float_as_uint(__uint_as_float(s1[j]) + __uint_as_float(h[j]));
                 tc::fence_before_sync();
             }
             __syncwarp();
-            if (lane == 0) tc::mbar_arrive(&s_free[sb]);                          // the accumulator may take S(t + 4)
+            if (lane == 0) tc::mbar_arrive(&s_free[b]);                           // the accumulators may take S(t + 2)
             if (live) {
                 if (tok0 < lo || tok0 + kTcTok - 1 > rp) {
 #pragma unroll

@@ -104,7 +104,15 @@ gemm_heads_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_consta
         }
     } else {
         cudaGridDependencySynchronize();                 // the gate, and the readers of the previous contents of `out`
-        const int quad = warp & 3, n = n0 + quad * 32 + lane;
+        const int quad = warp & 3, n = n0 + quad * 32 + lane, rows = min(kGhRows, g.M - m0);
+        // the gate values of 16 rows at once, asked for before the accumulator is waited for
+        float gate[16];
+        auto load_gate = [&](int c0) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j)
+                gate[j] = c0 + j < rows && n < g.N ? bf16_to_f32(g.gate[(size_t)(m0 + c0 + j) * g.ldg + (size_t)h * g.g_head + n]) : 0.f;
+        };
+        if (g.gate != nullptr) load_gate(0);
         const bool done = __all_sync(0xffffffffu, tc::mbar_wait_abortable(&acc_bar, 0, g.budget, &s_abort));
         tc::fence_after_sync();
         if (done && s_abort == 0) {
@@ -112,16 +120,14 @@ gemm_heads_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_consta
                 uint32_t r[16];
                 tc::tmem_ld_32x16(tmem + ((uint32_t)(quad * 32) << 16) + (uint32_t)c0, r);
                 tc::tmem_ld_wait();
-                if (n < g.N) {
+                if (g.gate != nullptr) {
 #pragma unroll
-                    for (int j = 0; j < 16; ++j) {
-                        const int m = m0 + c0 + j;
-                        if (m >= g.M || c0 + j >= kGhRows) break;
-                        float v = __uint_as_float(r[j]);
-                        if (g.gate != nullptr) v *= sigmoid_f(bf16_to_f32(g.gate[(size_t)m * g.ldg + (size_t)h * g.g_head + n]));
-                        g.out[(size_t)m * g.ldo + (size_t)h * g.o_head + n] = f32_to_bf16(v);
-                    }
+                    for (int j = 0; j < 16; ++j) r[j] = __float_as_uint(__uint_as_float(r[j]) * sigmoid_f(gate[j]));
+                    if (c0 + 16 < g.nb) load_gate(c0 + 16);
                 }
+#pragma unroll
+                for (int j = 0; j < 16; ++j)
+                    if (c0 + j < rows && n < g.N) g.out[(size_t)(m0 + c0 + j) * g.ldo + (size_t)h * g.o_head + n] = f32_to_bf16(__uint_as_float(r[j]));
             }
         }
     }
