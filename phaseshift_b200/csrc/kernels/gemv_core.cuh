@@ -428,7 +428,9 @@ template <> struct RowDot<W_MXFP8> {
     }
 };
 
-// Apply the epilogue for one quad (4 consecutive output rows) and one batch row.
+// Apply the epilogue for one quad (4 consecutive output rows) and one batch row.  GELU (the tanh form, on every output) is a
+// template parameter: as a run-time choice beside the others it slowed every streaming projection.
+template <bool GELU = false>
 __device__ __forceinline__ void quad_epilogue(const LinearSmallArgs& a, int n0, int m, const float (&v)[kQuadRows]) {
     if (a.epilogue == EPI_SWIGLU || a.epilogue == EPI_REGLU) {
         // rows (2j, 2j+1) hold (gate_j, up_j); both rounded to bf16 as separate projections would be
@@ -451,7 +453,7 @@ __device__ __forceinline__ void quad_epilogue(const LinearSmallArgs& a, int n0, 
         float y = v[r];
         if (a.epilogue == EPI_RESIDUAL)   // y rounded to bf16 before the add, like projection-then-add
             y = bf16_to_f32(f32_to_bf16(y)) + bf16_to_f32(a.residual[(size_t)m * a.ld_res + n]);
-        if (a.epilogue == EPI_GELU) y = gelu_tanh_f(y);
+        if constexpr (GELU) y = gelu_tanh_f(y);
         if (a.out_f32) reinterpret_cast<float*>(a.out)[(size_t)m * a.ldo + n] = y;
         else reinterpret_cast<__nv_bfloat16*>(a.out)[(size_t)m * a.ldo + n] = f32_to_bf16(y);
     }

@@ -27,9 +27,10 @@ __device__ __forceinline__ void bulk_g2s(void* smem_dst, const void* gsrc, uint3
                  ::"r"(tc::smem_u32(smem_dst)), "l"(gsrc), "r"(bytes), "r"(tc::smem_u32(bar)) : "memory");
 }
 
-// AMAX: greedy sampling fused into the epilogue (ps_linear_stream_argmax); a template parameter, so that the kernel every
-// other projection uses is compiled without a trace of it
-template <int WF, int MT, bool AMAX = false>
+// VARIANT: the common kernel, greedy sampling fused into the epilogue (ps_linear_stream_argmax), or the tanh form of gelu on every
+// output; a template parameter, so that the kernel every other projection runs compiles to what it is without them.
+enum StreamVariant : int { ST_PLAIN = 0, ST_ARGMAX = 1, ST_GELU = 2 };
+template <int WF, int MT, int VARIANT = ST_PLAIN>
 __global__ void __launch_bounds__(kStThreads, 1) linear_stream_kernel(const LinearSmallArgs a, uint32_t* status,
                                                                        const int n_slots, const long long budget) {
     extern __shared__ __align__(128) unsigned char smem_raw[];
@@ -94,6 +95,7 @@ __global__ void __launch_bounds__(kStThreads, 1) linear_stream_kernel(const Line
 
     int consumed = 0;
     bool timed_out = false;
+    constexpr bool AMAX = VARIANT == ST_ARGMAX;
     [[maybe_unused]] unsigned long long amax_mine = 0ull;      // AMAX: this thread's best key (its batch row is threadIdx.x % MT)
     [[maybe_unused]] bool amax_bad = false;
     for (int wave_q0 = quad_begin; wave_q0 < quad_end; wave_q0 += kStWaveQuads) {
@@ -177,7 +179,7 @@ __global__ void __launch_bounds__(kStThreads, 1) linear_stream_kernel(const Line
                             }
                         }
                     }
-                    if (!AMAX || a.out != nullptr) quad_epilogue(a, (wave_q0 + ql) * R, m, v);
+                    if (!AMAX || a.out != nullptr) quad_epilogue<VARIANT == ST_GELU>(a, (wave_q0 + ql) * R, m, v);
                 }
             }
         } else {
@@ -284,7 +286,7 @@ __global__ void __launch_bounds__(kStThreads, 1) linear_stream_kernel(const Line
 
 static int g_st_sm_count = 0, g_st_pdl = 1;
 
-template <int WF, int MT, bool AMAX = false>
+template <int WF, int MT, int VARIANT = ST_PLAIN>
 static int launch_stream(const LinearSmallArgs& a, uint32_t* status, cudaStream_t stream) {
     const int kpad = gemv_kpad<WF>(a.K);
     const size_t fixed = (size_t)kpad * MT * sizeof(typename WTraits<WF>::XS) +
@@ -296,7 +298,7 @@ static int launch_stream(const LinearSmallArgs& a, uint32_t* status, cudaStream_
     const size_t smem = fixed + (size_t)kStWarps * slots * slot_stride<WF>();
     static bool attr_set = false;
     if (!attr_set) {
-        cudaFuncSetAttribute(linear_stream_kernel<WF, MT, AMAX>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)budget);
+        cudaFuncSetAttribute(linear_stream_kernel<WF, MT, VARIANT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)budget);
         attr_set = true;
     }
     const int n_quads = (a.N + kQuadRows - 1) / kQuadRows;
@@ -307,24 +309,15 @@ static int launch_stream(const LinearSmallArgs& a, uint32_t* status, cudaStream_
     attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
     attr[0].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr; cfg.numAttrs = g_st_pdl ? 1 : 0;
-    return (int)cudaLaunchKernelEx(&cfg, linear_stream_kernel<WF, MT, AMAX>, a, status, slots, g_ps_wait_budget_cycles);
+    return (int)cudaLaunchKernelEx(&cfg, linear_stream_kernel<WF, MT, VARIANT>, a, status, slots, g_ps_wait_budget_cycles);
 }
 
-template <int WF>
+template <int WF, int VARIANT = ST_PLAIN>
 static int stream_dispatch_m(const LinearSmallArgs& a, uint32_t* status, cudaStream_t stream) {
-    if (a.M <= 1) return launch_stream<WF, 1>(a, status, stream);
-    if (a.M <= 2) return launch_stream<WF, 2>(a, status, stream);
-    if (a.M <= 4) return launch_stream<WF, 4>(a, status, stream);
-    if (a.M <= 8) return launch_stream<WF, 8>(a, status, stream);
-    return -1;
-}
-
-template <int WF>
-static int stream_dispatch_m_amax(const LinearSmallArgs& a, uint32_t* status, cudaStream_t stream) {
-    if (a.M <= 1) return launch_stream<WF, 1, true>(a, status, stream);
-    if (a.M <= 2) return launch_stream<WF, 2, true>(a, status, stream);
-    if (a.M <= 4) return launch_stream<WF, 4, true>(a, status, stream);
-    if (a.M <= 8) return launch_stream<WF, 8, true>(a, status, stream);
+    if (a.M <= 1) return launch_stream<WF, 1, VARIANT>(a, status, stream);
+    if (a.M <= 2) return launch_stream<WF, 2, VARIANT>(a, status, stream);
+    if (a.M <= 4) return launch_stream<WF, 4, VARIANT>(a, status, stream);
+    if (a.M <= 8) return launch_stream<WF, 8, VARIANT>(a, status, stream);
     return -1;
 }
 
@@ -365,6 +358,8 @@ PS_API int ps_linear_stream(int wfmt, const void* x, int M, int N, int K, int ld
     } else {
         a.tp.size = 0;
     }
+    if (epilogue == EPI_GELU)              // only unquantised models have it; no tensor-parallel combine
+        return wfmt == W_BF16 && tp_combine == nullptr ? stream_dispatch_m<W_BF16, ST_GELU>(a, (uint32_t*)status, stream) : (int)cudaErrorInvalidValue;
     switch (wfmt) {
         case W_BF16: return stream_dispatch_m<W_BF16>(a, (uint32_t*)status, stream);
         case W_NVFP4: return stream_dispatch_m<W_NVFP4>(a, (uint32_t*)status, stream);
@@ -393,9 +388,9 @@ PS_API int ps_linear_stream_argmax(int wfmt, const void* x, int M, int N, int K,
     a.out = out; a.ldo = ldo; a.out_f32 = 1; a.xn_out = nullptr; a.tp.size = 0;
     a.amax_best = (unsigned long long*)state; a.amax_ctl = (unsigned int*)((unsigned long long*)state + 8); a.amax_tokens = (int*)tokens;
     switch (wfmt) {
-        case W_BF16: return stream_dispatch_m_amax<W_BF16>(a, (uint32_t*)status, stream);
-        case W_NVFP4: return stream_dispatch_m_amax<W_NVFP4>(a, (uint32_t*)status, stream);
-        case W_MXFP8: return stream_dispatch_m_amax<W_MXFP8>(a, (uint32_t*)status, stream);
+        case W_BF16: return stream_dispatch_m<W_BF16, ST_ARGMAX>(a, (uint32_t*)status, stream);
+        case W_NVFP4: return stream_dispatch_m<W_NVFP4, ST_ARGMAX>(a, (uint32_t*)status, stream);
+        case W_MXFP8: return stream_dispatch_m<W_MXFP8, ST_ARGMAX>(a, (uint32_t*)status, stream);
     }
     return (int)cudaErrorInvalidValue;
 }

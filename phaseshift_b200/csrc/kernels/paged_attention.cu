@@ -127,6 +127,8 @@ __device__ __forceinline__ void tile_store(const PagedAttnArgs& a, const TileReg
     }
 }
 
+// TRANSFORM: query temperature and distance bias.
+template <bool TRANSFORM>
 __global__ void __launch_bounds__(kAttnThreads) paged_attn_split_kernel(const PagedAttnArgs a) {
     extern __shared__ __align__(16) unsigned char smem[];
     const int D = a.D, heads_per_kv = a.Hq / a.Hkv, kpitch = D + 8;
@@ -152,7 +154,7 @@ __global__ void __launch_bounds__(kAttnThreads) paged_attn_split_kernel(const Pa
     const int slot = a.row_slot[row];
     const int t = threadIdx.x, warp = t >> 5, lane = t & 31;
 
-    const float q_scale = a.sm_scale * attn_temperature(a.opt, visible - 1);
+    const float q_scale = TRANSFORM ? a.sm_scale * attn_temperature(a.opt, visible - 1) : a.sm_scale;
     for (int i = t; i < G * D; i += kAttnThreads) {
         const int g = i / D, d = i % D;
         qs[i] = bf16_to_f32(a.q[((size_t)row * a.Hq + h0 + g) * D + d]) * q_scale;
@@ -189,7 +191,7 @@ __global__ void __launch_bounds__(kAttnThreads) paged_attn_split_kernel(const Pa
             }
             s *= kscale[lane];
             const bool live = tok < tok_end;
-            if (live) s += attn_bias(a.opt, h0 + warp, visible - 1 - tok);
+            if (TRANSFORM && live) s += attn_bias(a.opt, h0 + warp, visible - 1 - tok);
             if (!live) s = -3.0e38f;
             const float m_new = fmaxf(m_run, warp_max(s));
             const float p = live ? __expf(s - m_new) : 0.f;
@@ -251,6 +253,7 @@ struct AttnMergeArgs {
 // parallel (thread s owns split s), then every thread adds its output dimension over the splits in
 // ascending order, so the result depends only on the row's position, never on the batch.
 constexpr int kAttnMaxSplits = 1024;
+template <bool RING>
 __global__ void paged_attn_merge_kernel(const AttnMergeArgs a) {
     __shared__ float s_w[kAttnMaxSplits];
     __shared__ float s_red[64];
@@ -261,27 +264,29 @@ __global__ void paged_attn_merge_kernel(const AttnMergeArgs a) {
     if (visible < 0) return;                                            // position -2: a row another kernel of the step owns
     const int n = (visible + a.split_tokens - 1) / a.split_tokens;      // 0 for a padding row
     const int s0 = visible > 0 ? attn_first(a.opt, visible - 1) / a.split_tokens : 0;
-    const int ring = a.ring > 0 ? a.ring : kAttnMaxSplits;
+    auto slot_of = [&](int s) { return RING ? s % a.ring : s; };
     const float sink = a.opt.sink != nullptr ? a.opt.sink[h] : -3.0e38f;
     const float* ml = a.part_ml + ((size_t)row * a.Hq + h) * a.max_splits * 2;
     const float* pa = a.part_acc + ((size_t)row * a.Hq + h) * a.max_splits * a.D;
     float m = sink;
-    for (int s = s0 + d; s < n; s += blockDim.x) m = fmaxf(m, ml[2 * (s % ring)]);
+    for (int s = s0 + d; s < n; s += blockDim.x) m = fmaxf(m, ml[2 * slot_of(s)]);
     m = block_max(m, s_red);
     float l = 0.f;
     for (int s = s0 + d; s < n; s += blockDim.x) {
-        const float w = __expf(ml[2 * (s % ring)] - m);
-        s_w[s % ring] = w;
-        l = fmaf(w, ml[2 * (s % ring) + 1], l);
+        const int at = slot_of(s);
+        const float w = __expf(ml[2 * at] - m);
+        s_w[at] = w;
+        l = fmaf(w, ml[2 * at + 1], l);
     }
     l = block_sum(l, s_red + 32);      // its barriers also publish s_w
     if (a.opt.sink != nullptr) l += __expf(sink - m);
     float o = 0.f;
-    int at = s0 % ring;
+    int at = slot_of(s0);
 #pragma unroll 4
     for (int s = s0; s < n; ++s) {
         o = fmaf(s_w[at], pa[(size_t)at * a.D + d], o);
-        at = at + 1 == ring ? 0 : at + 1;
+        ++at;
+        if (RING && at == a.ring) at = 0;
     }
     float v = l > 0.f ? o / l : 0.f;
     if (a.gate != nullptr) {
@@ -320,18 +325,20 @@ PS_API int ps_paged_attention_ex(const void* q, const void* k_pool, const void* 
                         sizeof(float) * (kAttnMaxG * D + kAttnMaxG * kAttnTile + kAttnMaxG + 2 * kAttnTile);
     static bool attr_set = false;
     if (!attr_set) {
-        cudaFuncSetAttribute(paged_attn_split_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024);
+        cudaFuncSetAttribute(paged_attn_split_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024);
+        cudaFuncSetAttribute(paged_attn_split_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024);
         attr_set = true;
     }
     dim3 grid(n_splits, Hkv * ((G + kAttnMaxG - 1) / kAttnMaxG), rows);
-    int err = launch_pdl(paged_attn_split_kernel, grid, dim3(kAttnThreads), smem, stream, a);
+    int err = launch_pdl(attn_transforms_scores(opt) ? paged_attn_split_kernel<true> : paged_attn_split_kernel<false>, grid, dim3(kAttnThreads),
+                         smem, stream, a);
     if (err) return err;
     AttnMergeArgs m;
     m.part_acc = a.part_acc; m.part_ml = a.part_ml; m.row_pos = a.row_pos; m.rows = rows; m.Hq = Hq; m.D = D;
     m.split_tokens = split_tokens; m.max_splits = max_splits; m.gate = (const __nv_bfloat16*)gate;
     m.ld_gate = ld_gate; m.gate_head_stride = gate_head_stride; m.gate_offset = gate_offset;
     m.out = (__nv_bfloat16*)out; m.opt = opt; m.ring = 0;
-    return launch_pdl(paged_attn_merge_kernel, dim3(Hq, rows), dim3(D), 0, stream, m);
+    return launch_pdl(paged_attn_merge_kernel<false>, dim3(Hq, rows), dim3(D), 0, stream, m);
 }
 
 PS_API int ps_paged_attention(const void* q, const void* k_pool, const void* v_pool, const void* k_scale,
@@ -361,7 +368,7 @@ PS_API int ps_paged_attention_merge_ex(const void* part_acc, const void* part_ml
     m.split_tokens = split_tokens; m.max_splits = max_splits; m.gate = (const __nv_bfloat16*)gate;
     m.ld_gate = ld_gate; m.gate_head_stride = gate_head_stride; m.gate_offset = gate_offset;
     m.out = (__nv_bfloat16*)out; m.opt = opt; m.ring = ring;
-    return launch_pdl(paged_attn_merge_kernel, dim3(Hq, rows), dim3(D), 0, stream, m);
+    return launch_pdl(ring > 0 ? paged_attn_merge_kernel<true> : paged_attn_merge_kernel<false>, dim3(Hq, rows), dim3(D), 0, stream, m);
 }
 
 PS_API int ps_paged_attention_merge(const void* part_acc, const void* part_ml, const void* row_pos, int rows, int Hq, int D,
