@@ -2,8 +2,9 @@
 
 The residual streams are 32-bit.  Writing a sublayer's output into all streams, reading the next sublayer's input from them
 and its norm are one launch (``ops.stream_norm``).  An attention layer decodes in nine launches: stream norm, in_proj, append,
-attention (split + merge), o, stream norm, up, down.  A latent layer decodes in twelve: stream norm, in_proj, latents (norms, rotation, append), uq, queries into the latent space, attention (split +
-merge), values out of it with the output gate, o, stream norm, up, down.
+attention (split + merge), o, stream norm, up, down.  A latent layer decodes in twelve: stream norm, in_proj, latents (norms,
+rotation, append), uq, queries into the latent space, attention (split + merge), values out of it with the output gate, o,
+stream norm, up, down.
 """
 from __future__ import annotations
 
