@@ -21,7 +21,7 @@ from ..models.qwen35.weights import AttnW, GdnW, LinearW
 from ..runtime.batch import StepBatch
 from ..runtime.state import GdnLayerState, KVLayer, ModelState
 from ..utils.sampling import sample_row_host
-from .specs import AttnSpec, GlaSpec, LatentSpec, Pending, StreamWrite
+from .specs import AttnSpec, ExpertSum, GlaSpec, HeadsSpec, LatentSpec, MoeSpec, Pending, Routed, StreamWrite
 
 
 class RefOps(OpTrace):
@@ -46,7 +46,7 @@ class RefOps(OpTrace):
         return self._dense(table)[b.ids[:rows].long()]
 
     def linear(self, x, W: LinearW, *, name: str, norm_w=None, eps: float = 0.0, residual=None, swiglu=False,
-               reglu=False, gelu=False, out_f32=False, out=None, ssq_in=None, ssq_out=None, prefetch=None, **_):
+               reglu=False, geglu=False, gelu=False, out_f32=False, out=None, ssq_in=None, ssq_out=None, prefetch=None, **_):
         x = x.float()
         if self.act_quant and W.fmt in ("nvfp4", "mxfp8"):
             # the tensor-core layout's arithmetic: quantise x (1 + w), apply the row factor 1/rms after the product
@@ -65,6 +65,8 @@ class RefOps(OpTrace):
             y = F.silu(y[:, 0::2]) * y[:, 1::2]
         if reglu:
             y = F.relu(y[:, 0::2]) * y[:, 1::2]
+        if geglu:
+            y = F.gelu(y[:, 0::2], approximate="tanh") * y[:, 1::2]
         if gelu:
             y = F.gelu(y, approximate="tanh")
         if residual is not None:
@@ -239,9 +241,15 @@ class RefOps(OpTrace):
         unit = lambda t: t.float() * torch.rsqrt(t.float().pow(2).mean(-1, keepdim=True) + eps)
         if pend is not None:
             W = x.shape[1]                       # projections may carry padding columns behind the width
-            y = pend.plain[:, :W].float() if pend.plain is not None else \
-                unit(pend.branch_a[:, :W]) * pend.weight_a + unit(pend.branch_b[:, :W]) * pend.weight_b
+            if pend.experts is not None:
+                y = self._expert_sum(pend.experts, W)
+            elif pend.plain is not None:
+                y = pend.plain[:, :W].float()
+            else:
+                y = unit(pend.branch_a[:, :W]) * pend.weight_a + unit(pend.branch_b[:, :W]) * pend.weight_b
             x = x + pend.coef * y
+            if pend.bias is not None:
+                x = x + pend.bias
         if add is not None:
             x = x + add
         if step is not None:
@@ -253,6 +261,124 @@ class RefOps(OpTrace):
             if one:
                 h[:, x.shape[1]] = 1.0
         return x, h
+
+    # ------------------------------------------------------------------ embedding of a token and the pair it ends
+    def embed_pairs(self, b: StepBatch, rows: int, table, pairs, mul_prev: int, mul_cur: int, norm_w, eps: float, st: ModelState):
+        """normed table[token] + pairs[(previous * mul_prev + token * mul_cur) mod buckets]; the last row of `pairs` belongs to
+        the first token of a sequence.  Keeps every sequence's last token."""
+        out = torch.empty(rows, table.shape[1])
+        buckets = pairs.shape[0] - 1
+        for s in range(b.n_seqs):
+            row0, n, slot, pos0 = (int(v) for v in b.seq_desc[s])
+            prev = int(st.last_token[slot])
+            for r in range(row0, row0 + n):
+                cur = int(b.ids[r])
+                at = buckets if pos0 + r - row0 == 0 else (prev * mul_prev + cur * mul_cur) % buckets
+                x = table[cur].float() + pairs[at].float()
+                out[r] = x * torch.rsqrt(x.pow(2).mean() + eps) * norm_w
+                prev = cur
+            if n > 0:
+                st.last_token[slot] = prev
+        return out
+
+    # ------------------------------------------------------------------ queries, keys and values of an attention
+    def attn_heads(self, proj, s: HeadsSpec, b: StepBatch, kv: KVLayer, st: ModelState, history=None, saved=None):
+        """Projection rows to queries (returned) and keys and values in their pages (ops/specs.py: HeadsSpec).  ``history``: the
+        layer's convolution rows in the state; ``saved``: buffer of the values that later layers mix in."""
+        rows, D, H, G = proj.shape[0], s.dim, s.heads, s.kv_heads
+        x = proj[:, :s.channels].float()
+        if s.conv is not None:
+            x = self._short_conv(x, s, b, history)
+        pos = b.row_pos[:rows].clamp(min=0)
+        unit = lambda t, n: t * torch.rsqrt(t.pow(2).sum(-1, keepdim=True) / n + s.eps)
+        q, k, v = x[:, :H * D], x[:, H * D:(H + G) * D], x[:, (H + G) * D:].reshape(rows, G, D)
+        if s.q_norm is not None:
+            q, k = unit(q, H * s.dim_true) * s.q_norm, unit(k, G * s.dim_true) * s.k_norm
+        q, k = (self._turn_heads(t.reshape(rows, -1, D), pos, s) for t in (q, k))
+        if s.unit:
+            q, k = unit(q, s.dim_true), unit(k, s.dim_true)
+        V = s.vdim_true
+        if s.save:
+            saved[:rows] = v[..., :V].reshape(rows, G * V)
+        if s.mix is not None:
+            v = v.clone()
+            v[..., :V] = (1.0 - s.mix) * v[..., :V] + s.mix * saved[:rows].reshape(rows, G, V)
+        for r in range(rows):
+            at = self._page_of(b, r, st)
+            if at is not None:
+                kv.k[at[0], :, at[1]], kv.v[at[0], :, at[1]] = k[r], v[r]
+        return q.reshape(rows, H * D)
+
+    @staticmethod
+    def _short_conv(x, s: HeadsSpec, b: StepBatch, history):
+        y, back = torch.zeros_like(x), s.taps - 1
+        for i in range(b.n_seqs):
+            row0, n, slot, pos0 = (int(v) for v in b.seq_desc[i])
+            if n <= 0:
+                continue
+            for r in range(n):
+                for j in range(s.taps):
+                    p = pos0 + r - j
+                    if p >= 0:
+                        u = x[row0 + r - j] if j <= r else history[slot, p % back]
+                        y[row0 + r] += s.conv[back - j].float() * u
+            for r in range(max(0, n - back), n):
+                history[slot, (pos0 + r) % back] = x[row0 + r]
+        return y
+
+    @staticmethod
+    def _turn_heads(t, pos, s: HeadsSpec):
+        n = s.freq.numel()
+        ang = pos.double()[:, None, None] * s.freq
+        c, w = (ang.cos() * s.turn_size), (ang.sin() * s.turn_size)
+        first, second = (slice(0, n), slice(n, 2 * n)) if s.halves else (slice(0, 2 * n, 2), slice(1, 2 * n, 2))
+        u, v = t[..., first].double(), t[..., second].double()
+        t = t.clone()
+        t[..., first], t[..., second] = (u * c - v * w).float(), (v * c + u * w).float()
+        return t
+
+    def saved_values(self, rows: int, width: int):
+        return torch.zeros(rows, width)
+
+    # ------------------------------------------------------------------ mixture of experts
+    def moe_route(self, logits, h, s: MoeSpec, b: StepBatch) -> Routed:
+        """Router logits to every row's experts and weights (ops/specs.py: MoeSpec), and the rows of `h` sorted by expert."""
+        rows, n = logits.shape[0], s.experts + s.identity
+        score = torch.softmax(logits[:, :n].float(), -1)
+        choice = score + s.correction
+        best = choice.reshape(rows, s.groups, -1).amax(-1).topk(s.keep, -1).indices
+        open_ = torch.zeros(rows, s.groups, dtype=torch.bool).scatter_(1, best, True).repeat_interleave(n // s.groups, 1)
+        ids = choice.masked_fill(~open_, -math.inf).topk(s.top, -1).indices
+        weight = score.gather(1, ids)
+        weight = weight / (weight.sum(-1, keepdim=True) + 1e-20)
+        real = ids < s.experts
+        order = sorted((int(ids[r, k]), r, k) for r in range(rows) for k in range(s.top) if real[r, k])
+        index = torch.full((rows, s.top), -1, dtype=torch.int32)
+        for at, (_, r, k) in enumerate(order):
+            index[r, k] = at
+        out = Routed(index, weight, (weight * ~real).sum(-1), h[[r for _, r, _ in order]])
+        out.tiles = torch.tensor([e for e, _, _ in order], dtype=torch.long)
+        return out
+
+    def moe_experts(self, routed: Routed, s: MoeSpec):
+        """Outputs of the sorted rows' experts, [sorted rows, n_out]."""
+        K = s.gate_up.shape[1]
+        out = torch.empty(routed.inputs.shape[0], s.n_out)
+        for e in routed.tiles.unique().tolist():
+            at = routed.tiles == e
+            y = routed.inputs[at].float() @ s.gate_up.reshape(s.experts, 2 * s.ff, K)[e].float().T
+            out[at] = (F.silu(y[:, 0::2]) * y[:, 1::2]) @ s.down.reshape(s.experts, s.n_out, s.ff)[e].float().T
+        return out
+
+    @staticmethod
+    def _expert_sum(e: ExpertSum, W: int):
+        r = e.routed
+        y = r.identity[:, None] * e.h[:, :W].float()
+        for k in range(r.index.shape[1]):
+            at = r.index[:, k].long()
+            got = at >= 0
+            y[got] = y[got] + r.weight[got, k][:, None] * e.y[at[got], :W]
+        return y if e.shared is None else y + e.shared[:, :W]
 
     # ------------------------------------------------------------------ parallel residual streams
     def stream_norm(self, x, pend: Optional[StreamWrite], *, read=None, norm_w=None, eps: float, width: int = 0, name: str = "",
@@ -303,7 +429,7 @@ class RefOps(OpTrace):
             slot, p = int(b.row_slot[r]), int(b.row_pos[r])
             if slot < 0:
                 continue
-            tok = torch.arange(spec.first_visible(p), p + 1)
+            tok = spec.visible(p)
             pages = st.block_table[slot, tok // pt].long()
             K = kv.k[pages, :, tok % pt].float().repeat_interleave(H // spec.kv_heads, 1)
             V = kv.v[pages, :, tok % pt].float().repeat_interleave(H // spec.kv_heads, 1)

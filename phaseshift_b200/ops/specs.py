@@ -3,7 +3,7 @@ from __future__ import annotations
 
 import math
 from dataclasses import dataclass
-from typing import Optional
+from typing import Optional, Tuple
 
 import torch
 
@@ -13,7 +13,8 @@ class AttnSpec:
     """Softmax attention over paged keys and values.
 
     ``chunk`` > 0: position i sees positions j <= i of its own block of `chunk` positions (blocks counted from position 0).
-    ``window`` > 0: position i sees positions j with i - j < window.
+    ``window`` > 0: position i sees positions j with i - j < window, and with ``keep_first`` > 0 the first `keep_first` positions of
+    its sequence as well.
     ``sink`` (f32 [heads]): one more term exp(sink[h]) in head h's denominator.
     ``temp_coef``, ``temp_every``: scores of a query at position p are multiplied by 1 + coef ln(floor((p + 1) / every) + 1).
     ``bias`` (f32 [heads, distances]): added to the score of a key at distance i - j; the last entry holds for every larger one.
@@ -33,10 +34,16 @@ class AttnSpec:
     temp_coef: float = 0.0
     temp_every: float = 1.0
     bias: Optional[torch.Tensor] = None
+    keep_first: int = 0
 
     def first_visible(self, pos: int) -> int:
+        """First position of the run that ends at `pos` itself (kept first positions lie before it)."""
         lo = pos // self.chunk * self.chunk if self.chunk > 0 else 0
         return max(lo, pos - self.window + 1) if self.window > 0 else lo
+
+    def visible(self, pos: int) -> torch.Tensor:
+        lo = self.first_visible(pos)
+        return torch.cat([torch.arange(min(self.keep_first, lo)), torch.arange(lo, pos + 1)])
 
 
 def distance_bias_table(table: torch.Tensor, far: float) -> torch.Tensor:
@@ -54,6 +61,110 @@ def distance_bias_table(table: torch.Tensor, far: float) -> torch.Tensor:
             buckets.append(min(rows - 1, half + math.floor(math.log(n / half) / math.log(far / half) * (rows - half))))
         n += 1
     return table.float()[torch.tensor(buckets, device=table.device)].T.contiguous()
+
+
+def rotation_frequencies(base: float, dims: int) -> torch.Tensor:
+    """f64 [dims / 2], radians per position of every rotated pair."""
+    return base ** (-torch.arange(dims // 2, dtype=torch.float64) * 2.0 / dims)
+
+
+def stepped_frequencies(freq: torch.Tensor, factor: float, low: float, high: float, original: float) -> torch.Tensor:
+    """Llama 3.1's scaling by wavelength: pairs that turn at least `high` times within the original length keep their frequency,
+    those that turn at most `low` times are slowed by the factor, the ones between are blended."""
+    turns = original * freq / (2.0 * math.pi)
+    if high == low:
+        return torch.where(turns > high, freq, freq / factor)
+    keep = ((turns - low) / (high - low)).clamp(0.0, 1.0)
+    return (1.0 - keep) * freq / factor + keep * freq
+
+
+def ramped_frequencies(freq: torch.Tensor, base: float, factor: float, original: float, fast: float, slow: float) -> Tuple[torch.Tensor, float]:
+    """YaRN's scaling by pair: a ramp from the pair that turns `fast` times within the original length (kept) to the one that
+    turns `slow` times (slowed by the factor).  Returns the frequencies and the factor on sine and cosine."""
+    dims = 2 * freq.numel()
+
+    def pair_of(turns: float) -> float:
+        return dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(base))
+    lo, hi = max(math.floor(pair_of(fast)), 0), min(math.ceil(pair_of(slow)), dims - 1)
+    ramp = ((torch.arange(freq.numel(), dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+    return freq / factor * ramp + freq * (1.0 - ramp), 0.1 * math.log(factor) + 1.0
+
+
+@dataclass
+class HeadsSpec:
+    """From a projection row [q heads | k heads | v heads] to the queries, keys and values of an attention, in this order, each
+    part optional:
+
+    ``conv`` ([taps, channels], the projection's type; the last tap is the row's own): a causal convolution over time on every
+    channel; the sequence's last taps - 1 rows are state (runtime/state.py: ConvSpec).
+    ``q_norm``, ``k_norm`` (f32 [heads * dim], [kv_heads * dim]): norm over all heads at once.
+    ``freq`` (f64 [pairs]): the first 2 * pairs dimensions of every query and key head turn, neighbours together or (``halves``)
+    dimension i with i + pairs; ``turn_size`` multiplies sine and cosine.
+    ``unit``: each query and key head is divided by its root mean square.
+    ``mix``: values become (1 - mix) v + mix (values that an earlier layer of the step has saved); ``save``: this layer's are
+    the ones that later layers mix in."""
+    heads: int
+    kv_heads: int
+    dim: int                    # the engine's (padded with zeros), as in AttnSpec
+    dim_true: int
+    vdim_true: int
+    eps: float
+    freq: torch.Tensor
+    halves: bool = False
+    turn_size: float = 1.0
+    unit: bool = False
+    conv: Optional[torch.Tensor] = None
+    q_norm: Optional[torch.Tensor] = None
+    k_norm: Optional[torch.Tensor] = None
+    mix: Optional[float] = None
+    save: bool = False
+
+    @property
+    def taps(self) -> int:
+        return 1 if self.conv is None else self.conv.shape[0]
+
+    @property
+    def channels(self) -> int:
+        return (self.heads + 2 * self.kv_heads) * self.dim
+
+
+@dataclass
+class MoeSpec:
+    """Mixture of feed-forward experts with (silu gate) * up.  A token's scores are the softmax of its router logits over
+    experts and, behind them, `identity` experts that return their input; it goes to the `top` largest of score + correction
+    among the `keep` best of `groups` equal groups of neighbours (a group counts as its best member), weighted by their scores
+    divided by the sum of these."""
+    experts: int
+    identity: int
+    top: int
+    groups: int
+    keep: int
+    ff: int                     # columns of an expert's activation (engine size)
+    n_out: int                  # output columns (engine size)
+    correction: torch.Tensor    # f32 [experts + identity]
+    gate_up: torch.Tensor       # [experts * 2 ff, K], rows alternate gate, up
+    down: torch.Tensor          # [experts * n_out, ff]
+
+
+@dataclass
+class Routed:
+    """Where the rows of a step go: expert contributions in rows sorted by expert."""
+    index: torch.Tensor         # int32 [rows, top]: sorted row of the contribution, -1: none
+    weight: torch.Tensor        # f32 [rows, top]
+    identity: torch.Tensor      # f32 [rows]: weight of the input itself
+    inputs: torch.Tensor        # [sorted rows, K]
+    tiles: Optional[torch.Tensor] = None     # kernel-side list of (expert, first row, rows)
+    tile_rows: int = 0
+    max_tiles: int = 0
+
+
+@dataclass
+class ExpertSum:
+    """Output of a mixture layer before its sum: sum_k weight[k] y[index[k]] + identity * h (+ shared)."""
+    routed: Routed
+    y: torch.Tensor             # f32 [sorted rows, width (+ padding columns)]
+    h: torch.Tensor             # the layer's normed input [rows, width (+ padding columns)]
+    shared: Optional[torch.Tensor] = None    # f32 [rows, width (+ padding columns)]
 
 
 @dataclass
@@ -131,13 +242,15 @@ class GlaSpec:
 @dataclass
 class Pending:
     """What the next residual update still has to add: the normed sum of two branches (each [rows, width] with its norm
-    weight) or a plain projection output, times `coef`."""
+    weight), a plain projection output or a mixture's sum, times `coef`; and a `bias` vector (f32 [width])."""
     coef: float
     branch_a: Optional[torch.Tensor] = None
     weight_a: Optional[torch.Tensor] = None
     branch_b: Optional[torch.Tensor] = None
     weight_b: Optional[torch.Tensor] = None
     plain: Optional[torch.Tensor] = None
+    experts: Optional[ExpertSum] = None
+    bias: Optional[torch.Tensor] = None
 
 
 @dataclass

@@ -4,8 +4,8 @@ Policy follows the reference (docs/developer/prefix_cache.md:27-141, src/phasesh
 prefix_cache.cpp): separate cache storage, no refcount / copy-on-write, restore = device-to-device copy
 into the request's own pages; lookup = longest stored sequence that is a strict prefix of the prompt;
 LRU eviction; entries shorter than ``min_tokens`` or larger than the capacity are skipped silently.
-A snapshot holds, for the first n tokens: every attention layer's K/V pages (and FP8 scales) and every
-GDN layer's recurrent state + conv history ring, stored in a pool that is allocated once and bounds the cache's
+A snapshot holds, for the first n tokens: every attention layer's K/V pages (and FP8 scales) and everything else the
+sequence keeps in its slot (recurrent state, convolution histories, the last token), stored in a pool that is allocated once and bounds the cache's
 device memory.  All copies are issued on the engine's stream, so no
 extra synchronisation is needed, and every tensor-parallel rank snapshots its own shard.
 """
@@ -23,7 +23,7 @@ from ..core.native import runtime
 class _Snapshot:
     tokens: int
     pages: List[int]  # pool pages holding this prefix's K/V, in block order
-    state_slot: int   # row of the pooled GDN state
+    state_slot: int   # row of the pooled per-slot state
     extra: object = None   # caller-owned companion state (e.g. a drafter's context ring), cloned by the caller
 
 
@@ -35,7 +35,7 @@ class PrefixHitInfo:
 
 class PrefixCache:
     """Storage is a POOL allocated once: ``capacity_tokens`` worth of K/V pages per attention layer (plus FP8 scales)
-    and ``max_entries`` recurrent-state rows per GDN layer -- the cache can never hold more device memory than that,
+    and ``max_entries`` rows of the per-slot state -- the cache can never hold more device memory than that,
     whatever is saved (the index evicts by LRU before the pool runs out; a save that still finds no room is skipped)."""
 
     def __init__(self, engine, capacity_tokens: int, max_entries: int = 16, min_tokens: int = 64):
@@ -49,7 +49,7 @@ class PrefixCache:
         self.free_pages: List[int] = list(range(self.pool_pages))
         self.free_slots: List[int] = list(range(max_entries))
         dev = st.device
-        self.kv_pool, self.gdn_pool = [], []
+        self.kv_pool = []
         for l in st.kv:
             if l is None:
                 continue
@@ -61,12 +61,7 @@ class PrefixCache:
             pk = torch.zeros(shp, dtype=l.k.dtype, device=dev)
             pv = pk if l.v is l.k else torch.zeros(shp, dtype=l.k.dtype, device=dev)       # keys that double as the values: one pool
             self.kv_pool.append((pk, pv, ks, vs))
-        for g in st.gdn:
-            if g is None:
-                continue
-            self.gdn_pool.append((torch.zeros((max_entries,) + tuple(g.rec.shape[1:]), dtype=g.rec.dtype, device=dev),
-                                  None if g.conv is None else torch.zeros((max_entries,) + tuple(g.conv.shape[1:]), dtype=g.conv.dtype,
-                                                                           device=dev)))
+        self.slot_pool = [torch.zeros((max_entries,) + tuple(t.shape[1:]), dtype=t.dtype, device=dev) for t in st.slot_tensors()]
         pin = dev.type == "cuda"
         self._h_idx = torch.zeros(2, max(1, st.max_blocks), dtype=torch.long, pin_memory=pin)
         self._d_idx = torch.zeros(2, max(1, st.max_blocks), dtype=torch.long, device=dev)
@@ -75,9 +70,7 @@ class PrefixCache:
         n = 0
         for k, v, ks, vs in self.kv_pool:
             n += (1 if v is k else 2) * k.numel() * k.element_size() + (2 * ks.numel() * ks.element_size() if ks is not None else 0)
-        for rec, conv in self.gdn_pool:
-            n += rec.numel() * rec.element_size() + (conv.numel() * conv.element_size() if conv is not None else 0)
-        return n
+        return n + sum(t.numel() * t.element_size() for t in self.slot_pool)
 
     def _index_pair(self, a: Sequence[int], b: Sequence[int]):
         """Two equally long page lists as device index tensors through one pinned staging buffer (no pageable copy)."""
@@ -130,15 +123,8 @@ class PrefixCache:
             if pks is not None:
                 pks.index_copy_(0, dst, l.k_scale.index_select(0, src))
                 pvs.index_copy_(0, dst, l.v_scale.index_select(0, src))
-        gi = 0
-        for g in st.gdn:
-            if g is None:
-                continue
-            rec, conv = self.gdn_pool[gi]
-            gi += 1
-            rec[ss].copy_(g.rec[slot])
-            if conv is not None:
-                conv[ss].copy_(g.conv[slot])
+        for pooled, t in zip(self.slot_pool, st.slot_tensors()):
+            pooled[ss].copy_(t[slot])
         self.snaps[entry] = _Snapshot(n, mine, ss, extra)
         self.stats["saved_tokens"] += n
         return True
@@ -161,15 +147,8 @@ class PrefixCache:
             if pks is not None:
                 l.k_scale.index_copy_(0, dst, pks.index_select(0, src))
                 l.v_scale.index_copy_(0, dst, pvs.index_select(0, src))
-        gi = 0
-        for g in st.gdn:
-            if g is None:
-                continue
-            rec, conv = self.gdn_pool[gi]
-            gi += 1
-            g.rec[slot].copy_(rec[snap.state_slot])
-            if conv is not None:
-                g.conv[slot].copy_(conv[snap.state_slot])
+        for pooled, t in zip(self.slot_pool, st.slot_tensors()):
+            t[slot].copy_(pooled[snap.state_slot])
         self.stats["restored_tokens"] += snap.tokens
         return snap.extra
 

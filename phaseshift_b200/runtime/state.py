@@ -14,6 +14,8 @@ include/phaseshift/models/qwen35/state/paged_kv_pool.h:59-140):
   A shared spec (values are the keys) has one pool: ``v`` is ``k``.
 * GDN conv history per GDN layer: ``[slots, Hv, ring, 2*Dk+Dv]`` bf16, position p in slot p % ring.
 * GDN recurrent state per GDN layer: ``[slots, Hv, Dk, Dv]`` f32 (reference: gdn_state_pool.h:16-105).
+* Short-convolution history of an attention layer: ``[slots, taps - 1, channels]``, position p in row p % (taps - 1).
+* Last token of every sequence, for models whose embedding looks back: ``[slots]`` int32.
 * Block table: ``[slots, max_blocks]`` int32, -1 = unmapped.
 
 Sizing rules follow docs/developer/runtime.md:109-119:
@@ -61,9 +63,17 @@ class RecurrentSpec:
 
 
 @dataclass(frozen=True)
+class ConvSpec:
+    """Rows before the current one that a short convolution over a layer's projection looks back to."""
+    channels: int
+    history: int
+
+
+@dataclass(frozen=True)
 class RunSpec:
     kv: Optional[KVSpec]
     rec: Optional[RecurrentSpec]
+    conv: Optional[ConvSpec] = None
 
 
 @dataclass
@@ -138,15 +148,18 @@ class ModelState:
         scaled = self.kv_fmt != 0                    # pools with an fp32 scale per (page, head, token)
         self.kv: List[Optional[KVLayer]] = []
         self.gdn: List[Optional[GdnLayerState]] = []
+        self.conv: List[Optional[torch.Tensor]] = []
         self.arenas = arenas
         esz = lambda dt: torch.empty(0, dtype=dt).element_size()
         row_elems = lambda s: kv_row_bytes("nvfp4", s.dim) if self.kv_fmt == 2 else s.dim       # last extent of the pools
         kv_need = sum((1 if s.shared else 2) * self.num_pages * s.heads * pt * (row_elems(s) * esz(kvt) + (4 if scaled else 0)) + 1024
                       for s in kv_specs)
-        st_need = sum(sc.max_slots * s.heads * (sc.conv_ring * s.conv_channels * esz(act_dtype)
+        conv_specs = [s.conv for s in self.specs if s.conv is not None and s.conv.history > 0]
+        st_need = sum(sc.max_slots * c.history * c.channels * esz(act_dtype) + 1024 for c in conv_specs)
+        st_need += sum(sc.max_slots * s.heads * (sc.conv_ring * s.conv_channels * esz(act_dtype)
                                                 + s.dk * s.dv * 4 * (2 if sc.spec_rows > 0 else 1)) + 1024 for s in rec_specs)
         kv_arena = arenas.get("kv", kv_need + (2 << 20)) if arenas is not None and kv_specs else None
-        st_arena = arenas.get("state", st_need + (2 << 20)) if arenas is not None and rec_specs else None
+        st_arena = arenas.get("state", st_need + (2 << 20)) if arenas is not None and (rec_specs or conv_specs) else None
 
         def pool(arena, shape, dtype, fill=0):
             if arena is None:
@@ -172,6 +185,10 @@ class ModelState:
                 rec = GdnLayerState(conv, main, alt)
             self.kv.append(kv)
             self.gdn.append(rec)
+            c = spec.conv
+            self.conv.append(pool(st_arena, (sc.max_slots, c.history, c.channels), act_dtype) if c is not None and c.history > 0 else None)
+        self.last_token = (torch.zeros(sc.max_slots, dtype=torch.int32, device=device)
+                           if getattr(cfg, "keeps_last_token", False) else None)
         self.block_table = torch.full((sc.max_slots, self.max_blocks), -1, dtype=torch.int32, device=device)
         self.status = torch.zeros(1, dtype=torch.int32, device=device)
 
@@ -184,16 +201,26 @@ class ModelState:
                     n += 2 * l.k_scale.numel() * 4
         return n
 
+    def slot_tensors(self) -> List[torch.Tensor]:
+        """Everything a sequence keeps outside its pages: tensors whose first extent is the slot."""
+        out = []
+        for g in self.gdn:
+            if g is not None:
+                out.append(g.rec)
+                if g.conv is not None:
+                    out.append(g.conv)
+        out += [c for c in self.conv if c is not None]
+        if self.last_token is not None:
+            out.append(self.last_token)
+        return out
+
     def reset_slot(self, slot: int) -> None:
-        """Fresh sequence: zero recurrent state (conv history needs no clearing: taps before position 0
-        are defined as zero by the kernels)."""
+        """Fresh sequence: zero recurrent state (convolution histories and the last token need no clearing: what lies before
+        position 0 is defined by the kernels)."""
         for g in self.gdn:
             if g is not None:
                 g.rec[slot].zero_()
 
     def copy_slot(self, dst: int, src: int) -> None:
-        for g in self.gdn:
-            if g is not None:
-                g.rec[dst].copy_(g.rec[src])
-                if g.conv is not None:
-                    g.conv[dst].copy_(g.conv[src])
+        for t in self.slot_tensors():
+            t[dst].copy_(t[src])
