@@ -15,14 +15,17 @@ struct AttnOptions {
     int bias_len;
     int gate_per_head;           // the sigmoid gate is one number per head instead of one per element
     const float* sink;           // [Hq] or null: exp(sink[h]) joins head h's denominator
+    int keep_first;              // > 0: the first `keep_first` positions of the sequence are seen besides the window or block
 };
 
-// First position that a query at `pos` sees.
+// First position of the run up to `pos` itself that a query at `pos` sees (kept first positions lie before it).
 __device__ __forceinline__ int attn_first(const AttnOptions& o, int pos) {
     int lo = o.chunk > 0 ? pos / o.chunk * o.chunk : 0;
     if (o.window > 0) lo = max(lo, pos - o.window + 1);
     return lo;
 }
+// Whether a query whose run begins at `lo` sees position `tok` (not later than the query).
+__device__ __forceinline__ bool attn_sees(const AttnOptions& o, int lo, int tok) { return tok >= lo || tok < o.keep_first; }
 __device__ __forceinline__ float attn_temperature(const AttnOptions& o, int pos) {
     if (o.temp_coef == 0.f) return 1.f;
     return 1.f + o.temp_coef * logf((float)(floor((double)(pos + 1) / (double)o.temp_every) + 1.0));
@@ -39,7 +42,7 @@ inline AttnOptions attn_options(const void* p) {
     return o;
 }
 inline bool attn_options_ok(const AttnOptions& o) {
-    return o.chunk >= 0 && o.window >= 0 && (o.bias == nullptr || o.bias_len > 0) && o.temp_every > 0.f;
+    return o.chunk >= 0 && o.window >= 0 && o.keep_first >= 0 && (o.bias == nullptr || o.bias_len > 0) && o.temp_every > 0.f;
 }
 // Scores need more than the scale before their maximum is taken.
 inline bool attn_transforms_scores(const AttnOptions& o) { return o.bias != nullptr || o.temp_coef != 0.f; }

@@ -193,7 +193,7 @@ PS_API int ps_latent_gather(const void* pool, int KR, int R, const void* block_t
                             cudaStream_t stream) {
     using namespace ps;
     const AttnOptions opt = attn_options(options);
-    if (rows <= 0 || rows % kTcTok || n_seqs <= 0 || KR % 8 || R % 8 || !attn_options_ok(opt)) return (int)cudaErrorInvalidValue;
+    if (rows <= 0 || rows % kTcTok || n_seqs <= 0 || KR % 8 || R % 8 || !attn_options_ok(opt) || opt.keep_first > 0) return (int)cudaErrorInvalidValue;
     LatentGatherArgs a;
     a.pool = (const uint4*)pool; a.row16 = (KR + R) / 8; a.lat16 = KR / 8; a.block_table = (const int*)block_table; a.max_blocks = max_blocks;
     a.page_tokens = page_tokens; a.num_pages = num_pages; a.seqs = (const int*)seqs; a.n_seqs = n_seqs; a.min_rows = min_rows; a.opt = opt;
@@ -215,7 +215,7 @@ PS_API int ps_latent_prefill(const void* q, int q_rows, const void* kv, const vo
     using namespace ps;
     const AttnOptions opt = attn_options(options);
     if (!ps_latent_prefill_ok(dim, R, vdim) || q_rows <= 0 || rows <= 0 || n_seqs <= 0 || max_seq_rows <= 0 || H <= 0 || H > 65535 ||
-        !attn_options_ok(opt) || attn_transforms_scores(opt) || (((uintptr_t)q | (uintptr_t)kv | (uintptr_t)rot) % 16) ||
+        !attn_options_ok(opt) || opt.keep_first > 0 || attn_transforms_scores(opt) || (((uintptr_t)q | (uintptr_t)kv | (uintptr_t)rot) % 16) ||
         (gate != nullptr && (opt.gate_per_head || ((uintptr_t)gate % 16) || ld_gate % 8 || gate_head_stride % 8 || gate_offset % 8)))
         return (int)cudaErrorInvalidValue;
     const int DK = dim + R;

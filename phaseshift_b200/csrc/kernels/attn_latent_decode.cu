@@ -388,7 +388,7 @@ PS_API int ps_latent_decode(const void* q, int q_rows, const void* pool, const v
     using namespace ps;
     const AttnOptions opt = attn_options(options);
     if (!ps_latent_decode_ok(KR, R, page_tokens) || q_rows <= 0 || n_seqs <= 0 || max_rows < 1 || max_rows > 16 || H <= 0 || split_tokens < kTcTok ||
-        split_tokens % kTcTok || splits < 1 || ring < 1 || splits > ring || !attn_options_ok(opt) || attn_transforms_scores(opt) || !(scale > 0.f) ||
+        split_tokens % kTcTok || splits < 1 || ring < 1 || splits > ring || !attn_options_ok(opt) || opt.keep_first > 0 || attn_transforms_scores(opt) || !(scale > 0.f) ||
         (((uintptr_t)q | (uintptr_t)pool | (uintptr_t)part_acc) % 16))
         return (int)cudaErrorInvalidValue;
     LatentDecodeArgs a;

@@ -295,7 +295,10 @@ __global__ void __launch_bounds__(kPfThreads) attn_prefill_async_kernel(const At
     const int t = threadIdx.x, warp = t >> 5, lane = t & 31;
     bool bad = false;
 
-    const int t_first = attn_first(a.opt, pos_q0) / kPfTok * kPfTok;      // tile of the first token the first row sees
+    const int t_run = attn_first(a.opt, pos_q0) / kPfTok * kPfTok;        // tile of the first token of the first row's run
+    const int keep = a.opt.keep_first;
+    const int t_first = keep > 0 ? 0 : t_run;
+    auto next_tile = [&](int t0) { return t0 + kPfTok >= keep && t0 + kPfTok < t_run ? t_run : t0 + kPfTok; };
     issue_tile<D>(a, a.k_pool, sK, slot, kvh, t_first, kv_end, bad);
     issue_tile<D>(a, a.v_pool, sV, slot, kvh, t_first, kv_end, bad);
     for (int p = t; p < kPfRows * (D / 8); p += kPfThreads) {
@@ -314,8 +317,9 @@ __global__ void __launch_bounds__(kPfThreads) attn_prefill_async_kernel(const At
     const float row_scale[2] = {a.scale_log2 * attn_temperature(a.opt, rpos0), a.scale_log2 * attn_temperature(a.opt, rpos0 + 8)};
     const int warp_lo = attn_first(a.opt, pos_q0 + warp * 16);              // no row of this warp sees an earlier token
 
-    for (int t0 = t_first; t0 < kv_end; t0 += kPfTok) {
-        const bool live = t0 <= pos_q0 + warp * 16 + 15 && t0 + kPfTok > warp_lo;       // some row of this warp sees this tile
+    for (int t0 = t_first, t1; t0 < kv_end; t0 = t1) {
+        t1 = next_tile(t0);
+        const bool live = t0 <= pos_q0 + warp * 16 + 15 && (t0 + kPfTok > warp_lo || t0 < keep);       // some row of this warp sees this tile
         cp_async_wait<1>();                                     // K(t) has landed (V(t) may still be in flight)
         __syncthreads();
         float s[kPfTok / 8][4];
@@ -336,7 +340,7 @@ __global__ void __launch_bounds__(kPfThreads) attn_prefill_async_kernel(const At
             }
         }
         __syncthreads();                                        // every warp is done with the K tile
-        issue_tile<D>(a, a.k_pool, sK, slot, kvh, t0 + kPfTok, kv_end, bad);
+        issue_tile<D>(a, a.k_pool, sK, slot, kvh, t1, kv_end, bad);
         uint32_t pf[kPfTok / 16][4];
         float alpha[2] = {1.f, 1.f};
         if (live) {
@@ -348,7 +352,7 @@ __global__ void __launch_bounds__(kPfThreads) attn_prefill_async_kernel(const At
                     const int tok = t0 + 8 * j + (lane & 3) * 2 + (e & 1);
                     float v = s[j][e] * row_scale[e >> 1];
                     if (a.transform) v = fmaf(attn_bias(a.opt, h, max(rpos0 + (e >> 1) * 8 - tok, 0)), 1.4426950408889634f, v);
-                    if (tok > rpos0 + (e >> 1) * 8 || tok < lo[e >> 1]) v = -1.0e30f;
+                    if (tok > rpos0 + (e >> 1) * 8 || !attn_sees(a.opt, lo[e >> 1], tok)) v = -1.0e30f;
                     s[j][e] = v;
                     mx[e >> 1] = fmaxf(mx[e >> 1], v);
                 }
@@ -391,7 +395,7 @@ __global__ void __launch_bounds__(kPfThreads) attn_prefill_async_kernel(const At
             }
         }
         __syncthreads();                                        // every warp is done with the V tile
-        issue_tile<D>(a, a.v_pool, sV, slot, kvh, t0 + kPfTok, kv_end, bad);
+        issue_tile<D>(a, a.v_pool, sV, slot, kvh, t1, kv_end, bad);
     }
     cp_async_wait<0>();
     if (bad) set_status(a.status, PS_DEV_BAD_INDEX);

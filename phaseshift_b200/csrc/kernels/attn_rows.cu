@@ -75,8 +75,11 @@ __global__ void __launch_bounds__(kArThreads) attn_rows_kernel(const AttnRowsArg
     const float scale = a.scale * attn_temperature(a.opt, pos);
     float m = a.opt.sink != nullptr ? a.opt.sink[h] : -3.0e38f;
     float l = a.opt.sink != nullptr ? 1.f : 0.f;
-    for (int t0 = lo; t0 <= pos; t0 += kArTile) {
-        const int n = min(kArTile, pos + 1 - t0);
+    // the kept first positions, then the run up to the query itself
+    const int kept = min(a.opt.keep_first, lo);
+    for (int t0 = kept > 0 ? 0 : lo, t1; t0 <= pos; t0 = t1) {
+        const int end = t0 < kept ? kept : pos + 1, n = min(kArTile, end - t0);
+        t1 = t0 + n == kept ? lo : t0 + n;
         __syncthreads();
         if (t < n) {
             const int tok = t0 + t, page = a.block_table[(size_t)slot * a.max_blocks + tok / a.page_tokens];

@@ -175,7 +175,9 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
     const int* sd = a.seqs + 4 * blockIdx.z;
     const int row_start = sd[0], n_rows = sd[1], slot = sd[2], pos_start = sd[3];
     const int G = a.Hq / a.Hkv;
-    int r_begin, nq, h, kvh, pos_q0, kv_end, t_first, T;
+    // tiles of the CTA: `n_keep` tiles of kept first positions from tile `keep0` on, then those from `t_first` on, T in all
+    int r_begin, nq, h, kvh, pos_q0, kv_end, t_first, T, keep0 = 0, n_keep = 0;
+    const int keep_tiles = EXPANDED ? 0 : (a.opt.keep_first + kTcTok - 1) / kTcTok;
     if constexpr (DEC) {
         if (slot < 0 || n_rows <= 0 || n_rows > a.dec_max_rows) return;
         r_begin = 0; nq = 8 * n_rows; kvh = blockIdx.y; h = kvh * G;
@@ -183,9 +185,11 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         const int tps = a.split_tokens / kTcTok;                         // tiles per split
         const int t_lo = attn_first(a.opt, pos_q0) / kTcTok;             // tile of the first token any row sees
         const int t_end = min((kv_end + kTcTok - 1) / kTcTok, ((int)blockIdx.x + 1) * tps);
-        t_first = max((int)blockIdx.x * tps, t_lo);
-        if (t_first >= t_end) return;
-        T = t_end - t_first;
+        keep0 = (int)blockIdx.x * tps;
+        t_first = max(keep0, t_lo);
+        n_keep = max(0, min(min(keep_tiles, t_lo), keep0 + tps) - keep0);
+        T = n_keep + max(0, t_end - t_first);
+        if (T <= 0) return;
     } else {
         const int tile = (int)gridDim.x - 1 - (int)blockIdx.x;
         r_begin = tile * kTcRows;
@@ -195,8 +199,10 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         pos_q0 = pos_start + r_begin;
         kv_end = pos_q0 + nq;
         t_first = attn_first(a.opt, pos_q0) / kTcTok;
-        T = (kv_end + kTcTok - 1) / kTcTok - t_first;
+        n_keep = min(keep_tiles, t_first);
+        T = n_keep + (kv_end + kTcTok - 1) / kTcTok - t_first;
     }
+    auto tile_of = [&](int t) { return t < n_keep ? keep0 + t : t_first - n_keep + t; };
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const bool cta_stamp = a.prof != nullptr && threadIdx.x == 0 && blockIdx.x == 0 && blockIdx.y == 0 && blockIdx.z == 0;
     if (cta_stamp) a.prof[15] = clock64();
@@ -270,7 +276,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         for (int t = 0; t < T; ++t) {
             const int b = t & kStageMask;
             int page = 0;
-            const int blk = (t_first + t) * ppt + pg;
+            const int blk = tile_of(t) * ppt + pg;
             if (!EXPANDED && active && blk * pt < kv_end) {
                 page = bt[blk];
                 if (page < 0 || page >= a.num_pages) { s_bad = 1; page = 0; }
@@ -355,6 +361,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         const float sc = a.scale_log2;
         const int lo = attn_first(a.opt, rp);                        // first token this row sees
         const int lo_max = attn_first(a.opt, kv_end - 1);            // ... and the largest of any row
+        const int keep = EXPANDED ? 0 : a.opt.keep_first;
         [[maybe_unused]] float row_scale = sc, bias_far = 0.f;
         [[maybe_unused]] const float* bias = nullptr;                // this row's head, by distance
         if constexpr (TRANSFORM) {
@@ -374,7 +381,7 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
         for (int t = 0; t < T; ++t) {
             const int b = t & 1;
             const uint32_t ph = (uint32_t)(t >> 1) & 1u;
-            const int tt = t_first + t;                               // tile index within the sequence
+            const int tt = tile_of(t);                                // tile index within the sequence
             const int t0 = tt * kTcTok + half * 32;                   // first token of this thread's columns
             const bool stamp = a.prof != nullptr && threadIdx.x == 0 && blockIdx.x == 0 && blockIdx.y == 0 && blockIdx.z == 0 && t < 32;
             if (stamp) a.prof[t * 16 + 0] = clock64();
@@ -412,8 +419,8 @@ attn_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant_
                 const int to = tt * kTcTok + (half ^ 1) * 32;
 #pragma unroll
                 for (int j = 0; j < 32; ++j) {
-                    if (t0 + j < lo) sr[j] = 0xff800000u;
-                    if (to + j < lo) so[j] = 0xff800000u;
+                    if (t0 + j < lo && t0 + j >= keep) sr[j] = 0xff800000u;
+                    if (to + j < lo && to + j >= keep) so[j] = 0xff800000u;
                 }
             }
             if (tt * kTcTok + kTcTok - 1 > pos_q0) {                  // some row of the tile does not see every token

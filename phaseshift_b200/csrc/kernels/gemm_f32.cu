@@ -7,9 +7,11 @@ namespace ps {
 
 constexpr int kFT = 64, kFK = 16;
 
+__device__ __forceinline__ float gelu_f32(float z) { return z / (1.f + expf(-1.5957691216057308f * fmaf(0.044715f * z * z, z, z))); }
+
 struct GemmF32Args {
     const float* a; int lda; const float* w; int ldw;
-    int M, N, K, epilogue;             // 0 store, 2 SwiGLU, 3 ReGLU, 4 tanh-gelu
+    int M, N, K, epilogue;             // 0 store, 2 SwiGLU, 3 ReGLU, 4 tanh-gelu, 5 GeGLU
     float* out; int ldo;
     long long stride_a, stride_w, stride_o;                   // elements from one product of the batch to the next
     const float* gate; int ldg; long long stride_g;           // optional: the stored value is multiplied by sigmoid(gate)
@@ -44,13 +46,13 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(GemmF32Args g) {
     for (int i = 0; i < 4; ++i) {
         const int m = m0 + ty * 4 + i;
         if (m >= g.M) continue;
-        if (g.epilogue == 2 || g.epilogue == 3) {
+        if (g.epilogue == 2 || g.epilogue == 3 || g.epilogue == 5) {
 #pragma unroll
             for (int j = 0; j < 4; j += 2) {
                 const int n = n0 + tx * 4 + j;
                 if (n + 1 < g.N) {
                     const float gate = acc[i][j];
-                    const float act = g.epilogue == 3 ? fmaxf(gate, 0.f) : gate / (1.f + expf(-gate));
+                    const float act = g.epilogue == 3 ? fmaxf(gate, 0.f) : g.epilogue == 5 ? gelu_f32(gate) : gate / (1.f + expf(-gate));
                     g.out[(size_t)m * g.ldo + (n >> 1)] = act * acc[i][j + 1];
                 }
             }
@@ -60,7 +62,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(GemmF32Args g) {
                 const int n = n0 + tx * 4 + j;
                 if (n >= g.N) continue;
                 float v = acc[i][j];
-                if (g.epilogue == 4) v = v / (1.f + expf(-1.5957691216057308f * fmaf(0.044715f * v * v, v, v)));
+                if (g.epilogue == 4) v = gelu_f32(v);
                 if (g.gate != nullptr) v *= 1.f / (1.f + expf(-g.gate[(size_t)m * g.ldg + n]));
                 g.out[(size_t)m * g.ldo + n] = v;
             }
@@ -73,7 +75,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(GemmF32Args g) {
 PS_API int ps_gemm_f32(const void* a, int lda, const void* w, int ldw, int M, int N, int K, int epilogue, void* out, int ldo,
                        cudaStream_t stream) {
     using namespace ps;
-    if (M <= 0 || N <= 0 || K <= 0 || epilogue < 0 || epilogue == 1 || epilogue > 4 || ((epilogue == 2 || epilogue == 3) && (N & 1)))
+    if (M <= 0 || N <= 0 || K <= 0 || epilogue < 0 || epilogue == 1 || epilogue > 5 || ((epilogue == 2 || epilogue == 3 || epilogue == 5) && (N & 1)))
         return (int)cudaErrorInvalidValue;
     GemmF32Args g{(const float*)a, lda, (const float*)w, ldw, M, N, K, epilogue, (float*)out, ldo, 0, 0, 0, nullptr, 0, 0};
     gemm_f32_kernel<<<dim3((N + kFT - 1) / kFT, (M + kFT - 1) / kFT), 256, 0, stream>>>(g);

@@ -144,7 +144,7 @@ gemm_smallm_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_const
 
 struct SmallMReduceArgs {
     const float* partial; int splits, M, N;
-    int epilogue;            // 0 store, 1 residual, 2 / 3 SwiGLU / ReGLU on interleaved (gate, up) columns, 4 tanh-gelu
+    int epilogue;            // 0 store, 1 residual, 2 / 3 / 5 SwiGLU / ReGLU / GeGLU on interleaved (gate, up) columns, 4 tanh-gelu
     const __nv_bfloat16* residual; int ld_res;
     void* out; int ldo; int out_f32;
 };
@@ -160,9 +160,9 @@ __global__ void gemm_smallm_reduce_kernel(const SmallMReduceArgs a) {
         const float2 p = *reinterpret_cast<const float2*>(a.partial + ((size_t)s * a.M + m) * a.N + c);
         v0 += p.x; v1 += p.y;
     }
-    if (a.epilogue == 2 || a.epilogue == 3) {
+    if (a.epilogue == 2 || a.epilogue == 3 || a.epilogue == 5) {
         const float gt = bf16_to_f32(f32_to_bf16(v0)), up = bf16_to_f32(f32_to_bf16(v1));
-        reinterpret_cast<__nv_bfloat16*>(a.out)[(size_t)m * a.ldo + (c >> 1)] = f32_to_bf16((a.epilogue == 3 ? fmaxf(gt, 0.f) : silu_f(gt)) * up);
+        reinterpret_cast<__nv_bfloat16*>(a.out)[(size_t)m * a.ldo + (c >> 1)] = f32_to_bf16((a.epilogue == 3 ? fmaxf(gt, 0.f) : a.epilogue == 5 ? gelu_tanh_f(gt) : silu_f(gt)) * up);
         return;
     }
     if (a.epilogue == 1) {
@@ -225,7 +225,7 @@ PS_API int ps_gemm_smallm(const void* a, int lda, const void* w, int ldw, int M,
     if (M < 1 || M > 64 || N <= 0 || (N & 1) || K <= 0 || (K % 8) || (lda % 8) || (ldw % 8) || ((uintptr_t)a % 16) ||
         ((uintptr_t)w % 16) || partial == nullptr)
         return (int)cudaErrorInvalidValue;
-    if ((epilogue == 2 || epilogue == 3) && out_f32) return (int)cudaErrorInvalidValue;
+    if ((epilogue == 2 || epilogue == 3 || epilogue == 5) && out_f32) return (int)cudaErrorInvalidValue;
     SmallMArgs g;
     g.M = M; g.N = N; g.K = K;
     g.nb = M <= 16 ? 16 : (M <= 32 ? 32 : 64);

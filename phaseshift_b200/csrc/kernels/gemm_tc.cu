@@ -21,7 +21,7 @@
 
 namespace ps {
 
-enum GemmEpilogue : int { GEPI_STORE = 0, GEPI_RESIDUAL = 1, GEPI_SWIGLU = 2, GEPI_REGLU = 3, GEPI_GELU = 4 };
+enum GemmEpilogue : int { GEPI_STORE = 0, GEPI_RESIDUAL = 1, GEPI_SWIGLU = 2, GEPI_REGLU = 3, GEPI_GELU = 4, GEPI_GEGLU = 5 };
 
 constexpr int kBM = 128, kBK = 64;
 constexpr int kGemmThreads = 192;
@@ -139,7 +139,7 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                 tc::tmem_ld_wait();
                 const int col0 = tile_n * BN + c0;
                 if (row < g.M) {
-                    if (g.epilogue == GEPI_SWIGLU || g.epilogue == GEPI_REGLU) {
+                    if (g.epilogue == GEPI_SWIGLU || g.epilogue == GEPI_REGLU || g.epilogue == GEPI_GEGLU) {
                         // columns (2j, 2j+1) = (gate_j, up_j), each rounded to bf16 like a stored projection
                         __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(g.out) + (size_t)row * g.ldo + (col0 >> 1);
 #pragma unroll
@@ -147,7 +147,7 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                             if (col0 + 2 * j + 1 < g.N) {
                                 const float gt = bf16_to_f32(f32_to_bf16(__uint_as_float(r[2 * j])));
                                 const float up = bf16_to_f32(f32_to_bf16(__uint_as_float(r[2 * j + 1])));
-                                o[j] = f32_to_bf16((g.epilogue == GEPI_REGLU ? fmaxf(gt, 0.f) : silu_f(gt)) * up);
+                                o[j] = f32_to_bf16((g.epilogue == GEPI_REGLU ? fmaxf(gt, 0.f) : g.epilogue == GEPI_GEGLU ? gelu_tanh_f(gt) : silu_f(gt)) * up);
                             }
                         }
                     } else if (g.vec && g.epilogue != GEPI_RESIDUAL && col0 + 31 < g.N) {
@@ -269,7 +269,7 @@ PS_API int ps_gemm_bf16_tc(const void* a, int lda, const void* w, int ldw, int M
     using namespace ps;
     if (M <= 0 || N <= 0 || K <= 0 || (lda % 8) || (ldw % 8) || (K % 8) || ((uintptr_t)a % 16) || ((uintptr_t)w % 16))
         return (int)cudaErrorInvalidValue;
-    if ((epilogue == GEPI_SWIGLU || epilogue == GEPI_REGLU) && ((N & 1) || out_f32)) return (int)cudaErrorInvalidValue;
+    if ((epilogue == GEPI_SWIGLU || epilogue == GEPI_REGLU || epilogue == GEPI_GEGLU) && ((N & 1) || out_f32)) return (int)cudaErrorInvalidValue;
     GemmArgs g;
     g.M = M; g.N = N; g.K = K; g.epilogue = epilogue; g.residual = (const __nv_bfloat16*)residual; g.ld_res = ld_res;
     g.out = out; g.ldo = ldo; g.out_f32 = out_f32; g.status = (uint32_t*)status;

@@ -32,7 +32,7 @@ namespace ps {
 
 enum WeightFormat : int { W_BF16 = 0, W_NVFP4 = 1, W_MXFP8 = 2 };
 enum LinearPrologue : int { PRO_NONE = 0, PRO_RMSNORM_ONEPLUS = 1, PRO_SIGMOID_GATE = 2 };
-enum LinearEpilogue : int { EPI_STORE = 0, EPI_RESIDUAL = 1, EPI_SWIGLU = 2, EPI_REGLU = 3, EPI_GELU = 4 };     // gated: silu / relu (gate) * up
+enum LinearEpilogue : int { EPI_STORE = 0, EPI_RESIDUAL = 1, EPI_SWIGLU = 2, EPI_REGLU = 3, EPI_GELU = 4, EPI_GEGLU = 5 };     // gated: silu / relu / gelu (gate) * up
 
 constexpr int kTpMaxRanks = 8;
 // Tensor-parallel combine fused into a row-parallel projection's epilogue (one-shot all-reduce over
@@ -428,17 +428,17 @@ template <> struct RowDot<W_MXFP8> {
     }
 };
 
-// Apply the epilogue for one quad (4 consecutive output rows) and one batch row.  GELU (the tanh form, on every output) is a
+// Apply the epilogue for one quad (4 consecutive output rows) and one batch row.  GELU (the tanh form, on every output or on gates) is a
 // template parameter: as a run-time choice beside the others it slowed every streaming projection.
 template <bool GELU = false>
 __device__ __forceinline__ void quad_epilogue(const LinearSmallArgs& a, int n0, int m, const float (&v)[kQuadRows]) {
-    if (a.epilogue == EPI_SWIGLU || a.epilogue == EPI_REGLU) {
+    if (a.epilogue == EPI_SWIGLU || a.epilogue == EPI_REGLU || (GELU && a.epilogue == EPI_GEGLU)) {
         // rows (2j, 2j+1) hold (gate_j, up_j); both rounded to bf16 as separate projections would be
 #pragma unroll
         for (int h = 0; h < kQuadRows / 2; ++h) {
             if (n0 + 2 * h + 1 < a.N) {
                 const float g = bf16_to_f32(f32_to_bf16(v[2 * h])), up = bf16_to_f32(f32_to_bf16(v[2 * h + 1]));
-                const float y = (a.epilogue == EPI_REGLU ? fmaxf(g, 0.f) : silu_f(g)) * up;
+                const float y = (GELU ? gelu_tanh_f(g) : a.epilogue == EPI_REGLU ? fmaxf(g, 0.f) : silu_f(g)) * up;
                 const int j = (n0 >> 1) + h;
                 if (a.out_f32) reinterpret_cast<float*>(a.out)[(size_t)m * a.ldo + j] = y;
                 else reinterpret_cast<__nv_bfloat16*>(a.out)[(size_t)m * a.ldo + j] = f32_to_bf16(y);

@@ -28,7 +28,7 @@ __device__ __forceinline__ void bulk_g2s(void* smem_dst, const void* gsrc, uint3
 }
 
 // VARIANT: the common kernel, greedy sampling fused into the epilogue (ps_linear_stream_argmax), or the tanh form of gelu on every
-// output; a template parameter, so that the kernel every other projection runs compiles to what it is without them.
+// output or gate; a template parameter, so that the kernel every other projection runs compiles to what it is without them.
 enum StreamVariant : int { ST_PLAIN = 0, ST_ARGMAX = 1, ST_GELU = 2 };
 template <int WF, int MT, int VARIANT = ST_PLAIN>
 __global__ void __launch_bounds__(kStThreads, 1) linear_stream_kernel(const LinearSmallArgs a, uint32_t* status,
@@ -342,7 +342,7 @@ PS_API int ps_linear_stream(int wfmt, const void* x, int M, int N, int K, int ld
     stream_init_once();
     if (M < 1 || M > 8 || (K % 32) != 0 || (ldx % 8) != 0 || ((uintptr_t)w_tiled % 16) != 0)
         return (int)cudaErrorInvalidValue;
-    if ((epilogue == EPI_SWIGLU || epilogue == EPI_REGLU) && (N & 1)) return (int)cudaErrorInvalidValue;
+    if ((epilogue == EPI_SWIGLU || epilogue == EPI_REGLU || epilogue == EPI_GEGLU) && (N & 1)) return (int)cudaErrorInvalidValue;
     LinearSmallArgs a;
     a.x = (const __nv_bfloat16*)x; a.M = M; a.N = N; a.K = K; a.ldx = ldx;
     a.w = (const uint8_t*)w_tiled; a.w_gscale = w_gscale;
@@ -358,7 +358,7 @@ PS_API int ps_linear_stream(int wfmt, const void* x, int M, int N, int K, int ld
     } else {
         a.tp.size = 0;
     }
-    if (epilogue == EPI_GELU)              // only unquantised models have it; no tensor-parallel combine
+    if (epilogue == EPI_GELU || epilogue == EPI_GEGLU)              // only unquantised models have it; no tensor-parallel combine
         return wfmt == W_BF16 && tp_combine == nullptr ? stream_dispatch_m<W_BF16, ST_GELU>(a, (uint32_t*)status, stream) : (int)cudaErrorInvalidValue;
     switch (wfmt) {
         case W_BF16: return stream_dispatch_m<W_BF16>(a, (uint32_t*)status, stream);

@@ -148,9 +148,12 @@ __global__ void __launch_bounds__(kAttnThreads) paged_attn_split_kernel(const Pa
     const int G = min(kAttnMaxG, heads_per_kv - g_first), h0 = kvh * heads_per_kv + g_first;
     const int visible = a.row_pos[row] + 1;
     const int lo = visible > 0 ? attn_first(a.opt, visible - 1) : 0;
-    const int tok_end = min(visible, (split + 1) * a.split_tokens);
-    const int tok_begin = max(split * a.split_tokens, lo);
-    if (tok_begin >= tok_end) return;
+    // the split's share of the kept first positions, then of the run up to the query itself
+    const int run_end = min(visible, (split + 1) * a.split_tokens), run_begin = max(split * a.split_tokens, lo);
+    const int kept_end = min(min(a.opt.keep_first, lo), run_end);
+    const bool kept = split * a.split_tokens < kept_end;
+    int tok0 = kept ? split * a.split_tokens : run_begin, tok_end = kept ? kept_end : run_end;
+    if (tok0 >= tok_end) return;
     const int slot = a.row_slot[row];
     const int t = threadIdx.x, warp = t >> 5, lane = t & 31;
 
@@ -167,12 +170,15 @@ __global__ void __launch_bounds__(kAttnThreads) paged_attn_split_kernel(const Pa
 
     bool bad = false;
     TileRegs regs;
-    tile_fetch(a, regs, slot, kvh, tok_begin, tok_end, bad);
-    for (int tok0 = tok_begin; tok0 < tok_end; tok0 += kAttnTile) {
+    tile_fetch(a, regs, slot, kvh, tok0, tok_end, bad);
+    for (bool more = true; more;) {
+        int next0 = tok0 + kAttnTile, next_end = tok_end;
+        if (next0 >= tok_end && tok_end != run_end) { next0 = run_begin; next_end = run_end; }
+        more = next0 < next_end;
         __syncthreads();                       // previous tile fully consumed
         tile_store(a, regs, ks, vs, kscale, vscale);
         __syncthreads();
-        if (tok0 + kAttnTile < tok_end) tile_fetch(a, regs, slot, kvh, tok0 + kAttnTile, tok_end, bad);
+        if (more) tile_fetch(a, regs, slot, kvh, next0, next_end, bad);
 
         // scores: warp g, lane = token
         if (warp < G) {
@@ -226,6 +232,7 @@ __global__ void __launch_bounds__(kAttnThreads) paged_attn_split_kernel(const Pa
                 }
             }
         }
+        tok0 = next0; tok_end = next_end;
     }
     if (bad && t == 0) set_status(a.status, PS_DEV_BAD_INDEX);
     // write partials
@@ -263,16 +270,19 @@ __global__ void paged_attn_merge_kernel(const AttnMergeArgs a) {
     const int visible = a.row_pos[row] + 1;
     if (visible < 0) return;                                            // position -2: a row another kernel of the step owns
     const int n = (visible + a.split_tokens - 1) / a.split_tokens;      // 0 for a padding row
-    const int s0 = visible > 0 ? attn_first(a.opt, visible - 1) / a.split_tokens : 0;
-    auto slot_of = [&](int s) { return RING ? s % a.ring : s; };
+    const int lo = visible > 0 ? attn_first(a.opt, visible - 1) : 0, s0 = lo / a.split_tokens;
+    // splits of kept first positions before those of the run (no ring then)
+    const int ks = RING ? 0 : min((min(a.opt.keep_first, lo) + a.split_tokens - 1) / a.split_tokens, s0);
+    const int first = s0 - ks;                                          // the i-th split of the row, i from `first` on
+    auto slot_of = [&](int i) { return RING ? i % a.ring : i < s0 ? i - first : i; };
     const float sink = a.opt.sink != nullptr ? a.opt.sink[h] : -3.0e38f;
     const float* ml = a.part_ml + ((size_t)row * a.Hq + h) * a.max_splits * 2;
     const float* pa = a.part_acc + ((size_t)row * a.Hq + h) * a.max_splits * a.D;
     float m = sink;
-    for (int s = s0 + d; s < n; s += blockDim.x) m = fmaxf(m, ml[2 * slot_of(s)]);
+    for (int s = first + d; s < n; s += blockDim.x) m = fmaxf(m, ml[2 * slot_of(s)]);
     m = block_max(m, s_red);
     float l = 0.f;
-    for (int s = s0 + d; s < n; s += blockDim.x) {
+    for (int s = first + d; s < n; s += blockDim.x) {
         const int at = slot_of(s);
         const float w = __expf(ml[2 * at] - m);
         s_w[at] = w;
@@ -281,6 +291,7 @@ __global__ void paged_attn_merge_kernel(const AttnMergeArgs a) {
     l = block_sum(l, s_red + 32);      // its barriers also publish s_w
     if (a.opt.sink != nullptr) l += __expf(sink - m);
     float o = 0.f;
+    for (int s = 0; s < ks; ++s) o = fmaf(s_w[s], pa[(size_t)s * a.D + d], o);
     int at = slot_of(s0);
 #pragma unroll 4
     for (int s = s0; s < n; ++s) {
@@ -361,7 +372,7 @@ PS_API int ps_paged_attention_merge_ex(const void* part_acc, const void* part_ml
     using namespace ps;
     const AttnOptions opt = attn_options(options);
     if (rows <= 0 || rows > 65535 || Hq <= 0 || D <= 0 || D > 1024 || max_splits > kAttnMaxSplits || ring < 0 || ring > max_splits ||
-        !attn_options_ok(opt))
+        !attn_options_ok(opt) || (ring > 0 && opt.keep_first > 0))
         return (int)cudaErrorInvalidValue;
     AttnMergeArgs m;
     m.part_acc = (const float*)part_acc; m.part_ml = (const float*)part_ml; m.row_pos = (const int*)row_pos; m.rows = rows; m.Hq = Hq; m.D = D;

@@ -21,19 +21,20 @@ from ..models.qwen35.weights import AttnW, GdnW, LinearW
 from ..runtime.batch import StepBatch
 from ..runtime.state import GdnLayerState, KVLayer, ModelState
 from . import _lib
-from .specs import AttnSpec, GlaSpec, LatentSpec, Pending, StreamWrite
+from .specs import AttnSpec, GlaSpec, HeadsSpec, LatentSpec, MoeSpec, Pending, Routed, StreamWrite
 from ._lib import c_float, c_int, c_ll, ptr
 
 WFMT = {"bf16": 0, "nvfp4": 1, "mxfp8": 2}
 PRO_NONE, PRO_RMSNORM, PRO_SIGMOID_GATE = 0, 1, 2
-EPI_STORE, EPI_RESIDUAL, EPI_SWIGLU, EPI_REGLU, EPI_GELU = 0, 1, 2, 3, 4
+EPI_STORE, EPI_RESIDUAL, EPI_SWIGLU, EPI_REGLU, EPI_GELU, EPI_GEGLU = 0, 1, 2, 3, 4, 5
+GATED = (EPI_SWIGLU, EPI_REGLU, EPI_GEGLU)
 SMALL_M_MAX = 8
 
 
 class AttnOptions(ctypes.Structure):
     """csrc/include/attn_options.cuh: AttnOptions."""
     _fields_ = [("chunk", ctypes.c_int), ("window", ctypes.c_int), ("temp_coef", ctypes.c_float), ("temp_every", ctypes.c_float),
-                ("bias", ctypes.c_void_p), ("bias_len", ctypes.c_int), ("gate_per_head", ctypes.c_int), ("sink", ctypes.c_void_p)]
+                ("bias", ctypes.c_void_p), ("bias_len", ctypes.c_int), ("gate_per_head", ctypes.c_int), ("sink", ctypes.c_void_p), ("keep_first", ctypes.c_int)]
 
     @staticmethod
     def of(s: AttnSpec) -> "AttnOptions":
@@ -41,7 +42,7 @@ class AttnOptions(ctypes.Structure):
             if t is not None and (t.dtype != torch.float32 or not t.is_contiguous() or t.shape[0] != s.heads):
                 raise ValueError("attention biases and sinks are contiguous f32 tensors, one row per head")
         return AttnOptions(s.chunk, s.window, s.temp_coef, s.temp_every, None if s.bias is None else s.bias.data_ptr(),
-                           0 if s.bias is None else s.bias.shape[1], int(s.gate_per_head), None if s.sink is None else s.sink.data_ptr())
+                           0 if s.bias is None else s.bias.shape[1], int(s.gate_per_head), None if s.sink is None else s.sink.data_ptr(), s.keep_first)
 
 
 class CudaOps(OpTrace):
@@ -140,7 +141,7 @@ class CudaOps(OpTrace):
 
     def linear(self, x: torch.Tensor, W: LinearW, *, name: str, norm_w: Optional[torch.Tensor] = None,
                eps: float = 0.0, residual: Optional[torch.Tensor] = None, swiglu: bool = False, reglu: bool = False, gelu: bool = False,
-               out_f32: bool = False, out: Optional[torch.Tensor] = None,
+               geglu: bool = False, out_f32: bool = False, out: Optional[torch.Tensor] = None,
                xn_out: Optional[torch.Tensor] = None, tp_combine=None, ssq_in=None,
                ssq_out: Optional[torch.Tensor] = None, prefetch: Optional[LinearW] = None, tp_scatter=None) -> torch.Tensor:
         """``tp_combine`` (a parallel.tp.TpCombineStruct): the projection is row-parallel and the kernel sums
@@ -152,14 +153,16 @@ class CudaOps(OpTrace):
         bytes of its weights while it drains.
         ``tp_scatter`` (a parallel.tp.TpScatterStruct; tensor-core path with streamed activations only): instead of
         storing to ``out`` the kernel pushes each bf16 output row to the receive buffer of the rank that owns it.
-        ``swiglu`` / ``reglu``: the weight's rows interleave (gate, up) and the output is silu / relu (gate) * up.
+        ``swiglu`` / ``reglu`` / ``geglu``: the weight's rows interleave (gate, up) and the output is silu / relu / tanh-gelu
+        (gate) * up.
         ``gelu``: the tanh form of gelu is applied to every output.
         32-bit weights run in fp32 on the CUDA cores (activation epilogues only)."""
         M, K = x.shape
         if W.fmt == "f32":
-            return self._linear_f32(x, W, name, swiglu, reglu, gelu, out, plain=norm_w is None and residual is None)
+            return self._linear_f32(x, W, name, self._epilogue(swiglu, reglu, gelu, geglu, residual), out, plain=norm_w is None and residual is None)
         assert K == W.K and x.dtype == torch.bfloat16 and x.stride(1) == 1, (x.shape, W.K, x.dtype)
-        n_out = W.N // 2 if swiglu or reglu else W.N
+        epi = self._epilogue(swiglu, reglu, gelu, geglu, residual)
+        n_out = W.N // 2 if epi in GATED else W.N
         if out is None:
             out = self.buf(name, M, n_out, torch.float32 if out_f32 else torch.bfloat16)
         assert out.shape[0] == M and out.shape[1] == n_out and out.stride(1) == 1
@@ -167,8 +170,8 @@ class CudaOps(OpTrace):
             raise ValueError(f"K={W.K} must be a multiple of 32 for the streaming / bf16 tensor-core kernels")
         sel = self.select_linear(W, M)
         if sel == "tc":
-            if reglu or gelu:
-                raise ValueError("the block-scaled projections have no ReGLU or gelu epilogue")
+            if reglu or gelu or geglu:
+                raise ValueError("the block-scaled projections have no ReGLU, GeGLU or gelu epilogue")
             # block-quantised codes straight into the tensor cores (any number of rows)
             return self.linear_bs(x, W, name=name, norm_w=norm_w, eps=eps, residual=residual, swiglu=swiglu,
                                   out_f32=out_f32, out=out, xn_out=xn_out, tp_combine=tp_combine, ssq_in=ssq_in,
@@ -183,10 +186,8 @@ class CudaOps(OpTrace):
                    and not self.exact_rows)
         self.sel_counts["gemm" if (sel == "gemm" or batched) else "stream"] += 1
         if sel == "gemm" or batched:
-            return self.linear_large(x, W, name=name, norm_w=norm_w, eps=eps, residual=residual, swiglu=swiglu,
-                                     reglu=reglu, gelu=gelu, out_f32=out_f32, out=out)
+            return self.linear_large(x, W, norm_w=norm_w, eps=eps, residual=residual, epi=epi, out_f32=out_f32, out=out)
         pro = PRO_RMSNORM if norm_w is not None else PRO_NONE
-        epi = self._epilogue(swiglu, reglu, gelu, residual)
         if W.tiled is None:
             W.make_tiled()
         L = _lib.lib()
@@ -208,10 +209,12 @@ class CudaOps(OpTrace):
         return out
 
     @staticmethod
-    def _epilogue(swiglu: bool, reglu: bool, gelu: bool, residual) -> int:
-        if gelu and residual is not None:
+    def _epilogue(swiglu: bool, reglu: bool, gelu: bool, geglu: bool, residual) -> int:
+        if (gelu or geglu) and residual is not None:
             raise ValueError("a projection has either an activation or a residual in its epilogue")
-        return EPI_SWIGLU if swiglu else EPI_REGLU if reglu else EPI_GELU if gelu else EPI_RESIDUAL if residual is not None else EPI_STORE
+        if swiglu or reglu or geglu:
+            return EPI_SWIGLU if swiglu else EPI_REGLU if reglu else EPI_GEGLU
+        return EPI_GELU if gelu else EPI_RESIDUAL if residual is not None else EPI_STORE
 
     def can_fuse_argmax(self, W: LinearW, M: int) -> bool:
         """True when ``linear_argmax`` can serve these rows: the streaming kernel would be chosen and holds them in one launch."""
@@ -239,21 +242,20 @@ class CudaOps(OpTrace):
         self.sel_counts["stream"] += 1
         return tokens.view(-1)[:M]
 
-    def _linear_f32(self, x: torch.Tensor, W: LinearW, name: str, swiglu: bool, reglu: bool, gelu: bool, out, plain: bool) -> torch.Tensor:
+    def _linear_f32(self, x: torch.Tensor, W: LinearW, name: str, epi: int, out, plain: bool) -> torch.Tensor:
         M, K = x.shape
         if not plain or x.dtype != torch.float32 or K != W.K or x.stride(1) != 1:
             raise ValueError("32-bit projections take fp32 rows and have no fused norm or residual")
         if out is None:
-            out = self.buf(name, M, W.N // 2 if swiglu or reglu else W.N, torch.float32)
+            out = self.buf(name, M, W.N // 2 if epi in GATED else W.N, torch.float32)
         w = W.q.codes
         _lib.call("ps_gemm_f32", ptr(x), c_int(x.stride(0)), ptr(w), c_int(w.stride(0)), c_int(M), c_int(W.N), c_int(K),
-                  c_int(self._epilogue(swiglu, reglu, gelu, None)), ptr(out), c_int(out.stride(0)))
+                  c_int(epi), ptr(out), c_int(out.stride(0)))
         self.launches += 1
         self.sel_counts["f32"] = self.sel_counts.get("f32", 0) + 1
         return out
 
-    def linear_large(self, x: torch.Tensor, W: LinearW, *, name: str, norm_w, eps, residual, swiglu, out_f32, out, reglu=False,
-                     gelu=False):
+    def linear_large(self, x: torch.Tensor, W: LinearW, *, norm_w, eps, residual, epi: int, out_f32, out):
         """Prefill-sized projection: (RMSNorm kernel) -> weight expansion to a bf16 scratch matrix -> tcgen05
         GEMM with the residual / SwiGLU / dtype epilogue fused."""
         M, K = x.shape
@@ -271,7 +273,6 @@ class CudaOps(OpTrace):
             _lib.call("ps_dequant_tiled", c_int(WFMT[W.fmt]), ptr(W.tiled), c_int(W.N), c_int(kp),
                       c_float(W.tensor_scale), ptr(wd), c_int(kp))
             self.launches += 1
-        epi = self._epilogue(swiglu, reglu, gelu, residual)
         if W.rowmajor_bf16 is not None and M <= 64 and W.N % 2 == 0:
             # batched decode: swap-AB split-K weight-streaming GEMM (gemm_smallm.cu)
             L = _lib.lib()
@@ -447,7 +448,7 @@ class CudaOps(OpTrace):
         opt = ctypes.byref(opts)
         gate_t = spec.gate if gate is None else gate
         gate = (ptr(gate_t), c_int(gate_t.stride(0) if gate_t is not None else 0), c_int(spec.gate_head_stride), c_int(spec.gate_offset))
-        if st.kv_fmt != 0 and (spec.chunk > 0 or spec.window > 0 or spec.sink is not None or spec.bias is not None or spec.temp_coef != 0.0
+        if st.kv_fmt != 0 and (spec.chunk > 0 or spec.window > 0 or spec.keep_first > 0 or spec.sink is not None or spec.bias is not None or spec.temp_coef != 0.0
                                or spec.gate_per_head):
             raise ValueError("masks, sinks, score transforms and per-head gates need bf16 or 32-bit pages")
         geom = f"{hq}x{D}"                      # layers of one model may differ in head geometry: one set of buffers for each
@@ -664,6 +665,10 @@ class CudaOps(OpTrace):
         Returns (residual, normed rows or None); the residual lives in one buffer of its own, `x` itself is only overwritten
         when it is that buffer."""
         rows, W = x.shape
+        if pend is not None and pend.bias is not None:
+            if step is not None:
+                raise ValueError("a residual update adds one vector: a step or a bias")
+            step = pend.bias
         changed = pend is not None or add is not None or step is not None
         xo = self.buf("x_res", rows, W, torch.float32) if changed else None
         h = self.buf(name, rows, width, self.act_dtype) if norm_w is not None else None
@@ -673,6 +678,15 @@ class CudaOps(OpTrace):
         if pend is not None:
             a, b, wa, wb, y = pend.branch_a, pend.branch_b, pend.weight_a, pend.weight_b, pend.plain
         ld = lambda t: c_int(t.stride(0) if t is not None else 0)
+        if pend is not None and pend.experts is not None:
+            if add is not None or one or scale != 1.0:
+                raise ValueError("a mixture's sum is followed by a plain norm")
+            e, r = pend.experts, pend.experts.routed
+            _lib.call("ps_residual_norm_experts", ptr(x), ptr(xo), c_int(rows), c_int(W), ptr(r.index), ptr(r.weight), ptr(r.identity),
+                      c_int(r.index.shape[1]), ptr(e.y), ld(e.y), ptr(e.h), ld(e.h), ptr(e.shared), ld(e.shared), c_float(pend.coef), ptr(step),
+                      ptr(norm_w), c_float(eps), ptr(h), c_int(1 if self.act_dtype == torch.float32 else 0), c_int(width))
+            self.launches += 1
+            return xo, h
         _lib.call("ps_residual_norm", ptr(x), ptr(xo), c_int(rows), c_int(W), ptr(a), ld(a), ptr(wa), ptr(b), ld(b), ptr(wb),
                   ptr(y), ld(y), c_float(pend.coef if pend is not None else 0.0), ptr(add), ptr(step), ptr(norm_w), c_float(eps),
                   c_float(scale), ptr(h), c_int(1 if self.act_dtype == torch.float32 else 0), c_int(width), c_int(1 if one else 0))
@@ -711,6 +725,89 @@ class CudaOps(OpTrace):
                   ptr(st.block_table), c_int(st.max_blocks), c_int(st.sc.page_tokens), c_int(st.num_pages), ptr(st.status))
         self.launches += 1
         return q
+
+    # ------------------------------------------------------------------ embedding of a token and the pair it ends
+    def embed_pairs(self, b: StepBatch, rows: int, table: torch.Tensor, pairs: torch.Tensor, mul_prev: int, mul_cur: int, norm_w, eps: float,
+                    st: ModelState) -> torch.Tensor:
+        """normed table[token] + pairs[(previous * mul_prev + token * mul_cur) mod buckets], fp32; the last row of `pairs` belongs
+        to the first token of a sequence.  Keeps every sequence's last token."""
+        W = table.shape[1]
+        out = self.buf("x_embed", rows, W, torch.float32)
+        _lib.call("ps_embed_pairs", ptr(b.ids), ptr(table), ptr(pairs), c_int(1 if table.dtype == torch.float32 else 0), c_int(rows),
+                  c_int(table.shape[0]), c_int(pairs.shape[0] - 1), c_ll(mul_prev), c_ll(mul_cur), ptr(norm_w), c_float(eps), c_int(W),
+                  ptr(b.row_slot), ptr(b.seq_desc), c_int(b.max_seqs if b.graph_static else b.n_seqs), ptr(st.last_token), ptr(out), ptr(st.status))
+        self.launches += 1
+        return out
+
+    # ------------------------------------------------------------------ queries, keys and values of an attention
+    def attn_heads(self, proj: torch.Tensor, s: HeadsSpec, b: StepBatch, kv: KVLayer, st: ModelState, history: Optional[torch.Tensor] = None,
+                   saved: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """Projection rows to queries (returned) and keys and values in their pages (ops/specs.py: HeadsSpec).  ``history``: the
+        layer's convolution rows in the state; ``saved``: buffer of the values that later layers mix in.  One launch."""
+        rows, dt = proj.shape[0], self.act_dtype
+        if st.kv_fmt != 0:
+            raise ValueError("attn_heads appends to bf16 or 32-bit pages")
+        if proj.dtype != dt or (s.conv is not None and s.conv.dtype != dt):
+            raise ValueError("projection rows and convolution weights have the engine's type")
+        q = self.buf(f"attn_q{s.heads}x{s.dim}", rows, s.heads * s.dim, dt)
+        _lib.call("ps_attn_heads", ptr(proj), c_int(proj.stride(0)), c_int(1 if dt == torch.float32 else 0), c_int(rows), c_int(s.heads),
+                  c_int(s.kv_heads), c_int(s.dim), c_int(s.dim_true), c_int(s.vdim_true), c_int(s.freq.numel()), c_int(int(s.halves)),
+                  c_int(int(s.unit)), c_float(s.eps), c_float(s.turn_size), ptr(s.freq), ptr(s.q_norm), ptr(s.k_norm), c_int(s.taps),
+                  ptr(s.conv), ptr(history), c_float(s.mix or 0.0), ptr(saved if s.mix is not None else None), ptr(saved if s.save else None),
+                  ptr(q), ptr(kv.k), ptr(kv.v), ptr(b.row_slot), ptr(b.row_pos), ptr(st.block_table), c_int(st.max_blocks),
+                  c_int(st.sc.page_tokens), c_int(st.num_pages), ptr(b.seq_desc), c_int(b.max_seqs if b.graph_static else b.n_seqs),
+                  ptr(st.status))
+        self.launches += 1
+        return q
+
+    def saved_values(self, rows: int, width: int) -> torch.Tensor:
+        return self.buf(f"saved_values{width}", rows, width, self.act_dtype)
+
+    # ------------------------------------------------------------------ mixture of experts
+    def moe_route(self, logits: torch.Tensor, h: torch.Tensor, s: MoeSpec, b: StepBatch) -> Routed:
+        """Router logits (fp32) to every row's experts and weights (ops/specs.py: MoeSpec), and the rows of `h` sorted by expert."""
+        rows, K = h.shape
+        R, i32, f32 = rows * s.top, torch.int32, torch.float32
+        tile = self._moe_tile(rows, s)
+        max_tiles = R // tile + min(s.experts, R)
+        out = Routed(self.buf(f"moe_index{s.top}", rows, s.top, i32), self.buf(f"moe_weight{s.top}", rows, s.top, f32),
+                     self.buf("moe_same", rows, 1, f32), self.buf(f"moe_x{K}", R + tile, K, self.act_dtype),
+                     self.buf("moe_tiles", 1 + max_tiles, 4, i32), tile, max_tiles)
+        small = rows <= 64
+        pairs = None if small else self.buf(f"moe_pairs{s.top}", rows, 2 * s.top, i32)
+        counts = None if small else self.buf(f"moe_counts{s.experts}", 1, s.experts, i32)
+        _lib.call("ps_moe_route", ptr(logits), c_int(logits.stride(0)), ptr(s.correction), ptr(b.row_slot), c_int(rows), c_int(s.experts),
+                  c_int(s.identity), c_int(s.top), c_int(s.groups), c_int(s.keep), ptr(out.index), ptr(out.weight), ptr(out.identity), ptr(h),
+                  c_int(K * h.element_size()), ptr(out.inputs), ptr(out.tiles), c_int(tile), ptr(pairs), ptr(counts), ptr(self.status))
+        self.launches += 1 if small else 3
+        return out
+
+    def _moe_tile(self, rows: int, s: MoeSpec) -> int:
+        """Rows per tile of the experts' products: all that one expert can get in a small step, else about what it gets on average."""
+        if self.act_dtype == torch.float32:
+            return 64
+        if rows <= 64:
+            return 16 if rows <= 16 else 32 if rows <= 32 else 64
+        return 64 if rows * s.top <= 64 * s.experts else 128
+
+    def moe_experts(self, routed: Routed, s: MoeSpec) -> torch.Tensor:
+        """Outputs of the sorted rows' experts, fp32 [sorted rows, n_out].  Two launches."""
+        x, K, dt = routed.inputs, s.gate_up.shape[1], self.act_dtype
+        R = x.shape[0] - routed.tile_rows
+        act = self.buf(f"moe_act{s.ff}", x.shape[0], s.ff, dt)
+        y = self.buf(f"moe_y{s.n_out}", R, s.n_out, torch.float32)
+
+        def product(a, w, N, K, gated, out):
+            if dt == torch.float32:
+                _lib.call("ps_moe_gemm_f32", ptr(a), ptr(w), c_int(N), c_int(K), c_int(gated), ptr(routed.tiles), c_int(routed.max_tiles), ptr(out),
+                          c_int(out.stride(0)))
+            else:
+                _lib.call("ps_moe_gemm", ptr(a), c_int(a.shape[0]), ptr(w), c_int(s.experts), c_int(N), c_int(K), c_int(gated), ptr(routed.tiles),
+                          c_int(routed.tile_rows), c_int(routed.max_tiles), ptr(out), c_int(out.stride(0)), ptr(self.status))
+            self.launches += 1
+        product(x, s.gate_up, 2 * s.ff, K, 1, act)
+        product(act, s.down, s.n_out, s.ff, 0, y)
+        return y
 
     # ------------------------------------------------------------------ latent attention
     def latent_down(self, proj: torch.Tensor, s: LatentSpec, b: StepBatch, kv: KVLayer, st: ModelState) -> torch.Tensor:
