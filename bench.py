@@ -55,9 +55,9 @@ def _parse():
     ap.add_argument("--serving-slots", type=int, default=32,
                     help="sequence slots of the serving block (fewer than the requests, so that later admissions can hit "
                          "the prefix cache the earlier ones filled)")
-    ap.add_argument("--compare", default="", choices=["", "gebuzen", "luvutar"],
+    ap.add_argument("--compare", default="", choices=["", "gebuzen", "luvutar", "fudulix"],
                     help="instead of the headline workload: prefill and decode of a model family beside the closest other one (Gebuzen: the "
-                         "hybrid decoder; Luvutar: Gebuzen) at equal layer shapes (random bf16 weights, 1 GPU), and the mixers' kernels "
+                         "hybrid decoder; Luvutar: Gebuzen; Fudulix: Luvutar) at equal layer shapes (random bf16 weights, 1 GPU), and the mixers' kernels "
                          "against their rooflines")
     ap.add_argument("--compare-layers", type=int, default=16)
     ap.add_argument("--watchdog", type=int, default=1500,

@@ -1,5 +1,5 @@
 """Throughput of a model family beside the closest other one at equal size (`bench.py --compare gebuzen`: the hybrid decoder;
-`--compare luvutar`: Gebuzen): prefill and decode of a stack of layers of real-model shapes with random bf16 weights, and the
+`--compare luvutar`: Gebuzen; `--compare fudulix`: Luvutar): prefill and decode of a stack of layers of real-model shapes with random bf16 weights, and the
 mixers' kernels alone against their rooflines.
 
 Every kernel row gives its time, the algorithmic bytes and FLOPs of one launch group, and the fraction of the roofline
@@ -37,6 +37,28 @@ def luvutar_pairs(layers: int) -> List[tuple]:
     small.layers = [Layer(narrow(L.mixer), L.ff) for L in small.layers]
     return [("4b", cut(luvutar_4b_config()), cut(gebuzen_4b_config())), ("4b, attention heads of 128, latents of 256", small, None),
             ("27b", cut(luvutar_27b_config()), cut(gebuzen_27b_config()))]
+
+
+def fudulix_pairs(layers: int) -> List[tuple]:
+    """(label, Fudulix configuration, Luvutar configuration) of equal width, attention heads, active feed-forward weights and depth."""
+    from ..models.fudulix.config import ConvAttention, Layer, Mixture, UnitAttention, fudulix_27b_config, fudulix_4b_config
+    from ..models.luvutar.config import luvutar_27b_config, luvutar_4b_config
+
+    def cut(cfg):
+        cfg.layers = cfg.layers[:layers]
+        return cfg
+
+    def narrow(L):
+        """Half the head size, twice the heads; half-size experts, twice as many."""
+        m, c = L.mixer, L.mlp
+        common = (32, 8, 128, 128, 128 ** -0.5, m.window, m.rot_base, m.rot_dims // 2, m.v_mix, m.scaling)
+        mixer = ConvAttention(*common, m.keep_first, m.taps) if isinstance(m, ConvAttention) else UnitAttention(*common)
+        return Layer(mixer, Mixture(512, 124, 16, 8, 4, 4, 1024) if isinstance(c, Mixture) else c)
+
+    small = cut(fudulix_4b_config(name="fudulix-4b-d128"))
+    small.layers = [narrow(L) for L in small.layers]
+    return [("4b", cut(fudulix_4b_config()), cut(luvutar_4b_config())), ("4b, attention heads of 128, experts of 512", small, None),
+            ("27b", cut(fudulix_27b_config()), cut(luvutar_27b_config()))]
 
 
 def gebuzen_pairs(layers: int) -> List[tuple]:
@@ -104,7 +126,7 @@ def model_times(eng: Engine, prompt_tokens: int, steps: int, warmup: int, batch:
         for s in seqs:
             eng.step([SeqRows(s.slot, 0, ids[:prompt_tokens], (prompt_tokens - 1,))], [s])
         for _ in range(3):
-            eng.step([SeqRows(s.slot, s.position, [7], (0,)) for s in seqs], seqs)
+            eng.step([SeqRows(s.slot, s.position, [7 + i], (0,)) for i, s in enumerate(seqs)], seqs)      # (rows that differ in their experts)
         from ..runtime.batch import resolve_row_bucket
         key = [k for k in eng.graphs if not isinstance(k, tuple) and eng.graph_key_bucket(k) == resolve_row_bucket(rows)][0]
         graph = eng.graphs[key]
@@ -279,6 +301,74 @@ def luvutar_kernel_times(eng: Engine, timer: _Flushed, peaks: dict, rows: int, c
     return res
 
 
+def fudulix_kernel_times(eng: Engine, timer: _Flushed, peaks: dict, rows: int, context: int, batch: int) -> Dict[str, dict]:
+    """As `kernel_times`, for both mixers and both feed-forwards.  What a mixture moves and multiplies is counted from the rows its
+    random router sends to every expert."""
+    from ..models.fudulix.weights import MixtureW
+    from ..ops.specs import ExpertSum, Pending
+    hbm, tc = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    ops, st, w = eng.ops, eng.state, eng.runner.w
+    res: Dict[str, dict] = {}
+
+    def add(name, fn, nbytes, flops):
+        us = timer(fn)
+        floor = max(nbytes / hbm, flops / tc) * 1e6
+        res[name] = {"us": round(us, 1), "gb": round(nbytes / 1e9, 4), "gflop": round(flops / 1e9, 2), "roofline_us": round(floor, 2),
+                     "roofline_frac": round(floor / us, 4)}
+
+    def rand(n, width, dtype=torch.bfloat16):
+        return torch.randn(n, width, device=eng.device, dtype=torch.float32).to(dtype)
+
+    W = eng.cfg.hidden_size
+    lc = next(i for i, L in enumerate(w.layers) if L.heads.conv is not None)
+    lu = next(i for i, L in enumerate(w.layers) if L.heads.conv is None)
+    dense = next(L.mlp for L in w.layers if not isinstance(L.mlp, MixtureW))
+    mix = next(L.mlp for L in w.layers if isinstance(L.mlp, MixtureW))
+    m = mix.moe
+    shapes = [("prefill", [(0, rows)]), ("prefill after context", [(context, rows)]), ("decode 1", [(context, 1)]),
+              (f"decode {batch}", [(context, 1)] * batch)]
+    for name, seqs in shapes:
+        b, opened = _batch(eng, seqs)
+        n = b.n_rows
+        for i, kind in ((lu, "attention"), (lc, "attention_2")):
+            L, f = w.layers[i], w.layers[i].attn
+            seen = [[min(q + 1, f.window + min(f.keep_first, max(0, q + 1 - f.window))) for q in range(p, p + k)] for p, k in seqs]
+            pairs, kv_tok = sum(map(sum, seen)), sum(min(p + k, s[0] + k - 1) for (p, k), s in zip(seqs, seen))
+            proj = rand(n, L.in_proj.N)
+            saved = ops.saved_values(n, eng.runner.saved_width)
+            q = ops.attn_heads(proj, L.heads, b, st.kv[i], st, st.conv[i], saved)
+            if name != "prefill after context":
+                io = n * 2 * L.in_proj.N * 2 + 2 * n * eng.runner.saved_width + (L.heads.conv.numel() * 2 if L.heads.conv is not None else 0)
+                add(f"heads of {kind}, {name}", lambda: ops.attn_heads(proj, L.heads, b, st.kv[i], st, st.conv[i], saved), io, 0.0)
+            add(f"{kind}, {name}", lambda: ops.attention(q, f, b, st.kv[i], st, b.max_visible_launch),
+                2 * n * f.heads * f.dim * 2 + kv_tok * 2 * f.kv_heads * f.dim * 2, 4.0 * pairs * f.heads * f.dim)
+        if name != "prefill after context":
+            x, y, h = rand(n, W, torch.float32), rand(n, W, torch.float32), rand(n, mix.router.K)
+            L = w.layers[lu]
+            add("residual + norm, " + name, lambda: ops.residual_norm(x, Pending(1.0, plain=y), norm_w=L.norm1, eps=1e-6, width=h.shape[1], name="bench_h"),
+                n * W * (3 * 4 + 2), 0.0)
+            xg = rand(n, dense.gate_up.K)
+            gu = dense.gate_up
+            add("gate_up, " + name, lambda: ops.linear(xg, gu, name="bench_act", geglu=True), gu.N * gu.k_padded * 2 + n * (gu.K + gu.N // 2) * 2,
+                2.0 * n * gu.N * gu.K)
+            add("router, " + name, lambda: ops.linear(h, mix.router, name="bench_z", out_f32=True),
+                mix.router.N * mix.router.K * 2 + n * (mix.router.K * 2 + mix.router.N * 4), 2.0 * n * mix.router.N * mix.router.K)
+            z = ops.linear(h, mix.router, name="bench_z", out_f32=True)
+            r = ops.moe_route(z, h, m, b)
+            R, used = int((r.index >= 0).sum()), len(set(r.tiles[1:1 + int(r.tiles[0, 0]), 0].tolist()))
+            add("routing, " + name, lambda: ops.moe_route(z, h, m, b), n * (z.shape[1] * 4 + h.shape[1] * 2 + m.top * 8) + R * h.shape[1] * 2, 0.0)
+            K = m.gate_up.shape[1]
+            add("experts, " + name, lambda: ops.moe_experts(r, m),
+                used * 3 * m.ff * K * 2 + R * (K * 2 + 2 * m.ff * 2 + m.n_out * 4), 2.0 * R * (2 * m.ff * K + m.n_out * m.ff))
+            ye = ops.moe_experts(r, m)
+            pend = Pending(1.0, experts=ExpertSum(r, ye, h, y))
+            add("expert sum + norm, " + name, lambda: ops.residual_norm(x, pend, norm_w=L.norm1, eps=1e-6, width=h.shape[1], name="bench_h"),
+                n * W * (3 * 4 + 2) + R * m.n_out * 4 + int((r.identity > 0).sum()) * W * 2, 0.0)
+        for o in opened:
+            eng.close_sequence(o)
+    return res
+
+
 def _prefill_core(ops, q, s, b, st, kv, gate):
     """The attention over keys and values that one call of `latent_attention` has gathered and expanded."""
     out = ops.latent_attention(q, s, b, kv, st, gate)
@@ -292,9 +382,12 @@ def run(peaks: dict, layers: int = 16, prompt_tokens: int = 2048, steps: int = 5
     dev = torch.device("cuda:0")
     timer = _Flushed(dev)
     out = {"layers": layers, "prompt_tokens": prompt_tokens, "batch": batch, "sizes": {}}
-    for label, *cfgs in (luvutar_pairs if which == "luvutar" else gebuzen_pairs)(layers):
+    pairs, names = {"gebuzen": (gebuzen_pairs, ("gebuzen", "hybrid")), "luvutar": (luvutar_pairs, ("luvutar", "gebuzen")),
+                    "fudulix": (fudulix_pairs, ("fudulix", "luvutar"))}[which]
+    kernels = {"luvutar": luvutar_kernel_times, "fudulix": fudulix_kernel_times}
+    for label, *cfgs in pairs(layers):
         row = out["sizes"][label] = {}
-        for name, cfg in zip(("luvutar", "gebuzen") if which == "luvutar" else ("gebuzen", "hybrid"), cfgs):
+        for name, cfg in zip(names, cfgs):
             if cfg is None:
                 continue
             with torch.no_grad():
@@ -305,7 +398,7 @@ def run(peaks: dict, layers: int = 16, prompt_tokens: int = 2048, steps: int = 5
                 if sampler is not None:
                     sampler.begin()
                 t = model_times(eng, prompt_tokens, steps, warmup, batch)
-                k = (luvutar_kernel_times if name == "luvutar" else kernel_times)(eng, timer, peaks, prompt_tokens, prompt_tokens, batch)
+                k = kernels.get(name, kernel_times)(eng, timer, peaks, prompt_tokens, prompt_tokens, batch)
             rd = ew.decode_read_bytes()
             row[name] = {**{a: round(v, 4) for a, v in t.items()},
                          "prefill_tok_s": round(prompt_tokens / t["prefill_ms"] * 1e3), "decode1_tok_s": round(1e3 / t["decode1_ms"], 1),

@@ -139,13 +139,13 @@ def attend(q, k, v, scale, allowed, weights):
 
 
 def mixed_values(v, w, p, m, shared):
-    """`shared` keeps the values of the first layer that takes part."""
+    """`shared` keeps the values of the first layer that takes part (all heads of a token in a row)."""
     if not m["v_mix"]:
         return v
     if "v" not in shared:
         shared["v"] = v
         return v
-    return mix_values(v, shared["v"], w[p + "vmix"])
+    return mix_values(v, shared["v"].reshape(v.shape), w[p + "vmix"])
 
 
 def attention(h, w, p, m, eps, shared):
