@@ -142,13 +142,21 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                     if (g.epilogue == GEPI_SWIGLU || g.epilogue == GEPI_REGLU || g.epilogue == GEPI_GEGLU) {
                         // columns (2j, 2j+1) = (gate_j, up_j), each rounded to bf16 like a stored projection
                         __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(g.out) + (size_t)row * g.ldo + (col0 >> 1);
+                        auto gated = [&](int j) {
+                            const float gt = bf16_to_f32(f32_to_bf16(__uint_as_float(r[2 * j])));
+                            const float up = bf16_to_f32(f32_to_bf16(__uint_as_float(r[2 * j + 1])));
+                            return (g.epilogue == GEPI_REGLU ? fmaxf(gt, 0.f) : g.epilogue == GEPI_GEGLU ? gelu_tanh_f(gt) : silu_f(gt)) * up;
+                        };
+                        if (g.vec && col0 + 31 < g.N) {
+                            uint32_t p[8];
 #pragma unroll
-                        for (int j = 0; j < 16; ++j) {
-                            if (col0 + 2 * j + 1 < g.N) {
-                                const float gt = bf16_to_f32(f32_to_bf16(__uint_as_float(r[2 * j])));
-                                const float up = bf16_to_f32(f32_to_bf16(__uint_as_float(r[2 * j + 1])));
-                                o[j] = f32_to_bf16((g.epilogue == GEPI_REGLU ? fmaxf(gt, 0.f) : g.epilogue == GEPI_GEGLU ? gelu_tanh_f(gt) : silu_f(gt)) * up);
-                            }
+                            for (int j = 0; j < 8; ++j) p[j] = f32x2_to_bf16x2_bits(gated(2 * j), gated(2 * j + 1));
+                            reinterpret_cast<uint4*>(o)[0] = make_uint4(p[0], p[1], p[2], p[3]);
+                            reinterpret_cast<uint4*>(o)[1] = make_uint4(p[4], p[5], p[6], p[7]);
+                        } else {
+#pragma unroll
+                            for (int j = 0; j < 16; ++j)
+                                if (col0 + 2 * j + 1 < g.N) o[j] = f32_to_bf16(gated(j));
                         }
                     } else if (g.vec && g.epilogue != GEPI_RESIDUAL && col0 + 31 < g.N) {
                         if (g.epilogue == GEPI_GELU) {

@@ -31,6 +31,8 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
     extern __shared__ __align__(1024) unsigned char smem_raw[];
     constexpr int kWBytes = kMgM * kMgK * 2, kXBytes = NB * kMgK * 2;
     constexpr uint32_t kCols = NB < 32 ? 32 : NB;
+    cudaTriggerProgrammaticLaunchCompletion();
+    cudaGridDependencySynchronize();
     if ((int)blockIdx.y >= g.tiles[0]) return;
     const int4 tile = reinterpret_cast<const int4*>(g.tiles)[1 + blockIdx.y];
     unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -73,7 +75,7 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
         }
     } else if (warp == 1) {
         if (lane == 0) {
-            constexpr uint32_t idesc = tc::idesc_bf16_f32(kMgM, NB);
+            const uint32_t idesc = tc::idesc_bf16_f32(kMgM, (tile.z + 15) / 16 * 16);
             bool ok = true;
             for (int it = 0; it < k_iters && ok; ++it) {
                 const int s = it % STAGES;
@@ -168,8 +170,7 @@ static int launch_moe_gemm(const CUtensorMap& map_w, const CUtensorMap& map_x, i
         cudaFuncSetAttribute(moe_gemm_kernel<NB, STAGES>, cudaFuncAttributePreferredSharedMemoryCarveout, (int)cudaSharedmemCarveoutMaxShared);
         set = true;
     }
-    moe_gemm_kernel<NB, STAGES><<<dim3((g.N + kMgM - 1) / kMgM, max_tiles), kMgThreads, smem, stream>>>(map_w, map_x, g);
-    return PS_LAUNCH_CHECK();
+    return launch_pdl(moe_gemm_kernel<NB, STAGES>, dim3((g.N + kMgM - 1) / kMgM, max_tiles), dim3(kMgThreads), smem, stream, map_w, map_x, g);
 }
 
 constexpr int kMfT = 64, kMfK = 16;

@@ -24,13 +24,37 @@ struct RouteArgs {
     uint32_t* status;
 };
 
-__device__ __forceinline__ void rt_argmax(float& v, int& i) {
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-        const float ov = __shfl_xor_sync(0xffffffffu, v, o);
-        const int oi = __shfl_xor_sync(0xffffffffu, i, o);
-        if (oi >= 0 && (i < 0 || ov > v || (ov == v && oi < i))) { v = ov; i = oi; }
+// Order-preserving integer of a float (NaN: below everything that counts).
+__device__ __forceinline__ uint32_t rt_key(float v) {
+    const uint32_t u = __float_as_uint(v);
+    return v == v ? (u & 0x80000000u ? ~u : u | 0x80000000u) : 0u;
+}
+constexpr uint32_t kRtNone = 0x007fffffu;            // rt_key(-infinity): nothing above it is left
+
+// The `k` largest of v[0 .. n), one after the other; ties go to the lower index.  Every lane keeps the best of its own elements
+// (lane, lane + 32, ...), only the lane that loses one looks again.  Taken elements become minus infinity; `take(place, index)` runs
+// on all lanes, index -1: nothing is left.
+template <typename F>
+__device__ __forceinline__ void rt_top(float* v, int n, int k, F take) {
+    const int lane = threadIdx.x & 31;
+    uint32_t best = 0;
+    int at = 0;
+    auto look = [&] {
+        best = 0;
+        for (int i = lane; i < n; i += 32) {
+            const uint32_t key = rt_key(v[i]);
+            if (key > best) { best = key; at = i; }
+        }
+    };
+    look();
+    for (int place = 0; place < k; ++place) {
+        const uint32_t top = __reduce_max_sync(0xffffffffu, best);
+        const uint32_t who = __reduce_min_sync(0xffffffffu, best == top ? (uint32_t)at : 0xffffffffu);
+        const bool some = top > kRtNone;
+        take(place, some ? (int)who : -1);
+        if (some && best == top && (uint32_t)at == who) { v[at] = -INFINITY; look(); }
     }
+    __syncwarp();
 }
 
 // One row by one warp; `s` is 3 n floats of its own.  Lane k < top returns place k's choice (-1 when the logits are not finite) and
@@ -57,36 +81,19 @@ __device__ __forceinline__ void route_row(const RouteArgs& a, int row, float* s,
             group[g] = b;
         }
         __syncwarp();
-        for (int k = 0; k < a.keep; ++k) {
-            float v = -INFINITY;
-            int at = -1;
-            for (int g = lane; g < a.groups; g += 32)
-                if (group[g] > v) { v = group[g]; at = g; }
-            rt_argmax(v, at);
-            __syncwarp();
-            if (lane == 0 && at >= 0) group[at] = -INFINITY;           // kept groups end as minus infinity
-            __syncwarp();
-        }
+        rt_top(group, a.groups, a.keep, [](int, int) {});              // kept groups end as minus infinity
         for (int i = lane; i < n; i += 32)
             if (group[i / size] != -INFINITY) choice[i] = -INFINITY;
         __syncwarp();
     }
     id = -1; weight = 0.f;
     float total = 0.f;
-    for (int k = 0; k < a.top; ++k) {
-        float v = -INFINITY;
-        int at = -1;
-        for (int i = lane; i < n; i += 32)
-            if (choice[i] > v) { v = choice[i]; at = i; }
-        rt_argmax(v, at);
-        __syncwarp();
-        if (at >= 0) {
-            if (lane == k) { id = at; weight = score[at]; }
-            total += score[at];
-            if (lane == 0) choice[at] = -INFINITY;
-        }
-        __syncwarp();
-    }
+    rt_top(choice, n, a.top, [&](int place, int at) {
+        if (at < 0) return;
+        const float w = score[at];
+        if (lane == place) { id = at; weight = w; }
+        total += w;
+    });
     if (lane < a.top && id < 0) set_status(a.status, PS_DEV_NONFINITE);
     weight /= total + 1e-20f;
 }
@@ -98,6 +105,7 @@ __device__ __forceinline__ void route_prefix(const RouteArgs& a, F count, int* f
     int rows = 0, tiles = 0;
     for (int e0 = 0; e0 < a.E; e0 += 32) {
         const int e = e0 + lane, c = e < a.E ? count(e) : 0, nt = (c + a.tile_rows - 1) / a.tile_rows;
+        const int per = nt > 0 ? ((c + nt - 1) / nt + 15) / 16 * 16 : 0;                 // an expert's tiles are about equal
         int r = c, t = nt;
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
@@ -108,7 +116,7 @@ __device__ __forceinline__ void route_prefix(const RouteArgs& a, F count, int* f
         if (write_tiles)
             for (int i = 0; i < nt; ++i)
                 reinterpret_cast<int4*>(a.tiles)[1 + tiles + t - nt + i] =
-                    make_int4(e, rows + r - c + i * a.tile_rows, min(a.tile_rows, c - i * a.tile_rows), 0);
+                    make_int4(e, rows + r - c + i * per, max(0, min(per, c - i * per)), 0);
         rows += __shfl_sync(0xffffffffu, r, 31);
         tiles += __shfl_sync(0xffffffffu, t, 31);
     }

@@ -165,12 +165,23 @@ __global__ void residual_norm_kernel(const ResidualNormArgs g) {
 #pragma unroll
                 for (int e = 0; e < VEC; ++e) s.v[e] = fmaf(same, u.v[e], s.v[e]);
             }
-#pragma unroll 4
-            for (int k = 0; k < g.top; ++k) {
-                if (s_at[k] < 0) continue;
-                const FVec<VEC> u = fload<VEC>(g.ye + (size_t)s_at[k] * g.ldye + i);
+            for (int k0 = 0; k0 < g.top; k0 += 4) {                      // four rows' loads in flight together
+                FVec<VEC> u[4];
+                float wk[4];
 #pragma unroll
-                for (int e = 0; e < VEC; ++e) s.v[e] = fmaf(s_w[k], u.v[e], s.v[e]);
+                for (int j = 0; j < 4; ++j) {
+                    const int at = k0 + j < g.top ? s_at[k0 + j] : -1;
+                    wk[j] = at >= 0 ? s_w[k0 + j] : 0.f;
+                    if (at >= 0) u[j] = fload<VEC>(g.ye + (size_t)at * g.ldye + i);
+                    else {
+#pragma unroll
+                        for (int e = 0; e < VEC; ++e) u[j].v[e] = 0.f;
+                    }
+                }
+#pragma unroll
+                for (int j = 0; j < 4; ++j)
+#pragma unroll
+                    for (int e = 0; e < VEC; ++e) s.v[e] = fmaf(wk[j], u[j].v[e], s.v[e]);
             }
 #pragma unroll
             for (int e = 0; e < VEC; ++e) v.v[e] = fmaf(g.coef, s.v[e], v.v[e]);

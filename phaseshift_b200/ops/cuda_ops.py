@@ -18,7 +18,7 @@ import torch
 
 from .trace import OpTrace
 from ..models.qwen35.weights import AttnW, GdnW, LinearW
-from ..runtime.batch import StepBatch
+from ..runtime.batch import ROW_BUCKETS, StepBatch
 from ..runtime.state import GdnLayerState, KVLayer, ModelState
 from . import _lib
 from .specs import AttnSpec, GlaSpec, HeadsSpec, LatentSpec, MoeSpec, Pending, Routed, StreamWrite
@@ -86,6 +86,7 @@ class CudaOps(OpTrace):
         self.force_tc = os.environ.get("PS_FORCE_TC", "0") == "1"   # single-row steps on the tensor-core kernel too
         self.bs_prefetch = os.environ.get("PS_BS_PREFETCH", "1") != "0"
         self._bs_plan_cache: Dict[tuple, bool] = {}
+        self.tickets = torch.zeros(ROW_BUCKETS[-1], dtype=torch.int32, device=device)      # one per sequence, zero between launches
         self.sel_counts: Dict[str, int] = {"tc_resident": 0, "tc_streamed": 0, "stream": 0, "gemm": 0}   # projection calls per kernel
         self.fallbacks: Dict[str, int] = {}
 
@@ -338,6 +339,7 @@ class CudaOps(OpTrace):
             self.bs_flags.zero_()
         if getattr(self, "_amax_state", None) is not None:
             self._amax_state.zero_()              # a fused arg-max launch that did not finish leaves its keys and counter
+        self.tickets.zero_()
         self.status.zero_()
 
     def leaves_row_stats(self, W: LinearW, M: int) -> bool:
@@ -756,7 +758,7 @@ class CudaOps(OpTrace):
                   ptr(s.conv), ptr(history), c_float(s.mix or 0.0), ptr(saved if s.mix is not None else None), ptr(saved if s.save else None),
                   ptr(q), ptr(kv.k), ptr(kv.v), ptr(b.row_slot), ptr(b.row_pos), ptr(st.block_table), c_int(st.max_blocks),
                   c_int(st.sc.page_tokens), c_int(st.num_pages), ptr(b.seq_desc), c_int(b.max_seqs if b.graph_static else b.n_seqs),
-                  ptr(st.status))
+                  ptr(self.tickets), ptr(st.status))
         self.launches += 1
         return q
 
@@ -788,7 +790,8 @@ class CudaOps(OpTrace):
             return 64
         if rows <= 64:
             return 16 if rows <= 16 else 32 if rows <= 32 else 64
-        return 64 if rows * s.top <= 64 * s.experts else 128
+        each = rows * s.top / (s.experts + s.identity)
+        return 64 if each <= 32 else 128
 
     def moe_experts(self, routed: Routed, s: MoeSpec) -> torch.Tensor:
         """Outputs of the sorted rows' experts, fp32 [sorted rows, n_out].  Two launches."""
