@@ -77,9 +77,9 @@ class FudulixRunner:
                 pend = Pending(1.0, plain=ops.linear(ctx, L.o, name="mix_out", out_f32=True))
             if L.mlp is not None:
                 dense = isinstance(L.mlp, DenseW)
+                width = (L.mlp.gate_up if dense else L.mlp.router).K          # (the two kinds have buffers of their own)
                 with ops.range("norm"):
-                    x, h = ops.residual_norm(x, pend, norm_w=L.norm2, eps=eps, width=(L.mlp.gate_up if dense else L.mlp.router).K, one=dense,
-                                             name="h_mlp")
+                    x, h = ops.residual_norm(x, pend, norm_w=L.norm2, eps=eps, width=width, one=dense, name=f"h_mlp{width}")
                 pend = self._dense(L.mlp, h) if dense else self._mixture(L.mlp, h, b)
             if i in tap_layers:
                 x, _ = ops.residual_norm(x, pend, eps=eps)
