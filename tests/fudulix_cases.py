@@ -45,7 +45,7 @@ MIXED = model(301, 75, [(conv(6, 2, 40, 24, 9, 5, 3), moe(10, 33, 3, 3, 2, 2, 50
 # shapes of the tensor-core kernels: heads of 64 to 256 columns, query heads that share key heads, many experts
 WIDE = model(520, 192, [(unit(6, 2, 128, 128, 150, 0.25, rot=32, original=60), dense(160)),
                         (conv(4, 2, 256, 128, 100, 40, 4, base=20.0), moe(30, 64, 4, 4, 2, 2, 96)),
-                        (unit(4, 2, 64, 128, 64, 0.4), moe(16, 96, 5, 1, 1, 4, 64)), (conv(8, 1, 192, 256, 70, 130, 2, original=50), dense(96))])
+                        (unit(4, 2, 64, 128, 64, 0.4), moe(15, 80, 5, 1, 1, 3, 64)), (conv(8, 1, 192, 256, 70, 130, 2, original=50), dense(96))])
 # one of everything: one head, a window of the position itself, one tap, no kept token, one expert, one group, one bucket
 UNIT = model(64, 64, [(conv(1, 1, 32, 32, 1, 0, 1), moe(1, 32, 1, shared=32)), (unit(1, 1, 32, 32, 1, 1.0, rot=2, factor=1.0), dense(32)),
                       (conv(1, 1, 2, 32, 1, 1, 1, factor=1.0), moe(1, 32, 1, 2, 1, 1, 64))], buckets=1)

@@ -75,7 +75,7 @@ def test_state_holds_what_the_layers_look_back_to():
     assert bool((st.conv[0][2] == 7).all()) and int(st.last_token[2]) == 5
 
 
-@pytest.mark.parametrize("base,dims,factor,original", [(900.0, 14, 4.0, 100), (20000.0, 64, 8.0, 512), (10.0, 8, 2.0, 4), (5e5, 128, 1.0, 8192)])
+@pytest.mark.parametrize("base,dims,factor,original", [(900.0, 14, 4.0, 100), (30000.0, 48, 6.0, 700), (10.0, 8, 2.0, 4), (5e5, 128, 1.0, 8192)])
 def test_scaled_frequencies(base, dims, factor, original):
     f = specs.rotation_frequencies(base, dims)
     rot = {"base": base, "dims": dims, "scaling": {"factor": factor, "low": 1.0, "high": 4.0, "original": original, "fast": 16.0, "slow": 1.0}}

@@ -237,7 +237,7 @@ def step_of(rows, padding=3):
     return b
 
 
-ROUTERS = [(16, 4, 2, 2, 1), (10, 2, 3, 3, 2), (1, 0, 1, 1, 1), (60, 4, 8, 4, 2), (200, 56, 10, 16, 3), (41, 4, 6, 9, 4), (8, 2, 2, 5, 2), (3, 5, 8, 1, 1)]
+ROUTERS = [(18, 6, 2, 4, 1), (10, 2, 3, 3, 2), (1, 0, 1, 1, 1), (60, 4, 8, 4, 2), (200, 56, 10, 16, 3), (41, 4, 6, 9, 4), (8, 2, 2, 5, 2), (3, 5, 8, 1, 1)]
 
 
 @pytest.mark.parametrize("rows", [1, 5, 64, 65, 300])
@@ -287,7 +287,7 @@ def test_logits_that_are_not_finite_are_reported():
 
 
 @pytest.mark.parametrize("rows", [1, 3, 16, 17, 40, 64, 65, 200, 700])
-@pytest.mark.parametrize("E,identity,top,ff,width,K", [(16, 4, 2, 96, 192, 192), (10, 2, 3, 64, 76, 96), (4, 0, 4, 160, 128, 128), (60, 4, 8, 96, 256, 320)])
+@pytest.mark.parametrize("E,identity,top,ff,width,K", [(14, 3, 2, 96, 224, 160), (10, 2, 3, 64, 76, 96), (4, 0, 4, 160, 128, 128), (60, 4, 8, 96, 256, 320)])
 @pytest.mark.parametrize("dtype", [BF, F32])
 def test_experts_and_their_sum(rows, E, identity, top, ff, width, K, dtype):
     """Router, experts, shared expert, residual update and norm against the plain mixture; unequal loads, experts without rows."""
