@@ -42,6 +42,11 @@ def pad_cols(t: torch.Tensor, to: int) -> torch.Tensor:
     return t if t.shape[1] == to else torch.cat([t, t.new_zeros(t.shape[0], to - t.shape[1])], 1)
 
 
+def alternate(a: torch.Tensor, b: torch.Tensor) -> torch.Tensor:
+    """Rows a0, b0, a1, b1, ..."""
+    return torch.stack([a, b], 1).flatten(0, 1)
+
+
 def plain_linear(w: torch.Tensor, n: int, k: int, fmt: str):
     """Unquantised projection of `n` x `k` (zero-padded from `w`): bf16 on CUDA keeps both kernel forms, streaming tiles for
     single rows and row-major for the tensor-core GEMMs."""

@@ -15,7 +15,7 @@ from typing import Callable, Dict, List, Optional
 import torch
 
 from ...ops.specs import AttnSpec, HeadsSpec, MoeSpec
-from ..common import pad, pad_heads, pad_rows, plain_linear
+from ..common import alternate, pad, pad_heads, pad_rows, plain_linear
 from ..qwen35.weights import LinearW
 from .config import ConvAttention, Dense, FudulixConfig, Mixer, Mixture
 
@@ -152,11 +152,6 @@ class FudulixWeights:
         return (n + sum(m.gate_up.numel() + m.down.numel() for m in self._mixtures())) * self.embed.element_size()
 
 
-def _alternate(a: torch.Tensor, b: torch.Tensor) -> torch.Tensor:
-    """Rows a0, b0, a1, b1, ..."""
-    return torch.stack([a, b], 1).flatten(0, 1)
-
-
 def build_engine_weights(cfg: FudulixConfig, get: Callable[[str], torch.Tensor], device="cpu",
                          dtype: Optional[torch.dtype] = None) -> FudulixWeights:
     """``dtype``: what projections and activations run in, bfloat16 or float32 (default: bfloat16 on a CUDA device)."""
@@ -205,7 +200,7 @@ def build_engine_weights(cfg: FudulixConfig, get: Callable[[str], torch.Tensor],
         def one(n: str) -> torch.Tensor:
             w = t(p + n)
             return pad_rows(torch.cat([w, t(f"{p}{n}.b")[:, None]], 1) if bias else w, ffp)
-        return _alternate(one("gate"), one("up"))
+        return alternate(one("gate"), one("up"))
 
     def mixture(c: Mixture, y: str) -> MixtureW:
         n, ffp = c.experts + c.identity, pad(c.ff, 32)

@@ -96,6 +96,7 @@ def _plain_family(name: str, architecture: str) -> ModelFamily:
 
 
 FAMILIES: List[ModelFamily] = [
+    _plain_family("rotutar", "Rotutar"),
     _plain_family("fudulix", "Fudulix"),
     _plain_family("luvutar", "Luvutar"),
     _plain_family("gebuzen", "Gebuzen"),

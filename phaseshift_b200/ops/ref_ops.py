@@ -21,7 +21,7 @@ from ..models.qwen35.weights import AttnW, GdnW, LinearW
 from ..runtime.batch import StepBatch
 from ..runtime.state import GdnLayerState, KVLayer, ModelState
 from ..utils.sampling import sample_row_host
-from .specs import AttnSpec, ExpertSum, GlaSpec, HeadsSpec, LatentSpec, MoeSpec, Pending, Routed, StreamWrite
+from .specs import AttnSpec, DeltaSpec, ExpertSum, GatedNorm, GlaSpec, HeadsSpec, LatentSpec, MoeSpec, Pending, Routed, StreamWrite, clamped_gate
 
 
 class RefOps(OpTrace):
@@ -344,13 +344,15 @@ class RefOps(OpTrace):
     def moe_route(self, logits, h, s: MoeSpec, b: StepBatch) -> Routed:
         """Router logits to every row's experts and weights (ops/specs.py: MoeSpec), and the rows of `h` sorted by expert."""
         rows, n = logits.shape[0], s.experts + s.identity
-        score = torch.softmax(logits[:, :n].float(), -1)
-        choice = score + s.correction
-        best = choice.reshape(rows, s.groups, -1).amax(-1).topk(s.keep, -1).indices
+        z = logits[:, :n].float()
+        score = torch.sigmoid(z) if s.sigmoid else torch.softmax(z, -1)
+        choice = score if s.correction is None else score + s.correction
+        best = choice.reshape(rows, s.groups, -1).topk(min(s.group_top, n // s.groups), -1).values.sum(-1).topk(s.keep, -1).indices
         open_ = torch.zeros(rows, s.groups, dtype=torch.bool).scatter_(1, best, True).repeat_interleave(n // s.groups, 1)
         ids = choice.masked_fill(~open_, -math.inf).topk(s.top, -1).indices
         weight = score.gather(1, ids)
-        weight = weight / (weight.sum(-1, keepdim=True) + 1e-20)
+        if s.renormalize:
+            weight = weight / (weight.sum(-1, keepdim=True) + 1e-20)
         real = ids < s.experts
         order = sorted((int(ids[r, k]), r, k) for r in range(rows) for k in range(s.top) if real[r, k])
         index = torch.full((rows, s.top), -1, dtype=torch.int32)
@@ -367,18 +369,49 @@ class RefOps(OpTrace):
         for e in routed.tiles.unique().tolist():
             at = routed.tiles == e
             y = routed.inputs[at].float() @ s.gate_up.reshape(s.experts, 2 * s.ff, K)[e].float().T
-            out[at] = (F.silu(y[:, 0::2]) * y[:, 1::2]) @ s.down.reshape(s.experts, s.n_out, s.ff)[e].float().T
+            act = F.silu(y[:, 0::2]) * y[:, 1::2] if s.limit is None else clamped_gate(y[:, 0::2], y[:, 1::2], s.limit)
+            out[at] = act @ s.down.reshape(s.experts, s.n_out, s.ff)[e].float().T
         return out
 
     @staticmethod
-    def _expert_sum(e: ExpertSum, W: int):
-        r = e.routed
-        y = r.identity[:, None] * e.h[:, :W].float()
+    def _weighted_experts(y, r: Routed, experts):
         for k in range(r.index.shape[1]):
             at = r.index[:, k].long()
             got = at >= 0
-            y[got] = y[got] + r.weight[got, k][:, None] * e.y[at[got], :W]
+            y[got] = y[got] + r.weight[got, k][:, None] * experts[at[got], :y.shape[1]]
+        return y
+
+    def _expert_sum(self, e: ExpertSum, W: int):
+        y = self._weighted_experts(e.routed.identity[:, None] * e.h[:, :W].float(), e.routed, e.y)
         return y if e.shared is None else y + e.shared[:, :W]
+
+    # ------------------------------------------------------------------ norms behind the sublayers
+    @staticmethod
+    def _group_norm(x, w, eps: float, groups: int):
+        p = x.reshape(x.shape[0], groups, -1)
+        return (p * torch.rsqrt(p.pow(2).mean(-1, keepdim=True) + eps)).reshape(x.shape) * w
+
+    def gated_norm(self, x, pend: Optional[GatedNorm], *, eps: float, groups: int, norm_w=None, width: int = 0, name: str = ""):
+        """x + the sublayer's gated and normed result, and the next projection's input: the new residual itself, or with `norm_w` its
+        norm in groups, padded to `width` columns.  Returns (new residual, rows or None)."""
+        W = x.shape[1]
+        if pend is not None:
+            if pend.routed is not None:
+                y = self._weighted_experts(torch.zeros_like(x), pend.routed, pend.experts)
+            else:
+                y = pend.scale_a * pend.a[:, :W].float()
+                if pend.b is not None:
+                    y = y + pend.scale_b * pend.b[:, :W].float()
+            x = x + self._group_norm(y * torch.sigmoid(pend.gate[:, :W].float() + pend.gate_bias), pend.norm_w, eps, groups)
+        if width == 0:
+            return x, None
+        h = x.new_zeros(x.shape[0], width)
+        h[:, :W] = x if norm_w is None else self._group_norm(x, norm_w, eps, groups)
+        return x, h
+
+    def soft_limit(self, logits, cap: float):
+        """cap * tanh(logits / cap), in place."""
+        return logits.div_(cap).tanh_().mul_(cap)
 
     # ------------------------------------------------------------------ parallel residual streams
     def stream_norm(self, x, pend: Optional[StreamWrite], *, read=None, norm_w=None, eps: float, width: int = 0, name: str = "",
@@ -487,12 +520,18 @@ class RefOps(OpTrace):
         H, dk, dv = g.heads, g.dk, g.dv
         out = proj.new_zeros(proj.shape[0], H * dv)
         p = proj.float()
-        z = p[:, g.a_off:g.a_off + g.rank] @ g.a2.float().T + g.a2_bias
-        alpha = torch.exp(F.logsigmoid(z) * g.inv_tau).reshape(-1, H, dk)
-        q = p[:, g.q_off:g.q_off + H * dk].reshape(-1, H, dk) * g.q_scale
-        k = p[:, g.k_off:g.k_off + H * dk].reshape(-1, H, dk)
+        q = p[:, g.q_off:g.q_off + H * dk].reshape(-1, H, dk)
+        if g.lower is not None:
+            z = p[:, g.a_off:g.a_off + H * dk] + g.a2_bias
+            k = ((1.0 - g.lower) * torch.sigmoid(-z)).reshape(-1, H, dk)
+            alpha, q = 1.0 - k, F.silu(q)
+        else:
+            z = p[:, g.a_off:g.a_off + g.rank] @ g.a2.float().T + g.a2_bias
+            alpha = torch.exp(F.logsigmoid(z) * g.inv_tau).reshape(-1, H, dk)
+            k = p[:, g.k_off:g.k_off + H * dk].reshape(-1, H, dk)
+        q = q * g.q_scale
         v = p[:, g.v_off:g.v_off + H * dv].reshape(-1, H, dv)
-        gate = F.silu(p[:, g.g_off:g.g_off + H * dv])
+        gate = F.silu(p[:, g.g_off:g.g_off + H * dv]) if g.g_off >= 0 else p.new_ones(p.shape[0], H * dv)
         for s in range(b.n_seqs):
             row0, n, slot, _ = (int(t) for t in b.seq_desc[s])
             S = gs.rec[slot]
@@ -503,4 +542,40 @@ class RefOps(OpTrace):
                 out[row] = o.reshape(-1) * gate[row]
             if n > 0:
                 gs.rec[slot] = S
+        return out
+
+    # ------------------------------------------------------------------ delta rule with a decay per channel
+    def delta(self, proj, d: DeltaSpec, b: StepBatch, gs: GdnLayerState, st: ModelState, history):
+        H, G, dk, dv, taps = d.heads, d.kv_heads, d.dk, d.dv, d.taps
+        p, out = proj.float(), proj.new_zeros(proj.shape[0], H * dv)
+        head = torch.arange(H)[:, None]
+        # every value head's own channels: columns of the projection, and of the convolution
+        cols = torch.cat([d.q_off + head // (H // G) * dk + torch.arange(dk), d.k_off + head // (H // G) * dk + torch.arange(dk),
+                          d.v_off + head * dv + torch.arange(dv)], 1)
+        w = d.conv.float()[:, cols - d.q_off]                     # [taps, heads, 2 dk + dv] (the three parts lie side by side)
+        g = torch.exp(-d.rate[:, None] * F.softplus(p[:, d.a_off:d.a_off + d.a2.shape[1]] @ d.a2.float().T + d.dt_bias).reshape(-1, H, dk))
+        beta = torch.sigmoid(p[:, d.b_off:d.b_off + H])
+        gate = torch.sigmoid(p[:, d.g_off:d.g_off + d.g2.shape[1]] @ d.g2.float().T)
+        for s in range(b.n_seqs):
+            row0, n, slot, pos0 = (int(t) for t in b.seq_desc[s])
+            if n <= 0:
+                continue
+            S = gs.rec[slot]
+            hist = None if history is None else history[slot].reshape(taps - 1, H, 2 * dk + dv)
+            for r in range(n):
+                x = torch.zeros(H, 2 * dk + dv)
+                for j in range(min(taps, pos0 + r + 1)):
+                    x = x + w[taps - 1 - j] * (p[row0 + r - j][cols] if j <= r else hist[(pos0 + r - j) % (taps - 1)].float())
+                x = F.silu(x)
+                unit = lambda t: t * torch.rsqrt(t.pow(2).sum(-1, keepdim=True) + 1e-6)
+                q, k, v = unit(x[:, :dk]) * d.dk_true ** -0.5, unit(x[:, dk:2 * dk]), x[:, 2 * dk:]
+                S = S * g[row0 + r][:, :, None]
+                u = beta[row0 + r][:, None] * (v - torch.einsum("hkv,hk->hv", S, k))
+                S = S + k[:, :, None] * u[:, None, :]
+                o = torch.einsum("hkv,hk->hv", S, q)
+                o = o * torch.rsqrt(o.pow(2).sum(-1, keepdim=True) / d.dv_true + d.eps) * d.norm_w
+                out[row0 + r] = o.reshape(-1) * gate[row0 + r]
+            gs.rec[slot] = S
+            for r in range(max(0, n - taps + 1), n):
+                hist[(pos0 + r) % (taps - 1)] = proj[row0 + r][cols]
         return out

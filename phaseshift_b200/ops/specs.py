@@ -130,10 +130,11 @@ class HeadsSpec:
 
 @dataclass
 class MoeSpec:
-    """Mixture of feed-forward experts with (silu gate) * up.  A token's scores are the softmax of its router logits over
-    experts and, behind them, `identity` experts that return their input; it goes to the `top` largest of score + correction
-    among the `keep` best of `groups` equal groups of neighbours (a group counts as its best member), weighted by their scores
-    divided by the sum of these."""
+    """Mixture of feed-forward experts.  A token's scores are the softmax (or the sigmoids) of its router logits over experts and,
+    behind them, `identity` experts that return their input; it goes to the `top` largest of score + correction among the `keep`
+    best of `groups` equal groups of neighbours (a group counts as the sum of its `group_top` best members), weighted by their
+    scores, divided by the sum of these if `renormalize`.  An expert's activation is silu(gate) * up, or with a `limit` that of
+    `clamped_gate`."""
     experts: int
     identity: int
     top: int
@@ -141,9 +142,19 @@ class MoeSpec:
     keep: int
     ff: int                     # columns of an expert's activation (engine size)
     n_out: int                  # output columns (engine size)
-    correction: torch.Tensor    # f32 [experts + identity]
+    correction: Optional[torch.Tensor]       # f32 [experts + identity]; None: zero
     gate_up: torch.Tensor       # [experts * 2 ff, K], rows alternate gate, up
     down: torch.Tensor          # [experts * n_out, ff]
+    sigmoid: bool = False
+    group_top: int = 1          # 1 or 2
+    renormalize: bool = True
+    limit: Optional[float] = None
+
+
+def clamped_gate(gate: torch.Tensor, up: torch.Tensor, limit: float) -> torch.Tensor:
+    """g sigmoid(1.702 g) (u + 1) with g = min(gate, limit) and u = up clamped to [-limit, limit]."""
+    g = gate.clamp(max=limit)
+    return g * torch.sigmoid(1.702 * g) * (up.clamp(-limit, limit) + 1.0)
 
 
 @dataclass
@@ -220,7 +231,11 @@ class LatentSpec:
 @dataclass
 class GlaSpec:
     """Gated linear attention over one projection row: column offsets of q, k, v, the output gate and the low-rank decay input,
-    head geometry (engine sizes, and the true value size the head norm averages over) and the decay's constants."""
+    head geometry (engine sizes, and the true value size the head norm averages over) and the decay's constants.
+
+    With `lower` the decay is a gate of its own that also decides what is written: f = lower + (1 - lower) sigmoid(z), z a column per
+    head and channel of the projection (at `a_off`) + `a2_bias`; the key is 1 - f and the query silu(q).  There is no `a2` then.
+    `g_off` -1: no output gate."""
     heads: int
     dk: int
     dv: int
@@ -234,9 +249,60 @@ class GlaSpec:
     q_scale: float
     inv_tau: float
     eps: float
-    a2: torch.Tensor            # [heads * dk, rank]
+    a2: Optional[torch.Tensor]  # [heads * dk, rank]
     a2_bias: torch.Tensor       # f32 [heads * dk]
     norm_w: torch.Tensor        # f32 [dv]
+    lower: Optional[torch.Tensor] = None     # f32 [heads * dk]
+
+
+@dataclass
+class DeltaSpec:
+    """Delta rule with a decay per head and key channel, between a projection row and the output projection.  Projection columns:
+    q and k heads (`kv_heads`; consecutive value heads share one), v heads, the input of the step size (a column per head) and the
+    low-rank inputs of decay and output gate.
+
+    q, k and v pass a causal convolution over time (`conv`, the last tap is the row's own; the sequence's last taps - 1 rows are
+    state, a copy per value head: [slots, taps - 1, heads, 2 dk + dv], position p in row p % (taps - 1)) and silu; q and k are divided
+    by their length, q also by sqrt(dk_true).  g = exp(-rate softplus(a2 a + dt_bias)), beta = sigmoid(b), and per head
+    S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q.  The output is rms(o) norm_w sigmoid(g2 g)."""
+    heads: int
+    kv_heads: int
+    dk: int                     # the engine's sizes (padded with zeros), and the model's
+    dv: int
+    dk_true: int
+    dv_true: int
+    q_off: int
+    k_off: int
+    v_off: int
+    b_off: int
+    a_off: int
+    g_off: int
+    eps: float
+    conv: torch.Tensor          # [taps, q | k | v channels], the projection's type
+    a2: torch.Tensor            # [heads * dk, a rank]
+    dt_bias: torch.Tensor       # f32 [heads * dk]
+    rate: torch.Tensor          # f32 [heads]
+    g2: torch.Tensor            # [heads * dv, g rank]
+    norm_w: torch.Tensor        # f32 [dv]
+
+    @property
+    def taps(self) -> int:
+        return self.conv.shape[0]
+
+
+@dataclass
+class GatedNorm:
+    """A sublayer's result on its way into the residual: y = scale_a a + scale_b b (projection outputs, f32) or the weighted sum of a
+    mixture's experts; y * sigmoid(gate + gate_bias) is normed in groups, times `norm_w`, and added."""
+    gate: torch.Tensor          # [rows, width (+ padding columns)], bf16 or f32
+    gate_bias: torch.Tensor     # f32 [width]
+    norm_w: torch.Tensor        # f32 [width]
+    a: Optional[torch.Tensor] = None
+    scale_a: float = 1.0
+    b: Optional[torch.Tensor] = None
+    scale_b: float = 1.0
+    routed: Optional[Routed] = None
+    experts: Optional[torch.Tensor] = None   # f32 [sorted rows, width (+ padding columns)]
 
 
 @dataclass
