@@ -3,6 +3,9 @@
 // Per head, with log-decay la = log(sigmoid(z)) / tau, z = a2 . a1 + bias (a1 = the row's low-rank decay input):
 //     S_t = diag(exp(la_t)) S_{t-1} + k_t v_t^T ,   o_t = S_t^T (q_t * q_scale) ,   out = (rms(o) * w) * silu(g)
 // The decays, their logarithms and sums, the state and everything multiplied into it are fp32.
+// FORGET variants (linear attention whose forget gate is its key): z is a column of the projection per head and channel (+ bias),
+//     f = lower + (1 - lower) sigmoid(z),  la = log(f),  k = 1 - f,  q = silu(q) * q_scale
+// and there may be no output gate.
 //
 // ps_gla_rows     row-sequential: one CTA per (sequence, head), state read and written once per launch.  Decode, short
 //                 portions, and the 32-bit engines.  Sizes 128 x 128 and 64 x 64 keep the state in registers, others update
@@ -31,6 +34,7 @@ struct GlaArgs {
     int q_off, k_off, v_off, g_off, a_off, rank;
     float q_scale, inv_tau, eps;
     const void* a2; const float* a2_bias; const float* norm_w;
+    const float* lower;                // FORGET: [H * dk]
     float* state;                      // [slots, H, dk, dv]
     const GlaSeq* seqs; int n_seqs;
     void* out;                         // [rows, H * dv]
@@ -45,13 +49,20 @@ struct GlaArgs {
 __device__ __forceinline__ float gla_log_decay(float z, float inv_tau) {
     return (fminf(z, 0.f) - log1pf(expf(-fabsf(z)))) * inv_tau;
 }
+// Forget gate: how much is written, and the logarithm of what is kept (bounded, so that sums stay finite).
+__device__ __forceinline__ float gla_forget(float z, float lower, float& log_keep) {
+    const float e = expf(-fabsf(z)), s = 1.f / (1.f + e), neg = z > 0.f ? e * s : s;            // sigmoid(-z)
+    const float k = (1.f - lower) * neg;
+    log_keep = fmaxf(k < 0.5f ? log1pf(-k) : logf(lower + (1.f - lower) * (z > 0.f ? s : e * s)), -100.f);
+    return k;
+}
 template <typename T> __device__ __forceinline__ T gla_cast(float v);
 template <> __device__ __forceinline__ float gla_cast<float>(float v) { return v; }
 template <> __device__ __forceinline__ __nv_bfloat16 gla_cast<__nv_bfloat16>(float v) { return f32_to_bf16(v); }
 __device__ __forceinline__ float gla_silu(float x) { return x / (1.f + expf(-x)); }
 
 // ------------------------------------------------------------------------------------------------ row-sequential form
-template <typename T, int DK, int DV>
+template <typename T, int DK, int DV, bool FORGET>
 __global__ void __launch_bounds__(256) gla_rows_kernel(const GlaArgs a) {
     extern __shared__ __align__(16) float gla_smem[];
     const int dk = DK > 0 ? DK : a.dk, dv = DV > 0 ? DV : a.dv;
@@ -85,12 +96,22 @@ __global__ void __launch_bounds__(256) gla_rows_kernel(const GlaArgs a) {
         const int row = sd.row_start + i;
         const T* pr = reinterpret_cast<const T*>(a.proj) + (size_t)row * a.ld;
         for (int d = t; d < dk; d += 256) {
-            const T* w = reinterpret_cast<const T*>(a.a2) + (size_t)(h * dk + d) * a.rank;
             float z = a.a2_bias[h * dk + d];
-            for (int r = 0; r < a.rank; ++r) z = fmaf((float)w[r], (float)pr[a.a_off + r], z);
-            s_al[d] = expf(gla_log_decay(z, a.inv_tau));
-            s_q[d] = (float)pr[a.q_off + h * dk + d] * a.q_scale;
-            s_k[d] = (float)pr[a.k_off + h * dk + d];
+            const float q = (float)pr[a.q_off + h * dk + d];
+            if constexpr (FORGET) {
+                float la;
+                z += (float)pr[a.a_off + h * dk + d];
+                const float k = gla_forget(z, a.lower[h * dk + d], la);
+                s_k[d] = k;
+                s_al[d] = 1.f - k;
+                s_q[d] = gla_silu(q) * a.q_scale;
+            } else {
+                const T* w = reinterpret_cast<const T*>(a.a2) + (size_t)(h * dk + d) * a.rank;
+                for (int r = 0; r < a.rank; ++r) z = fmaf((float)w[r], (float)pr[a.a_off + r], z);
+                s_al[d] = expf(gla_log_decay(z, a.inv_tau));
+                s_q[d] = q * a.q_scale;
+                s_k[d] = (float)pr[a.k_off + h * dk + d];
+            }
         }
         for (int d = t; d < dv; d += 256) s_v[d] = (float)pr[a.v_off + h * dv + d];
         __syncthreads();
@@ -132,7 +153,7 @@ __global__ void __launch_bounds__(256) gla_rows_kernel(const GlaArgs a) {
         const float inv = rsqrtf(ss / (float)a.dv_true + a.eps);
         T* out = reinterpret_cast<T*>(a.out) + (size_t)row * a.H * dv + h * dv;
         for (int d = t; d < dv; d += 256)
-            out[d] = gla_cast<T>(s_v[d] * inv * a.norm_w[d] * gla_silu((float)pr[a.g_off + h * dv + d]));
+            out[d] = gla_cast<T>(s_v[d] * inv * a.norm_w[d] * (FORGET && a.g_off < 0 ? 1.f : gla_silu((float)pr[a.g_off + h * dv + d])));
         __syncthreads();
     }
     if constexpr (DK > 0) {
@@ -183,7 +204,7 @@ __host__ __device__ inline size_t gla_prep_smem_floats(int dk, int dv) {
 }
 
 // grid = (blocks, H)
-template <int DKT, int DVT>
+template <int DKT, int DVT, bool FORGET>
 __global__ void __launch_bounds__(kGPrepThreads) gla_prepare_kernel(const GlaArgs a) {
     extern __shared__ __align__(16) float gla_smem[];
     const int dk = DKT > 0 ? DKT : a.dk, dv = DVT > 0 ? DVT : a.dv;
@@ -200,6 +221,30 @@ __global__ void __launch_bounds__(kGPrepThreads) gla_prepare_kernel(const GlaArg
     const size_t bh = (size_t)blockIdx.x * a.H + h;
     const __nv_bfloat16* proj = reinterpret_cast<const __nv_bfloat16*>(a.proj) + (size_t)row0 * a.ld;
 
+    if constexpr (FORGET) {
+        // ---- log-decays and keys from the gate's columns
+        for (int i = t; i < kGC * (dk / 8); i += kGPrepThreads) {
+            const int r = i / (dk / 8), c = (i % (dk / 8)) * 8;
+            float la[8], k[8];
+            if (r < n) {
+                const uint4 zr = *reinterpret_cast<const uint4*>(proj + (size_t)r * a.ld + a.a_off + h * dk + c);
+                const uint32_t zw[4] = {zr.x, zr.y, zr.z, zr.w};
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const float2 z = bf16x2_bits_to_f32x2(zw[e]);
+                    const int d = h * dk + c + 2 * e;
+                    k[2 * e] = gla_forget(z.x + a.a2_bias[d], a.lower[d], la[2 * e]);
+                    k[2 * e + 1] = gla_forget(z.y + a.a2_bias[d + 1], a.lower[d + 1], la[2 * e + 1]);
+                }
+            } else {
+#pragma unroll
+                for (int e = 0; e < 8; ++e) la[e] = k[e] = 0.f;
+            }
+#pragma unroll
+            for (int e = 0; e < 8; ++e) { sB[r * PQ + c + e] = la[e]; sK[r * PK + c + e] = k[e]; }
+        }
+        __syncthreads();
+    } else
     // ---- log-decays: a1 rows and this head's slice of a2 share the q / k buffers, which are not filled yet
     {
         float* s1 = sQ;                                 // [64][rank]
@@ -264,14 +309,19 @@ __global__ void __launch_bounds__(kGPrepThreads) gla_prepare_kernel(const GlaArg
         uint4 q = make_uint4(0, 0, 0, 0), k = q;
         if (r < n) {
             q = *reinterpret_cast<const uint4*>(proj + (size_t)r * a.ld + a.q_off + h * dk + c);
-            k = *reinterpret_cast<const uint4*>(proj + (size_t)r * a.ld + a.k_off + h * dk + c);
+            if constexpr (!FORGET) k = *reinterpret_cast<const uint4*>(proj + (size_t)r * a.ld + a.k_off + h * dk + c);
         }
         const uint32_t qw[4] = {q.x, q.y, q.z, q.w}, kw[4] = {k.x, k.y, k.z, k.w};
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-            const float2 qf = bf16x2_bits_to_f32x2(qw[e]), kf = bf16x2_bits_to_f32x2(kw[e]);
-            sQ[r * PQ + c + 2 * e] = qf.x * a.q_scale; sQ[r * PQ + c + 2 * e + 1] = qf.y * a.q_scale;
-            sK[r * PK + c + 2 * e] = kf.x; sK[r * PK + c + 2 * e + 1] = kf.y;
+            const float2 qf = bf16x2_bits_to_f32x2(qw[e]);
+            if constexpr (FORGET) {
+                sQ[r * PQ + c + 2 * e] = silu_f(qf.x) * a.q_scale; sQ[r * PQ + c + 2 * e + 1] = silu_f(qf.y) * a.q_scale;
+            } else {
+                const float2 kf = bf16x2_bits_to_f32x2(kw[e]);
+                sQ[r * PQ + c + 2 * e] = qf.x * a.q_scale; sQ[r * PQ + c + 2 * e + 1] = qf.y * a.q_scale;
+                sK[r * PK + c + 2 * e] = kf.x; sK[r * PK + c + 2 * e + 1] = kf.y;
+            }
         }
     }
     __syncthreads();
@@ -483,7 +533,7 @@ __device__ __forceinline__ void gla_cp_async16(void* dst, const void* src) {
 }
 
 // grid = (blocks, H)
-template <int DKT, int DVT>
+template <int DKT, int DVT, bool FORGET>
 __global__ void __launch_bounds__(kGOutThreads) gla_output_kernel(const GlaArgs a) {
     extern __shared__ __align__(16) float gla_smem[];
     __shared__ float s_ss[2][kGC];
@@ -564,32 +614,52 @@ __global__ void __launch_bounds__(kGOutThreads) gla_output_kernel(const GlaArgs 
         for (int j = 0; j < kNT; ++j) {
             if (j < nt) {
                 const int d = half * (dv / 2) + j * 8 + 2 * tq;
-                const float2 gv = bf16x2_bits_to_f32x2(*reinterpret_cast<const uint32_t*>(gp + d));
                 const float2 wv = *reinterpret_cast<const float2*>(a.norm_w + d);
-                *reinterpret_cast<uint32_t*>(out + d) = f32x2_to_bf16x2_bits(acc[j][2 * r] * inv * wv.x * silu_f(gv.x),
-                                                                             acc[j][2 * r + 1] * inv * wv.y * silu_f(gv.y));
+                float gx = 1.f, gy = 1.f;
+                if (!FORGET || a.g_off >= 0) {
+                    const float2 gv = bf16x2_bits_to_f32x2(*reinterpret_cast<const uint32_t*>(gp + d));
+                    gx = silu_f(gv.x); gy = silu_f(gv.y);
+                }
+                *reinterpret_cast<uint32_t*>(out + d) = f32x2_to_bf16x2_bits(acc[j][2 * r] * inv * wv.x * gx, acc[j][2 * r + 1] * inv * wv.y * gy);
             }
         }
     }
 }
 
-template <int DKT, int DVT>
+template <int DKT, int DVT, bool FORGET>
 static int launch_gla_chunked(const GlaArgs& a, int blocks, cudaStream_t stream) {
     const size_t s1 = gla_prep_smem_floats(a.dk, a.dv) * 4, s2 = ((size_t)kGC * (a.dk + 4) + (size_t)a.dk * (a.dv + 8)) * 4;
     static bool set = false;
     if (!set) {
-        cudaFuncSetAttribute(gla_prepare_kernel<DKT, DVT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024);
-        cudaFuncSetAttribute(gla_output_kernel<DKT, DVT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024);
+        cudaFuncSetAttribute(gla_prepare_kernel<DKT, DVT, FORGET>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024);
+        cudaFuncSetAttribute(gla_output_kernel<DKT, DVT, FORGET>, cudaFuncAttributeMaxDynamicSharedMemorySize, 226 * 1024);
         set = true;
     }
-    gla_prepare_kernel<DKT, DVT><<<dim3(blocks, a.H), kGPrepThreads, s1, stream>>>(a);
+    gla_prepare_kernel<DKT, DVT, FORGET><<<dim3(blocks, a.H), kGPrepThreads, s1, stream>>>(a);
     int e = PS_LAUNCH_CHECK();
     if (e) return e;
     const long long groups = (long long)a.H * a.dk * a.dv / 4;
     gla_scan_kernel<<<dim3((unsigned)((groups + 255) / 256), a.n_seqs), 256, 0, stream>>>(a);
     if ((e = PS_LAUNCH_CHECK())) return e;
-    gla_output_kernel<DKT, DVT><<<dim3(blocks, a.H), kGOutThreads, s2, stream>>>(a);
+    gla_output_kernel<DKT, DVT, FORGET><<<dim3(blocks, a.H), kGOutThreads, s2, stream>>>(a);
     return PS_LAUNCH_CHECK();
+}
+
+template <bool FORGET>
+static int launch_gla(const GlaArgs& a, int chunked, int f32, int blocks, cudaStream_t stream) {
+    const int dk = a.dk, dv = a.dv;
+    if (chunked) {
+        if (dk == 128 && dv == 128) return launch_gla_chunked<128, 128, FORGET>(a, blocks, stream);
+        if (dk == 64 && dv == 64) return launch_gla_chunked<64, 64, FORGET>(a, blocks, stream);
+        return launch_gla_chunked<0, 0, FORGET>(a, blocks, stream);
+    }
+    const size_t smem = ((size_t)3 * dk + dv + 1024) * 4;
+    if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
+    const dim3 grid(a.H, a.n_seqs);
+    if (f32) return launch_pdl(gla_rows_kernel<float, 0, 0, FORGET>, grid, dim3(256), smem, stream, a);
+    if (dk == 128 && dv == 128) return launch_pdl(gla_rows_kernel<__nv_bfloat16, 128, 128, FORGET>, grid, dim3(256), smem, stream, a);
+    if (dk == 64 && dv == 64) return launch_pdl(gla_rows_kernel<__nv_bfloat16, 64, 64, FORGET>, grid, dim3(256), smem, stream, a);
+    return launch_pdl(gla_rows_kernel<__nv_bfloat16, 0, 0, FORGET>, grid, dim3(256), smem, stream, a);
 }
 
 }  // namespace ps
@@ -599,7 +669,7 @@ PS_DEFINE_LIMITS_SETTER(gla)
 // Rows of the chunked path's blocks, and whether it takes a head geometry (shared-memory plan and tile multiples).
 PS_API int ps_gla_block_rows() { return ps::kGC; }
 PS_API int ps_gla_chunked_ok(int dk, int dv, int rank) {
-    if (dk % 16 || dv % 32 || dk > 256 || dv > 256 || rank < 1) return 0;
+    if (dk % 16 || dv % 32 || dk > 256 || dv > 256 || rank < 0) return 0;
     if (ps::gla_prep_smem_floats(dk, dv) * 4 > 226 * 1024 || ((size_t)ps::kGC * (dk + 4) + (size_t)dk * (dv + 8)) * 4 > 226 * 1024) return 0;
     return (size_t)ps::kGC * rank + (size_t)dk * (rank + 1) <= (size_t)ps::kGC * (2 * dk + 12) ? 1 : 0;
 }
@@ -607,32 +677,22 @@ PS_API int ps_gla_chunked_ok(int dk, int dv, int rank) {
 // `chunked` = 0: every sequence with at most `rows_limit` rows (0 = all) row by row, bf16 or (`f32`) 32-bit;
 // `chunked` = 1: the sequences with more than `rows_limit` rows, `blocks` = the sum of their ceil(rows / 64), bf16 only, scratch
 // sizes as in GlaArgs.  dk a multiple of 16, dv of 32 (at most 1024), row pitch and offsets multiples of 8 elements.
+// `lower` not null: the FORGET variants (`rank` 0, `a2` null, z at `a_off`, `k_off` unused); `g_off` -1 there: no output gate.
 // Both forms may load a slot's state before the stream predecessor has finished (see ps_gdn_rows).
 PS_API int ps_gla(int chunked, const void* proj, int ld, int f32, int H, int dk, int dv, int dv_true, int q_off, int k_off, int v_off,
                   int g_off, int a_off, int rank, float q_scale, float inv_tau, float eps, const void* a2, const void* a2_bias,
-                  const void* norm_w, void* state, const void* seqs, int n_seqs, int rows_limit, void* out, int blocks, void* qd,
+                  const void* norm_w, const void* lower, void* state, const void* seqs, int n_seqs, int rows_limit, void* out, int blocks, void* qd,
                   void* oi, void* u, void* dec, cudaStream_t stream) {
     using namespace ps;
-    if (n_seqs <= 0 || H <= 0 || dk <= 0 || dk % 16 || dv <= 0 || dv % 32 || dv > 1024 || dv_true < 1 || dv_true > dv || rank < 1 ||
-        rank % 8 || ((ld | q_off | k_off | v_off | g_off | a_off) % 8) || ((uintptr_t)proj | (uintptr_t)state) % 16)
+    if (n_seqs <= 0 || H <= 0 || dk <= 0 || dk % 16 || dv <= 0 || dv % 32 || dv > 1024 || dv_true < 1 || dv_true > dv || rank < (lower != nullptr ? 0 : 1) ||
+        rank % 8 || ((ld | q_off | k_off | v_off | a_off) % 8) || (lower != nullptr && g_off < 0 ? false : g_off % 8 != 0) || ((uintptr_t)proj | (uintptr_t)state) % 16)
         return (int)cudaErrorInvalidValue;
     GlaArgs a;
     a.proj = proj; a.ld = ld; a.H = H; a.dk = dk; a.dv = dv; a.dv_true = dv_true; a.q_off = q_off; a.k_off = k_off; a.v_off = v_off;
     a.g_off = g_off; a.a_off = a_off; a.rank = rank; a.q_scale = q_scale; a.inv_tau = inv_tau; a.eps = eps; a.a2 = a2;
-    a.a2_bias = (const float*)a2_bias; a.norm_w = (const float*)norm_w; a.state = (float*)state; a.seqs = (const GlaSeq*)seqs;
+    a.a2_bias = (const float*)a2_bias; a.norm_w = (const float*)norm_w; a.lower = (const float*)lower; a.state = (float*)state; a.seqs = (const GlaSeq*)seqs;
     a.n_seqs = n_seqs; a.out = out; a.rows_limit = rows_limit; a.qd = (float*)qd; a.oi = (float*)oi; a.u = (float*)u; a.dec = (float*)dec;
-    if (chunked) {
-        if (f32 || blocks <= 0 || !ps_gla_chunked_ok(dk, dv, rank) || qd == nullptr || oi == nullptr || u == nullptr || dec == nullptr)
-            return (int)cudaErrorInvalidValue;
-        if (dk == 128 && dv == 128) return launch_gla_chunked<128, 128>(a, blocks, stream);
-        if (dk == 64 && dv == 64) return launch_gla_chunked<64, 64>(a, blocks, stream);
-        return launch_gla_chunked<0, 0>(a, blocks, stream);
-    }
-    const size_t smem = ((size_t)3 * dk + dv + 1024) * 4;
-    if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;
-    const dim3 grid(H, n_seqs);
-    if (f32) return launch_pdl(gla_rows_kernel<float, 0, 0>, grid, dim3(256), smem, stream, a);
-    if (dk == 128 && dv == 128) return launch_pdl(gla_rows_kernel<__nv_bfloat16, 128, 128>, grid, dim3(256), smem, stream, a);
-    if (dk == 64 && dv == 64) return launch_pdl(gla_rows_kernel<__nv_bfloat16, 64, 64>, grid, dim3(256), smem, stream, a);
-    return launch_pdl(gla_rows_kernel<__nv_bfloat16, 0, 0>, grid, dim3(256), smem, stream, a);
+    if (chunked && (f32 || blocks <= 0 || !ps_gla_chunked_ok(dk, dv, rank) || qd == nullptr || oi == nullptr || u == nullptr || dec == nullptr))
+        return (int)cudaErrorInvalidValue;
+    return lower != nullptr ? launch_gla<true>(a, chunked, f32, blocks, stream) : launch_gla<false>(a, chunked, f32, blocks, stream);
 }

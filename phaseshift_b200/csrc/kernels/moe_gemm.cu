@@ -5,8 +5,8 @@
 // `tcgen05.mma`, up to NB sorted rows the N side, so that a tile with few rows (decode: every active expert has a handful)
 // streams weights at full width and one with many is an ordinary tensor-core product.  Both operands come by TMA (128-byte swizzle,
 // no multicast) into a ring; the accumulator (128 lanes = output features, NB columns = rows) lives in tensor memory.  The
-// epilogue reads it with `tcgen05.ld`, a lane per feature: SwiGLU takes its (gate, up) pair from two neighbouring lanes, which
-// share the work of two rows; stores of a warp are whole sectors.  Columns behind a tile's rows hold other experts' rows and are not
+// epilogue reads it with `tcgen05.ld`, a lane per feature: a gated activation (SwiGLU, or g sigmoid(1.702 g) (u + 1) with g and u
+// limited) takes its (gate, up) pair from two neighbouring lanes, which share the work of two rows; stores of a warp are whole sectors.  Columns behind a tile's rows hold other experts' rows and are not
 // stored.  Every wait is bounded (abort flag, bounded drain, tensor memory freed).
 //
 // 32-bit: the same list on the CUDA cores, 64 x 64 tiles.
@@ -18,11 +18,17 @@ constexpr int kMgM = 128, kMgK = 64, kMgThreads = 192;
 
 struct MoeGemmArgs {
     const int* tiles;            // [0]: number of tiles; from [4] on (expert, first row, rows, 0)
-    int N, K, swiglu;            // N: weight rows per expert
-    void* out; int ldo;          // SwiGLU: bf16 [rows, N / 2]; else fp32 [rows, N]
+    int N, K, gated;             // N: weight rows per expert; gated 0 store, 1 SwiGLU, 2 limited gate
+    void* out; int ldo;          // gated: bf16 [rows, N / 2]; else fp32 [rows, N]
+    float limit;
     uint32_t* status;
     long long budget;
 };
+
+__device__ __forceinline__ float mg_limited(float gate, float up, float limit) {
+    const float g = fminf(gate, limit);
+    return g / (1.f + expf(-1.702f * g)) * (fminf(fmaxf(up, -limit), limit) + 1.f);
+}
 
 // grid = (weight tiles, tiles of the list at most)
 template <int NB, int STAGES>
@@ -104,7 +110,7 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
                 if constexpr (CW == 16) tc::tmem_ld_32x16(tmem_acc + ((uint32_t)(quad * 32) << 16) + (uint32_t)c0, r);
                 else tc::tmem_ld_32x32(tmem_acc + ((uint32_t)(quad * 32) << 16) + (uint32_t)c0, r);
                 tc::tmem_ld_wait();
-                if (g.swiglu) {
+                if (g.gated) {
                     // lanes 2i, 2i + 1 hold gate and up of one feature: the even lane finishes row c, the odd one row c + 1
                     __nv_bfloat16* o = reinterpret_cast<__nv_bfloat16*>(g.out) + (n >> 1);
                     const bool odd = lane & 1;
@@ -114,7 +120,7 @@ moe_gemm_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant
                         const float got = __shfl_xor_sync(0xffffffffu, give, 1);
                         const float gt = bf16_to_f32(f32_to_bf16(odd ? got : mine)), up = bf16_to_f32(f32_to_bf16(odd ? mine : got));
                         const int row = c0 + c + (odd ? 1 : 0);
-                        if (row < tile.z && n < g.N) o[(size_t)(tile.y + row) * g.ldo] = f32_to_bf16(silu_f(gt) * up);
+                        if (row < tile.z && n < g.N) o[(size_t)(tile.y + row) * g.ldo] = f32_to_bf16(g.gated == 2 ? mg_limited(gt, up, g.limit) : silu_f(gt) * up);
                     }
                 } else {
                     float* o = reinterpret_cast<float*>(g.out) + n;
@@ -176,7 +182,7 @@ static int launch_moe_gemm(const CUtensorMap& map_w, const CUtensorMap& map_x, i
 constexpr int kMfT = 64, kMfK = 16;
 
 struct MoeGemmF32Args {
-    const int* tiles; const float* x; const float* w; int N, K, swiglu; float* out; int ldo;
+    const int* tiles; const float* x; const float* w; int N, K, gated; float* out; int ldo; float limit;
 };
 
 // grid = (column tiles, tiles of the list at most)
@@ -216,8 +222,8 @@ __global__ void __launch_bounds__(256) moe_gemm_f32_kernel(const MoeGemmF32Args 
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx * 4 + j;
             if (n >= g.N) continue;
-            if (!g.swiglu) o[n] = acc[i][j];
-            else if (!(j & 1)) o[n >> 1] = acc[i][j] / (1.f + expf(-acc[i][j])) * acc[i][j + 1];
+            if (!g.gated) o[n] = acc[i][j];
+            else if (!(j & 1)) o[n >> 1] = g.gated == 2 ? mg_limited(acc[i][j], acc[i][j + 1], g.limit) : acc[i][j] / (1.f + expf(-acc[i][j])) * acc[i][j + 1];
         }
     }
 }
@@ -225,8 +231,8 @@ __global__ void __launch_bounds__(256) moe_gemm_f32_kernel(const MoeGemmF32Args 
 }  // namespace ps
 
 // Sorted rows `x` [x_rows, K] (x_rows: at least the last tile's first row + tile_rows, whatever lies behind the sorted rows), weights
-// `w` [E * N, K], both bf16 and contiguous, K a multiple of 8, N even.  `tile_rows` (16, 32, 64 or 128): the list's tile size.
-PS_API int ps_moe_gemm(const void* x, int x_rows, const void* w, int E, int N, int K, int swiglu, const void* tiles, int tile_rows,
+// `w` [E * N, K], both bf16 and contiguous, K a multiple of 8, N even; `gated` and `limit` as in MoeGemmArgs.  `tile_rows` (16, 32, 64 or 128): the list's tile size.
+PS_API int ps_moe_gemm(const void* x, int x_rows, const void* w, int E, int N, int K, int gated, float limit, const void* tiles, int tile_rows,
                        int max_tiles, void* out, int ldo, void* status, cudaStream_t stream) {
     using namespace ps;
     if (x_rows <= 0 || E <= 0 || N <= 0 || (N & 1) || K <= 0 || K % 8 || max_tiles < 1 || max_tiles > 65535 ||
@@ -236,7 +242,7 @@ PS_API int ps_moe_gemm(const void* x, int x_rows, const void* w, int E, int N, i
     int err = mg_map_2d(&mw, w, (uint64_t)E * N, K, kMgM);
     if (err) return err;
     if ((err = mg_map_2d(&mx, x, (uint64_t)x_rows, K, (uint32_t)tile_rows))) return err;
-    MoeGemmArgs g{(const int*)tiles, N, K, swiglu, out, ldo, (uint32_t*)status, g_ps_wait_budget_cycles};
+    MoeGemmArgs g{(const int*)tiles, N, K, gated, out, ldo, limit, (uint32_t*)status, g_ps_wait_budget_cycles};
     switch (tile_rows) {
         case 16: return launch_moe_gemm<16, 5>(mw, mx, max_tiles, g, stream);
         case 32: return launch_moe_gemm<32, 5>(mw, mx, max_tiles, g, stream);
@@ -246,12 +252,12 @@ PS_API int ps_moe_gemm(const void* x, int x_rows, const void* w, int E, int N, i
     }
 }
 
-// The same in fp32 over tiles of 64 rows; the SwiGLU output is fp32 too.
-PS_API int ps_moe_gemm_f32(const void* x, const void* w, int N, int K, int swiglu, const void* tiles, int max_tiles, void* out, int ldo,
+// The same in fp32 over tiles of 64 rows; the gated output is fp32 too.
+PS_API int ps_moe_gemm_f32(const void* x, const void* w, int N, int K, int gated, float limit, const void* tiles, int max_tiles, void* out, int ldo,
                            cudaStream_t stream) {
     using namespace ps;
     if (N <= 0 || (N & 1) || K <= 0 || max_tiles < 1 || max_tiles > 65535 || (uintptr_t)tiles % 16) return (int)cudaErrorInvalidValue;
-    MoeGemmF32Args g{(const int*)tiles, (const float*)x, (const float*)w, N, K, swiglu, (float*)out, ldo};
+    MoeGemmF32Args g{(const int*)tiles, (const float*)x, (const float*)w, N, K, gated, (float*)out, ldo, limit};
     moe_gemm_f32_kernel<<<dim3((N + kMfT - 1) / kMfT, max_tiles), 256, 0, stream>>>(g);
     return PS_LAUNCH_CHECK();
 }

@@ -1,8 +1,8 @@
 // Routing of a mixture of experts: router logits to every row's experts and weights, and the rows sorted by expert.
 //
-// Per row (a warp): scores = softmax over experts and, behind them, identity experts; choice = score + correction; only experts of
-// the best groups (a group counts as its best member) can be chosen; the `top` largest choices are taken and weighted by their
-// scores divided by the sum of these.  All in 32-bit; ties go to the lower index.
+// Per row (a warp): scores = softmax (or sigmoids) over experts and, behind them, identity experts; choice = score + correction; only
+// experts of the best groups (a group counts as its best member, or as the sum of its two best) can be chosen; the `top` largest
+// choices are taken and weighted by their scores, which may be divided by their sum.  All in 32-bit; ties go to the lower index.
 //
 // Steps of at most 64 rows run one launch: every CTA routes all rows (a bit per row and expert, so that ranks are population
 // counts and every CTA computes the same order) and copies its share of the input rows to their sorted places.  Longer steps
@@ -17,6 +17,7 @@ constexpr int kRtSmallRows = 64, kRtMaxTop = 32, kRtMaxChoices = 1024, kRtWarps 
 struct RouteArgs {
     const float* z; int ldz; const float* correction; const int* row_slot;
     int rows, E, n, top, groups, keep;           // E experts, n = E + identity experts
+    int sigmoid, group_top, renormalize;
     int* index; float* weight; float* identity;  // [rows, top], [rows, top], [rows]
     const uint4* h; int h16; uint4* xs;          // input rows of h16 16-byte units, sorted copies
     int* tiles; int tile_rows;                   // [0]: number of tiles; from [4] on (expert, first row, rows, 0)
@@ -65,20 +66,28 @@ __device__ __forceinline__ void route_row(const RouteArgs& a, int row, float* s,
     float* choice = s + n;
     float* group = s + 2 * n;
     const float* z = a.z + (size_t)row * a.ldz;
-    float m = -INFINITY;
-    for (int i = lane; i < n; i += 32) m = fmaxf(m, z[i]);
-    m = warp_max(m);
-    float sum = 0.f;
-    for (int i = lane; i < n; i += 32) { const float e = expf(z[i] - m); score[i] = e; sum += e; }
-    sum = warp_sum(sum);
-    for (int i = lane; i < n; i += 32) { const float p = score[i] / sum; score[i] = p; choice[i] = p + a.correction[i]; }
+    float sum = 1.f;
+    if (a.sigmoid) {
+        for (int i = lane; i < n; i += 32) score[i] = 1.f / (1.f + expf(-z[i]));
+    } else {
+        float m = -INFINITY;
+        for (int i = lane; i < n; i += 32) m = fmaxf(m, z[i]);
+        m = warp_max(m);
+        sum = 0.f;
+        for (int i = lane; i < n; i += 32) { const float e = expf(z[i] - m); score[i] = e; sum += e; }
+        sum = warp_sum(sum);
+    }
+    for (int i = lane; i < n; i += 32) { const float p = score[i] / sum; score[i] = p; choice[i] = a.correction != nullptr ? p + a.correction[i] : p; }
     __syncwarp();
     if (a.keep < a.groups) {
         const int size = n / a.groups;
         for (int g = lane; g < a.groups; g += 32) {
-            float b = -INFINITY;
-            for (int i = g * size; i < (g + 1) * size; ++i) b = fmaxf(b, choice[i]);
-            group[g] = b;
+            float b = -INFINITY, second = -INFINITY;
+            for (int i = g * size; i < (g + 1) * size; ++i) {
+                second = fmaxf(second, fminf(b, choice[i]));
+                b = fmaxf(b, choice[i]);
+            }
+            group[g] = a.group_top > 1 && size > 1 ? b + second : b;
         }
         __syncwarp();
         rt_top(group, a.groups, a.keep, [](int, int) {});              // kept groups end as minus infinity
@@ -95,7 +104,7 @@ __device__ __forceinline__ void route_row(const RouteArgs& a, int row, float* s,
         total += w;
     });
     if (lane < a.top && id < 0) set_status(a.status, PS_DEV_NONFINITE);
-    weight /= total + 1e-20f;
+    if (a.renormalize) weight /= total + 1e-20f;
 }
 
 // Exclusive prefix sums of rows and tiles per expert by one warp; `count(e)` gives an expert's rows.
@@ -203,18 +212,18 @@ __global__ void __launch_bounds__(256) moe_sort_kernel(const RouteArgs a) {
 }  // namespace ps
 
 // `h`, `xs`: rows of `row_bytes` (a multiple of 16); `tiles`: 4 + 4 * (rows * top / tile_rows + min(E, rows * top)) ints; `pairs`
-// (2 ints per row and place) and `counts` ([E]) are scratch of steps longer than 64 rows.
+// (2 ints per row and place) and `counts` ([E]) are scratch of steps longer than 64 rows.  `correction` may be null; `group_top` 1 or 2.
 PS_API int ps_moe_route(const void* z, int ldz, const void* correction, const void* row_slot, int rows, int E, int identity, int top,
-                        int groups, int keep, void* index, void* weight, void* same, const void* h, int row_bytes, void* xs, void* tiles,
+                        int groups, int keep, int sigmoid, int group_top, int renormalize, void* index, void* weight, void* same, const void* h, int row_bytes, void* xs, void* tiles,
                         int tile_rows, void* pairs, void* counts, void* status, cudaStream_t stream) {
     using namespace ps;
     const int n = E + identity;
     if (rows <= 0 || E <= 0 || identity < 0 || n > kRtMaxChoices || top < 1 || top > kRtMaxTop || groups < 1 || n % groups || keep < 1 || keep > groups ||
-        top > keep * (n / groups) || ldz < n || row_bytes % 16 || tile_rows < 1 || ((uintptr_t)h | (uintptr_t)xs | (uintptr_t)tiles) % 16)
+        group_top < 1 || group_top > 2 || top > keep * (n / groups) || ldz < n || row_bytes % 16 || tile_rows < 1 || ((uintptr_t)h | (uintptr_t)xs | (uintptr_t)tiles) % 16)
         return (int)cudaErrorInvalidValue;
     RouteArgs a;
     a.z = (const float*)z; a.ldz = ldz; a.correction = (const float*)correction; a.row_slot = (const int*)row_slot; a.rows = rows; a.E = E;
-    a.n = n; a.top = top; a.groups = groups; a.keep = keep; a.index = (int*)index; a.weight = (float*)weight; a.identity = (float*)same;
+    a.n = n; a.top = top; a.groups = groups; a.keep = keep; a.sigmoid = sigmoid; a.group_top = group_top; a.renormalize = renormalize; a.index = (int*)index; a.weight = (float*)weight; a.identity = (float*)same;
     a.h = (const uint4*)h; a.h16 = row_bytes / 16; a.xs = (uint4*)xs; a.tiles = (int*)tiles; a.tile_rows = tile_rows;
     a.pairs = (int2*)pairs; a.counts = (int*)counts; a.status = (uint32_t*)status;
     static bool set = false;

@@ -219,16 +219,14 @@ def build_engine_weights(cfg: RotutarConfig, get: Callable[[str], torch.Tensor],
         dk, dv = r.dim_padded, r.vdim_padded
         parts = (("q", r.kv_heads, r.dim, dk), ("k", r.kv_heads, r.dim, dk), ("v", r.heads, r.vdim, dv))
         q = (H + 2 * G) * D
-        k = q + r.kv_heads * dk
-        v = k + r.kv_heads * dk
-        b = v + r.heads * dv
+        b = q + 2 * r.kv_heads * dk + r.heads * dv
         a1, g1 = t(y + "a1"), t(y + "g1")
         ra, rg = pad(a1.shape[0], 16), pad(g1.shape[0], 16)
         a = b + pad(r.heads, 16)
         rows += [pad_heads(t(y + n), h, d, to) for n, h, d, to in parts]
         rows += [pad_rows(t(y + "b"), pad(r.heads, 16)), pad_rows(a1, ra), pad_rows(g1, rg)]
         conv = torch.cat([pad_heads(t(f"{y}{n}.conv"), h, d, to) for n, h, d, to in parts], 0).T.contiguous()
-        delta = DeltaSpec(r.heads, r.kv_heads, dk, dv, r.dim, r.vdim, q, k, v, b, a, a + ra, cfg.norm_eps, conv,
+        delta = DeltaSpec(r.heads, r.kv_heads, dk, dv, r.dim, r.vdim, q, b, a, a + ra, cfg.norm_eps, conv,
                           pad_cols(pad_heads(t(y + "a2"), r.heads, r.dim, dk), ra).contiguous(),
                           pad_heads(f32(y + "dt_bias"), r.heads, r.dim, dk).contiguous(), torch.exp(f32(y + "A_log")),
                           pad_cols(pad_heads(t(y + "g2"), r.heads, r.vdim, dv), rg).contiguous(),

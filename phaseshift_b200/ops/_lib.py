@@ -53,7 +53,7 @@ def checked_build() -> bool:
 def set_limits(max_slots: int, max_rows: int, status) -> None:
     """Checked build: register the descriptor limits and the status word with every kernel file that asserts on them."""
     L = lib()
-    for tag in ("gdn_recurrent", "gdn_chunked", "gla"):
+    for tag in ("gdn_recurrent", "gdn_chunked", "gla", "delta_rule"):
         fn = getattr(L, "ps_set_limits_" + tag, None)
         if fn is not None:
             fn.restype = ctypes.c_int

@@ -21,7 +21,7 @@ from ..models.qwen35.weights import AttnW, GdnW, LinearW
 from ..runtime.batch import ROW_BUCKETS, StepBatch
 from ..runtime.state import GdnLayerState, KVLayer, ModelState
 from . import _lib
-from .specs import AttnSpec, GlaSpec, HeadsSpec, LatentSpec, MoeSpec, Pending, Routed, StreamWrite
+from .specs import AttnSpec, DeltaSpec, GatedNorm, GlaSpec, HeadsSpec, LatentSpec, MoeSpec, Pending, Routed, StreamWrite
 from ._lib import c_float, c_int, c_ll, ptr
 
 WFMT = {"bf16": 0, "nvfp4": 1, "mxfp8": 2}
@@ -695,6 +695,39 @@ class CudaOps(OpTrace):
         self.launches += 1
         return (xo if changed else x), h
 
+    # ------------------------------------------------------------------ norms behind the sublayers
+    def gated_norm(self, x: torch.Tensor, pend: Optional[GatedNorm], *, eps: float, groups: int, norm_w: Optional[torch.Tensor] = None,
+                   width: int = 0, name: str = ""):
+        """x + the sublayer's gated and normed result (ops/specs.py: GatedNorm), and the next projection's input: the new residual
+        itself, or with `norm_w` its norm in groups, zero-padded to `width` columns (0: none).  One launch.  Returns (residual, rows or
+        None); the residual lives in one buffer of its own, `x` itself is only overwritten when it is that buffer."""
+        rows, W = x.shape
+        f32 = self.act_dtype == torch.float32
+        xo = self.buf("x_res", rows, W, torch.float32) if pend is not None else None
+        h = self.buf(name, rows, width, self.act_dtype) if width else None
+        if xo is None and h is None:
+            return x, None
+        p = pend if pend is not None else GatedNorm(None, None, None)
+        r = p.routed
+        if p.gate is not None and f32 and p.gate.dtype != torch.float32:
+            raise ValueError("32-bit engines have 32-bit gates")
+        ld = lambda t: c_int(t.stride(0) if t is not None else 0)
+        _lib.call("ps_gated_norm", ptr(x), ptr(xo), c_int(rows), c_int(W), c_int(groups), c_float(eps), ptr(p.a), ld(p.a), c_float(p.scale_a),
+                  ptr(p.b), ld(p.b), c_float(p.scale_b), c_int(r.index.shape[1] if r is not None else 0), ptr(r.index if r is not None else None),
+                  ptr(r.weight if r is not None else None), ptr(p.experts), ld(p.experts), ptr(p.gate), ld(p.gate),
+                  c_int(1 if p.gate is not None and p.gate.dtype == torch.float32 else 0), ptr(p.gate_bias), ptr(p.norm_w), ptr(norm_w), ptr(h),
+                  c_int(1 if f32 else 0), c_int(width))
+        self.launches += 1
+        return (xo if xo is not None else x), h
+
+    def soft_limit(self, logits: torch.Tensor, cap: float) -> torch.Tensor:
+        """cap * tanh(logits / cap), in place."""
+        if not logits.is_contiguous() or logits.dtype != torch.float32:
+            raise ValueError("soft_limit takes contiguous fp32 logits")
+        _lib.call("ps_soft_limit", ptr(logits), c_ll(logits.numel()), c_float(cap))
+        self.launches += 1
+        return logits
+
     # ------------------------------------------------------------------ parallel residual streams
     def stream_norm(self, x: torch.Tensor, pend: Optional[StreamWrite], *, read: Optional[torch.Tensor] = None,
                     norm_w: Optional[torch.Tensor] = None, eps: float, width: int = 0, name: str = "", last: bool = False):
@@ -779,7 +812,8 @@ class CudaOps(OpTrace):
         pairs = None if small else self.buf(f"moe_pairs{s.top}", rows, 2 * s.top, i32)
         counts = None if small else self.buf(f"moe_counts{s.experts}", 1, s.experts, i32)
         _lib.call("ps_moe_route", ptr(logits), c_int(logits.stride(0)), ptr(s.correction), ptr(b.row_slot), c_int(rows), c_int(s.experts),
-                  c_int(s.identity), c_int(s.top), c_int(s.groups), c_int(s.keep), ptr(out.index), ptr(out.weight), ptr(out.identity), ptr(h),
+                  c_int(s.identity), c_int(s.top), c_int(s.groups), c_int(s.keep), c_int(int(s.sigmoid)), c_int(s.group_top), c_int(int(s.renormalize)),
+                  ptr(out.index), ptr(out.weight), ptr(out.identity), ptr(h),
                   c_int(K * h.element_size()), ptr(out.inputs), ptr(out.tiles), c_int(tile), ptr(pairs), ptr(counts), ptr(self.status))
         self.launches += 1 if small else 3
         return out
@@ -799,16 +833,17 @@ class CudaOps(OpTrace):
         R = x.shape[0] - routed.tile_rows
         act = self.buf(f"moe_act{s.ff}", x.shape[0], s.ff, dt)
         y = self.buf(f"moe_y{s.n_out}", R, s.n_out, torch.float32)
+        limit = 0.0 if s.limit is None else s.limit
 
         def product(a, w, N, K, gated, out):
             if dt == torch.float32:
-                _lib.call("ps_moe_gemm_f32", ptr(a), ptr(w), c_int(N), c_int(K), c_int(gated), ptr(routed.tiles), c_int(routed.max_tiles), ptr(out),
-                          c_int(out.stride(0)))
+                _lib.call("ps_moe_gemm_f32", ptr(a), ptr(w), c_int(N), c_int(K), c_int(gated), c_float(limit), ptr(routed.tiles),
+                          c_int(routed.max_tiles), ptr(out), c_int(out.stride(0)))
             else:
-                _lib.call("ps_moe_gemm", ptr(a), c_int(a.shape[0]), ptr(w), c_int(s.experts), c_int(N), c_int(K), c_int(gated), ptr(routed.tiles),
-                          c_int(routed.tile_rows), c_int(routed.max_tiles), ptr(out), c_int(out.stride(0)), ptr(self.status))
+                _lib.call("ps_moe_gemm", ptr(a), c_int(a.shape[0]), ptr(w), c_int(s.experts), c_int(N), c_int(K), c_int(gated), c_float(limit),
+                          ptr(routed.tiles), c_int(routed.tile_rows), c_int(routed.max_tiles), ptr(out), c_int(out.stride(0)), ptr(self.status))
             self.launches += 1
-        product(x, s.gate_up, 2 * s.ff, K, 1, act)
+        product(x, s.gate_up, 2 * s.ff, K, 1 if s.limit is None else 2, act)
         product(act, s.down, s.n_out, s.ff, 0, y)
         return y
 
@@ -959,9 +994,9 @@ class CudaOps(OpTrace):
 
         def call(chunked: int, limit: int, blocks: int, scratch) -> None:
             _lib.call("ps_gla", c_int(chunked), ptr(proj), c_int(proj.stride(0)), c_int(1 if f32 else 0), c_int(g.heads), c_int(g.dk),
-                      c_int(g.dv), c_int(g.dv_true), c_int(g.q_off), c_int(g.k_off), c_int(g.v_off), c_int(g.g_off), c_int(g.a_off),
+                      c_int(g.dv), c_int(g.dv_true), c_int(g.q_off), c_int(max(g.k_off, 0)), c_int(g.v_off), c_int(g.g_off), c_int(g.a_off),
                       c_int(g.rank), c_float(g.q_scale), c_float(g.inv_tau), c_float(g.eps), ptr(g.a2), ptr(g.a2_bias), ptr(g.norm_w),
-                      ptr(gs.rec), ptr(b.seq_desc), c_int(n_seqs), c_int(limit), ptr(out), c_int(blocks), *[ptr(t) for t in scratch])
+                      ptr(g.lower), ptr(gs.rec), ptr(b.seq_desc), c_int(n_seqs), c_int(limit), ptr(out), c_int(blocks), *[ptr(t) for t in scratch])
         if long:
             C = int(L.ps_gla_block_rows())
             blocks = sum(-(-n // C) for n in long)
@@ -980,3 +1015,20 @@ class CudaOps(OpTrace):
         if t is None or t.numel() < sum(sizes):
             t = self._gla_buf = torch.empty(sum(sizes), dtype=torch.float32, device=self.device)
         return torch.split(t[:sum(sizes)], sizes)
+
+    # ------------------------------------------------------------------ delta rule with a decay per channel
+    def delta(self, proj: torch.Tensor, d: DeltaSpec, b: StepBatch, gs: GdnLayerState, st: ModelState,
+              history: Optional[torch.Tensor]) -> torch.Tensor:
+        """ops/specs.py: DeltaSpec.  ``history``: the layer's convolution rows in the state."""
+        rows, f32 = proj.shape[0], self.act_dtype == torch.float32
+        for t in (proj, d.conv, d.a2, d.g2):
+            if t.dtype != self.act_dtype:
+                raise ValueError("projection rows, convolution and low-rank weights have the engine's type")
+        out = self.buf(f"delta_o{d.heads}x{d.dv}", rows, d.heads * d.dv, self.act_dtype)
+        n_seqs = b.max_seqs if b.graph_static else b.n_seqs
+        args = (c_int(d.heads), c_int(d.kv_heads), c_int(d.dk), c_int(d.dv), c_int(d.dk_true), c_int(d.dv_true), c_int(d.q_off), c_int(d.b_off),
+                c_int(d.a_off), c_int(d.g_off), c_int(d.a2.shape[1]), c_int(d.g2.shape[1]), c_int(d.taps), c_float(d.eps), ptr(d.conv), ptr(d.a2),
+                ptr(d.dt_bias), ptr(d.rate), ptr(d.g2), ptr(d.norm_w), ptr(history), ptr(gs.rec), ptr(b.seq_desc), c_int(n_seqs), ptr(out))
+        _lib.call("ps_delta_rows", ptr(proj), c_int(proj.stride(0)), c_int(1 if f32 else 0), *args, c_int(0))
+        self.launches += 1
+        return out

@@ -552,7 +552,7 @@ class RefOps(OpTrace):
         # every value head's own channels: columns of the projection, and of the convolution
         cols = torch.cat([d.q_off + head // (H // G) * dk + torch.arange(dk), d.k_off + head // (H // G) * dk + torch.arange(dk),
                           d.v_off + head * dv + torch.arange(dv)], 1)
-        w = d.conv.float()[:, cols - d.q_off]                     # [taps, heads, 2 dk + dv] (the three parts lie side by side)
+        w = d.conv.float()[:, cols - d.q_off]                     # [taps, heads, 2 dk + dv]
         g = torch.exp(-d.rate[:, None] * F.softplus(p[:, d.a_off:d.a_off + d.a2.shape[1]] @ d.a2.float().T + d.dt_bias).reshape(-1, H, dk))
         beta = torch.sigmoid(p[:, d.b_off:d.b_off + H])
         gate = torch.sigmoid(p[:, d.g_off:d.g_off + d.g2.shape[1]] @ d.g2.float().T)

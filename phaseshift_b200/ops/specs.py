@@ -271,9 +271,7 @@ class DeltaSpec:
     dv: int
     dk_true: int
     dv_true: int
-    q_off: int
-    k_off: int
-    v_off: int
+    q_off: int                  # the k and v heads lie behind the q heads
     b_off: int
     a_off: int
     g_off: int
@@ -288,6 +286,14 @@ class DeltaSpec:
     @property
     def taps(self) -> int:
         return self.conv.shape[0]
+
+    @property
+    def k_off(self) -> int:
+        return self.q_off + self.kv_heads * self.dk
+
+    @property
+    def v_off(self) -> int:
+        return self.k_off + self.kv_heads * self.dk
 
 
 @dataclass
