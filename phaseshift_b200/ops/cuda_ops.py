@@ -1029,6 +1029,30 @@ class CudaOps(OpTrace):
         args = (c_int(d.heads), c_int(d.kv_heads), c_int(d.dk), c_int(d.dv), c_int(d.dk_true), c_int(d.dv_true), c_int(d.q_off), c_int(d.b_off),
                 c_int(d.a_off), c_int(d.g_off), c_int(d.a2.shape[1]), c_int(d.g2.shape[1]), c_int(d.taps), c_float(d.eps), ptr(d.conv), ptr(d.a2),
                 ptr(d.dt_bias), ptr(d.rate), ptr(d.g2), ptr(d.norm_w), ptr(history), ptr(gs.rec), ptr(b.seq_desc), c_int(n_seqs), ptr(out))
-        _lib.call("ps_delta_rows", ptr(proj), c_int(proj.stride(0)), c_int(1 if f32 else 0), *args, c_int(0))
-        self.launches += 1
+        T, L = self.GDN_CHUNKED_MIN_ROWS, _lib.lib()
+        chunk_ok = (not f32 and not b.graph_static
+                    and bool(L.ps_delta_chunked_ok(c_int(d.dk), c_int(d.dv), c_int(d.a2.shape[1]), c_int(d.g2.shape[1]))))
+        seq_rows = [len(sq.token_ids) for sq in b.seqs] if chunk_ok else []
+        long = [n for n in seq_rows if n > T]
+        if long:
+            C = int(L.ps_delta_block_rows())
+            blocks = sum(-(-n // C) for n in long)
+            _lib.call("ps_delta_chunked", ptr(proj), c_int(proj.stride(0)), *args, c_int(T), c_int(blocks),
+                      *[ptr(t) for t in self._delta_scratch(blocks, rows, C, d)])
+            self.launches += 3
+        if not long or len(long) < len(seq_rows):
+            _lib.call("ps_delta_rows", ptr(proj), c_int(proj.stride(0)), c_int(1 if f32 else 0), *args, c_int(T if long else 0))
+            self.launches += 1
         return out
+
+    def _delta_scratch(self, blocks: int, rows: int, C: int, d: DeltaSpec):
+        """Scratch of the chunked delta rule (its matrices as bf16 pairs, U, block decays, outputs before the head norm); one
+        allocation that grows to the largest step seen."""
+        L = _lib.lib()
+        L.ps_delta_mats.restype = ctypes.c_longlong
+        n = blocks * d.heads
+        sizes = [n * int(L.ps_delta_mats(c_int(d.dk))) // 2, n * C * d.dv, n * d.dk, rows * d.heads * d.dv]
+        t = getattr(self, "_delta_buf", None)
+        if t is None or t.numel() < sum(sizes):
+            t = self._delta_buf = torch.empty(sum(sizes), dtype=torch.float32, device=self.device)
+        return torch.split(t[:sum(sizes)], sizes)
