@@ -55,7 +55,7 @@ def _parse():
     ap.add_argument("--serving-slots", type=int, default=32,
                     help="sequence slots of the serving block (fewer than the requests, so that later admissions can hit "
                          "the prefix cache the earlier ones filled)")
-    ap.add_argument("--compare", default="", choices=["", "gebuzen", "luvutar", "fudulix"],
+    ap.add_argument("--compare", default="", choices=["", "gebuzen", "luvutar", "fudulix", "rotutar"],
                     help="instead of the headline workload: prefill and decode of a model family beside the closest other one (Gebuzen: the "
                          "hybrid decoder; Luvutar: Gebuzen; Fudulix: Luvutar) at equal layer shapes (random bf16 weights, 1 GPU), and the mixers' kernels "
                          "against their rooflines")

@@ -1,6 +1,7 @@
 """Throughput of a model family beside the closest other one at equal size (`bench.py --compare gebuzen`: the hybrid decoder;
-`--compare luvutar`: Gebuzen; `--compare fudulix`: Luvutar): prefill and decode of a stack of layers of real-model shapes with random bf16 weights, and the
-mixers' kernels alone against their rooflines.
+`--compare luvutar`: Gebuzen; `--compare fudulix`: Luvutar; `--compare rotutar`: Gebuzen, with Fudulix for the mixtures and the hybrid
+decoder for the delta rule): prefill and decode of a stack of layers of real-model shapes with random bf16 weights, and the mixers'
+kernels alone against their rooflines.
 
 Every kernel row gives its time, the algorithmic bytes and FLOPs of one launch group, and the fraction of the roofline
 max(bytes / measured copy bandwidth, FLOPs / measured bf16 throughput) it reaches.  Kernel timings flush L2 between samples.
@@ -59,6 +60,36 @@ def fudulix_pairs(layers: int) -> List[tuple]:
     small.layers = [narrow(L) for L in small.layers]
     return [("4b", cut(fudulix_4b_config()), cut(luvutar_4b_config())), ("4b, attention heads of 128, experts of 512", small, None),
             ("27b", cut(fudulix_27b_config()), cut(luvutar_27b_config()))]
+
+
+def rotutar_pairs(layers: int) -> List[tuple]:
+    """(label, Rotutar, Gebuzen, Fudulix and hybrid configurations) of equal width, attention heads, recurrent heads, active
+    feed-forward weights and depth."""
+    from ..models.fudulix.config import fudulix_27b_config, fudulix_4b_config
+    from ..models.gebuzen.config import gebuzen_27b_config, gebuzen_4b_config
+    from ..models.qwen35.config import qwen35_27b_config, qwen35_4b_config
+    from ..models.rotutar.config import ForgetLinear, GatedDelta, Layer, Mixture, Parallel, WindowAttention, rotutar_27b_config, rotutar_4b_config
+
+    def cut(cfg):
+        cfg.layers = cfg.layers[:layers]
+        return cfg
+
+    def narrow(L):
+        """Half the head sizes, twice the heads; half-size experts, twice as many."""
+        m, c = L.mixer, L.mlp
+        if isinstance(m, Parallel):
+            l, r = m.left, m.right
+            m = Parallel(WindowAttention(32, 8, 128, 128, 128 ** -0.5, l.window, l.rot_base, 32), m.left_scale,
+                         GatedDelta(2 * r.heads, 2 * r.kv_heads, 64, 64, r.taps), m.right_scale)
+        else:
+            m = ForgetLinear(2 * m.heads, 64, 64)
+        return Layer(m, Mixture(c.ff // 2, c.limit, 2 * c.experts, 2 * c.top, 2 * c.groups, 2 * c.keep) if isinstance(c, Mixture) else c)
+
+    small = cut(rotutar_4b_config(name="rotutar-4b-narrow"))
+    small.layers = [narrow(L) for L in small.layers]
+    return [("4b", cut(rotutar_4b_config()), cut(gebuzen_4b_config()), cut(fudulix_4b_config()), qwen35_4b_config(num_hidden_layers=layers)),
+            ("4b, attention heads of 128, recurrent heads of 64, experts of 576", small, None, None, None),
+            ("27b", cut(rotutar_27b_config()), cut(gebuzen_27b_config()), cut(fudulix_27b_config()), qwen35_27b_config(num_hidden_layers=layers))]
 
 
 def gebuzen_pairs(layers: int) -> List[tuple]:
@@ -369,6 +400,80 @@ def fudulix_kernel_times(eng: Engine, timer: _Flushed, peaks: dict, rows: int, c
     return res
 
 
+def rotutar_kernel_times(eng: Engine, timer: _Flushed, peaks: dict, rows: int, context: int, batch: int) -> Dict[str, dict]:
+    """As `kernel_times`, for the mixers, both feed-forwards and the norms behind them."""
+    from ..models.rotutar.weights import DenseW, MixtureW, ParallelW
+    from ..ops.specs import GatedNorm
+    hbm, tc = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    ops, st, w = eng.ops, eng.state, eng.runner.w
+    res: Dict[str, dict] = {}
+
+    def add(name, fn, nbytes, flops):
+        us = timer(fn)
+        floor = max(nbytes / hbm, flops / tc) * 1e6
+        res[name] = {"us": round(us, 1), "gb": round(nbytes / 1e9, 4), "gflop": round(flops / 1e9, 2), "roofline_us": round(floor, 2),
+                     "roofline_frac": round(floor / us, 4)}
+
+    def rand(n, width, dtype=torch.bfloat16):
+        return torch.randn(n, width, device=eng.device, dtype=torch.float32).to(dtype)
+
+    W, groups, kin = eng.cfg.hidden_size, eng.cfg.norm_groups, w.lm_head.K
+    lp = next(i for i, L in enumerate(w.layers) if isinstance(L.mixer, ParallelW))
+    lf = next(i for i, L in enumerate(w.layers) if not isinstance(L.mixer, ParallelW))
+    P, F = w.layers[lp], w.layers[lf]
+    dense = next(L.mlp for L in w.layers if isinstance(L.mlp, DenseW))
+    mix = next(L.mlp for L in w.layers if isinstance(L.mlp, MixtureW))
+    a, d, f, m = P.mixer.attn, P.mixer.delta, F.mixer.gla, mix.moe
+    shapes = [("prefill", [(0, rows)]), ("prefill after context", [(context, rows)]), ("decode 1", [(context, 1)]),
+              (f"decode {batch}", [(context, 1)] * batch)]
+    for name, seqs in shapes:
+        b, opened = _batch(eng, seqs)
+        n = b.n_rows
+        pairs = sum(min(q + 1, a.window) for p, k in seqs for q in range(p, p + k))
+        kv_tok = sum(min(p + k, a.window + k - 1) for p, k in seqs)
+        proj = rand(n, P.in_proj.N)
+        q = ops.attn_heads(proj, P.mixer.heads, b, st.kv[lp], st)
+        add("attention, " + name, lambda: ops.attention(q, a, b, st.kv[lp], st, b.max_visible_launch),
+            2 * n * a.heads * a.dim * 2 + kv_tok * 2 * a.kv_heads * a.dim * 2, 4.0 * pairs * a.heads * a.dim)
+        ra, rg = d.a2.shape[1], d.g2.shape[1]
+        state = len(seqs) * d.heads * d.dk * d.dv * 4 * 2
+        io = n * (2 * d.kv_heads * d.dk + 2 * d.heads * d.dv + d.heads + ra + rg) * 2 + (d.a2.numel() + d.g2.numel()) * 2
+        flops = n * d.heads * (6.0 * d.dk * d.dv + 64.0 * (2 * d.dk + d.dv)) + 2.0 * n * (d.a2.numel() + d.g2.numel())
+        add("delta rule, " + name, lambda: ops.delta(proj, d, b, st.gdn[lp], st, st.conv[lp]), io + state, flops)
+        fproj = rand(n, F.in_proj.N)
+        state = len(seqs) * f.heads * f.dk * f.dv * 4 * 2
+        add("forget-gate linear attention, " + name, lambda: ops.gla(fproj, f, b, st.gdn[lf], st), n * f.heads * 2 * (f.dk + f.dv) * 2 + state,
+            n * f.heads * (4.0 * f.dk * f.dv + 64.0 * (f.dk + f.dv)))
+        if name != "prefill after context":
+            h = rand(n, kin)
+            add("heads, " + name, lambda: ops.attn_heads(proj, P.mixer.heads, b, st.kv[lp], st), n * 2 * P.mixer.heads.channels * 2, 0.0)
+            for what, lw, kw in (("in_proj", P.in_proj, {}), ("gate_up", dense.gate_up, {"swiglu": True}), ("gate of the result", dense.gate, {}),
+                                 ("router and gate", mix.router, {"out_f32": True})):
+                cols = lw.N // 2 if kw.get("swiglu") else lw.N
+                add(f"{what}, {name}", lambda: ops.linear(h, lw, name="bench_" + what, **kw),
+                    lw.N * lw.k_padded * 2 + n * (lw.K * 2 + cols * (4 if kw.get("out_f32") else 2)), 2.0 * n * lw.N * lw.K)
+            x, ya, yb = (rand(n, W, torch.float32) for _ in range(3))
+            pend = GatedNorm(proj[:, P.gate_off:], P.gate1, P.norm1, ya, 0.7, yb, 0.7)
+            add("gated norm, " + name, lambda: ops.gated_norm(x, pend, eps=1e-6, groups=groups, width=kin, name="bench_h"), n * W * (4 * 4 + 2 + 2), 0.0)
+            z = ops.linear(h, mix.router, name="bench_z", out_f32=True)
+            r = ops.moe_route(z, h, m, b)
+            R, used = int((r.index >= 0).sum()), len(set(r.tiles[1:1 + int(r.tiles[0, 0]), 0].tolist()))
+            add("routing, " + name, lambda: ops.moe_route(z, h, m, b), n * (m.experts * 4 + kin * 2 + m.top * 8) + R * kin * 2, 0.0)
+            K = m.gate_up.shape[1]
+            add("experts, " + name, lambda: ops.moe_experts(r, m), used * 3 * m.ff * K * 2 + R * (K * 2 + 2 * m.ff * 2 + m.n_out * 4),
+                2.0 * R * (2 * m.ff * K + m.n_out * m.ff))
+            ye = ops.moe_experts(r, m)
+            pend2 = GatedNorm(z[:, mix.gate_off:], F.gate2, F.norm2, routed=r, experts=ye)
+            add("gated norm of a mixture, " + name, lambda: ops.gated_norm(x, pend2, eps=1e-6, groups=groups, width=kin, name="bench_h"),
+                n * W * (2 * 4 + 4 + 2) + R * m.n_out * 4, 0.0)
+        if name.startswith("decode"):
+            lg = rand(n, w.lm_head.N, torch.float32)
+            add("soft limit, " + name, lambda: ops.soft_limit(lg, 30.0), n * w.lm_head.N * 8, 0.0)
+        for o in opened:
+            eng.close_sequence(o)
+    return res
+
+
 def _prefill_core(ops, q, s, b, st, kv, gate):
     """The attention over keys and values that one call of `latent_attention` has gathered and expanded."""
     out = ops.latent_attention(q, s, b, kv, st, gate)
@@ -383,8 +488,8 @@ def run(peaks: dict, layers: int = 16, prompt_tokens: int = 2048, steps: int = 5
     timer = _Flushed(dev)
     out = {"layers": layers, "prompt_tokens": prompt_tokens, "batch": batch, "sizes": {}}
     pairs, names = {"gebuzen": (gebuzen_pairs, ("gebuzen", "hybrid")), "luvutar": (luvutar_pairs, ("luvutar", "gebuzen")),
-                    "fudulix": (fudulix_pairs, ("fudulix", "luvutar"))}[which]
-    kernels = {"luvutar": luvutar_kernel_times, "fudulix": fudulix_kernel_times}
+                    "fudulix": (fudulix_pairs, ("fudulix", "luvutar")), "rotutar": (rotutar_pairs, ("rotutar", "gebuzen", "fudulix", "hybrid"))}[which]
+    kernels = {"luvutar": luvutar_kernel_times, "fudulix": fudulix_kernel_times, "rotutar": rotutar_kernel_times}
     for label, *cfgs in pairs(layers):
         row = out["sizes"][label] = {}
         for name, cfg in zip(names, cfgs):

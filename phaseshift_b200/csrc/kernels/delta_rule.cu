@@ -18,14 +18,13 @@
 // S_end = diag(exp(B_end)) S0 + (k exp(B_end - B))^T Delta.  With T = (I + A)^-1 everything but the state is independent of it:
 //   delta_prepare  per (block, head): convolutions, unit vectors, decays; M, T, W = T diag(beta) (k exp(B)), U = T diag(beta) V and the
 //                  decayed queries and keys
-//   delta_scan     per (sequence, head, 32 value columns): Delta = U - W S0,  o = Qd S0 + M Delta,  S = diag(dec) S0 + Kd^T Delta
+//   delta_scan     per (sequence, head, 32 or 64 value columns): Delta = U - W S0,  o = Qd S0 + M Delta,  S = diag(dec) S0 + Kd^T Delta
 //   delta_finish   per (block, head): head norm, output gate, and the convolution's history
 // No exponential of a positive number is formed, whatever the decays: the triangles are cut into 16-row sub-blocks; off the diagonal
 // exp(B_t - B_s) factors through the end of the key's sub-block and of the sub-block before the query's, on the diagonal it is
 // evaluated pair by pair.  (The triangular form is that of "Parallelizing Linear Transformers with the Delta Rule over Sequence Length"
 // by Songlin Yang, Bailin Wang, Yu Zhang, Yikang Shen and Yoon Kim; sub-blocks as in gla.cu.)
-// The products of delta_prepare run on TF32 mma.sync with both operands split into two terms, those of the scan on bf16 mma.sync with
-// both operands split into two bf16 terms (16 bits of mantissa); sums and the state are fp32.
+// The products run on bf16 mma.sync with both operands split into two terms (16 bits of mantissa); sums and the state are fp32.
 #include "ps_common.cuh"
 
 namespace ps {
@@ -236,9 +235,9 @@ __global__ void __launch_bounds__(256, 2) delta_rows_kernel(const DeltaArgs a) {
 
 // ------------------------------------------------------------------------------------------------ chunked form (bf16 engines)
 constexpr int kDC = 64;                 // rows of a block
-constexpr int kDPrepThreads = 512, kDScanThreads = 256, kDFinThreads = 256;
-constexpr int kDSlice = 32;             // value columns of a scan CTA
+constexpr int kDPrepThreads = 512, kDScanThreads = 512, kDFinThreads = 256;
 constexpr int kDTP = kDC + 4;
+template <int N> struct DeltaInt { static constexpr int value = N; };
 
 struct DeltaChunkArgs {
     DeltaArgs a;
@@ -262,16 +261,6 @@ __device__ __forceinline__ bool delta_find_block(const DeltaArgs& a, int blk, De
     return false;
 }
 
-__device__ __forceinline__ uint32_t dr_tf32(float x) { uint32_t r; asm("cvt.rna.tf32.f32 %0, %1;" : "=r"(r) : "f"(x)); return r; }
-__device__ __forceinline__ void dr_split(float x, uint32_t& hi, uint32_t& lo) {
-    hi = dr_tf32(x);
-    lo = dr_tf32(x - __uint_as_float(hi));
-}
-__device__ __forceinline__ void dr_mma_tf32(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-                 : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
 __device__ __forceinline__ void dr_mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};\n"
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
@@ -300,131 +289,239 @@ __device__ __forceinline__ void dr_widen(const uint4& v, float (&f)[8]) {
     for (int i = 0; i < 4; ++i) { const float2 t = bf16x2_bits_to_f32x2(u[i]); f[2 * i] = t.x; f[2 * i + 1] = t.y; }
 }
 
-// Convolution + silu of eight channels over four consecutive rows of a block.  `src`: row 0 of the block at the channels, `hist`: the
-// head's history at the channels (rows of `hist_ld`), `w`: the taps at the channels (rows of C); rows from n on become zero.
-template <int TAPS>
-__device__ __forceinline__ void delta_conv(const __nv_bfloat16* src, int ld, const __nv_bfloat16* hist, size_t hist_ld, const __nv_bfloat16* w, int C,
-                                           int taps, int r0, int n, int before, int pos0, float* dst, int pitch) {
-    constexpr int kRun = 4;
-    const int T = TAPS > 0 ? TAPS : taps, back = T - 1;
-    auto row = [&](int r) {                            // `before`: rows of the portion ahead of the block
-        if (r >= n || pos0 + r < 0) return make_uint4(0, 0, 0, 0);
-        if (r + before >= 0) return *reinterpret_cast<const uint4*>(src + (ptrdiff_t)r * ld);
-        return *reinterpret_cast<const uint4*>(hist + (size_t)((pos0 + r) % back) * hist_ld);
-    };
-    float y[kRun][8];
+__device__ __forceinline__ float dr_ex2(float x) { float r; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x)); return r; }
+// Products with operands split into a high and a low part, n column tiles of eight; the low parts' product is left out.  Every round
+// runs over all accumulators, so that neighbouring instructions do not wait for each other.
+template <int N>
+__device__ __forceinline__ void dr_mma3(float (&acc)[N][4], const uint32_t (&ah)[4], const uint32_t (&al)[4], const uint32_t (&bh)[N / 2][4],
+                                        const uint32_t (&bl)[N / 2][4]) {
 #pragma unroll
-    for (int i = 0; i < kRun; ++i)
+    for (int j = 0; j < N; ++j) dr_mma_bf16(acc[j], al, bh[j / 2][j % 2 * 2], bh[j / 2][j % 2 * 2 + 1]);
+#pragma unroll
+    for (int j = 0; j < N; ++j) dr_mma_bf16(acc[j], ah, bl[j / 2][j % 2 * 2], bl[j / 2][j % 2 * 2 + 1]);
+#pragma unroll
+    for (int j = 0; j < N; ++j) dr_mma_bf16(acc[j], ah, bh[j / 2][j % 2 * 2], bh[j / 2][j % 2 * 2 + 1]);
+}
+
+// log(1 + exp(x)) from the series of the inverse hyperbolic tangent: log(1 + e) = 2 artanh(e / (2 + e)), e <= 1
+__device__ __forceinline__ float dr_softplus_fast(float x) {
+    const float e = __expf(-fabsf(x)), s = __fdividef(e, 2.f + e), q = s * s;
+    float p = 1.f / 15.f;
+    p = fmaf(p, q, 1.f / 13.f); p = fmaf(p, q, 1.f / 11.f); p = fmaf(p, q, 1.f / 9.f); p = fmaf(p, q, 1.f / 7.f);
+    p = fmaf(p, q, 1.f / 5.f); p = fmaf(p, q, 1.f / 3.f); p = fmaf(p, q, 1.f);
+    return fmaf(2.f * s, p, fmaxf(x, 0.f));
+}
+
+// Convolution + silu of eight channels over the RUN rows from r0 on of a block; rows from n on become zero.  `row(r)`: the projected
+// channels of row r (negative: before the block; zero before the sequence), `weight(j)`: those of tap j.
+template <int TAPS, int RUN, typename Row, typename Weight>
+__device__ __forceinline__ void delta_conv(int taps, int r0, int n, Row row, Weight weight, float (&y)[RUN][8]) {
+    const int T = TAPS > 0 ? TAPS : taps;
+#pragma unroll
+    for (int i = 0; i < RUN; ++i)
 #pragma unroll
         for (int e = 0; e < 8; ++e) y[i][e] = 0.f;
     if constexpr (TAPS > 0) {
-        uint4 x[kRun + TAPS - 1];
+        uint4 x[RUN - 1 + TAPS];
+        float wv[TAPS][8];
 #pragma unroll
-        for (int i = 0; i < kRun + TAPS - 1; ++i) x[i] = row(r0 + i - (TAPS - 1));
+        for (int i = 0; i < RUN - 1 + TAPS; ++i) x[i] = row(r0 + i - (TAPS - 1));
 #pragma unroll
-        for (int j = 0; j < TAPS; ++j) {               // tap j meets the row TAPS - 1 - j before
-            float wv[8];
-            dr_widen(*reinterpret_cast<const uint4*>(w + (size_t)j * C), wv);
+        for (int j = 0; j < TAPS; ++j) dr_widen(weight(j), wv[j]);
 #pragma unroll
-            for (int i = 0; i < kRun; ++i) {
-                float xv[8];
-                dr_widen(x[i + j], xv);
+        for (int k = 0; k < RUN - 1 + TAPS; ++k) {           // row k of the run meets tap k - i of output i
+            float xv[8];
+            dr_widen(x[k], xv);
 #pragma unroll
-                for (int e = 0; e < 8; ++e) y[i][e] = fmaf(wv[e], xv[e], y[i][e]);
+            for (int i = 0; i < RUN; ++i) {
+                const int j = k - i;
+                if (j < 0 || j >= TAPS) continue;
+#pragma unroll
+                for (int e = 0; e < 8; ++e) y[i][e] = fmaf(wv[j][e], xv[e], y[i][e]);
             }
         }
     } else {
-        for (int j = 0; j < T; ++j) {
+        for (int j = 0; j < T; ++j) {                  // tap j meets the row T - 1 - j before
             float wv[8];
-            dr_widen(*reinterpret_cast<const uint4*>(w + (size_t)j * C), wv);
+            dr_widen(weight(j), wv);
 #pragma unroll
-            for (int i = 0; i < kRun; ++i) {
+            for (int i = 0; i < RUN; ++i) {
                 float xv[8];
-                dr_widen(row(r0 + i - (back - j)), xv);
+                dr_widen(row(r0 + i - (T - 1 - j)), xv);
 #pragma unroll
                 for (int e = 0; e < 8; ++e) y[i][e] = fmaf(wv[e], xv[e], y[i][e]);
             }
         }
     }
 #pragma unroll
-    for (int i = 0; i < kRun; ++i) {
-        if (r0 + i >= n) {
+    for (int i = 0; i < RUN; ++i)
 #pragma unroll
-            for (int e = 0; e < 8; ++e) y[i][e] = 0.f;
-        }
-#pragma unroll
-        for (int e = 0; e < 8; e += 4)
-            *reinterpret_cast<float4*>(dst + (r0 + i) * pitch + e) = make_float4(silu_f(y[i][e]), silu_f(y[i][e + 1]), silu_f(y[i][e + 2]), silu_f(y[i][e + 3]));
-    }
+        for (int e = 0; e < 8; ++e) y[i][e] = r0 + i < n ? __fdividef(y[i][e], 1.f + __expf(-y[i][e])) : 0.f;
 }
 
-__host__ __device__ constexpr size_t delta_prep_floats(int dk, int dv) {
-    return (size_t)3 * kDC * (dk + 4) + (size_t)kDC * (dv + 8) + 3 * kDC * kDTP + 3 * 16 * 17 + 4 * dk + kDC;
+// Shared memory of delta_prepare in bytes: [fp32 q, k, decays | later their bf16 pairs], v pairs, A, M, T, small tables.
+constexpr int kDRel = 6;                // (query sub-block, key sub-block) below the diagonal
+constexpr int kDStageTaps = 7;          // longest convolution whose rows are staged in shared memory
+constexpr int kDLow = 128;              // low-rank columns staged at a time
+constexpr int kDLowPitch = kDLow + 8;
+__host__ __device__ constexpr size_t delta_prep_region(int dk, int dv) {
+    const size_t f = (size_t)3 * kDC * (dk + 4) * 4, h = (size_t)2 * 2 * (2 * kDC + kDRel * 16) * (dk + 8);
+    const size_t r = (size_t)2 * kDC * (dk + 4) * 4 + (size_t)(kDC + kDStageTaps - 1) * (2 * dk + dv) * 2;
+    return f > h ? (f > r ? f : r) : (h > r ? h : r);
+}
+__host__ __device__ constexpr size_t delta_prep_bytes(int dk, int dv) {
+    return delta_prep_region(dk, dv) + (size_t)2 * 2 * kDC * (dv + 8) + 4 * ((size_t)3 * kDC * kDTP + 3 * 16 * 17 + 4 * dk + 10 * dk + kDC);
 }
 
 // grid = (blocks, H)
 template <int DK, int DV, int TAPS>
 __global__ void __launch_bounds__(kDPrepThreads, 1) delta_prepare_kernel(const DeltaChunkArgs c) {
-    extern __shared__ __align__(16) float dr_smem[];
+    extern __shared__ __align__(16) unsigned char dp_smem[];
+    typedef __nv_bfloat16 bf;
     const DeltaArgs& a = c.a;
-    constexpr int P = DK + 4, PV = DV + 8, NW = kDPrepThreads / 32;
-    float* sQ = dr_smem;                                // [64][P]
-    float* sK = sQ + kDC * P;                           // [64][P]  k, later decayed to the end of its sub-block
-    float* sB = sK + kDC * P;                           // [64][P]  running log-decays, later k decayed from the start
-    float* sV = sB + kDC * P;                           // [64][PV]
-    float* sA = sV + kDC * PV;                          // [64][68]
+    constexpr int P = DK + 4, PB = DK + 8, PV = DV + 8, NW = kDPrepThreads / 32, PT = kDC + 8;
+    float* sQ = reinterpret_cast<float*>(dp_smem);      // [64][P]
+    float* sK = sQ + kDC * P;                           // [64][P]
+    float* sB = sK + kDC * P;                           // [64][P]  log2-decays, then their running sums in a sub-block
+    bf* hQ = reinterpret_cast<bf*>(dp_smem);            // later [2][64][PB]: q decayed from the start of its sub-block, high and low part
+    bf* hR = hQ + 2 * kDC * PB;                         // [2][64][PB]: k likewise, then from the start of the block
+    bf* hC = hR + 2 * kDC * PB;                         // [2][96][PB]: k decayed to the start of a later sub-block
+    bf* hT = hQ;                                        // [2][64][PT]: T diag(beta), when hQ has been used up
+    bf* sRaw = reinterpret_cast<bf*>(sB);               // first of all [64 + taps - 1][CH]: projected rows, from taps - 1 before the block on
+    bf* hV = reinterpret_cast<bf*>(dp_smem + delta_prep_region(DK, DV));  // [2][64][PV]
+    float* sA = reinterpret_cast<float*>(hV + 2 * kDC * PV);              // [64][68]
     float* sM = sA + kDC * kDTP;                        // [64][68]
     float* sT = sM + kDC * kDTP;                        // [64][68]
+    bf* sLow = reinterpret_cast<bf*>(sA);               // at first [64][136] low-rank inputs and [DK][136] rows of a2
     float* sX = sT + kDC * kDTP;                        // [3][16][17]
-    float* sE = sX + 3 * 16 * 17;                       // [4][DK]  log-decay sums of the sub-blocks, then up to their ends
-    float* sBeta = sE + 4 * DK;                         // [64]
+    bf* sConv = reinterpret_cast<bf*>(sX);              // at first [taps][CH]: the convolutions
+    float* sE = sX + 3 * 16 * 17;                       // [4][DK]  log2-decay sums of the sub-blocks
+    float* sF = sE + 4 * DK;                            // [4][DK] decay up to a sub-block's start, [6][DK] between two sub-blocks' ends
+    float* sBeta = sF + 10 * DK;                        // [64]
     DeltaSeq sd; int chunk;
     if (!delta_find_block(a, blockIdx.x, sd, chunk)) return;
     PS_CHECK(PS_SLOT_OK(sd.slot) && PS_ROWS_OK(sd.row_start, sd.n_rows) && sd.pos_start >= 0);
     const int h = blockIdx.y, t = threadIdx.x, warp = t >> 5, lane = t & 31, g = lane >> 2, tq = lane & 3;
     const int before = chunk * kDC, n = min(kDC, sd.n_rows - before), pos0 = sd.pos_start + before, back = a.taps - 1;
     const size_t bh = (size_t)blockIdx.x * a.H + h;
-    const __nv_bfloat16* proj = reinterpret_cast<const __nv_bfloat16*>(a.proj) + (size_t)(sd.row_start + before) * a.ld;
-    const __nv_bfloat16* conv = reinterpret_cast<const __nv_bfloat16*>(a.conv);
-    const int CH = 2 * DK + DV, C = 2 * a.G * DK + a.H * DV;
+    const bf* proj = reinterpret_cast<const bf*>(a.proj) + (size_t)(sd.row_start + before) * a.ld;
+    const bf* conv = reinterpret_cast<const bf*>(a.conv);
+    constexpr int CH = 2 * DK + DV;
+    const int C = 2 * a.G * DK + a.H * DV;
 
-    // ---- convolutions
-    for (int i = t; i < kDC / 4 * (CH / 8); i += kDPrepThreads) {
-        const int ch = i % (CH / 8) * 8, r0 = i / (CH / 8) * 4, col = dr_column(a, h, ch);
-        const __nv_bfloat16* hist = reinterpret_cast<const __nv_bfloat16*>(a.history) + ((size_t)sd.slot * back * a.H + h) * CH + ch;
-        const bool is_v = ch >= 2 * DK;
-        float* dst = is_v ? sV + ch - 2 * DK : ch < DK ? sQ + ch : sK + ch - DK;
-        delta_conv<TAPS>(proj + a.q_off + col, a.ld, hist, (size_t)a.H * CH, conv + col, C, a.taps, r0, n, before, pos0, dst, is_v ? PV : P);
+    static_assert((size_t)kDStageTaps * CH * 2 <= (size_t)4 * (3 * 16 * 17 + 4 * DK + 10 * DK) && (kDC + DK) * kDLowPitch * 2 <= 4 * 3 * kDC * kDTP,
+                  "staged operands");
+    const bf* a2 = reinterpret_cast<const bf*>(a.a2) + (size_t)h * DK * a.ra;
+    auto stage_low = [&](int k0) {                      // columns k0 .. of the low-rank inputs (rows behind the last are not used) and of a2
+        const int d = lane * 8;
+        if (d >= min(kDLow, a.ra - k0)) return;
+        for (int r = warp; r < kDC; r += NW) dr_cp16(sLow + r * kDLowPitch + d, proj + (size_t)min(r, n - 1) * a.ld + a.a_off + k0 + d);
+        for (int r = warp; r < DK; r += NW) dr_cp16(sLow + (kDC + r) * kDLowPitch + d, a2 + (size_t)r * a.ra + k0 + d);
+    };
+    // ---- convolutions, out of staged rows
+    const bf* hist = reinterpret_cast<const bf*>(a.history) + ((size_t)sd.slot * back * a.H + h) * CH;
+    // columns of the head's three runs of channels, less the channel
+    const int hk = h / (a.H / a.G), col_q = hk * DK, col_k = (a.G + hk - 1) * DK, col_v = 2 * a.G * DK + h * DV - 2 * DK;
+    auto column = [&](int ch) { return ch + (ch < DK ? col_q : ch < 2 * DK ? col_k : col_v); };
+    auto row_source = [&](int r, bool& mine) -> const bf* {              // row r: null: zero, `mine`: the projection's columns
+        mine = r + before >= 0;
+        if (r >= n || pos0 + r < 0) return nullptr;
+        return mine ? proj + (ptrdiff_t)r * a.ld + a.q_off : hist + (size_t)((pos0 + r) % back) * a.H * CH;
+    };
+    const bool staged = a.taps <= kDStageTaps;
+    if (staged) {
+        for (int r = warp; r < kDC + back; r += NW) {
+            bool mine;
+            const bf* src = row_source(r - back, mine);
+            for (int ch = lane * 8; ch < CH; ch += 256) {
+                if (src != nullptr) dr_cp16(sRaw + r * CH + ch, src + (mine ? column(ch) : ch));
+                else *reinterpret_cast<uint4*>(sRaw + r * CH + ch) = make_uint4(0, 0, 0, 0);
+            }
+        }
+        for (int j = warp; j < a.taps; j += NW)
+            for (int ch = lane * 8; ch < CH; ch += 256) dr_cp16(sConv + j * CH + ch, conv + (size_t)j * C + column(ch));
     }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    stage_low(0);
+    asm volatile("cp.async.commit_group;" ::: "memory");
     if (t < kDC) sBeta[t] = t < n ? dr_sigmoid(bf16_to_f32(proj[(size_t)t * a.ld + a.b_off + h])) : 0.f;
-    // ---- log-decays: rows of low-rank inputs times the head's rows of a2, on the tensor cores; a warp has 16 rows and DK / 4 channels
+    asm volatile("cp.async.wait_group 1;" ::: "memory");
+    __syncthreads();
+    auto convolve = [&](auto run, int r0, int ch, float (&y)[decltype(run)::value][8]) {
+        if (TAPS > 0 || staged)
+            delta_conv<TAPS>(a.taps, r0, n, [&](int r) { return *reinterpret_cast<const uint4*>(sRaw + (r + back) * CH + ch); },
+                             [&](int j) { return *reinterpret_cast<const uint4*>(sConv + j * CH + ch); }, y);
+        else
+            delta_conv<0>(a.taps, r0, n, [&](int r) {
+                bool mine;
+                const bf* p = row_source(r, mine);
+                return p != nullptr ? *reinterpret_cast<const uint4*>(p + (mine ? column(ch) : ch)) : make_uint4(0, 0, 0, 0);
+            }, [&](int j) { return *reinterpret_cast<const uint4*>(conv + (size_t)j * C + column(ch)); }, y);
+    };
+    for (int i = t; i < kDC / 4 * (2 * DK / 8); i += kDPrepThreads) {        // queries and keys
+        const int ch = i % (2 * DK / 8) * 8, r0 = i / (2 * DK / 8) * 4;
+        float y[4][8];
+        convolve(DeltaInt<4>{}, r0, ch, y);
+        float* dst = (ch < DK ? sQ + ch : sK + ch - DK) + r0 * P;
+#pragma unroll
+        for (int r = 0; r < 4; ++r) {
+            *reinterpret_cast<float4*>(dst + r * P) = make_float4(y[r][0], y[r][1], y[r][2], y[r][3]);
+            *reinterpret_cast<float4*>(dst + r * P + 4) = make_float4(y[r][4], y[r][5], y[r][6], y[r][7]);
+        }
+    }
+    for (int i = t; i < kDC / 2 * (DV / 8); i += kDPrepThreads) {            // values
+        const int ch = i % (DV / 8) * 8, r0 = i / (DV / 8) * 2;
+        float y[2][8];
+        convolve(DeltaInt<2>{}, r0, 2 * DK + ch, y);
+        bf* dst = hV + r0 * PV + ch;
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+            uint4 hi, lo;
+            dr_halves(y[r][0], y[r][1], hi.x, lo.x); dr_halves(y[r][2], y[r][3], hi.y, lo.y);
+            dr_halves(y[r][4], y[r][5], hi.z, lo.z); dr_halves(y[r][6], y[r][7], hi.w, lo.w);
+            *reinterpret_cast<uint4*>(dst + r * PV) = hi;
+            *reinterpret_cast<uint4*>(dst + (kDC + r) * PV) = lo;
+        }
+    }
+    asm volatile("cp.async.wait_all;" ::: "memory");
+    __syncthreads();                                    // (the staged rows have been read too)
+    // ---- log2-decays: rows of low-rank inputs times the head's rows of a2, on the tensor cores; a warp has 16 rows and DK / 4 channels
     {
         constexpr int kNT = DK / 32;
         const int m = warp & 3, n0 = (warp >> 2) * (DK / 4);
         float z[kNT][4];
 #pragma unroll
         for (int j = 0; j < kNT; ++j) z[j][0] = z[j][1] = z[j][2] = z[j][3] = 0.f;
-        const int rlo = min(m * 16 + g, n - 1), rhi = min(m * 16 + g + 8, n - 1);        // (rows behind the last are not used)
-        const __nv_bfloat16* lo = proj + (size_t)rlo * a.ld + a.a_off + 2 * tq;
-        const __nv_bfloat16* hi = proj + (size_t)rhi * a.ld + a.a_off + 2 * tq;
-        const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(a.a2) + ((size_t)h * DK + n0 + g) * a.ra + 2 * tq;
-        for (int k = 0; k < a.ra; k += 16) {
-            const uint32_t af[4] = {*reinterpret_cast<const uint32_t*>(lo + k), *reinterpret_cast<const uint32_t*>(hi + k),
-                                    *reinterpret_cast<const uint32_t*>(lo + k + 8), *reinterpret_cast<const uint32_t*>(hi + k + 8)};
+        const bf* ap = sLow + (16 * m + (lane & 15)) * kDLowPitch + (lane >> 4) * 8;
+        const bf* bp = sLow + (kDC + n0 + (lane & 7) + (lane >> 4) * 8) * kDLowPitch + ((lane >> 3) & 1) * 8;
+        for (int k0 = 0; k0 < a.ra; k0 += kDLow) {
+            if (k0 > 0) {
+                __syncthreads();
+                stage_low(k0);
+                asm volatile("cp.async.wait_all;" ::: "memory");
+                __syncthreads();
+            }
+            const int cols = min(kDLow, a.ra - k0);
+            for (int k = 0; k < cols; k += 16) {
+                uint32_t af[4];
+                dr_ldsm(af, ap + k);
 #pragma unroll
-            for (int j = 0; j < kNT; ++j) {
-                const __nv_bfloat16* wp = w + (size_t)j * 8 * a.ra + k;
-                dr_mma_bf16(z[j], af, *reinterpret_cast<const uint32_t*>(wp), *reinterpret_cast<const uint32_t*>(wp + 8));
+                for (int j = 0; j < kNT; j += 2) {
+                    uint32_t wf[4];
+                    dr_ldsm(wf, bp + j * 8 * kDLowPitch + k);
+                    dr_mma_bf16(z[j], af, wf[0], wf[1]);
+                    dr_mma_bf16(z[j + 1], af, wf[2], wf[3]);
+                }
             }
         }
-        const float rate = a.rate[h];
+        const float rate = -1.4426950408889634f * a.rate[h];
 #pragma unroll
         for (int j = 0; j < kNT; ++j) {
             const int d = n0 + j * 8 + 2 * tq;
             const float b0 = a.dt_bias[h * DK + d], b1 = a.dt_bias[h * DK + d + 1];
             const int r0 = m * 16 + g, r1 = r0 + 8;
-            *reinterpret_cast<float2*>(sB + r0 * P + d) = r0 < n ? make_float2(-rate * dr_softplus(z[j][0] + b0), -rate * dr_softplus(z[j][1] + b1)) : make_float2(0.f, 0.f);
-            *reinterpret_cast<float2*>(sB + r1 * P + d) = r1 < n ? make_float2(-rate * dr_softplus(z[j][2] + b0), -rate * dr_softplus(z[j][3] + b1)) : make_float2(0.f, 0.f);
+            *reinterpret_cast<float2*>(sB + r0 * P + d) = r0 < n ? make_float2(rate * dr_softplus_fast(z[j][0] + b0), rate * dr_softplus_fast(z[j][1] + b1)) : make_float2(0.f, 0.f);
+            *reinterpret_cast<float2*>(sB + r1 * P + d) = r1 < n ? make_float2(rate * dr_softplus_fast(z[j][2] + b0), rate * dr_softplus_fast(z[j][3] + b1)) : make_float2(0.f, 0.f);
         }
     }
     __syncthreads();
@@ -454,11 +551,43 @@ __global__ void __launch_bounds__(kDPrepThreads, 1) delta_prepare_kernel(const D
         }
     }
     __syncthreads();
-    // ---- diagonal sub-blocks, pair by pair, two keys at a time (sums local to the sub-block suffice: only differences enter)
+    // ---- diagonal sub-blocks (sums local to the sub-block suffice: only differences enter).  Rows 8 - 15 against keys 0 - 7: both
+    // sides factor through row 7; a warp has a quarter of the channels of one sub-block, rows 0 - 7 of its tile are queries, 8 - 15 keys
+    {
+        const int blk = warp >> 2, part = warp & 3;
+        const float* ref = sB + (blk * 16 + 7) * P;
+        const float* q = sQ + (blk * 16 + 8 + g) * P;
+        const float* k = sK + (blk * 16 + 8 + g) * P;
+        const float* bi = sB + (blk * 16 + 8 + g) * P;
+        const float* kj = sK + (blk * 16 + g) * P;
+        const float* bj = sB + (blk * 16 + g) * P;
+        float acc[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int k0 = part * (DK / 4); k0 < (part + 1) * (DK / 4); k0 += 16) {
+            uint32_t ah[4], al[4], xh[2], xl[2];
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int d = k0 + 8 * e + 2 * tq;
+                const float2 r = *reinterpret_cast<const float2*>(ref + d), b = *reinterpret_cast<const float2*>(bi + d), u = *reinterpret_cast<const float2*>(bj + d);
+                const float2 qv = *reinterpret_cast<const float2*>(q + d), kv = *reinterpret_cast<const float2*>(k + d), jv = *reinterpret_cast<const float2*>(kj + d);
+                const float f0 = dr_ex2(b.x - r.x), f1 = dr_ex2(b.y - r.y);
+                dr_halves(qv.x * f0, qv.y * f1, ah[2 * e], al[2 * e]);
+                dr_halves(kv.x * f0, kv.y * f1, ah[2 * e + 1], al[2 * e + 1]);
+                dr_halves(jv.x * dr_ex2(r.x - u.x), jv.y * dr_ex2(r.y - u.y), xh[e], xl[e]);
+            }
+            dr_mma_bf16(acc, al, xh[0], xh[1]);
+            dr_mma_bf16(acc, ah, xl[0], xl[1]);
+            dr_mma_bf16(acc, ah, xh[0], xh[1]);
+        }
+        float* dst = sT + (warp * 16 + g) * 8 + 2 * tq;      // partial sums of the four quarters
+        *reinterpret_cast<float2*>(dst) = make_float2(acc[0], acc[1]);
+        *reinterpret_cast<float2*>(dst + 64) = make_float2(acc[2], acc[3]);
+    }
+    // the eight 8 x 8 triangles on the diagonal pair by pair, two keys at a time
 #pragma unroll 1
-    for (int blk = 0; blk < 4; ++blk) {
+    for (int u = 0; u < 4; ++u) {
         constexpr int kU = DK / 32;
-        const int il = (blk & 1) ? 15 - warp : warp, i = blk * 16 + il, d = lane * kU;
+        const int il = (u & 1) ? 7 - (warp & 7) : warp & 7, first = ((warp >> 3) + 2 * u) * 8, i = first + il, d = lane * kU;
         auto load = [&](const float* p, float (&v)[kU]) {
             if constexpr (kU == 4) *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(p);
             else *reinterpret_cast<float2*>(v) = *reinterpret_cast<const float2*>(p);
@@ -469,79 +598,125 @@ __global__ void __launch_bounds__(kDPrepThreads, 1) delta_prepare_kernel(const D
             float v[4];
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
-                const int j = blk * 16 + min(jl + e, il);
+                const int j = first + min(jl + e, il);
                 float kj[kU], bj[kU], s0 = 0.f, s1 = 0.f;
                 load(sK + j * P + d, kj); load(sB + j * P + d, bj);
 #pragma unroll
-                for (int u = 0; u < kU; ++u) {
-                    const float f = kj[u] * __expf(bi[u] - bj[u]);
-                    s0 = fmaf(qi[u], f, s0); s1 = fmaf(ki[u], f, s1);
+                for (int x = 0; x < kU; ++x) {
+                    const float f = kj[x] * dr_ex2(bi[x] - bj[x]);
+                    s0 = fmaf(qi[x], f, s0); s1 = fmaf(ki[x], f, s1);
                 }
                 v[2 * e] = s0; v[2 * e + 1] = s1;
             }
             // four sums over the warp at once: lanes 0, 8, 16, 24 end with one each
             const bool up = lane & 16, odd = lane & 8;
-            float x = (up ? v[2] : v[0]) + __shfl_xor_sync(0xffffffffu, up ? v[0] : v[2], 16);
-            float y = (up ? v[3] : v[1]) + __shfl_xor_sync(0xffffffffu, up ? v[1] : v[3], 16);
+            const float x = (up ? v[2] : v[0]) + __shfl_xor_sync(0xffffffffu, up ? v[0] : v[2], 16);
+            const float y = (up ? v[3] : v[1]) + __shfl_xor_sync(0xffffffffu, up ? v[1] : v[3], 16);
             float s = (odd ? y : x) + __shfl_xor_sync(0xffffffffu, odd ? x : y, 8);
             s += __shfl_xor_sync(0xffffffffu, s, 4);
             s += __shfl_xor_sync(0xffffffffu, s, 2);
             s += __shfl_xor_sync(0xffffffffu, s, 1);
-            const int j = jl + (up ? 1 : 0);
-            if ((lane & 7) == 0 && j <= il) {
-                if (!odd) sM[i * kDTP + blk * 16 + j] = s;
-                else sA[i * kDTP + blk * 16 + j] = sBeta[i] * s;
+            const int jj = jl + (up ? 1 : 0), j = first + jj;
+            if ((lane & 7) == 0 && jj <= il) {
+                if (!odd) sM[i * kDTP + j] = s;
+                else sA[i * kDTP + j] = sBeta[i] * s;
             }
         }
     }
-    __syncthreads();
-    // ---- queries and keys decayed from the start of their sub-block, keys decayed to its end
-    for (int i = t; i < kDC * DK / 4; i += kDPrepThreads) {
-        const int r = i / (DK / 4), d = i % (DK / 4) * 4;
-        float4 b = *reinterpret_cast<float4*>(sB + r * P + d), q = *reinterpret_cast<float4*>(sQ + r * P + d), k = *reinterpret_cast<float4*>(sK + r * P + d);
-        const float4 e = *reinterpret_cast<const float4*>(sE + (r >> 4) * DK + d);
-        const float4 f = make_float4(__expf(b.x), __expf(b.y), __expf(b.z), __expf(b.w));
-        *reinterpret_cast<float4*>(sQ + r * P + d) = make_float4(q.x * f.x, q.y * f.y, q.z * f.z, q.w * f.w);
-        *reinterpret_cast<float4*>(sB + r * P + d) = make_float4(k.x * f.x, k.y * f.y, k.z * f.z, k.w * f.w);
-        *reinterpret_cast<float4*>(sK + r * P + d) = make_float4(k.x * __expf(e.x - b.x), k.y * __expf(e.y - b.y), k.z * __expf(e.z - b.z), k.w * __expf(e.w - b.w));
+    // ---- decay factors: up to the sub-blocks' starts, and between the ends of two sub-blocks
+    if (t < DK) {
+        const float e0 = sE[t], e1 = sE[DK + t], e2 = sE[2 * DK + t], e3 = sE[3 * DK + t];
+        sF[t] = 1.f; sF[DK + t] = dr_ex2(e0); sF[2 * DK + t] = dr_ex2(e0 + e1); sF[3 * DK + t] = dr_ex2(e0 + e1 + e2);
+        float* rel = sF + 4 * DK + t;                   // ends of sub-blocks (1, 0), (2, 0), (2, 1), (3, 0), (3, 1), (3, 2)
+        rel[0] = dr_ex2(e1); rel[DK] = dr_ex2(e1 + e2); rel[2 * DK] = dr_ex2(e2);
+        rel[3 * DK] = dr_ex2(e1 + e2 + e3); rel[4 * DK] = dr_ex2(e2 + e3); rel[5 * DK] = dr_ex2(e3);
+        c.dec[bh * DK + t] = exp2f(e0 + e1 + e2 + e3);
+    }
+    // ---- a thread's elements of q, k and the sums move to registers; their place takes the bf16 pairs
+    constexpr int kQ4 = kDC * DK / 4 / kDPrepThreads;
+    float4 rq[kQ4], rk[kQ4], rb[kQ4];
+#pragma unroll
+    for (int u = 0; u < kQ4; ++u) {
+        const int i = t + u * kDPrepThreads, at = i / (DK / 4) * P + i % (DK / 4) * 4;
+        rq[u] = *reinterpret_cast<const float4*>(sQ + at); rk[u] = *reinterpret_cast<const float4*>(sK + at); rb[u] = *reinterpret_cast<const float4*>(sB + at);
     }
     __syncthreads();
-    if (t < DK) {                                       // sub-block totals -> sums up to the sub-blocks' ends
-        const float e1 = sE[t] + sE[DK + t], e2 = e1 + sE[2 * DK + t], e3 = e2 + sE[3 * DK + t];
-        sE[DK + t] = e1; sE[2 * DK + t] = e2; sE[3 * DK + t] = e3;
-        c.dec[bh * DK + t] = expf(e3);
+    if (t < 256) {                                      // the quarters of the 8 x 8 squares
+        const int blk = t >> 6, il = (t >> 3) & 7, j = t & 7, i = blk * 16 + 8 + il, at = i * kDTP + blk * 16 + j;
+        float m = 0.f, k = 0.f;
+#pragma unroll
+        for (int p = 0; p < 4; ++p) {
+            m += sT[((blk * 4 + p) * 16 + il) * 8 + j];
+            k += sT[((blk * 4 + p) * 16 + 8 + il) * 8 + j];
+        }
+        sM[at] = m;
+        sA[at] = sBeta[i] * k;
+    }
+    bf* mats = c.mats + bh * delta_mats(DK);
+    constexpr int kMat = kDC * DK / 2;                  // pairs of columns; the high part, then the low part
+    uint32_t* gW = reinterpret_cast<uint32_t*>(mats);
+    uint32_t* gQ = gW + 2 * kMat;
+    uint32_t* gK = gQ + 2 * kMat;
+    uint32_t* gM = gK + 2 * kMat;
+    auto pair4 = [](float4 v, uint2& hi, uint2& lo) { dr_halves(v.x, v.y, hi.x, lo.x); dr_halves(v.z, v.w, hi.y, lo.y); };
+    auto mul4 = [](float4 x, float4 y) { return make_float4(x.x * y.x, x.y * y.y, x.z * y.z, x.w * y.w); };
+    auto put = [&](bf* dst, int part, float4 v) {
+        uint2 hi, lo;
+        pair4(v, hi, lo);
+        *reinterpret_cast<uint2*>(dst) = hi;
+        *reinterpret_cast<uint2*>(dst + part) = lo;
+    };
+#pragma unroll
+    for (int u = 0; u < kQ4; ++u) {
+        const int i = t + u * kDPrepThreads, r = i / (DK / 4), d = i % (DK / 4) * 4, blk = r >> 4;
+        const float4 b = rb[u], e = *reinterpret_cast<const float4*>(sE + blk * DK + d);
+        const float4 f = make_float4(dr_ex2(b.x), dr_ex2(b.y), dr_ex2(b.z), dr_ex2(b.w));
+        const float4 q = mul4(rq[u], f), k = mul4(rk[u], make_float4(dr_ex2(e.x - b.x), dr_ex2(e.y - b.y), dr_ex2(e.z - b.z), dr_ex2(e.w - b.w)));
+        put(hQ + r * PB + d, kDC * PB, q);
+        put(hR + r * PB + d, kDC * PB, mul4(rk[u], f));
+        uint2 hi, lo;
+        pair4(mul4(q, *reinterpret_cast<const float4*>(sF + blk * DK + d)), hi, lo);
+        reinterpret_cast<uint2*>(gQ)[i] = hi; reinterpret_cast<uint2*>(gQ + kMat)[i] = lo;
+        const float* rel = sF + 4 * DK + d;
+        if (blk < 3) {
+            // to the start of sub-block qi = blk + 1, ..., 3 (places qi (qi - 1) / 2 + blk), and to the block's end
+            bf* dst = hC + (r & 15) * PB + d;
+            constexpr int part = kDRel * 16 * PB;
+            put(dst + (blk + 1) * (blk) / 2 * 16 * PB + blk * 16 * PB, part, k);
+            for (int qi = blk + 2; qi <= 3; ++qi) {
+                const int x = (qi - 1) * (qi - 2) / 2 + blk;                       // (qi - 1, blk) among the pairs of ends
+                put(dst + (qi * (qi - 1) / 2 + blk) * 16 * PB, part, mul4(k, *reinterpret_cast<const float4*>(rel + x * DK)));
+            }
+            pair4(mul4(k, *reinterpret_cast<const float4*>(rel + (3 + blk) * DK)), hi, lo);
+        } else {
+            pair4(k, hi, lo);
+        }
+        reinterpret_cast<uint2*>(gK)[i] = hi; reinterpret_cast<uint2*>(gK + kMat)[i] = lo;
     }
     __syncthreads();
-    // ---- below the diagonal: (query sub-block, key sub-block) x two halves of eight keys, for queries and keys at once; the solve of
-    // the diagonal sub-blocks of T (thread: sub-block, column) by the last two warps
+    // ---- below the diagonal: a warp has one (query sub-block, key sub-block) for queries or for keys; the solve of T's diagonal
+    // sub-blocks (thread: sub-block, column) by the last two warps
     if (warp < 12) {
-        const int pair = warp >> 1, half = warp & 1;
-        const int qi = pair < 1 ? 1 : (pair < 3 ? 2 : 3), kj = pair < 1 ? 0 : (pair < 3 ? pair - 1 : pair - 3);
-        float am[4] = {0.f, 0.f, 0.f, 0.f}, aa[4] = {0.f, 0.f, 0.f, 0.f};
-        const float* q0 = sQ + (qi * 16 + g) * P + tq;
-        const float* p0 = sB + (qi * 16 + g) * P + tq;
-        const float* k0 = sK + (kj * 16 + half * 8 + g) * P + tq;
-#pragma unroll 2
-        for (int k = 0; k < DK; k += 8) {
-            float f0 = 1.f, f1 = 1.f;                   // decay from the end of the key's sub-block to the start of the query's
-            if (qi - 1 > kj) {
-                f0 = __expf(sE[(qi - 1) * DK + k + tq] - sE[kj * DK + k + tq]);
-                f1 = __expf(sE[(qi - 1) * DK + k + tq + 4] - sE[kj * DK + k + tq + 4]);
-            }
-            uint32_t bh2[2], bl2[2], ah[4], al[4];
-            dr_split(k0[k] * f0, bh2[0], bl2[0]);
-            dr_split(k0[k + 4] * f1, bh2[1], bl2[1]);
-            dr_split(q0[k], ah[0], al[0]); dr_split(q0[8 * P + k], ah[1], al[1]);
-            dr_split(q0[k + 4], ah[2], al[2]); dr_split(q0[8 * P + k + 4], ah[3], al[3]);
-            dr_mma_tf32(am, al, bh2[0], bh2[1]); dr_mma_tf32(am, ah, bl2[0], bl2[1]); dr_mma_tf32(am, ah, bh2[0], bh2[1]);
-            dr_split(p0[k], ah[0], al[0]); dr_split(p0[8 * P + k], ah[1], al[1]);
-            dr_split(p0[k + 4], ah[2], al[2]); dr_split(p0[8 * P + k + 4], ah[3], al[3]);
-            dr_mma_tf32(aa, al, bh2[0], bh2[1]); dr_mma_tf32(aa, ah, bl2[0], bl2[1]); dr_mma_tf32(aa, ah, bh2[0], bh2[1]);
+        const int x = warp >> 1, qi = x < 1 ? 1 : (x < 3 ? 2 : 3), kj = x - qi * (qi - 1) / 2;
+        const bool keys = warp & 1;
+        float acc[2][4] = {};
+        const bf* ap = (keys ? hR : hQ) + (qi * 16 + (lane & 15)) * PB + (lane >> 4) * 8;
+        const bf* bp = hC + (x * 16 + (lane & 7) + (lane >> 4) * 8) * PB + ((lane >> 3) & 1) * 8;
+#pragma unroll
+        for (int k = 0; k < DK; k += 16) {
+            uint32_t ah[4], al[4], bh[1][4], bl[1][4];
+            dr_ldsm(ah, ap + k); dr_ldsm(al, ap + kDC * PB + k);
+            dr_ldsm(bh[0], bp + k); dr_ldsm(bl[0], bp + kDRel * 16 * PB + k);
+            dr_mma3<2>(acc, ah, al, bh, bl);
         }
-        const int r0 = qi * 16 + g, at = r0 * kDTP + kj * 16 + half * 8 + 2 * tq;
-        const float b0 = sBeta[r0], b1 = sBeta[r0 + 8];
-        sM[at] = am[0]; sM[at + 1] = am[1]; sM[at + 8 * kDTP] = am[2]; sM[at + 8 * kDTP + 1] = am[3];
-        sA[at] = b0 * aa[0]; sA[at + 1] = b0 * aa[1]; sA[at + 8 * kDTP] = b1 * aa[2]; sA[at + 8 * kDTP + 1] = b1 * aa[3];
+        const int r0 = qi * 16 + g;
+        const float f0 = keys ? sBeta[r0] : 1.f, f1 = keys ? sBeta[r0 + 8] : 1.f;
+        float* dst = (keys ? sA : sM) + r0 * kDTP + kj * 16 + 2 * tq;
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+            *reinterpret_cast<float2*>(dst + 8 * j) = make_float2(f0 * acc[j][0], f0 * acc[j][1]);
+            *reinterpret_cast<float2*>(dst + 8 * kDTP + 8 * j) = make_float2(f1 * acc[j][2], f1 * acc[j][3]);
+        }
     } else if (warp >= 14) {
         const int b = (t - 14 * 32) >> 4, j = t & 15;
         const float* Ab = sA + (16 * b) * kDTP + 16 * b;
@@ -557,36 +732,19 @@ __global__ void __launch_bounds__(kDPrepThreads, 1) delta_prepare_kernel(const D
         for (int i = 0; i < 16; ++i) sT[(16 * b + i) * kDTP + 16 * b + j] = x[i];
     }
     __syncthreads();
-    // ---- everything that is ready goes out: Qd, Kd, M; k decayed from the block's start replaces k decayed from the sub-block's
-    __nv_bfloat16* mats = c.mats + bh * delta_mats(DK);
-    uint32_t* gW = reinterpret_cast<uint32_t*>(mats);                   // pairs of columns; high part, then low part
-    constexpr int kMat = kDC * DK / 2;
-    uint32_t* gQ = gW + 2 * kMat;
-    uint32_t* gK = gQ + 2 * kMat;
-    uint32_t* gM = gK + 2 * kMat;
-    for (int i = t; i < kMat / 2; i += kDPrepThreads) {
-        const int r = i / (DK / 4), d = i % (DK / 4) * 4, blk = r >> 4;
-        const float4 q = *reinterpret_cast<const float4*>(sQ + r * P + d), k = *reinterpret_cast<const float4*>(sK + r * P + d);
-        float f[4], e[4];
-#pragma unroll
-        for (int u = 0; u < 4; ++u) {
-            f[u] = blk > 0 ? __expf(sE[(blk - 1) * DK + d + u]) : 1.f;
-            e[u] = blk < 3 ? __expf(sE[3 * DK + d + u] - sE[blk * DK + d + u]) : 1.f;
-        }
+    // ---- M goes out; k decayed from the block's start replaces k decayed from the sub-block's
+    for (int i = t; i < kDC * kDC / 4; i += kDPrepThreads) {
+        const int r = i / (kDC / 4), s = i % (kDC / 4) * 4;
+        const float* p = sM + r * kDTP + s;
         uint2 hi, lo;
-        dr_halves(q.x * f[0], q.y * f[1], hi.x, lo.x); dr_halves(q.z * f[2], q.w * f[3], hi.y, lo.y);
-        reinterpret_cast<uint2*>(gQ)[i] = hi; reinterpret_cast<uint2*>(gQ + kMat)[i] = lo;
-        dr_halves(k.x * e[0], k.y * e[1], hi.x, lo.x); dr_halves(k.z * e[2], k.w * e[3], hi.y, lo.y);
-        reinterpret_cast<uint2*>(gK)[i] = hi; reinterpret_cast<uint2*>(gK + kMat)[i] = lo;
-        float4* p = reinterpret_cast<float4*>(sB + r * P + d);
-        const float4 b = *p;
-        *p = make_float4(b.x * f[0], b.y * f[1], b.z * f[2], b.w * f[3]);
+        pair4(make_float4(s <= r ? p[0] : 0.f, s + 1 <= r ? p[1] : 0.f, s + 2 <= r ? p[2] : 0.f, s + 3 <= r ? p[3] : 0.f), hi, lo);
+        reinterpret_cast<uint2*>(gM)[i] = hi; reinterpret_cast<uint2*>(gM + kDC * kDC / 2)[i] = lo;
     }
-    for (int i = t; i < kDC * kDC / 2; i += kDPrepThreads) {
-        const int r = i / (kDC / 2), s = i % (kDC / 2) * 2;
-        uint32_t hi, lo;
-        dr_halves(s <= r ? sM[r * kDTP + s] : 0.f, s + 1 <= r ? sM[r * kDTP + s + 1] : 0.f, hi, lo);
-        gM[i] = hi; gM[kDC * kDC / 2 + i] = lo;
+#pragma unroll
+    for (int u = 0; u < kQ4; ++u) {
+        const int i = t + u * kDPrepThreads, r = i / (DK / 4), d = i % (DK / 4) * 4, blk = r >> 4;
+        const float4 b = rb[u], p = *reinterpret_cast<const float4*>(sF + blk * DK + d);
+        put(hR + r * PB + d, kDC * PB, mul4(mul4(rk[u], make_float4(dr_ex2(b.x), dr_ex2(b.y), dr_ex2(b.z), dr_ex2(b.w))), p));
     }
     // ---- T, block rows 1 .. 3: T_ij = -T_ii (sum_{k = j .. i-1} A_ik T_kj) for all j < i at once
     for (int bi = 1; bi < 4; ++bi) {
@@ -594,9 +752,10 @@ __global__ void __launch_bounds__(kDPrepThreads, 1) delta_prepare_kernel(const D
             const int bj = e >> 8, r = (e >> 4) & 15, cc = e & 15;
             const float* Ar = sA + (16 * bi + r) * kDTP;
             float s0 = 0.f, s1 = 0.f;
-            for (int k = 16 * bj; k < 16 * bi; k += 2) {
-                s0 = fmaf(Ar[k], sT[k * kDTP + 16 * bj + cc], s0);
-                s1 = fmaf(Ar[k + 1], sT[(k + 1) * kDTP + 16 * bj + cc], s1);
+            for (int k = 16 * bj; k < 16 * bi; k += 4) {
+                const float4 x = *reinterpret_cast<const float4*>(Ar + k);
+                const float* tp = sT + k * kDTP + 16 * bj + cc;
+                s0 = fmaf(x.x, tp[0], s0); s1 = fmaf(x.y, tp[kDTP], s1); s0 = fmaf(x.z, tp[2 * kDTP], s0); s1 = fmaf(x.w, tp[3 * kDTP], s1);
             }
             sX[(bj * 16 + r) * 17 + cc] = s0 + s1;
         }
@@ -606,176 +765,174 @@ __global__ void __launch_bounds__(kDPrepThreads, 1) delta_prepare_kernel(const D
             const float* Tr = sT + (16 * bi + r) * kDTP + 16 * bi;
             float s = 0.f;
 #pragma unroll
-            for (int k = 0; k < 16; ++k) s = fmaf(Tr[k], sX[(bj * 16 + k) * 17 + cc], s);        // T_ii is zero above its diagonal
+            for (int k = 0; k < 16; k += 4) {                        // T_ii is zero above its diagonal
+                const float4 x = *reinterpret_cast<const float4*>(Tr + k);
+                const float* xp = sX + (bj * 16 + k) * 17 + cc;
+                s = fmaf(x.x, xp[0], s); s = fmaf(x.y, xp[17], s); s = fmaf(x.z, xp[34], s); s = fmaf(x.w, xp[51], s);
+            }
             sT[(16 * bi + r) * kDTP + 16 * bj + cc] = -s;
         }
         __syncthreads();
     }
+    for (int i = t; i < kDC * kDC / 4; i += kDPrepThreads) {
+        const int r = i / (kDC / 4), s = i % (kDC / 4) * 4;
+        if (s >> 4 > r >> 4) continue;                  // blocks above the diagonal are not read
+        put(hT + r * PT + s, kDC * PT, mul4(*reinterpret_cast<const float4*>(sT + r * kDTP + s), *reinterpret_cast<const float4*>(sBeta + s)));
+    }
+    __syncthreads();
     // ---- W = T diag(beta) K (warps 0-7) and U = T diag(beta) V (warps 8-15): a warp has 16 rows and half the columns; T is lower
     // triangular, so steps beyond the row tile are skipped
-    {
-        const int m = warp & 3, half = (warp >> 2) & 1;
-        const bool isW = warp < NW / 2;
-        constexpr int kNT = (DK > DV ? DK : DV) / 16;
-        const int nt = (isW ? DK : DV) / 16, col0 = half * (isW ? DK : DV) / 2;
-        const float* src = isW ? sB : sV;
-        const int pitch = isW ? P : PV;
-        float acc[kNT][4];
+    auto product = [&](auto cols, const bf* src, auto store) {
+        constexpr int D = decltype(cols)::value, pitch = D + 8, kN = D / 16;
+        const int m = warp & 3, col0 = ((warp >> 2) & 1) * (D / 2);
+        float acc[kN][4];
 #pragma unroll
-        for (int j = 0; j < kNT; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
-        const float* tr = sT + (16 * m + g) * kDTP + tq;
-        for (int k = 0; k < 16 * (m + 1); k += 8) {
-            uint32_t ah[4], al[4];
-            dr_split(tr[k], ah[0], al[0]); dr_split(tr[8 * kDTP + k], ah[1], al[1]);
-            dr_split(tr[k + 4], ah[2], al[2]); dr_split(tr[8 * kDTP + k + 4], ah[3], al[3]);
-            const float f0 = sBeta[k + tq], f1 = sBeta[k + tq + 4];
-            const float* b0p = src + (k + tq) * pitch + col0 + g;
-            const float* b1p = b0p + 4 * pitch;
+        for (int j = 0; j < kN; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+        const bf* ap = hT + (16 * m + (lane & 15)) * PT + (lane >> 4) * 8;
+        const bf* bp = src + (lane & 15) * pitch + col0 + (lane >> 4) * 8;
+        for (int k = 0; k < 16 * (m + 1); k += 16) {
+            uint32_t ah[4], al[4], bh[kN / 2][4], bl[kN / 2][4];
+            dr_ldsm(ah, ap + k); dr_ldsm(al, ap + kDC * PT + k);
 #pragma unroll
-            for (int j = 0; j < kNT; ++j) {
-                if (j < nt) {
-                    uint32_t bh0, bl0, bh1, bl1;
-                    dr_split(b0p[8 * j] * f0, bh0, bl0);
-                    dr_split(b1p[8 * j] * f1, bh1, bl1);
-                    dr_mma_tf32(acc[j], al, bh0, bh1);
-                    dr_mma_tf32(acc[j], ah, bl0, bl1);
-                    dr_mma_tf32(acc[j], ah, bh0, bh1);
-                }
-            }
+            for (int j = 0; j < kN / 2; ++j) { dr_ldsm_t(bh[j], bp + k * pitch + 16 * j); dr_ldsm_t(bl[j], bp + (kDC + k) * pitch + 16 * j); }
+            dr_mma3<kN>(acc, ah, al, bh, bl);
         }
-        const int r0 = 16 * m + g;
 #pragma unroll
-        for (int j = 0; j < kNT; ++j) {
-            if (j >= nt) continue;
-            const int d = col0 + 8 * j + 2 * tq;
-            if (isW) {
-                uint32_t hi, lo;
-                dr_halves(acc[j][0], acc[j][1], hi, lo);
-                gW[(r0 * DK + d) / 2] = hi; gW[kMat + (r0 * DK + d) / 2] = lo;
-                dr_halves(acc[j][2], acc[j][3], hi, lo);
-                gW[((r0 + 8) * DK + d) / 2] = hi; gW[kMat + ((r0 + 8) * DK + d) / 2] = lo;
-            } else {
-                float* u = c.u + bh * kDC * DV;
-                *reinterpret_cast<float2*>(u + (size_t)r0 * DV + d) = make_float2(acc[j][0], acc[j][1]);
-                *reinterpret_cast<float2*>(u + (size_t)(r0 + 8) * DV + d) = make_float2(acc[j][2], acc[j][3]);
-            }
+        for (int j = 0; j < kN; ++j) {
+            store(16 * m + g, col0 + 8 * j + 2 * tq, acc[j][0], acc[j][1]);
+            store(16 * m + g + 8, col0 + 8 * j + 2 * tq, acc[j][2], acc[j][3]);
         }
+    };
+    if (warp < NW / 2) {
+        product(DeltaInt<DK>{}, hR, [&](int r, int d, float x, float y) {
+            uint32_t hi, lo;
+            dr_halves(x, y, hi, lo);
+            gW[(r * DK + d) / 2] = hi; gW[kMat + (r * DK + d) / 2] = lo;
+        });
+    } else {
+        float* u = c.u + bh * kDC * DV;
+        product(DeltaInt<DV>{}, hV, [&](int r, int d, float x, float y) { *reinterpret_cast<float2*>(u + (size_t)r * DV + d) = make_float2(x, y); });
     }
 }
 
 // Shared-memory rows of the scan are padded so that eight rows of a fragment load fall into different banks.
 __host__ __device__ constexpr int delta_pk(int dk) { return dk + 8; }
-__host__ __device__ constexpr size_t delta_scan_bytes(int dk) {
-    return (size_t)2 * 2 * (3 * kDC * delta_pk(dk) + kDC * (kDC + 8) + (dk + kDC) * (kDSlice + 8)) + (size_t)4 * kDC * (kDSlice + 8);
+__host__ __device__ constexpr int delta_late(int slice) { return slice <= 32 ? 2 : 1; }          // buffers of Kd and M
+__host__ __device__ constexpr size_t delta_scan_bytes(int dk, int slice) {
+    return (size_t)2 * 2 * (2 * kDC * delta_pk(dk) + delta_late(slice) * (kDC * delta_pk(dk) + kDC * (kDC + 8)) + (dk + kDC) * (slice + 8)) +
+           (size_t)4 * kDC * (slice + 8);
 }
 
-// grid = (DV / 32, H, n_seqs): a CTA walks the sequence's blocks with 32 columns of the state in its accumulator registers.
-template <int DK>
+// grid = (DV / SLICE, H, n_seqs): a CTA walks the sequence's blocks with SLICE columns of the state in its accumulator registers.  A warp
+// has 16 rows and half the columns of every product.
+template <int DK, int SLICE>
 __global__ void __launch_bounds__(kDScanThreads, 1) delta_scan_kernel(const DeltaChunkArgs c) {
     extern __shared__ __align__(16) unsigned char ds_smem[];
     typedef __nv_bfloat16 bf;
     const DeltaArgs& a = c.a;
-    constexpr int PK = delta_pk(DK), PM = kDC + 8, PS = kDSlice + 8, NT = kDSlice / 8, PU = kDSlice + 8;
+    constexpr int PK = delta_pk(DK), PM = kDC + 8, PS = SLICE + 8, NT = SLICE / 16, PU = SLICE + 8, LATE = delta_late(SLICE);
     bf* sW = reinterpret_cast<bf*>(ds_smem);            // [2][64][PK], high and low part
     bf* sQ = sW + 2 * kDC * PK;
-    bf* sK = sQ + 2 * kDC * PK;
-    bf* sM = sK + 2 * kDC * PK;                         // [2][64][PM]
-    bf* sS = sM + 2 * kDC * PM;                         // [2][DK][PS]  operand copy of the state
+    bf* sK = sQ + 2 * kDC * PK;                         // LATE x [2][64][PK]
+    bf* sM = sK + LATE * 2 * kDC * PK;                  // LATE x [2][64][PM]
+    bf* sS = sM + LATE * 2 * kDC * PM;                  // [2][DK][PS]  operand copy of the state
     bf* sD = sS + 2 * DK * PS;                          // [2][64][PS]  Delta
     float* sU = reinterpret_cast<float*>(sD + 2 * kDC * PS);             // [64][PU]
     const DeltaSeq sd = a.seqs[blockIdx.z];
     if (sd.slot < 0 || sd.n_rows <= a.rows_limit) return;
     PS_CHECK(PS_SLOT_OK(sd.slot) && PS_ROWS_OK(sd.row_start, sd.n_rows));
-    int blk = 0;
+    int first = 0;
     for (int s = 0; s < (int)blockIdx.z; ++s) {
         const DeltaSeq d = a.seqs[s];
-        if (d.n_rows > a.rows_limit && d.slot >= 0) blk += (d.n_rows + kDC - 1) / kDC;
+        if (d.n_rows > a.rows_limit && d.slot >= 0) first += (d.n_rows + kDC - 1) / kDC;
     }
     const int h = blockIdx.y, t = threadIdx.x, warp = t >> 5, lane = t & 31, g = lane >> 2, tq = lane & 3;
-    const int c0 = blockIdx.x * kDSlice, dv = a.dv, m = warp & 3;
-    const bool own = warp < DK / 16;                    // this warp keeps state rows 16 warp .. 16 warp + 15
-    float* state = a.state + ((size_t)sd.slot * a.H + h) * DK * dv + c0;
+    const int c0 = blockIdx.x * SLICE, dv = a.dv, m = warp & 3, cols = (warp >> 3) * (SLICE / 2), srow = (warp & 7) * 16;
+    const bool own = srow < DK, queries = (warp >> 2) & 1;      // keeps state rows srow .. srow + 15; has Qd's side of the first product
+    const int n_blocks = (sd.n_rows + kDC - 1) / kDC;
+    float* state = a.state + ((size_t)sd.slot * a.H + h) * DK * dv + c0 + cols;
     float S[NT][4];
     auto publish = [&]() {                              // the state as a high and a low part
 #pragma unroll
         for (int j = 0; j < NT; ++j) {
             uint32_t hi, lo;
-            bf* p = sS + (16 * warp + g) * PS + 8 * j + 2 * tq;
+            bf* p = sS + (srow + g) * PS + cols + 8 * j + 2 * tq;
             dr_halves(S[j][0], S[j][1], hi, lo);
             *reinterpret_cast<uint32_t*>(p) = hi; *reinterpret_cast<uint32_t*>(p + DK * PS) = lo;
             dr_halves(S[j][2], S[j][3], hi, lo);
             *reinterpret_cast<uint32_t*>(p + 8 * PS) = hi; *reinterpret_cast<uint32_t*>(p + (DK + 8) * PS) = lo;
         }
     };
+    auto copy = [&](bf* dst, const bf* src, int width, int pitch) {      // both parts of a [64, width] matrix
+        const int per = width / 8;
+        for (int i = t; i < 2 * kDC * per; i += kDScanThreads) dr_cp16(dst + (i / per) * pitch + i % per * 8, src + (size_t)i * 8);
+    };
+    auto matrices = [&](int i) { return c.mats + ((size_t)(first + i) * a.H + h) * delta_mats(DK); };
+    auto fetch_early = [&](int i) {                     // what the first products of a block read
+        copy(sW, matrices(i), DK, PK);
+        copy(sQ, matrices(i) + 2 * kDC * DK, DK, PK);
+        const float* u = c.u + ((size_t)(first + i) * a.H + h) * kDC * dv + c0;
+        for (int x = t; x < kDC * SLICE / 4; x += kDScanThreads) {
+            const int r = x / (SLICE / 4), cc = x % (SLICE / 4) * 4;
+            dr_cp16(sU + r * PU + cc, u + (size_t)r * dv + cc);
+        }
+    };
+    auto fetch_late = [&](int i) {
+        copy(sK + (i % LATE) * 2 * kDC * PK, matrices(i) + 4 * kDC * DK, DK, PK);
+        copy(sM + (i % LATE) * 2 * kDC * PM, matrices(i) + 6 * kDC * DK, kDC, PM);
+    };
+    // lines of a later block towards L2; the CTAs of a head share the work
+    auto prefetch = [&](int i) {
+        const char* p = reinterpret_cast<const char*>(matrices(i));
+        for (int x = (blockIdx.x * kDScanThreads + t) * 128; x < (int)(delta_mats(DK) * 2); x += gridDim.x * kDScanThreads * 128)
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(p + x));
+    };
+    // acc += A B with split operands: 16 rows, this warp's columns; A at `ap` (parts `da` apart), B rows of the pitch PS at `bp` (parts
+    // `db` apart)
+    auto step = [&](float (&acc)[NT][4], const bf* ap, int da, bool trans, const bf* bp, int db) {
+        uint32_t ah[4], al[4], bh[NT / 2][4], bl[NT / 2][4];
+        if (trans) { dr_ldsm_t(ah, ap); dr_ldsm_t(al, ap + da); }
+        else { dr_ldsm(ah, ap); dr_ldsm(al, ap + da); }
+#pragma unroll
+        for (int j = 0; j < NT / 2; ++j) { dr_ldsm_t(bh[j], bp + 16 * j); dr_ldsm_t(bl[j], bp + db + 16 * j); }
+        dr_mma3<NT>(acc, ah, al, bh, bl);
+    };
+    fetch_early(0);
+    if (LATE > 1) fetch_late(0);
+    if (n_blocks > 1) prefetch(1);
     if (own) {
 #pragma unroll
         for (int j = 0; j < NT; ++j) {
-            const float2 x = *reinterpret_cast<const float2*>(state + (size_t)(16 * warp + g) * dv + 8 * j + 2 * tq);
-            const float2 y = *reinterpret_cast<const float2*>(state + (size_t)(16 * warp + g + 8) * dv + 8 * j + 2 * tq);
+            const float2 x = *reinterpret_cast<const float2*>(state + (size_t)(srow + g) * dv + 8 * j + 2 * tq);
+            const float2 y = *reinterpret_cast<const float2*>(state + (size_t)(srow + g + 8) * dv + 8 * j + 2 * tq);
             S[j][0] = x.x; S[j][1] = x.y; S[j][2] = y.x; S[j][3] = y.y;
         }
         publish();
     }
-    auto copy = [&](bf* dst, const bf* src, int cols, int pitch) {       // both parts of a [64, cols] matrix
-        const int per = cols / 8;
-        for (int i = t; i < 2 * kDC * per; i += kDScanThreads) dr_cp16(dst + (i / per) * pitch + i % per * 8, src + (size_t)i * 8);
-    };
-    auto commit = []() { asm volatile("cp.async.commit_group;" ::: "memory"); };
-    auto fetch_first = [&](int b) {                     // what the first products of a block read
-        const bf* src = c.mats + ((size_t)b * a.H + h) * delta_mats(DK);
-        copy(sW, src, DK, PK);
-        copy(sQ, src + 2 * kDC * DK, DK, PK);
-        const float* u = c.u + ((size_t)b * a.H + h) * kDC * dv + c0;
-        for (int i = t; i < kDC * kDSlice / 4; i += kDScanThreads) {
-            const int r = i / (kDSlice / 4), cc = i % (kDSlice / 4) * 4;
-            dr_cp16(sU + r * PU + cc, u + (size_t)r * dv + cc);
-        }
-        commit();
-    };
-    // one product with split operands: the low parts' product is left out
-    auto mma3 = [](float (&acc)[4], const uint32_t (&ah)[4], const uint32_t (&al)[4], uint32_t bh0, uint32_t bh1, uint32_t bl0, uint32_t bl1) {
-        dr_mma_bf16(acc, al, bh0, bh1);
-        dr_mma_bf16(acc, ah, bl0, bl1);
-        dr_mma_bf16(acc, ah, bh0, bh1);
-    };
-    fetch_first(blk);
-    for (int r0 = 0; r0 < sd.n_rows; r0 += kDC, ++blk) {
-        const int n = min(kDC, sd.n_rows - r0);
-        const float* dec = c.dec + ((size_t)blk * a.H + h) * DK;
+    for (int i = 0; i < n_blocks; ++i) {
+        const int n = min(kDC, sd.n_rows - i * kDC);
+        const float* dec = c.dec + ((size_t)(first + i) * a.H + h) * DK;
         float d0 = 0.f, d1 = 0.f;
-        if (own) { d0 = dec[16 * warp + g]; d1 = dec[16 * warp + g + 8]; }
+        if (own) { d0 = dec[srow + g]; d1 = dec[srow + g + 8]; }
+        if (i + 2 < n_blocks) prefetch(i + 2);
         asm volatile("cp.async.wait_all;" ::: "memory");
         __syncthreads();                                // W, Qd, U and the state's copy are there; Kd and M of the last block are free
-        {
-            const bf* src = c.mats + ((size_t)blk * a.H + h) * delta_mats(DK) + 4 * kDC * DK;
-            copy(sM, src + 2 * kDC * DK, kDC, PM);
-            copy(sK, src, DK, PK);
-            commit();
-        }
-        // ---- warps 0-3: W S0, warps 4-7: Qd S0; 16 rows x 32 columns each
+        if (LATE == 1) fetch_late(i);
+        else if (i + 1 < n_blocks) fetch_late(i + 1);
+        // ---- W S0 and Qd S0
         float acc[NT][4];
 #pragma unroll
         for (int j = 0; j < NT; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
         {
-            const bf* ap = (warp < 4 ? sW : sQ) + (16 * m + (lane & 15)) * PK + (lane >> 4) * 8;
-            const bf* bp = sS + (lane & 15) * PS + (lane >> 4) * 8;
+            const bf* ap = (queries ? sQ : sW) + (16 * m + (lane & 15)) * PK + (lane >> 4) * 8;
+            const bf* bp = sS + (lane & 15) * PS + cols + (lane >> 4) * 8;
 #pragma unroll
-            for (int k = 0; k < DK; k += 16) {
-                uint32_t ah[4], al[4];
-                dr_ldsm(ah, ap + k); dr_ldsm(al, ap + kDC * PK + k);
-#pragma unroll
-                for (int j = 0; j < NT; j += 2) {
-                    uint32_t bh[4], bl[4];
-                    dr_ldsm_t(bh, bp + k * PS + j * 8); dr_ldsm_t(bl, bp + (DK + k) * PS + j * 8);
-                    mma3(acc[j], ah, al, bh[0], bh[1], bl[0], bl[1]);
-                    mma3(acc[j + 1], ah, al, bh[2], bh[3], bl[2], bl[3]);
-                }
-            }
+            for (int k = 0; k < DK; k += 16) step(acc, ap + k, kDC * PK, false, bp + k * PS, DK * PS);
         }
-        if (warp < 4) {
+        if (!queries) {
 #pragma unroll
             for (int j = 0; j < NT; ++j) {
-                const int r = 16 * m + g, cc = 8 * j + 2 * tq;
+                const int r = 16 * m + g, cc = cols + 8 * j + 2 * tq;
                 const float2 u0 = *reinterpret_cast<const float2*>(sU + r * PU + cc), u1 = *reinterpret_cast<const float2*>(sU + (r + 8) * PU + cc);
                 uint32_t hi, lo;
                 bf* p = sD + r * PS + cc;
@@ -785,66 +942,48 @@ __global__ void __launch_bounds__(kDScanThreads, 1) delta_scan_kernel(const Delt
                 *reinterpret_cast<uint32_t*>(p + 8 * PS) = hi; *reinterpret_cast<uint32_t*>(p + (kDC + 8) * PS) = lo;
             }
         }
-        asm volatile("cp.async.wait_all;" ::: "memory");
+        if (LATE == 1) asm volatile("cp.async.wait_all;" ::: "memory");
         __syncthreads();                                // Delta, Kd and M are there; W, Qd, U and the state's copy are free
-        if (r0 + kDC < sd.n_rows) fetch_first(blk + 1);
+        if (i + 1 < n_blocks) fetch_early(i + 1);
+        const bf* bp = sD + (lane & 15) * PS + cols + (lane >> 4) * 8;
         // ---- o = Qd S0 + M Delta (steps above the diagonal are skipped)
-        if (warp >= 4) {
-            const bf* ap = sM + (16 * m + (lane & 15)) * PM + (lane >> 4) * 8;
-            const bf* bp = sD + (lane & 15) * PS + (lane >> 4) * 8;
-            for (int k = 0; k < 16 * (m + 1); k += 16) {
-                uint32_t ah[4], al[4];
-                dr_ldsm(ah, ap + k); dr_ldsm(al, ap + kDC * PM + k);
-#pragma unroll
-                for (int j = 0; j < NT; j += 2) {
-                    uint32_t bh[4], bl[4];
-                    dr_ldsm_t(bh, bp + k * PS + j * 8); dr_ldsm_t(bl, bp + (kDC + k) * PS + j * 8);
-                    mma3(acc[j], ah, al, bh[0], bh[1], bl[0], bl[1]);
-                    mma3(acc[j + 1], ah, al, bh[2], bh[3], bl[2], bl[3]);
-                }
-            }
+        if (queries) {
+            const bf* ap = sM + (i % LATE) * 2 * kDC * PM + (16 * m + (lane & 15)) * PM + (lane >> 4) * 8;
+            for (int k = 0; k < 16 * (m + 1); k += 16) step(acc, ap + k, kDC * PM, false, bp + k * PS, kDC * PS);
             const int lo = 16 * m + g, hi = lo + 8;
-            float* o = c.o + (size_t)(sd.row_start + r0) * a.H * dv + (size_t)h * dv + c0;
+            float* o = c.o + (size_t)(sd.row_start + i * kDC) * a.H * dv + (size_t)h * dv + c0 + cols + 2 * tq;
 #pragma unroll
             for (int j = 0; j < NT; ++j) {
-                const int cc = 8 * j + 2 * tq;
-                if (lo < n) *reinterpret_cast<float2*>(o + (size_t)lo * a.H * dv + cc) = make_float2(acc[j][0], acc[j][1]);
-                if (hi < n) *reinterpret_cast<float2*>(o + (size_t)hi * a.H * dv + cc) = make_float2(acc[j][2], acc[j][3]);
+                if (lo < n) *reinterpret_cast<float2*>(o + (size_t)lo * a.H * dv + 8 * j) = make_float2(acc[j][0], acc[j][1]);
+                if (hi < n) *reinterpret_cast<float2*>(o + (size_t)hi * a.H * dv + 8 * j) = make_float2(acc[j][2], acc[j][3]);
             }
         }
         // ---- S = diag(dec) S0 + Kd^T Delta
         if (own) {
 #pragma unroll
             for (int j = 0; j < NT; ++j) { S[j][0] *= d0; S[j][1] *= d0; S[j][2] *= d1; S[j][3] *= d1; }
-            const bf* ap = sK + ((lane & 7) + ((lane >> 4) & 1) * 8) * PK + 16 * warp + ((lane >> 3) & 1) * 8;
-            const bf* bp = sD + (lane & 15) * PS + (lane >> 4) * 8;
+            const bf* ap = sK + (i % LATE) * 2 * kDC * PK + ((lane & 7) + ((lane >> 4) & 1) * 8) * PK + srow + ((lane >> 3) & 1) * 8;
 #pragma unroll
-            for (int k = 0; k < kDC; k += 16) {
-                uint32_t ah[4], al[4];
-                dr_ldsm_t(ah, ap + k * PK); dr_ldsm_t(al, ap + (kDC + k) * PK);
-#pragma unroll
-                for (int j = 0; j < NT; j += 2) {
-                    uint32_t bh[4], bl[4];
-                    dr_ldsm_t(bh, bp + k * PS + j * 8); dr_ldsm_t(bl, bp + (kDC + k) * PS + j * 8);
-                    mma3(S[j], ah, al, bh[0], bh[1], bl[0], bl[1]);
-                    mma3(S[j + 1], ah, al, bh[2], bh[3], bl[2], bl[3]);
-                }
-            }
+            for (int k = 0; k < kDC; k += 16) step(S, ap + k * PK, kDC * PK, true, bp + k * PS, kDC * PS);
             publish();                                  // (nobody reads the copy between the two barriers)
         }
     }
     if (own) {
 #pragma unroll
         for (int j = 0; j < NT; ++j) {
-            *reinterpret_cast<float2*>(state + (size_t)(16 * warp + g) * dv + 8 * j + 2 * tq) = make_float2(S[j][0], S[j][1]);
-            *reinterpret_cast<float2*>(state + (size_t)(16 * warp + g + 8) * dv + 8 * j + 2 * tq) = make_float2(S[j][2], S[j][3]);
+            *reinterpret_cast<float2*>(state + (size_t)(srow + g) * dv + 8 * j + 2 * tq) = make_float2(S[j][0], S[j][1]);
+            *reinterpret_cast<float2*>(state + (size_t)(srow + g + 8) * dv + 8 * j + 2 * tq) = make_float2(S[j][2], S[j][3]);
         }
     }
 }
 
 // grid = (blocks, H): head norm and output gate (low-rank inputs times the head's rows of g2, on the tensor cores)
 template <int DV>
-__global__ void __launch_bounds__(kDFinThreads) delta_finish_kernel(const DeltaChunkArgs c) {
+__global__ void __launch_bounds__(kDFinThreads, 2) delta_finish_kernel(const DeltaChunkArgs c) {
+    extern __shared__ __align__(16) unsigned char df_smem[];
+    constexpr int PG = kDLowPitch;
+    __nv_bfloat16* s_in = reinterpret_cast<__nv_bfloat16*>(df_smem);      // [64][136]
+    __nv_bfloat16* s_w = s_in + kDC * PG;                                 // [DV][136]
     __shared__ float s_ss[2][kDC];
     const DeltaArgs& a = c.a;
     DeltaSeq sd; int chunk;
@@ -856,6 +995,16 @@ __global__ void __launch_bounds__(kDFinThreads) delta_finish_kernel(const DeltaC
     constexpr int kNT = DV / 16;
     const int m = warp & 3, half = warp >> 2, col0 = half * (DV / 2);
     const int rlo = m * 16 + g, rhi = rlo + 8;
+    const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(a.g2) + (size_t)h * DV * a.rg;
+    auto stage = [&](int k0) {                          // (rows behind the last are not used)
+        const int per = min(kDLow, a.rg - k0) / 8;
+        for (int i = t; i < (kDC + DV) * per; i += kDFinThreads) {
+            const int r = i / per, d = i % per * 8;
+            if (r < kDC) dr_cp16(s_in + r * PG + d, proj + (size_t)min(r, n - 1) * a.ld + a.g_off + k0 + d);
+            else dr_cp16(s_w + (r - kDC) * PG + d, w + (size_t)(r - kDC) * a.rg + k0 + d);
+        }
+    };
+    stage(0);
     const float* o = c.o + row0 * a.H * DV + (size_t)h * DV + col0 + 2 * tq;
     float2 v[kNT][2];
     float ss[2] = {0.f, 0.f};
@@ -869,16 +1018,26 @@ __global__ void __launch_bounds__(kDFinThreads) delta_finish_kernel(const DeltaC
     float z[kNT][4];
 #pragma unroll
     for (int j = 0; j < kNT; ++j) z[j][0] = z[j][1] = z[j][2] = z[j][3] = 0.f;
-    const __nv_bfloat16* lo = proj + (size_t)min(rlo, n - 1) * a.ld + a.g_off + 2 * tq;
-    const __nv_bfloat16* hi = proj + (size_t)min(rhi, n - 1) * a.ld + a.g_off + 2 * tq;
-    const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(a.g2) + ((size_t)h * DV + col0 + g) * a.rg + 2 * tq;
-    for (int k = 0; k < a.rg; k += 16) {
-        const uint32_t af[4] = {*reinterpret_cast<const uint32_t*>(lo + k), *reinterpret_cast<const uint32_t*>(hi + k),
-                                *reinterpret_cast<const uint32_t*>(lo + k + 8), *reinterpret_cast<const uint32_t*>(hi + k + 8)};
+    for (int k0 = 0; k0 < a.rg; k0 += kDLow) {
+        const int cols = min(kDLow, a.rg - k0);
+        if (k0 > 0) {
+            __syncthreads();
+            stage(k0);
+        }
+        asm volatile("cp.async.wait_all;" ::: "memory");
+        __syncthreads();
+        const __nv_bfloat16* ap = s_in + (16 * m + (lane & 15)) * PG + (lane >> 4) * 8;
+        const __nv_bfloat16* bp = s_w + (col0 + (lane & 7) + (lane >> 4) * 8) * PG + ((lane >> 3) & 1) * 8;
+        for (int k = 0; k < cols; k += 16) {
+            uint32_t af[4];
+            dr_ldsm(af, ap + k);
 #pragma unroll
-        for (int j = 0; j < kNT; ++j) {
-            const __nv_bfloat16* wp = w + (size_t)j * 8 * a.rg + k;
-            dr_mma_bf16(z[j], af, *reinterpret_cast<const uint32_t*>(wp), *reinterpret_cast<const uint32_t*>(wp + 8));
+            for (int j = 0; j < kNT; j += 2) {
+                uint32_t wf[4];
+                dr_ldsm(wf, bp + j * 8 * PG + k);
+                dr_mma_bf16(z[j], af, wf[0], wf[1]);
+                dr_mma_bf16(z[j + 1], af, wf[2], wf[3]);
+            }
         }
     }
 #pragma unroll
@@ -906,13 +1065,15 @@ __global__ void __launch_bounds__(kDFinThreads) delta_finish_kernel(const DeltaC
 
 template <int DK, int DV>
 static int launch_delta_chunked(const DeltaChunkArgs& c, int blocks, cudaStream_t stream) {
-    constexpr size_t s1 = delta_prep_floats(DK, DV) * 4, s2 = delta_scan_bytes(DK);
-    static_assert(s1 <= 226 * 1024 && s2 <= 226 * 1024, "shared memory of the chunked kernels");
+    constexpr size_t s1 = delta_prep_bytes(DK, DV), s2 = delta_scan_bytes(DK, 32), s3 = delta_scan_bytes(DK, 64), s4 = (size_t)(kDC + DV) * kDLowPitch * 2;
+    static_assert(s1 <= 226 * 1024 && s3 <= 226 * 1024, "shared memory of the chunked kernels");
     static bool set = false;
     if (!set) {
         cudaFuncSetAttribute(delta_prepare_kernel<DK, DV, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1);
         cudaFuncSetAttribute(delta_prepare_kernel<DK, DV, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1);
-        cudaFuncSetAttribute(delta_scan_kernel<DK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2);
+        cudaFuncSetAttribute(delta_finish_kernel<DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s4);
+        cudaFuncSetAttribute(delta_scan_kernel<DK, 32>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2);
+        cudaFuncSetAttribute(delta_scan_kernel<DK, 64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s3);
         set = true;
     }
     const DeltaArgs& a = c.a;
@@ -920,9 +1081,11 @@ static int launch_delta_chunked(const DeltaChunkArgs& c, int blocks, cudaStream_
     else delta_prepare_kernel<DK, DV, 0><<<dim3(blocks, a.H), kDPrepThreads, s1, stream>>>(c);
     int e = PS_LAUNCH_CHECK();
     if (e) return e;
-    delta_scan_kernel<DK><<<dim3(DV / kDSlice, a.H, a.n_seqs), kDScanThreads, s2, stream>>>(c);
+    // one CTA per SM: narrow slices while all of them are resident at once
+    if (a.H * a.n_seqs * (DV / 32) <= 148) delta_scan_kernel<DK, 32><<<dim3(DV / 32, a.H, a.n_seqs), kDScanThreads, s2, stream>>>(c);
+    else delta_scan_kernel<DK, 64><<<dim3(DV / 64, a.H, a.n_seqs), kDScanThreads, s3, stream>>>(c);
     if ((e = PS_LAUNCH_CHECK())) return e;
-    delta_finish_kernel<DV><<<dim3(blocks, a.H), kDFinThreads, 0, stream>>>(c);
+    delta_finish_kernel<DV><<<dim3(blocks, a.H), kDFinThreads, s4, stream>>>(c);
     return PS_LAUNCH_CHECK();
 }
 
