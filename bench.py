@@ -57,7 +57,7 @@ def _parse():
                          "the prefix cache the earlier ones filled)")
     ap.add_argument("--compare", default="", choices=["", "gebuzen", "luvutar", "fudulix", "rotutar"],
                     help="instead of the headline workload: prefill and decode of a model family beside the closest other one (Gebuzen: the "
-                         "hybrid decoder; Luvutar: Gebuzen; Fudulix: Luvutar) at equal layer shapes (random bf16 weights, 1 GPU), and the mixers' kernels "
+                         "hybrid decoder; Luvutar: Gebuzen; Fudulix: Luvutar; Rotutar: Gebuzen, Fudulix and the hybrid decoder) at equal layer shapes (random bf16 weights, 1 GPU), and the mixers' kernels "
                          "against their rooflines")
     ap.add_argument("--compare-layers", type=int, default=16)
     ap.add_argument("--watchdog", type=int, default=1500,

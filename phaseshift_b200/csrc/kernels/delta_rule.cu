@@ -18,14 +18,14 @@
 // S_end = diag(exp(B_end)) S0 + (k exp(B_end - B))^T Delta.  With T = (I + A)^-1 everything but the state is independent of it:
 //   delta_prepare  per (block, head): convolutions, unit vectors, decays; M, T, W = T diag(beta) (k exp(B)), U = T diag(beta) V and the
 //                  decayed queries and keys
-//   delta_scan     per (sequence, head, 32 or 64 value columns): Delta = U - W S0,  o = Qd S0 + M Delta,  S = diag(dec) S0 + Kd^T Delta
+//   delta_scan     per (sequence, head, 16 value columns): Delta = U - W S0,  o = Qd S0 + M Delta,  S = diag(dec) S0 + Kd^T Delta
 //   delta_finish   per (block, head): head norm, output gate, and the convolution's history
 // No exponential of a positive number is formed, whatever the decays: the triangles are cut into 16-row sub-blocks; off the diagonal
 // exp(B_t - B_s) factors through the end of the key's sub-block and of the sub-block before the query's, on the diagonal it is
 // evaluated pair by pair.  (The triangular form is that of "Parallelizing Linear Transformers with the Delta Rule over Sequence Length"
 // by Songlin Yang, Bailin Wang, Yu Zhang, Yikang Shen and Yoon Kim; sub-blocks as in gla.cu.)
 // The products run on bf16 mma.sync with both operands split into two terms (16 bits of mantissa); sums and the state are fp32.
-#include "ps_common.cuh"
+#include "ps_tcgen05.cuh"
 
 namespace ps {
 
@@ -235,18 +235,24 @@ __global__ void __launch_bounds__(256, 2) delta_rows_kernel(const DeltaArgs a) {
 
 // ------------------------------------------------------------------------------------------------ chunked form (bf16 engines)
 constexpr int kDC = 64;                 // rows of a block
-constexpr int kDPrepThreads = 512, kDScanThreads = 512, kDFinThreads = 256;
+constexpr int kDPrepThreads = 512, kDFinThreads = 256;
 constexpr int kDTP = kDC + 4;
 template <int N> struct DeltaInt { static constexpr int value = N; };
 
 struct DeltaChunkArgs {
     DeltaArgs a;
-    __nv_bfloat16* mats;                // per (block, head): W, Qd, Kd [64, dk] and M [64, 64], each as a high and a low part
-    float* u;                           // per (block, head): [64, dv]
-    float* dec;                         // per (block, head): [dk]
+    unsigned char* mats;                // per (block, head), as the scan's shared memory holds it: -W and Qd, then Kd, M and the decay
+    float* u;                           // per (block, head): U transposed, [dv, 64]
     float* o;                           // [rows, H * dv]
+    uint32_t* status; long long budget;
 };
-__host__ __device__ constexpr size_t delta_mats(int dk) { return (size_t)2 * (3 * kDC * dk + kDC * kDC); }
+// -W, Qd, Kd [64, dk] and M [64, 64] as a high and a low part of bf16, rows padded by eight elements so that eight rows of a fragment
+// load fall into different banks; dec [dk] fp32.
+constexpr int kDMPitch = kDC + 8;
+__host__ __device__ constexpr size_t delta_mat_bytes(int dk) { return (size_t)2 * 2 * kDC * (dk + 8); }
+__host__ __device__ constexpr size_t delta_early_bytes(int dk) { return 2 * delta_mat_bytes(dk); }
+__host__ __device__ constexpr size_t delta_late_bytes(int dk) { return delta_mat_bytes(dk) + (size_t)2 * 2 * kDC * kDMPitch + (size_t)4 * dk; }
+__host__ __device__ constexpr size_t delta_mats(int dk) { return delta_early_bytes(dk) + delta_late_bytes(dk); }
 
 // Which sequence and block of it a global block index is; false: none.
 __device__ __forceinline__ bool delta_find_block(const DeltaArgs& a, int blk, DeltaSeq& sd, int& chunk) {
@@ -630,7 +636,7 @@ __global__ void __launch_bounds__(kDPrepThreads, 1) delta_prepare_kernel(const D
         float* rel = sF + 4 * DK + t;                   // ends of sub-blocks (1, 0), (2, 0), (2, 1), (3, 0), (3, 1), (3, 2)
         rel[0] = dr_ex2(e1); rel[DK] = dr_ex2(e1 + e2); rel[2 * DK] = dr_ex2(e2);
         rel[3 * DK] = dr_ex2(e1 + e2 + e3); rel[4 * DK] = dr_ex2(e2 + e3); rel[5 * DK] = dr_ex2(e3);
-        c.dec[bh * DK + t] = exp2f(e0 + e1 + e2 + e3);
+        reinterpret_cast<float*>(c.mats + (bh + 1) * delta_mats(DK))[t - DK] = exp2f(e0 + e1 + e2 + e3);
     }
     // ---- a thread's elements of q, k and the sums move to registers; their place takes the bf16 pairs
     constexpr int kQ4 = kDC * DK / 4 / kDPrepThreads;
@@ -652,12 +658,11 @@ __global__ void __launch_bounds__(kDPrepThreads, 1) delta_prepare_kernel(const D
         sM[at] = m;
         sA[at] = sBeta[i] * k;
     }
-    bf* mats = c.mats + bh * delta_mats(DK);
-    constexpr int kMat = kDC * DK / 2;                  // pairs of columns; the high part, then the low part
-    uint32_t* gW = reinterpret_cast<uint32_t*>(mats);
-    uint32_t* gQ = gW + 2 * kMat;
-    uint32_t* gK = gQ + 2 * kMat;
-    uint32_t* gM = gK + 2 * kMat;
+    constexpr int kMat = kDC * PB;                      // elements of a matrix: the high part, then the low part
+    bf* gW = reinterpret_cast<bf*>(c.mats + bh * delta_mats(DK));
+    bf* gQ = gW + 2 * kMat;
+    bf* gK = gQ + 2 * kMat;
+    bf* gM = gK + 2 * kMat;
     auto pair4 = [](float4 v, uint2& hi, uint2& lo) { dr_halves(v.x, v.y, hi.x, lo.x); dr_halves(v.z, v.w, hi.y, lo.y); };
     auto mul4 = [](float4 x, float4 y) { return make_float4(x.x * y.x, x.y * y.y, x.z * y.z, x.w * y.w); };
     auto put = [&](bf* dst, int part, float4 v) {
@@ -674,9 +679,7 @@ __global__ void __launch_bounds__(kDPrepThreads, 1) delta_prepare_kernel(const D
         const float4 q = mul4(rq[u], f), k = mul4(rk[u], make_float4(dr_ex2(e.x - b.x), dr_ex2(e.y - b.y), dr_ex2(e.z - b.z), dr_ex2(e.w - b.w)));
         put(hQ + r * PB + d, kDC * PB, q);
         put(hR + r * PB + d, kDC * PB, mul4(rk[u], f));
-        uint2 hi, lo;
-        pair4(mul4(q, *reinterpret_cast<const float4*>(sF + blk * DK + d)), hi, lo);
-        reinterpret_cast<uint2*>(gQ)[i] = hi; reinterpret_cast<uint2*>(gQ + kMat)[i] = lo;
+        put(gQ + r * PB + d, kMat, mul4(q, *reinterpret_cast<const float4*>(sF + blk * DK + d)));
         const float* rel = sF + 4 * DK + d;
         if (blk < 3) {
             // to the start of sub-block qi = blk + 1, ..., 3 (places qi (qi - 1) / 2 + blk), and to the block's end
@@ -687,11 +690,9 @@ __global__ void __launch_bounds__(kDPrepThreads, 1) delta_prepare_kernel(const D
                 const int x = (qi - 1) * (qi - 2) / 2 + blk;                       // (qi - 1, blk) among the pairs of ends
                 put(dst + (qi * (qi - 1) / 2 + blk) * 16 * PB, part, mul4(k, *reinterpret_cast<const float4*>(rel + x * DK)));
             }
-            pair4(mul4(k, *reinterpret_cast<const float4*>(rel + (3 + blk) * DK)), hi, lo);
-        } else {
-            pair4(k, hi, lo);
-        }
-        reinterpret_cast<uint2*>(gK)[i] = hi; reinterpret_cast<uint2*>(gK + kMat)[i] = lo;
+            put(gK + r * PB + d, kMat, mul4(k, *reinterpret_cast<const float4*>(rel + (3 + blk) * DK)));
+        } else
+            put(gK + r * PB + d, kMat, k);
     }
     __syncthreads();
     // ---- below the diagonal: a warp has one (query sub-block, key sub-block) for queries or for keys; the solve of T's diagonal
@@ -736,9 +737,7 @@ __global__ void __launch_bounds__(kDPrepThreads, 1) delta_prepare_kernel(const D
     for (int i = t; i < kDC * kDC / 4; i += kDPrepThreads) {
         const int r = i / (kDC / 4), s = i % (kDC / 4) * 4;
         const float* p = sM + r * kDTP + s;
-        uint2 hi, lo;
-        pair4(make_float4(s <= r ? p[0] : 0.f, s + 1 <= r ? p[1] : 0.f, s + 2 <= r ? p[2] : 0.f, s + 3 <= r ? p[3] : 0.f), hi, lo);
-        reinterpret_cast<uint2*>(gM)[i] = hi; reinterpret_cast<uint2*>(gM + kDC * kDC / 2)[i] = lo;
+        put(gM + r * kDMPitch + s, kDC * kDMPitch, make_float4(s <= r ? p[0] : 0.f, s + 1 <= r ? p[1] : 0.f, s + 2 <= r ? p[2] : 0.f, s + 3 <= r ? p[3] : 0.f));
     }
 #pragma unroll
     for (int u = 0; u < kQ4; ++u) {
@@ -806,38 +805,27 @@ __global__ void __launch_bounds__(kDPrepThreads, 1) delta_prepare_kernel(const D
     if (warp < NW / 2) {
         product(DeltaInt<DK>{}, hR, [&](int r, int d, float x, float y) {
             uint32_t hi, lo;
-            dr_halves(x, y, hi, lo);
-            gW[(r * DK + d) / 2] = hi; gW[kMat + (r * DK + d) / 2] = lo;
+            dr_halves(-x, -y, hi, lo);
+            *reinterpret_cast<uint32_t*>(gW + r * PB + d) = hi; *reinterpret_cast<uint32_t*>(gW + kMat + r * PB + d) = lo;
         });
     } else {
         float* u = c.u + bh * kDC * DV;
-        product(DeltaInt<DV>{}, hV, [&](int r, int d, float x, float y) { *reinterpret_cast<float2*>(u + (size_t)r * DV + d) = make_float2(x, y); });
+        product(DeltaInt<DV>{}, hV, [&](int r, int d, float x, float y) { u[d * kDC + r] = x; u[(d + 1) * kDC + r] = y; });
     }
 }
 
-// Shared-memory rows of the scan are padded so that eight rows of a fragment load fall into different banks.
-__host__ __device__ constexpr int delta_pk(int dk) { return dk + 8; }
-__host__ __device__ constexpr int delta_late(int slice) { return slice <= 32 ? 2 : 1; }          // buffers of Kd and M
-__host__ __device__ constexpr size_t delta_scan_bytes(int dk, int slice) {
-    return (size_t)2 * 2 * (2 * kDC * delta_pk(dk) + delta_late(slice) * (kDC * delta_pk(dk) + kDC * (kDC + 8)) + (dk + kDC) * (slice + 8)) +
-           (size_t)4 * kDC * (slice + 8);
-}
-
-// grid = (DV / SLICE, H, n_seqs): a CTA walks the sequence's blocks with SLICE columns of the state in its accumulator registers.  A warp
-// has 16 rows and half the columns of every product.
-template <int DK, int SLICE>
-__global__ void __launch_bounds__(kDScanThreads, 1) delta_scan_kernel(const DeltaChunkArgs c) {
+// grid = (DV / (16 NW), H, n_seqs).  Everything runs transposed: a warp has 16 value columns of a sequence's head and keeps their state,
+// Delta and outputs in accumulator registers, which are also the left operands of the next products; only W, Qd, Kd and M come from
+// shared memory.  One more warp copies them there: -W and Qd of two blocks, Kd, M and the decays of one.
+template <int DK, int NW>
+__global__ void __launch_bounds__(32 * NW + 32, 1) delta_scan_kernel(const DeltaChunkArgs c) {
     extern __shared__ __align__(16) unsigned char ds_smem[];
     typedef __nv_bfloat16 bf;
     const DeltaArgs& a = c.a;
-    constexpr int PK = delta_pk(DK), PM = kDC + 8, PS = SLICE + 8, NT = SLICE / 16, PU = SLICE + 8, LATE = delta_late(SLICE);
-    bf* sW = reinterpret_cast<bf*>(ds_smem);            // [2][64][PK], high and low part
-    bf* sQ = sW + 2 * kDC * PK;
-    bf* sK = sQ + 2 * kDC * PK;                         // LATE x [2][64][PK]
-    bf* sM = sK + LATE * 2 * kDC * PK;                  // LATE x [2][64][PM]
-    bf* sS = sM + LATE * 2 * kDC * PM;                  // [2][DK][PS]  operand copy of the state
-    bf* sD = sS + 2 * DK * PS;                          // [2][64][PS]  Delta
-    float* sU = reinterpret_cast<float*>(sD + 2 * kDC * PS);             // [64][PU]
+    constexpr int PB = DK + 8, kMat = kDC * PB, ND = DK / 8;
+    constexpr uint32_t kEarly = (uint32_t)delta_early_bytes(DK), kLate = (uint32_t)delta_late_bytes(DK);
+    __shared__ __align__(8) uint64_t full_e[2], empty_e[2], full_l, empty_l;
+    __shared__ int s_abort;
     const DeltaSeq sd = a.seqs[blockIdx.z];
     if (sd.slot < 0 || sd.n_rows <= a.rows_limit) return;
     PS_CHECK(PS_SLOT_OK(sd.slot) && PS_ROWS_OK(sd.row_start, sd.n_rows));
@@ -846,135 +834,164 @@ __global__ void __launch_bounds__(kDScanThreads, 1) delta_scan_kernel(const Delt
         const DeltaSeq d = a.seqs[s];
         if (d.n_rows > a.rows_limit && d.slot >= 0) first += (d.n_rows + kDC - 1) / kDC;
     }
-    const int h = blockIdx.y, t = threadIdx.x, warp = t >> 5, lane = t & 31, g = lane >> 2, tq = lane & 3;
-    const int c0 = blockIdx.x * SLICE, dv = a.dv, m = warp & 3, cols = (warp >> 3) * (SLICE / 2), srow = (warp & 7) * 16;
-    const bool own = srow < DK, queries = (warp >> 2) & 1;      // keeps state rows srow .. srow + 15; has Qd's side of the first product
+    const int h = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, tq = lane & 3, dv = a.dv;
     const int n_blocks = (sd.n_rows + kDC - 1) / kDC;
-    float* state = a.state + ((size_t)sd.slot * a.H + h) * DK * dv + c0 + cols;
-    float S[NT][4];
-    auto publish = [&]() {                              // the state as a high and a low part
-#pragma unroll
-        for (int j = 0; j < NT; ++j) {
-            uint32_t hi, lo;
-            bf* p = sS + (srow + g) * PS + cols + 8 * j + 2 * tq;
-            dr_halves(S[j][0], S[j][1], hi, lo);
-            *reinterpret_cast<uint32_t*>(p) = hi; *reinterpret_cast<uint32_t*>(p + DK * PS) = lo;
-            dr_halves(S[j][2], S[j][3], hi, lo);
-            *reinterpret_cast<uint32_t*>(p + 8 * PS) = hi; *reinterpret_cast<uint32_t*>(p + (DK + 8) * PS) = lo;
-        }
-    };
-    auto copy = [&](bf* dst, const bf* src, int width, int pitch) {      // both parts of a [64, width] matrix
-        const int per = width / 8;
-        for (int i = t; i < 2 * kDC * per; i += kDScanThreads) dr_cp16(dst + (i / per) * pitch + i % per * 8, src + (size_t)i * 8);
-    };
-    auto matrices = [&](int i) { return c.mats + ((size_t)(first + i) * a.H + h) * delta_mats(DK); };
-    auto fetch_early = [&](int i) {                     // what the first products of a block read
-        copy(sW, matrices(i), DK, PK);
-        copy(sQ, matrices(i) + 2 * kDC * DK, DK, PK);
-        const float* u = c.u + ((size_t)(first + i) * a.H + h) * kDC * dv + c0;
-        for (int x = t; x < kDC * SLICE / 4; x += kDScanThreads) {
-            const int r = x / (SLICE / 4), cc = x % (SLICE / 4) * 4;
-            dr_cp16(sU + r * PU + cc, u + (size_t)r * dv + cc);
-        }
-    };
-    auto fetch_late = [&](int i) {
-        copy(sK + (i % LATE) * 2 * kDC * PK, matrices(i) + 4 * kDC * DK, DK, PK);
-        copy(sM + (i % LATE) * 2 * kDC * PM, matrices(i) + 6 * kDC * DK, kDC, PM);
-    };
-    // lines of a later block towards L2; the CTAs of a head share the work
-    auto prefetch = [&](int i) {
-        const char* p = reinterpret_cast<const char*>(matrices(i));
-        for (int x = (blockIdx.x * kDScanThreads + t) * 128; x < (int)(delta_mats(DK) * 2); x += gridDim.x * kDScanThreads * 128)
-            asm volatile("prefetch.global.L2 [%0];" ::"l"(p + x));
-    };
-    // acc += A B with split operands: 16 rows, this warp's columns; A at `ap` (parts `da` apart), B rows of the pitch PS at `bp` (parts
-    // `db` apart)
-    auto step = [&](float (&acc)[NT][4], const bf* ap, int da, bool trans, const bf* bp, int db) {
-        uint32_t ah[4], al[4], bh[NT / 2][4], bl[NT / 2][4];
-        if (trans) { dr_ldsm_t(ah, ap); dr_ldsm_t(al, ap + da); }
-        else { dr_ldsm(ah, ap); dr_ldsm(al, ap + da); }
-#pragma unroll
-        for (int j = 0; j < NT / 2; ++j) { dr_ldsm_t(bh[j], bp + 16 * j); dr_ldsm_t(bl[j], bp + db + 16 * j); }
-        dr_mma3<NT>(acc, ah, al, bh, bl);
-    };
-    fetch_early(0);
-    if (LATE > 1) fetch_late(0);
-    if (n_blocks > 1) prefetch(1);
-    if (own) {
-#pragma unroll
-        for (int j = 0; j < NT; ++j) {
-            const float2 x = *reinterpret_cast<const float2*>(state + (size_t)(srow + g) * dv + 8 * j + 2 * tq);
-            const float2 y = *reinterpret_cast<const float2*>(state + (size_t)(srow + g + 8) * dv + 8 * j + 2 * tq);
-            S[j][0] = x.x; S[j][1] = x.y; S[j][2] = y.x; S[j][3] = y.y;
-        }
-        publish();
+    if (threadIdx.x == 0) {
+        for (int i = 0; i < 2; ++i) { tc::mbar_init(&full_e[i], 1); tc::mbar_init(&empty_e[i], NW); }
+        tc::mbar_init(&full_l, 1);
+        tc::mbar_init(&empty_l, NW);
+        tc::fence_barrier_init();
+        s_abort = 0;
     }
-    for (int i = 0; i < n_blocks; ++i) {
-        const int n = min(kDC, sd.n_rows - i * kDC);
-        const float* dec = c.dec + ((size_t)(first + i) * a.H + h) * DK;
-        float d0 = 0.f, d1 = 0.f;
-        if (own) { d0 = dec[srow + g]; d1 = dec[srow + g + 8]; }
-        if (i + 2 < n_blocks) prefetch(i + 2);
-        asm volatile("cp.async.wait_all;" ::: "memory");
-        __syncthreads();                                // W, Qd, U and the state's copy are there; Kd and M of the last block are free
-        if (LATE == 1) fetch_late(i);
-        else if (i + 1 < n_blocks) fetch_late(i + 1);
-        // ---- W S0 and Qd S0
-        float acc[NT][4];
-#pragma unroll
-        for (int j = 0; j < NT; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
-        {
-            const bf* ap = (queries ? sQ : sW) + (16 * m + (lane & 15)) * PK + (lane >> 4) * 8;
-            const bf* bp = sS + (lane & 15) * PS + cols + (lane >> 4) * 8;
-#pragma unroll
-            for (int k = 0; k < DK; k += 16) step(acc, ap + k, kDC * PK, false, bp + k * PS, DK * PS);
-        }
-        if (!queries) {
-#pragma unroll
-            for (int j = 0; j < NT; ++j) {
-                const int r = 16 * m + g, cc = cols + 8 * j + 2 * tq;
-                const float2 u0 = *reinterpret_cast<const float2*>(sU + r * PU + cc), u1 = *reinterpret_cast<const float2*>(sU + (r + 8) * PU + cc);
-                uint32_t hi, lo;
-                bf* p = sD + r * PS + cc;
-                dr_halves(u0.x - acc[j][0], u0.y - acc[j][1], hi, lo);
-                *reinterpret_cast<uint32_t*>(p) = hi; *reinterpret_cast<uint32_t*>(p + kDC * PS) = lo;
-                dr_halves(u1.x - acc[j][2], u1.y - acc[j][3], hi, lo);
-                *reinterpret_cast<uint32_t*>(p + 8 * PS) = hi; *reinterpret_cast<uint32_t*>(p + (kDC + 8) * PS) = lo;
+    __syncthreads();
+    unsigned char* late = ds_smem + 2 * kEarly;
+    if (warp == NW) {
+        if (lane == 0) {
+            int early = 0, lates = 0;                   // copies handed out
+            bool ok = true;
+            auto fetch_early = [&](int i) {
+                ok = ok && (i < 2 || tc::mbar_wait_abortable(&empty_e[i & 1], (uint32_t)((i >> 1) - 1) & 1u, c.budget, &s_abort));
+                if (!ok) return;
+                tc::mbar_expect_tx(&full_e[i & 1], kEarly);
+                tc::bulk_load(ds_smem + (i & 1) * kEarly, c.mats + ((size_t)(first + i) * a.H + h) * delta_mats(DK), kEarly, &full_e[i & 1]);
+                ++early;
+            };
+            fetch_early(0);
+            for (int i = 0; i < n_blocks && ok; ++i) {
+                if (i + 1 < n_blocks) fetch_early(i + 1);
+                ok = ok && (i < 1 || tc::mbar_wait_abortable(&empty_l, (uint32_t)(i - 1) & 1u, c.budget, &s_abort));
+                if (!ok) break;
+                tc::mbar_expect_tx(&full_l, kLate);
+                tc::bulk_load(late, c.mats + ((size_t)(first + i) * a.H + h) * delta_mats(DK) + kEarly, kLate, &full_l);
+                ++lates;
+            }
+            if (!ok) {
+                // copies still in flight get a bounded chance to land before the shared memory goes back to the next CTA
+                const long long b = c.budget < 4000000ll ? c.budget : 4000000ll;
+                for (int i = max(0, early - 2); i < early; ++i) tc::mbar_wait(&full_e[i & 1], (uint32_t)(i >> 1) & 1u, b);
+                if (lates > 0) tc::mbar_wait(&full_l, (uint32_t)(lates - 1) & 1u, b);
             }
         }
-        if (LATE == 1) asm volatile("cp.async.wait_all;" ::: "memory");
-        __syncthreads();                                // Delta, Kd and M are there; W, Qd, U and the state's copy are free
-        if (i + 1 < n_blocks) fetch_early(i + 1);
-        const bf* bp = sD + (lane & 15) * PS + cols + (lane >> 4) * 8;
-        // ---- o = Qd S0 + M Delta (steps above the diagonal are skipped)
-        if (queries) {
-            const bf* ap = sM + (i % LATE) * 2 * kDC * PM + (16 * m + (lane & 15)) * PM + (lane >> 4) * 8;
-            for (int k = 0; k < 16 * (m + 1); k += 16) step(acc, ap + k, kDC * PM, false, bp + k * PS, kDC * PS);
-            const int lo = 16 * m + g, hi = lo + 8;
-            float* o = c.o + (size_t)(sd.row_start + i * kDC) * a.H * dv + (size_t)h * dv + c0 + cols + 2 * tq;
+    } else {
+        const int v0 = (blockIdx.x * NW + warp) * 16 + g;            // this thread's value columns: v0 and v0 + 8
+        float* state = a.state + ((size_t)sd.slot * a.H + h) * DK * dv + v0;
+        float S[ND][4], D[8][4], R[8][4];
 #pragma unroll
-            for (int j = 0; j < NT; ++j) {
-                if (lo < n) *reinterpret_cast<float2*>(o + (size_t)lo * a.H * dv + 8 * j) = make_float2(acc[j][0], acc[j][1]);
-                if (hi < n) *reinterpret_cast<float2*>(o + (size_t)hi * a.H * dv + 8 * j) = make_float2(acc[j][2], acc[j][3]);
+        for (int j = 0; j < ND; ++j) {
+            const float* p = state + (size_t)(8 * j + 2 * tq) * dv;
+            S[j][0] = p[0]; S[j][1] = p[dv]; S[j][2] = p[8]; S[j][3] = p[dv + 8];
+        }
+        auto load_u = [&](int i) {
+            const float* u = c.u + (((size_t)(first + i) * a.H + h) * dv + v0) * kDC + 2 * tq;
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                const float2 x = *reinterpret_cast<const float2*>(u + 8 * j), y = *reinterpret_cast<const float2*>(u + 8 * kDC + 8 * j);
+                D[j][0] = x.x; D[j][1] = x.y; D[j][2] = y.x; D[j][3] = y.y;
+            }
+        };
+        // accumulator tiles 2 k and 2 k + 1 as the left operand of a product's step k
+        auto operand = [](const float (&x)[4], const float (&y)[4], uint32_t (&hi)[4], uint32_t (&lo)[4]) {
+            dr_halves(x[0], x[1], hi[0], lo[0]); dr_halves(x[2], x[3], hi[1], lo[1]);
+            dr_halves(y[0], y[1], hi[2], lo[2]); dr_halves(y[2], y[3], hi[3], lo[3]);
+        };
+        load_u(0);
+        const int row_n = (lane & 7) + (lane >> 4) * 8, col_n = ((lane >> 3) & 1) * 8;     // right operand from rows of columns
+        bool ok = true;
+        for (int i = 0; i < n_blocks; ++i) {
+            const int n = min(kDC, sd.n_rows - i * kDC);
+            ok = __all_sync(0xffffffffu, tc::mbar_wait_abortable(&full_e[i & 1], (uint32_t)(i >> 1) & 1u, c.budget, &s_abort));
+            if (!ok) break;
+            // ---- Delta^T = U^T - S^T W^T, and the state's part of the outputs
+#pragma unroll
+            for (int j = 0; j < 8; ++j) R[j][0] = R[j][1] = R[j][2] = R[j][3] = 0.f;
+            {
+                const bf* wp = reinterpret_cast<const bf*>(ds_smem + (i & 1) * kEarly) + row_n * PB + col_n;
+                const bf* qp = wp + 2 * kMat;
+#pragma unroll
+                for (int k = 0; k < DK / 16; ++k) {
+                    uint32_t ah[4], al[4], bh[4][4], bl[4][4];
+                    operand(S[2 * k], S[2 * k + 1], ah, al);
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) { dr_ldsm(bh[j], wp + 16 * j * PB + 16 * k); dr_ldsm(bl[j], wp + kMat + 16 * j * PB + 16 * k); }
+                    dr_mma3<8>(D, ah, al, bh, bl);
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) { dr_ldsm(bh[j], qp + 16 * j * PB + 16 * k); dr_ldsm(bl[j], qp + kMat + 16 * j * PB + 16 * k); }
+                    dr_mma3<8>(R, ah, al, bh, bl);
+                }
+            }
+            __syncwarp();
+            if (lane == 0) tc::mbar_arrive(&empty_e[i & 1]);
+            uint32_t dh[4][4], dl[4][4];
+#pragma unroll
+            for (int k = 0; k < 4; ++k) operand(D[2 * k], D[2 * k + 1], dh[k], dl[k]);
+            if (i + 1 < n_blocks) load_u(i + 1);
+            ok = __all_sync(0xffffffffu, tc::mbar_wait_abortable(&full_l, (uint32_t)i & 1u, c.budget, &s_abort));
+            if (!ok) break;
+            // ---- o^T += Delta^T M^T (tokens after the row are skipped)
+            {
+                const bf* mp = reinterpret_cast<const bf*>(late) + 2 * kMat + row_n * kDMPitch + col_n;
+#pragma unroll
+                for (int k = 0; k < 4; ++k) {
+                    uint32_t bh[4][4], bl[4][4];
+#pragma unroll
+                    for (int j = k; j < 4; ++j) {
+                        dr_ldsm(bh[j], mp + 16 * j * kDMPitch + 16 * k);
+                        dr_ldsm(bl[j], mp + kDC * kDMPitch + 16 * j * kDMPitch + 16 * k);
+                    }
+#pragma unroll
+                    for (int j = 2 * k; j < 8; ++j) dr_mma_bf16(R[j], dl[k], bh[j / 2][j % 2 * 2], bh[j / 2][j % 2 * 2 + 1]);
+#pragma unroll
+                    for (int j = 2 * k; j < 8; ++j) dr_mma_bf16(R[j], dh[k], bl[j / 2][j % 2 * 2], bl[j / 2][j % 2 * 2 + 1]);
+#pragma unroll
+                    for (int j = 2 * k; j < 8; ++j) dr_mma_bf16(R[j], dh[k], bh[j / 2][j % 2 * 2], bh[j / 2][j % 2 * 2 + 1]);
+                }
+            }
+            {
+                float* o = c.o + (size_t)(sd.row_start + i * kDC) * a.H * dv + (size_t)h * dv + v0;
+                const size_t ld = (size_t)a.H * dv;
+#pragma unroll
+                for (int j = 0; j < 8; ++j) {
+                    const int r = 8 * j + 2 * tq;
+                    if (r < n) { o[r * ld] = R[j][0]; o[r * ld + 8] = R[j][2]; }
+                    if (r + 1 < n) { o[(r + 1) * ld] = R[j][1]; o[(r + 1) * ld + 8] = R[j][3]; }
+                }
+            }
+            // ---- S^T = S^T diag(dec) + Delta^T Kd
+            {
+                const float* dec = reinterpret_cast<const float*>(late + kLate) - DK;
+#pragma unroll
+                for (int j = 0; j < ND; ++j) {
+                    const float2 d = *reinterpret_cast<const float2*>(dec + 8 * j + 2 * tq);
+                    S[j][0] *= d.x; S[j][1] *= d.y; S[j][2] *= d.x; S[j][3] *= d.y;
+                }
+                const bf* kp = reinterpret_cast<const bf*>(late) + (lane & 15) * PB + (lane >> 4) * 8;
+#pragma unroll
+                for (int x = 0; x < ND; x += 8) {
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) {
+                        uint32_t bh[4][4], bl[4][4];
+#pragma unroll
+                        for (int j = 0; j < 4; ++j) {
+                            dr_ldsm_t(bh[j], kp + 16 * k * PB + 8 * x + 16 * j);
+                            dr_ldsm_t(bl[j], kp + kMat + 16 * k * PB + 8 * x + 16 * j);
+                        }
+                        dr_mma3<8>(reinterpret_cast<float (&)[8][4]>(S[x]), dh[k], dl[k], bh, bl);
+                    }
+                }
+            }
+            __syncwarp();
+            if (lane == 0) tc::mbar_arrive(&empty_l);
+        }
+        if (ok) {
+#pragma unroll
+            for (int j = 0; j < ND; ++j) {
+                float* p = state + (size_t)(8 * j + 2 * tq) * dv;
+                p[0] = S[j][0]; p[dv] = S[j][1]; p[8] = S[j][2]; p[dv + 8] = S[j][3];
             }
         }
-        // ---- S = diag(dec) S0 + Kd^T Delta
-        if (own) {
-#pragma unroll
-            for (int j = 0; j < NT; ++j) { S[j][0] *= d0; S[j][1] *= d0; S[j][2] *= d1; S[j][3] *= d1; }
-            const bf* ap = sK + (i % LATE) * 2 * kDC * PK + ((lane & 7) + ((lane >> 4) & 1) * 8) * PK + srow + ((lane >> 3) & 1) * 8;
-#pragma unroll
-            for (int k = 0; k < kDC; k += 16) step(S, ap + k * PK, kDC * PK, true, bp + k * PS, kDC * PS);
-            publish();                                  // (nobody reads the copy between the two barriers)
-        }
     }
-    if (own) {
-#pragma unroll
-        for (int j = 0; j < NT; ++j) {
-            *reinterpret_cast<float2*>(state + (size_t)(srow + g) * dv + 8 * j + 2 * tq) = make_float2(S[j][0], S[j][1]);
-            *reinterpret_cast<float2*>(state + (size_t)(srow + g + 8) * dv + 8 * j + 2 * tq) = make_float2(S[j][2], S[j][3]);
-        }
-    }
+    __syncthreads();
+    if (threadIdx.x == 0 && s_abort != 0) set_status(c.status, PS_DEV_WAIT_TIMEOUT);
 }
 
 // grid = (blocks, H): head norm and output gate (low-rank inputs times the head's rows of g2, on the tensor cores)
@@ -1065,15 +1082,15 @@ __global__ void __launch_bounds__(kDFinThreads, 2) delta_finish_kernel(const Del
 
 template <int DK, int DV>
 static int launch_delta_chunked(const DeltaChunkArgs& c, int blocks, cudaStream_t stream) {
-    constexpr size_t s1 = delta_prep_bytes(DK, DV), s2 = delta_scan_bytes(DK, 32), s3 = delta_scan_bytes(DK, 64), s4 = (size_t)(kDC + DV) * kDLowPitch * 2;
-    static_assert(s1 <= 226 * 1024 && s3 <= 226 * 1024, "shared memory of the chunked kernels");
+    constexpr size_t s1 = delta_prep_bytes(DK, DV), s2 = 2 * delta_early_bytes(DK) + delta_late_bytes(DK), s4 = (size_t)(kDC + DV) * kDLowPitch * 2;
+    static_assert(s1 <= 226 * 1024 && s2 <= 226 * 1024, "shared memory of the chunked kernels");
     static bool set = false;
     if (!set) {
         cudaFuncSetAttribute(delta_prepare_kernel<DK, DV, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1);
         cudaFuncSetAttribute(delta_prepare_kernel<DK, DV, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s1);
         cudaFuncSetAttribute(delta_finish_kernel<DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s4);
-        cudaFuncSetAttribute(delta_scan_kernel<DK, 32>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2);
-        cudaFuncSetAttribute(delta_scan_kernel<DK, 64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s3);
+        cudaFuncSetAttribute(delta_scan_kernel<DK, 2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2);
+        cudaFuncSetAttribute(delta_scan_kernel<DK, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)s2);
         set = true;
     }
     const DeltaArgs& a = c.a;
@@ -1081,9 +1098,9 @@ static int launch_delta_chunked(const DeltaChunkArgs& c, int blocks, cudaStream_
     else delta_prepare_kernel<DK, DV, 0><<<dim3(blocks, a.H), kDPrepThreads, s1, stream>>>(c);
     int e = PS_LAUNCH_CHECK();
     if (e) return e;
-    // one CTA per SM: narrow slices while all of them are resident at once
-    if (a.H * a.n_seqs * (DV / 32) <= 148) delta_scan_kernel<DK, 32><<<dim3(DV / 32, a.H, a.n_seqs), kDScanThreads, s2, stream>>>(c);
-    else delta_scan_kernel<DK, 64><<<dim3(DV / 64, a.H, a.n_seqs), kDScanThreads, s3, stream>>>(c);
+    // one CTA per SM: two warps each while all CTAs are resident at once
+    if (a.H * a.n_seqs * (DV / 32) <= 148) delta_scan_kernel<DK, 2><<<dim3(DV / 32, a.H, a.n_seqs), 96, s2, stream>>>(c);
+    else delta_scan_kernel<DK, 4><<<dim3(DV / 64, a.H, a.n_seqs), 160, s2, stream>>>(c);
     if ((e = PS_LAUNCH_CHECK())) return e;
     delta_finish_kernel<DV><<<dim3(blocks, a.H), kDFinThreads, s4, stream>>>(c);
     return PS_LAUNCH_CHECK();
@@ -1146,22 +1163,22 @@ PS_API int ps_delta_chunked_ok(int dk, int dv, int ra, int rg) {
 }
 PS_API long long ps_delta_mats(int dk) { return (long long)ps::delta_mats(dk); }
 
-// The sequences with more than `rows_limit` rows, `blocks` = the sum of their ceil(rows / 64); bf16.  `mats`: ps_delta_mats(dk) bf16 per
-// block and head, `u`: 64 * dv, `dec`: dk floats per block and head, `o`: [rows, H * dv] floats; all 16-byte aligned.
+// The sequences with more than `rows_limit` rows, `blocks` = the sum of their ceil(rows / 64); bf16.  `mats`: ps_delta_mats(dk) bytes per
+// block and head, `u`: 64 * dv floats per block and head, `o`: [rows, H * dv] floats; all 16-byte aligned.
 PS_API int ps_delta_chunked(const void* proj, int ld, int H, int G, int dk, int dv, int dk_true, int dv_true, int q_off, int b_off, int a_off,
                             int g_off, int ra, int rg, int taps, float eps, const void* conv, const void* a2, const void* dt_bias, const void* rate,
                             const void* g2, const void* norm_w, void* history, void* state, const void* seqs, int n_seqs, void* out, int rows_limit,
-                            int blocks, void* mats, void* u, void* dec, void* o, cudaStream_t stream) {
+                            int blocks, void* mats, void* u, void* o, void* status, cudaStream_t stream) {
     using namespace ps;
     DeltaChunkArgs c;
     const int err = delta_args(c.a, proj, ld, H, G, dk, dv, dk_true, dv_true, q_off, b_off, a_off, g_off, ra, rg, taps, eps, conv, a2, dt_bias, rate,
                                g2, norm_w, history, state, seqs, n_seqs, out);
     if (err) return err;
-    if (blocks <= 0 || rows_limit < 1 || !ps_delta_chunked_ok(dk, dv, ra, rg) || mats == nullptr || u == nullptr || dec == nullptr || o == nullptr ||
+    if (blocks <= 0 || rows_limit < 1 || !ps_delta_chunked_ok(dk, dv, ra, rg) || mats == nullptr || u == nullptr || o == nullptr ||
         ((uintptr_t)mats | (uintptr_t)u | (uintptr_t)o) % 16)
         return (int)cudaErrorInvalidValue;
     c.a.rows_limit = rows_limit;
-    c.mats = (__nv_bfloat16*)mats; c.u = (float*)u; c.dec = (float*)dec; c.o = (float*)o;
+    c.mats = (unsigned char*)mats; c.u = (float*)u; c.o = (float*)o; c.status = (uint32_t*)status; c.budget = g_ps_wait_budget_cycles;
     if (dk == 128) return dv == 128 ? launch_delta_chunked<128, 128>(c, blocks, stream) : launch_delta_chunked<128, 64>(c, blocks, stream);
     return dv == 128 ? launch_delta_chunked<64, 128>(c, blocks, stream) : launch_delta_chunked<64, 64>(c, blocks, stream);
 }

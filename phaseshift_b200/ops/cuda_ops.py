@@ -1038,7 +1038,7 @@ class CudaOps(OpTrace):
             C = int(L.ps_delta_block_rows())
             blocks = sum(-(-n // C) for n in long)
             _lib.call("ps_delta_chunked", ptr(proj), c_int(proj.stride(0)), *args, c_int(T), c_int(blocks),
-                      *[ptr(t) for t in self._delta_scratch(blocks, rows, C, d)])
+                      *[ptr(t) for t in self._delta_scratch(blocks, rows, C, d)], ptr(self.status))
             self.launches += 3
         if not long or len(long) < len(seq_rows):
             _lib.call("ps_delta_rows", ptr(proj), c_int(proj.stride(0)), c_int(1 if f32 else 0), *args, c_int(T if long else 0))
@@ -1046,12 +1046,12 @@ class CudaOps(OpTrace):
         return out
 
     def _delta_scratch(self, blocks: int, rows: int, C: int, d: DeltaSpec):
-        """Scratch of the chunked delta rule (its matrices as bf16 pairs, U, block decays, outputs before the head norm); one
+        """Scratch of the chunked delta rule (its matrices as bf16 pairs with the decays, U, outputs before the head norm); one
         allocation that grows to the largest step seen."""
         L = _lib.lib()
         L.ps_delta_mats.restype = ctypes.c_longlong
         n = blocks * d.heads
-        sizes = [n * int(L.ps_delta_mats(c_int(d.dk))) // 2, n * C * d.dv, n * d.dk, rows * d.heads * d.dv]
+        sizes = [n * int(L.ps_delta_mats(c_int(d.dk))) // 4, n * C * d.dv, rows * d.heads * d.dv]
         t = getattr(self, "_delta_buf", None)
         if t is None or t.numel() < sum(sizes):
             t = self._delta_buf = torch.empty(sum(sizes), dtype=torch.float32, device=self.device)

@@ -30,7 +30,7 @@ def test_library_gemm_only_in_reference_and_optional_paths():
     """`@` / matmul / einsum on activations is allowed in the CPU reference ops, the fp32 oracle, quantiser tooling, the
     optional torch drafters and tests -- not in the CUDA op set, the engine, the native drafter or the transport."""
     hot = ["ops/cuda_ops.py", "runtime/engine.py", "runtime/serving.py", "runtime/spec_serving.py", "parallel/tp.py",
-           "models/dflash2/native.py", "models/qwen35/model.py", "models/gebuzen/model.py"]
+           "models/dflash2/native.py", "models/qwen35/model.py", "models/gebuzen/model.py", "models/rotutar/model.py"]
     bad = []
     for rel in hot:
         txt = (PKG / rel).read_text()
